@@ -213,6 +213,47 @@ rcu_status rcu_index_write(rcu_device* dev, rcu_tensor* dst, const rcu_tensor* s
 rcu_status rcu_conv1d(rcu_device* dev, const rcu_tensor* x, const rcu_tensor* w, const rcu_tensor* bias,
                       uint32_t stride, uint32_t padding, rcu_tensor* dst);
 
+/* ------------------------------------------------------------------ ops of models with a 32-bit residual stream
+ * No counterpart in the reference, whose models keep activations in one dtype between ops (ratchet-nn/src/norm.rs:37-69).
+ * The residual stream, norms, gates, attention scores and recurrent states are f32; matrix products take bf16 or f16
+ * operands (or f32: then everything is true f32). */
+/* dst[M, N] = resid + alpha * (x[:, x_col : x_col + K] . w[N, K]^T + bias): x's last dimension may be wider than K.  w and x
+ * have one float dtype; dst has it too (resid NULL, alpha 1) or is F32.  bias [N] in dst's dtype, resid F32 (may be dst);
+ * both nullable. */
+rcu_status rcu_linear(rcu_device* dev, const rcu_tensor* w, const rcu_tensor* x, uint32_t x_col, const rcu_tensor* bias, const rcu_tensor* resid,
+                      float alpha, rcu_tensor* dst);
+/* LayerNorm without bias / RMSNorm over columns [x_col, x_col + N) of f32 rows (N = scale's length), statistics in f32 (the
+ * variance from the deviations), times sigmoid of columns [gate_col, gate_col + N) of `gate` (nullable, dst's dtype).  dst
+ * [rows, N] in any float dtype. */
+rcu_status rcu_norm_rows(rcu_device* dev, int kind, const rcu_tensor* x, uint32_t x_col, const rcu_tensor* scale, const rcu_tensor* gate,
+                         uint32_t gate_col, float eps, rcu_tensor* dst);
+/* Gated feed-forward activation: x [.., 2F] holds gate then up, dst [.., F] = act(gate) * up; act is RCU_GELU (tanh form) or
+ * RCU_SILU, evaluated in f32. */
+rcu_status rcu_glu(rcu_device* dev, int act, const rcu_tensor* x, rcu_tensor* dst);
+/* Frequencies of rotary pairs on the host: host_freqs [2, dims / 2] receives base^(-2i/dims) as f32 value and remainder,
+ * *magnitude the factor on cos and sin.  factor > 0 applies YaRN (Peng et al., "YaRN: Efficient Context Window Extension of
+ * Large Language Models"): frequencies blended with themselves over `factor` by a ramp between the pairs that turn `fast` and
+ * `slow` times over `original` positions, magnitude 0.1 ln(factor) + 1.  factor 0: plain.  Touches no device. */
+rcu_status rcu_rotary_frequencies(uint32_t dims, double base, double factor, double original, double fast, double slow, float* host_freqs,
+                                  float* magnitude);
+/* Rotation of interleaved pairs (first + 2i, first + 2i + 1) of every head by position * freqs[i]: x [tokens, heads, dim], token
+ * t at `position` + t, freqs F32 [2, pairs] (value and remainder).  dst may alias x.  (rcu_rope rotates half-split pairs.) */
+rcu_status rcu_rotary(rcu_device* dev, const rcu_tensor* x, uint32_t first, const rcu_tensor* freqs, float magnitude, uint32_t position, rcu_tensor* dst);
+/* Linear attention with a fixed decay per head: S <- d S + k v^T, o = S^T q over the rows of x, whose columns are q [H, D], k
+ * [H, D], v [H, E] (further columns are ignored), passed through silu first when `silu` is set.  decay_pow F32 [H, n >= 2]: d^0,
+ * d^1, ... (64 or more of them let long blocks run in chunks); state F32 [H, D, E], updated in place; dst F32 [tokens, H * E]. */
+rcu_status rcu_lightning(rcu_device* dev, const rcu_tensor* x, const rcu_tensor* decay_pow, rcu_tensor* state, int silu, rcu_tensor* dst);
+/* Latent cache of a sliding-window layer: columns [x_col, x_col + C) of the f32 rows x are RMS-normed with `scale` [C], the
+ * R = ring width - C columns behind them rotated (rcu_rotary); the rows go into `ring` [ring rows, C + R] (position p in row p mod
+ * ring rows) and dst [L, C + R] receives the L rows the block sees: L - T older ones from the ring, then the block's T. */
+rcu_status rcu_latent_append(rcu_device* dev, const rcu_tensor* x, uint32_t x_col, const rcu_tensor* scale, float eps, const rcu_tensor* freqs,
+                             float magnitude, uint32_t position, rcu_tensor* ring, rcu_tensor* dst);
+/* Softmax attention with a sliding window and a key part shared by the heads: q [T, H, D + R]; kv [L, H * D + H * vdim] (every
+ * head's keys, then its values); columns [shared_col, ..) of `shared` [L, ..] are the R shared key features.  Query i is row
+ * L - T + i of the keys and sees itself and the window - 1 rows before it.  dst [T, H * vdim]. */
+rcu_status rcu_window_attention(rcu_device* dev, const rcu_tensor* q, const rcu_tensor* kv, const rcu_tensor* shared, uint32_t shared_col, uint32_t vdim,
+                                uint32_t window, float scale, rcu_tensor* dst);
+
 /* ------------------------------------------------------------------ lazy tensor graph (tensor.rs)
  * rcu_lazy is ratchet-core's `Tensor` (tensor.rs:45-47): a reference-counted node of a lazy DAG.
  * Builders validate their arguments and compute the output view exactly when the reference's
@@ -256,6 +297,20 @@ rcu_status rcu_lazy_concat(rcu_lazy* const* inputs, uint32_t n, uint32_t dim, rc
 rcu_status rcu_lazy_index_select(rcu_lazy* src, rcu_lazy* ids, uint32_t dim, rcu_lazy** out);
 rcu_status rcu_lazy_cache(rcu_lazy* cache, rcu_lazy* src, uint32_t dim, uint32_t offset, rcu_lazy** out);
 rcu_status rcu_lazy_index_write(rcu_lazy* dst, rcu_lazy* src, const uint64_t* start, rcu_lazy** out);
+
+/* The ops of models with a 32-bit residual stream as nodes (arguments as their eager forms; nullable handles are NULL).
+ * rcu_lazy_linear writes into `resid` when it is its sole owner; rcu_lazy_lightning and rcu_lazy_latent_append update their
+ * state / ring as a side effect, as rcu_lazy_cache does. */
+rcu_status rcu_lazy_linear(rcu_lazy* w, rcu_lazy* x, uint32_t x_col, rcu_lazy* bias, rcu_lazy* resid, float alpha, int32_t dst_dt, rcu_lazy** out);
+rcu_status rcu_lazy_norm_rows(int kind, rcu_lazy* x, uint32_t x_col, rcu_lazy* scale, rcu_lazy* gate, uint32_t gate_col, float eps, int32_t dst_dt,
+                              rcu_lazy** out);
+rcu_status rcu_lazy_glu(int act, rcu_lazy* x, rcu_lazy** out);
+rcu_status rcu_lazy_rotary(rcu_lazy* x, uint32_t first, rcu_lazy* freqs, float magnitude, uint32_t position, rcu_lazy** out);
+rcu_status rcu_lazy_lightning(rcu_lazy* x, rcu_lazy* decay_pow, rcu_lazy* state, int silu, rcu_lazy** out);
+rcu_status rcu_lazy_latent_append(rcu_lazy* x, uint32_t x_col, rcu_lazy* scale, float eps, rcu_lazy* freqs, float magnitude, uint32_t position,
+                                  rcu_lazy* ring, uint32_t rows, rcu_lazy** out);
+rcu_status rcu_lazy_window_attention(rcu_lazy* q, rcu_lazy* kv, rcu_lazy* shared, uint32_t shared_col, uint32_t vdim, uint32_t window, float scale,
+                                     rcu_lazy** out);
 
 /* Tensor::id (tensor.rs:100-104): process-wide unique, increasing with creation. */
 uint64_t rcu_lazy_id(const rcu_lazy* t);
@@ -358,6 +413,52 @@ rcu_status rcu_attn_decode(rcu_device* dev, const void* qkv, void* k_cache, void
 rcu_status rcu_attn_decode_static(rcu_device* dev, const void* qkv, void* k_cache, void* v_cache, uint32_t n_heads,
                                   uint32_t n_kv_heads, uint32_t head_dim, uint32_t max_cache, uint32_t rope_dim,
                                   float rope_base, uint32_t position, void* out);
+
+/* ------------------------------------------------------------------ fused decode step of a layer stack
+ * The batch-1 step of models built from parallel-residual layers x <- x + m (mixer(norm1 x) + ff(norm2 x)) (LayerNorm without bias,
+ * gelu-gated feed-forward) whose mixers are linear attention (rcu_lightning) or latent attention with a sliding window
+ * (rcu_latent_append, rcu_window_attention): three or six kernels per layer run, replayed from a CUDA graph.  No counterpart in
+ * the reference.  Runs are listed in execution order; a layer that is run several times appears once per run, each with a state of
+ * its own.  Weights are weight_dt (BF16 or F32), norm scales, biases, decays and frequencies F32, activations f32.  All
+ * pointers are device memory owned by the caller and must outlive the stack. */
+typedef struct rcu_stack rcu_stack;
+typedef enum { RCU_MIXER_LIGHTNING = 0, RCU_MIXER_LATENT = 1 } rcu_mixer_kind;
+typedef struct {
+    uint32_t width, vocab, n_runs;
+    float eps, residual_mult;
+    int32_t weight_dt;
+} rcu_stack_config;
+typedef struct {
+    int32_t mixer;           /* rcu_mixer_kind */
+    uint32_t heads, dim, vdim, ff;   /* ff 0: no feed-forward */
+    uint32_t q_rank, kv_rank, rot_dim, rot_pairs, window, ring_rows;   /* latent mixer */
+    float scale, rot_magnitude;
+    const void* enter;       /* nullable [width, 2 width]: x <- enter . [x; embedding output] + enter_bias before this run */
+    const void* enter_bias;  /* F32 [width] */
+    const void* norm1;       /* F32 [width] */
+    const void* norm2;
+    const void* mix_in;      /* lightning: q, k, v, gate rows; latent: query-latent, latent, rotated-key rows */
+    const void* mix_norm;    /* F32: lightning [heads * vdim], latent [q_rank] */
+    const void* kv_norm;     /* F32 [kv_rank] */
+    const void* uq;          /* [heads * (dim + rot_dim), q_rank] */
+    const void* ukv;         /* key rows [heads * dim, kv_rank], then value rows [heads * vdim, kv_rank] */
+    const void* freqs;       /* F32 [2, rot_pairs] */
+    const void* decay;       /* F32 [heads] */
+    const void* out;         /* [width, heads * vdim] */
+    const void* gate_up;     /* [2 ff, width]: gate rows, then up rows */
+    const void* down;        /* [width, ff] */
+    void* state;             /* lightning: F32 [heads, dim, vdim]; latent: ring [ring_rows, kv_rank + rot_dim] in weight_dt */
+} rcu_stack_run;
+rcu_status rcu_stack_create(rcu_device* dev, const rcu_stack_config* cfg, const rcu_stack_run* runs, const void* embed, const void* final_norm,
+                            const void* head, rcu_stack** out);
+void rcu_stack_destroy(rcu_stack* stack);
+/* Position of the next token (a prompt that ran through the lazy graph over the same states moves it here). */
+rcu_status rcu_stack_set_position(rcu_stack* stack, uint32_t position);
+uint32_t rcu_stack_position(const rcu_stack* stack);
+/* One token: id from device memory, f32 logits [vocab] and (argmax_dev not NULL) the arg-max id to device memory; argmax_dev
+ * may be token_dev.  Advances the position.  Asynchronous on the device stream. */
+rcu_status rcu_stack_step(rcu_stack* stack, const int32_t* token_dev, float* logits_dev, int32_t* argmax_dev);
+uint32_t rcu_stack_kernels_per_step(const rcu_stack* stack);
 
 /* ------------------------------------------------------------------ row-sharded Linear over the GPUs of a node
  * No counterpart in the reference, which is single-device (gpu/device.rs:15-16).  A Linear's weight

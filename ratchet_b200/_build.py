@@ -17,6 +17,8 @@ HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
 OBJ = os.path.join(CSRC, "_obj")
 LIB = os.path.join(HERE, "libratchet_cuda.so")
+CORE_LIB = os.path.join(HERE, "libratchet_cuda_core.so")
+NOT_CORE = {"decode.cu", "comm.cu", "gguf.cu"}
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a",
@@ -62,15 +64,37 @@ def build(force: bool = False, verbose: bool = False) -> str:
     if force:
         for f in glob.glob(os.path.join(OBJ, "*.o")):
             os.remove(f)
-    sources = sorted(glob.glob(os.path.join(CSRC, "*.cu")))
-    with cf.ThreadPoolExecutor(max_workers=min(8, len(sources))) as ex:
-        objs = list(ex.map(lambda s: _compile(s, verbose), sources))
-    if _stale(LIB, objs):
-        cmd = [nvcc(), "-shared", "-o", LIB] + objs + ["-gencode", "arch=compute_100a,code=sm_100a", "-lcudart", "-ldl"]
+    return _link(LIB, _sources(), verbose)
+
+
+def _sources(core: bool = False):
+    return [s for s in sorted(glob.glob(os.path.join(CSRC, "*.cu"))) if not (core and os.path.basename(s) in NOT_CORE)]
+
+
+def _link(lib: str, sources, verbose: bool) -> str:
+    # the longest translation units first: they decide how long a parallel build takes
+    by_size = sorted(sources, key=os.path.getsize, reverse=True)
+    with cf.ThreadPoolExecutor(max_workers=min(len(sources), max(8, os.cpu_count() or 8))) as ex:
+        objs = sorted(ex.map(lambda s: _compile(s, verbose), by_size))
+    if _stale(lib, objs):
+        part = f"{lib}.{os.getpid()}"
+        cmd = [nvcc(), "-shared", "-o", part] + objs + ["-gencode", "arch=compute_100a,code=sm_100a", "-lcudart", "-ldl"]
         proc = subprocess.run(cmd, capture_output=True, text=True)
         if proc.returncode != 0:
             raise RuntimeError(f"link failed:\n{proc.stdout}\n{proc.stderr}")
-    return LIB
+        os.replace(part, lib)
+    return lib
+
+
+def ensure_runtime() -> str:
+    """Path of a library that is newer than its sources: the full one where it has been built, else the core library,
+    built first if need be."""
+    if not _stale(LIB, _sources() + _headers()):
+        return LIB
+    if _stale(CORE_LIB, _sources(core=True) + _headers()):
+        os.makedirs(OBJ, exist_ok=True)
+        _link(CORE_LIB, _sources(core=True), False)
+    return CORE_LIB
 
 
 if __name__ == "__main__":

@@ -3,7 +3,10 @@ scheduled through the lazy ``Tensor`` API exactly as the reference schedules the
 
 * Phi-3 decoder (crates/ratchet-models/src/phi3/{attn,mlp,model}.rs),
 * the Phi-2 MLP block inside its parallel-residual layer (phi2/mlp.rs:13-15, phi2/model.rs:78-89),
-* the Whisper encoder (whisper/{encoder,residual_block,mha,mlp}.rs).
+* the Whisper encoder (whisper/{encoder,residual_block,mha,mlp}.rs);
+
+and one decoder the reference does not have, Dadezen: parallel layers over linear attention and windowed latent
+attention, with a loop of layers that runs several times.
 
 They only call ``Tensor`` builder methods, as ``Module::schedule`` does in the reference; no device
 code lives here.
@@ -13,6 +16,7 @@ from __future__ import annotations
 from typing import List, Optional
 
 from . import capi
+from .nn import GatedMLP, RotaryTable, SequenceState, StreamNorm
 from .nn import KVCache, KVEntry, LayerNorm, Linear, RMSNorm, RotaryEmbedding, Embedding
 
 
@@ -180,3 +184,86 @@ class WhisperEncoder:
         for blk in self.blocks:
             x = blk.schedule(x)
         return self.ln_post.schedule(x)
+
+
+# ---------------------------------------------------------------------------------------- Dadezen
+class LightningMixer:
+    """Linear attention with a fixed decay per head; the output, RMS-normed over all heads and gated, goes through the output
+    projection into the residual stream.  ``proj`` stacks the q, k, v and gate rows; ``decay`` [heads] serves single tokens, its
+    powers ``decay_pow`` [heads, n] blocks."""
+
+    def __init__(self, proj, decay, decay_pow, norm: StreamNorm, out, heads: int, dim: int, vdim: int):
+        self.proj, self.decay, self.decay_pow, self.norm, self.out = proj, decay, decay_pow, norm, out
+        self.heads, self.dim, self.vdim = heads, dim, vdim
+
+    def schedule(self, h, resid, alpha: float, state, position: int):
+        rows = self.proj.linear(h)
+        o = rows.lightning(self.decay_pow, state, True)
+        y = self.norm.schedule(o, gate=rows, gate_col=self.heads * (2 * self.dim + self.vdim))
+        return self.out.linear(y, resid=resid, alpha=alpha, dt=capi.F32)
+
+
+class LatentMixer:
+    """Sliding-window attention whose keys and values are linear images of a cached latent; one rotated key part is shared
+    by the heads.  ``low`` stacks the query-latent, latent and rotated-key rows, ``ukv`` the key and value rows."""
+
+    def __init__(self, low, q_norm: StreamNorm, uq, kv_norm: StreamNorm, ukv, rot: RotaryTable, out, heads: int, dim: int, rot_dim: int,
+                 vdim: int, window: int, scale: float):
+        self.low, self.q_norm, self.uq, self.kv_norm, self.ukv, self.rot, self.out = low, q_norm, uq, kv_norm, ukv, rot, out
+        self.heads, self.dim, self.rot_dim, self.vdim, self.window, self.scale = heads, dim, rot_dim, vdim, window, scale
+
+    def schedule(self, h, resid, alpha: float, ring, position: int):
+        tokens = h.shape()[0]
+        q_rank, kv_rank = self.uq.shape()[1], self.ukv.shape()[1]
+        low = self.low.linear(h, dt=capi.F32)
+        q = self.uq.linear(self.q_norm.schedule(low)).view([tokens, self.heads, self.dim + self.rot_dim])
+        q = q.rotary(self.rot.freqs, self.rot.magnitude, position, first=self.dim)
+        rows = tokens + min(position, self.window - 1)
+        seen = low.latent_append(self.kv_norm.weight, self.kv_norm.eps, self.rot.freqs, self.rot.magnitude, position, ring, rows, col=q_rank)
+        o = q.window_attention(self.ukv.linear(seen), seen, kv_rank, self.vdim, self.window, self.scale)
+        return self.out.linear(o, resid=resid, alpha=alpha, dt=capi.F32)
+
+
+class ParallelLayer:
+    """x + alpha * (mixer(norm1 x) + mlp(norm2 x)), both branches from the same x; no mlp: the mixer alone."""
+
+    def __init__(self, norm1: StreamNorm, mixer, norm2: Optional[StreamNorm], mlp: Optional[GatedMLP], alpha: float):
+        self.norm1, self.mixer, self.norm2, self.mlp, self.alpha = norm1, mixer, norm2, mlp, alpha
+
+    def schedule(self, x, state, position: int):
+        y = self.mixer.schedule(self.norm1.schedule(x), x, self.alpha, state, position)
+        return y if self.mlp is None else self.mlp.schedule(self.norm2.schedule(x), y, self.alpha)
+
+
+class LoopEntry:
+    """x <- W [x; x0] + step, before the first layer of a pass."""
+
+    def __init__(self, w, steps: List):
+        self.w, self.steps = w, steps
+
+    def schedule(self, x, x0, t: int):
+        both = type(x).cat([x.cast(x0.dt()), x0], 1)
+        return self.w.linear(both, bias=self.steps[t], dt=capi.F32)
+
+
+class Dadezen:
+    """``runs``: (layer index, pass or None) in execution order; ``first``: the layer a pass begins with."""
+
+    def __init__(self, embedding: Embedding, layers: List[ParallelLayer], runs, first: Optional[int], entry: Optional[LoopEntry],
+                 norm: StreamNorm, head):
+        self.embedding, self.layers, self.runs, self.first, self.entry, self.norm, self.head = embedding, layers, runs, first, entry, norm, head
+
+    def schedule(self, ids, state: SequenceState, want=None, streams: Optional[list] = None):
+        """ids: a block of token ids, following `state.position` earlier ones.  Logits f32 [len(want), vocab] of the places in
+        the i32 tensor `want`, or - without one - the residual stream (which still runs every layer)."""
+        x0 = self.embedding.schedule(ids)
+        x = x0.full()
+        for k, (i, t) in enumerate(self.runs):
+            if t is not None and i == self.first:
+                x = self.entry.schedule(x, x0, t)
+            x = self.layers[i].schedule(x, state.runs[k], state.position)
+            if streams is not None:
+                streams.append(x)
+        if want is None:
+            return x
+        return self.head.linear(self.norm.schedule(x.index_select(want, 0)), dt=capi.F32)

@@ -13,6 +13,7 @@ import numpy as np
 
 _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_HERE, "libratchet_cuda.so")
+CORE_LIB_PATH = os.path.join(_HERE, "libratchet_cuda_core.so")     # without the symbols of _NOT_CORE
 
 RCU_MAX_RANK = 4
 
@@ -33,6 +34,7 @@ UNARY_OPS = {"gelu": 0, "tanh": 1, "exp": 2, "log": 3, "sin": 4, "cos": 5, "abs"
 LAYER_NORM, RMS_NORM, GROUP_NORM = 0, 1, 2
 DEBUG_NO_REUSE, DEBUG_PROFILE, DEBUG_LOG = 1, 2, 4
 REDUCE_SUM, REDUCE_MAX, REDUCE_MEAN = 0, 1, 2
+MIXER_LIGHTNING, MIXER_LATENT = 0, 1
 
 
 class RatchetCudaError(RuntimeError):
@@ -65,6 +67,19 @@ class rcu_gguf_tensor_info(C.Structure):
 class rcu_decoder_layer(C.Structure):
     _fields_ = [("attn_norm", C.c_void_p), ("qkv", C.c_void_p), ("o", C.c_void_p), ("ffn_norm", C.c_void_p),
                 ("gate_up", C.c_void_p), ("down", C.c_void_p), ("k_cache", C.c_void_p), ("v_cache", C.c_void_p)]
+
+
+class rcu_stack_config(C.Structure):
+    _fields_ = [("width", C.c_uint32), ("vocab", C.c_uint32), ("n_runs", C.c_uint32), ("eps", C.c_float), ("residual_mult", C.c_float),
+                ("weight_dt", C.c_int32)]
+
+
+class rcu_stack_run(C.Structure):
+    _fields_ = ([("mixer", C.c_int32)] +
+                [(n, C.c_uint32) for n in ("heads", "dim", "vdim", "ff", "q_rank", "kv_rank", "rot_dim", "rot_pairs", "window", "ring_rows")] +
+                [("scale", C.c_float), ("rot_magnitude", C.c_float)] +
+                [(n, C.c_void_p) for n in ("enter", "enter_bias", "norm1", "norm2", "mix_in", "mix_norm", "kv_norm", "uq", "ukv", "freqs", "decay",
+                                           "out", "gate_up", "down", "state")])
 
 
 _T = C.POINTER(rcu_tensor)
@@ -119,6 +134,15 @@ SIGNATURES = {
     "rcu_cache": (C.c_int, [_DEV, _T, _T, C.c_uint32, C.c_uint32, _T]),
     "rcu_index_write": (C.c_int, [_DEV, _T, _T, _u64p]),
     "rcu_conv1d": (C.c_int, [_DEV, _T, _T, _T, C.c_uint32, C.c_uint32, _T]),
+    # models with a 32-bit residual stream
+    "rcu_linear": (C.c_int, [_DEV, _T, _T, C.c_uint32, _T, _T, C.c_float, _T]),
+    "rcu_norm_rows": (C.c_int, [_DEV, C.c_int, _T, C.c_uint32, _T, _T, C.c_uint32, C.c_float, _T]),
+    "rcu_glu": (C.c_int, [_DEV, C.c_int, _T, _T]),
+    "rcu_rotary_frequencies": (C.c_int, [C.c_uint32] + [C.c_double] * 5 + [C.POINTER(C.c_float), C.POINTER(C.c_float)]),
+    "rcu_rotary": (C.c_int, [_DEV, _T, C.c_uint32, _T, C.c_float, C.c_uint32, _T]),
+    "rcu_lightning": (C.c_int, [_DEV, _T, _T, _T, C.c_int, _T]),
+    "rcu_latent_append": (C.c_int, [_DEV, _T, C.c_uint32, _T, C.c_float, _T, C.c_float, C.c_uint32, _T, _T]),
+    "rcu_window_attention": (C.c_int, [_DEV, _T, _T, _T, C.c_uint32, C.c_uint32, C.c_uint32, C.c_float, _T]),
     # lazy tensor graph
     "rcu_lazy_from_host": (C.c_int, [_DEV, C.c_int32, C.c_uint32, _u64p, C.c_void_p, C.c_uint64, C.POINTER(_LZ)]),
     "rcu_lazy_zeros": (C.c_int, [_DEV, C.c_int32, C.c_uint32, _u64p, C.POINTER(_LZ)]),
@@ -143,6 +167,13 @@ SIGNATURES = {
     "rcu_lazy_index_select": (C.c_int, [_LZ, _LZ, C.c_uint32, C.POINTER(_LZ)]),
     "rcu_lazy_cache": (C.c_int, [_LZ, _LZ, C.c_uint32, C.c_uint32, C.POINTER(_LZ)]),
     "rcu_lazy_index_write": (C.c_int, [_LZ, _LZ, _u64p, C.POINTER(_LZ)]),
+    "rcu_lazy_linear": (C.c_int, [_LZ, _LZ, C.c_uint32, _LZ, _LZ, C.c_float, C.c_int32, C.POINTER(_LZ)]),
+    "rcu_lazy_norm_rows": (C.c_int, [C.c_int, _LZ, C.c_uint32, _LZ, _LZ, C.c_uint32, C.c_float, C.c_int32, C.POINTER(_LZ)]),
+    "rcu_lazy_glu": (C.c_int, [C.c_int, _LZ, C.POINTER(_LZ)]),
+    "rcu_lazy_rotary": (C.c_int, [_LZ, C.c_uint32, _LZ, C.c_float, C.c_uint32, C.POINTER(_LZ)]),
+    "rcu_lazy_lightning": (C.c_int, [_LZ, _LZ, _LZ, C.c_int, C.POINTER(_LZ)]),
+    "rcu_lazy_latent_append": (C.c_int, [_LZ, C.c_uint32, _LZ, C.c_float, _LZ, C.c_float, C.c_uint32, _LZ, C.c_uint32, C.POINTER(_LZ)]),
+    "rcu_lazy_window_attention": (C.c_int, [_LZ, _LZ, _LZ, C.c_uint32, C.c_uint32, C.c_uint32, C.c_float, C.POINTER(_LZ)]),
     "rcu_lazy_id": (C.c_uint64, [_LZ]),
     "rcu_lazy_execution_order": (C.c_int, [_LZ, _u64p, C.c_uint32, _u32p]),
     "rcu_lazy_resolve": (C.c_int, [_LZ]),
@@ -174,6 +205,13 @@ SIGNATURES = {
     "rcu_decoder_profile_step": (C.c_int, [C.c_void_p, C.c_void_p, C.c_void_p, _u64p, C.c_uint32, _u32p]),
     "rcu_attn_decode_static": (C.c_int, [_DEV, C.c_void_p, C.c_void_p, C.c_void_p, C.c_uint32, C.c_uint32, C.c_uint32, C.c_uint32,
                                          C.c_uint32, C.c_float, C.c_uint32, C.c_void_p]),
+    "rcu_stack_create": (C.c_int, [_DEV, C.POINTER(rcu_stack_config), C.POINTER(rcu_stack_run), C.c_void_p, C.c_void_p, C.c_void_p,
+                                   C.POINTER(C.c_void_p)]),
+    "rcu_stack_destroy": (None, [C.c_void_p]),
+    "rcu_stack_set_position": (C.c_int, [C.c_void_p, C.c_uint32]),
+    "rcu_stack_position": (C.c_uint32, [C.c_void_p]),
+    "rcu_stack_step": (C.c_int, [C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p]),
+    "rcu_stack_kernels_per_step": (C.c_uint32, [C.c_void_p]),
     "rcu_comm_create": (C.c_int, [_DEV, C.c_int, C.c_int, C.c_uint64, C.POINTER(C.c_void_p)]),
     "rcu_comm_export": (C.c_int, [C.c_void_p, C.c_void_p]),
     "rcu_comm_import": (C.c_int, [C.c_void_p, C.c_int, C.c_void_p]),
@@ -186,18 +224,27 @@ SIGNATURES = {
                                   C.c_uint32, C.c_float, C.c_uint32, C.c_void_p]),
 }
 
+# prefixes of what only the full library exports
+_NOT_CORE = ("rcu_decoder_", "rcu_attn_", "rcu_comm_", "rcu_gemv_q8_allgather", "rcu_gguf_")
+
 _lib = None
 
 
-def lib() -> C.CDLL:
-    """Load the shared library (built in-tree by ``ratchet_b200._build``). Fails loudly if absent."""
+def lib(path: str = None) -> C.CDLL:
+    """Load the shared library (built in-tree by ``ratchet_b200._build``; `path`: this one, if none is loaded yet).  Fails
+    loudly if absent."""
     global _lib
     if _lib is None:
-        if not os.path.exists(LIB_PATH):
-            raise RatchetCudaError(ERR_CUDA, f"{LIB_PATH} is missing: run `python -m ratchet_b200._build` "
+        if path is None:
+            path = LIB_PATH if os.path.exists(LIB_PATH) or not os.path.exists(CORE_LIB_PATH) else CORE_LIB_PATH
+        if not os.path.exists(path):
+            raise RatchetCudaError(ERR_CUDA, f"{path} is missing: run `python -m ratchet_b200._build` "
                                              "(there is no CPU fallback)")
-        handle = C.CDLL(LIB_PATH)
+        handle = C.CDLL(path)
+        core = os.path.basename(path) == os.path.basename(CORE_LIB_PATH)
         for name, (res, args) in SIGNATURES.items():
+            if core and name.startswith(_NOT_CORE):
+                continue
             fn = getattr(handle, name)  # AttributeError here = the library does not export a declared symbol
             fn.restype = res
             fn.argtypes = args
@@ -227,6 +274,28 @@ def quantize(x: np.ndarray) -> np.ndarray:
     if st != OK:
         raise RatchetCudaError(st, f"rcu_quantize({DTYPE_NAMES[dt]}, numel={x.size})")
     return out
+
+
+def to_bf16(x: np.ndarray) -> np.ndarray:
+    """f32 -> bf16 bit patterns (uint16), round to nearest even; NaN stays NaN."""
+    u = np.ascontiguousarray(x, np.float32).view(np.uint32)
+    r = ((u >> 16) & 1) + 0x7FFF
+    out = ((u.astype(np.uint64) + r) >> 16).astype(np.uint16)
+    return np.where(np.isnan(x), np.uint16(0x7FC0), out)
+
+
+def from_bf16(u: np.ndarray) -> np.ndarray:
+    """bf16 bit patterns (uint16) -> f32."""
+    return (np.ascontiguousarray(u, np.uint16).astype(np.uint32) << 16).view(np.float32)
+
+
+def rotary_frequencies(dims: int, base: float, factor: float = 0.0, original: float = 0.0, fast: float = 0.0, slow: float = 0.0):
+    """(f32 [2, dims / 2] table of frequencies as value and remainder, factor on cos and sin); factor > 0: YaRN."""
+    out, mag = np.empty((2, dims // 2), np.float32), C.c_float()
+    st = lib().rcu_rotary_frequencies(dims, base, factor, original, fast, slow, out.ctypes.data_as(C.POINTER(C.c_float)), C.byref(mag))
+    if st != OK:
+        raise RatchetCudaError(st, f"rotary_frequencies(dims={dims}, base={base}, factor={factor})")
+    return out, mag.value
 
 
 def activation_dtype(dt: int) -> int:

@@ -55,10 +55,10 @@ __host__ __device__ constexpr int conv_warps(int bn) { return bn >= 128 ? 8 : 4;
 
 // Two CTAs share an SM (half of its shared memory and at most half of its tensor memory each), so one
 // CTA's pipeline fill and epilogue overlap the other's main loop.
-template <int BN, int WK, int STAGES>
+template <int BN, int WK, int STAGES, class Out>
 __global__ void __launch_bounds__(WK == WK_F16 ? kThreadsTc : kThreadsTc + conv_warps(BN) * 32, 2)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant__ CUtensorMap wmap, const QuantArgs qa,
-               const __half* __restrict__ bias, __half* __restrict__ out, int M, int N, int K, int* status, int splits, float* __restrict__ partial) {
+               const GemmEpilogue<Out> epi, Out* out, int M, int N, int K, int* status, int splits, float* __restrict__ partial, uint32_t idesc) {
     rcu_kernel_entry_wait_only();
     constexpr int A_BYTES = TM * TK * 2;          // 16 KiB
     constexpr int B_BYTES = BN * TK * 2;
@@ -126,7 +126,6 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant__
         }
     } else if (warp == 1) {
         if (lane == 0) {
-            constexpr uint32_t idesc = umma_idesc_f16(TM, BN);
             bool ok = true;
             for (int it = 0; it < nk && ok; ++it) {
                 const int s = it % STAGES;
@@ -162,30 +161,21 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant__
                     for (int j = 0; j < 32; j += 4)
                         if (n0 + c + j + 4 <= N) *reinterpret_cast<float4*>(prow + j) = make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]);
                 } else if (row < M) {
-                    __half* orow = out + (size_t)row * N + n0 + c;
+                    const size_t base = (size_t)row * N + n0 + c;
                     if ((N & 7) == 0) {              // rows start on 16-byte boundaries
 #pragma unroll
-                        for (int j = 0; j < 32; j += 8) {
-                            const int col = n0 + c + j;
-                            if (col + 8 <= N) {
-                                __align__(16) __half h[8];
-#pragma unroll
-                                for (int e = 0; e < 8; ++e) h[e] = __float2half_rn(v[j + e] + (bias ? __half2float(bias[col + e]) : 0.f));
-                                *reinterpret_cast<uint4*>(orow + j) = *reinterpret_cast<const uint4*>(h);
-                            } else {
-                                for (int e = 0; e < 8 && col + e < N; ++e)
-                                    orow[j + e] = __float2half_rn(v[j + e] + (bias ? __half2float(bias[col + e]) : 0.f));
-                            }
-                        }
-                    } else {                         // N a multiple of 4 (checked by the host): 8-byte stores
+                        for (int j = 0; j < 32; j += 8)
+                            if (n0 + c + j + 8 <= N) epi.store8(out, base + j, v + j, n0 + c + j);
+                    } else {                         // N a multiple of 4 (checked by the host): 4-element stores
 #pragma unroll
                         for (int j = 0; j < 32; j += 4) {
                             const int col = n0 + c + j;
                             if (col + 4 <= N) {
-                                __align__(8) __half h[4];
+                                __align__(16) Out h[4];
 #pragma unroll
-                                for (int e = 0; e < 4; ++e) h[e] = __float2half_rn(v[j + e] + (bias ? __half2float(bias[col + e]) : 0.f));
-                                *reinterpret_cast<uint2*>(orow + j) = *reinterpret_cast<const uint2*>(h);
+                                for (int e = 0; e < 4; ++e) h[e] = epi(v[j + e], col + e, base + j + e);
+#pragma unroll
+                                for (int e = 0; e < (int)sizeof(Out) / 2; ++e) reinterpret_cast<uint2*>(out + base + j)[e] = reinterpret_cast<const uint2*>(h)[e];
                             }
                         }
                     }
@@ -330,9 +320,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant__
     }
 }
 
-// out[m, n] = f16(sum over slices, in order, of partial[s, m, n] + bias[n]); eight outputs per thread
-__global__ void __launch_bounds__(256) sum_k_slices_kernel(const float* __restrict__ partial, const __half* __restrict__ bias, __half* __restrict__ out,
-                                                          size_t MN, int N, int splits) {
+// out[m, n] = epilogue(sum over slices, in order, of partial[s, m, n]); eight outputs per thread
+template <class Out>
+__global__ void __launch_bounds__(256) sum_k_slices_kernel(const float* __restrict__ partial, const GemmEpilogue<Out> epi, Out* out, size_t MN, int N,
+                                                          int splits) {
     rcu_kernel_entry();
     const size_t i = ((size_t)blockIdx.x * blockDim.x + threadIdx.x) * 8;
     if (i >= MN) return;
@@ -344,21 +335,18 @@ __global__ void __launch_bounds__(256) sum_k_slices_kernel(const float* __restri
         acc[0] += a.x; acc[1] += a.y; acc[2] += a.z; acc[3] += a.w;
         acc[4] += b.x; acc[5] += b.y; acc[6] += b.z; acc[7] += b.w;
     }
-    __align__(16) __half h[8];
-    const int col = (int)(i % (size_t)N);
-#pragma unroll
-    for (int e = 0; e < 8; ++e) h[e] = __float2half_rn(acc[e] + (bias ? __half2float(bias[col + e]) : 0.f));
-    *reinterpret_cast<uint4*>(out + i) = *reinterpret_cast<const uint4*>(h);
+    epi.store8(out, i, acc, (int)(i % (size_t)N));
 }
 
-template <int BN, int WK>
-rcu_status launch_tc(rcu_device* dev, const CUtensorMap& xmap, const CUtensorMap& wmap, const QuantArgs& qa, const void* bias, void* out,
-                     int M, int N, int K, int batch = 1) {
+template <int BN, int WK, class Out = __half>
+rcu_status launch_tc(rcu_device* dev, const CUtensorMap& xmap, const CUtensorMap& wmap, const QuantArgs& qa, const GemmEpilogue<Out>& epi, void* out,
+                     int M, int N, int K, int batch = 1, bool bf16 = false) {
     constexpr int STAGE = TM * TK * 2 + BN * TK * 2;
     constexpr int STAGES = (100 * 1024) / STAGE;     // two CTAs per SM
     const size_t smem = (size_t)STAGES * STAGE + 1024 + 512;
-    auto kern = gemm_tc_kernel<BN, WK, STAGES>;
+    auto kern = gemm_tc_kernel<BN, WK, STAGES, Out>;
     RCU_CUDA(dev, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    const uint32_t idesc = umma_idesc_f16(TM, BN, bf16);
     dim3 grid((N + BN - 1) / BN, (M + TM - 1) / TM, batch);
     const int threads = WK == WK_F16 ? kThreadsTc : kThreadsTc + conv_warps(BN) * 32;
     // Few tiles and a long K (a Linear at a few hundred token rows): every CTA's k loop is a chain of TMA -> convert -> MMA
@@ -375,22 +363,23 @@ rcu_status launch_tc(rcu_device* dev, const CUtensorMap& xmap, const CUtensorMap
         rcu_status st = rcu_alloc(dev, (uint64_t)splits * M * N * 4, &partial);
         if (st != RCU_OK) return st;
         grid.z = splits;
-        rcu_launch(dev, kern, grid, threads, smem, xmap, wmap, qa, nullptr, (__half*)out, M, N, K, dev->d_status, splits, (float*)partial);
+        rcu_launch(dev, kern, grid, threads, smem, xmap, wmap, qa, GemmEpilogue<Out>{nullptr, nullptr, 1.f}, (Out*)out, M, N, K, dev->d_status, splits,
+                   (float*)partial, idesc);
         dev->launches++;
         const size_t MN = (size_t)M * N;
-        rcu_launch(dev, sum_k_slices_kernel, (unsigned)((MN / 8 + 255) / 256), 256, 0, (const float*)partial, (const __half*)bias, (__half*)out, MN, N, splits);
+        rcu_launch(dev, sum_k_slices_kernel<Out>, (unsigned)((MN / 8 + 255) / 256), 256, 0, (const float*)partial, epi, (Out*)out, MN, N, splits);
         rcu_free(dev, partial);      // the pool reuses blocks in stream order
         RCU_LAUNCH_CHECK(dev);
         return RCU_OK;
     }
-    rcu_launch(dev, kern, grid, threads, smem, xmap, wmap, qa, (const __half*)bias, (__half*)out, M, N, K, dev->d_status, 1, nullptr);
+    rcu_launch(dev, kern, grid, threads, smem, xmap, wmap, qa, epi, (Out*)out, M, N, K, dev->d_status, 1, nullptr, idesc);
     RCU_LAUNCH_CHECK(dev);
     return RCU_OK;
 }
 
 // [batch, rows, K] f16, rows `pitch` elements apart (a multiple of 8: tensor-map strides are 16-byte multiples), box =
 // box_rows x 64 elements of one problem, 128-byte swizzle; reads beyond K or rows are filled with zeros
-bool make_map_f16_sw128(CUtensorMap* map, const void* base, uint64_t rows, uint64_t K, uint32_t box_rows, uint64_t batch = 1, uint64_t pitch = 0) {
+bool make_map_f16_sw128(CUtensorMap* map, const void* base, uint64_t rows, uint64_t K, uint32_t box_rows, uint64_t batch = 1, uint64_t pitch = 0, bool bf16 = false) {
     gemvq8::EncodeTiledFn fn = gemvq8::encode_tiled_fn();
     if (!fn) return false;
     if (pitch == 0) pitch = K;
@@ -398,7 +387,7 @@ bool make_map_f16_sw128(CUtensorMap* map, const void* base, uint64_t rows, uint6
     cuuint64_t strides[2] = {pitch * 2, rows * pitch * 2};
     cuuint32_t box[3] = {(cuuint32_t)TK, box_rows, 1};
     cuuint32_t estr[3] = {1, 1, 1};
-    return fn(map, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+    return fn(map, bf16 ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
               CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
@@ -415,14 +404,15 @@ bool rcu_gemm_tc_eligible(int lhs_dt, int act_dt, uint64_t M, uint64_t N, uint64
 
 // gemm_tc2.cu: the CTA-pair kernel for f16 weights
 bool rcu_gemm_tc2_eligible(rcu_device* dev, uint64_t M, uint64_t N, uint64_t K);
-rcu_status rcu_gemm_tc2_launch(rcu_device* dev, const void* w, const void* x, const void* bias, void* y, uint64_t M, uint64_t N, uint64_t K);
+rcu_status rcu_gemm_tc2_launch(rcu_device* dev, const void* w, const void* x, const void* bias, void* y, uint64_t M, uint64_t N, uint64_t K,
+                               const TcLinear& t);
 
 rcu_status rcu_gemm_tc_dispatch(rcu_device* dev, int lhs_dt, const void* w, int act_dt, const void* x, const void* bias, void* y,
                                 uint64_t M, uint64_t N, uint64_t K) {
     if (!rcu_gemm_tc_eligible(lhs_dt, act_dt, M, N, K)) return RCU_ERR_UNSUPPORTED;
     if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(w)) & 15) return RCU_ERR_UNSUPPORTED;
     DevGuard g(dev->ordinal);
-    if (lhs_dt == RCU_F16 && rcu_gemm_tc2_eligible(dev, M, N, K)) return rcu_gemm_tc2_launch(dev, w, x, bias, y, M, N, K);
+    if (lhs_dt == RCU_F16 && rcu_gemm_tc2_eligible(dev, M, N, K)) return rcu_gemm_tc2_launch(dev, w, x, bias, y, M, N, K, TcLinear{});
     // Quantised weights.  The fused kernel converts a weight tile once per 128-row token tile, i.e.
     // M/128 times over the whole problem, and it is the one-CTA kernel.  Beyond kFusedMaxM token rows it
     // is cheaper to convert the matrix once into pooled f16 scratch (which stays in L2) and run the f16
@@ -477,7 +467,7 @@ rcu_status rcu_gemm_tc_dispatch(rcu_device* dev, int lhs_dt, const void* w, int 
     if (!maps)
         st = rcu_fail(dev, RCU_ERR_CUDA, "gemm_tc: cuTensorMapEncodeTiled failed (M=%llu N=%llu K=%llu)", (unsigned long long)M,
                       (unsigned long long)N, (unsigned long long)K);
-#define RCU_TC(BN_, WK_) launch_tc<BN_, WK_>(dev, xmap, wmap, qa, bias, y, (int)M, (int)N, (int)K)
+#define RCU_TC(BN_, WK_) launch_tc<BN_, WK_>(dev, xmap, wmap, qa, GemmEpilogue<__half>{(const __half*)bias, nullptr, 1.f}, y, (int)M, (int)N, (int)K)
     if (st == RCU_OK) {
         if (wk == WK_F16) st = bn == 256 ? RCU_TC(256, WK_F16) : bn == 128 ? RCU_TC(128, WK_F16) : RCU_TC(64, WK_F16);
         else if (wk == WK_Q8) st = bn == 128 ? RCU_TC(128, WK_Q8) : RCU_TC(64, WK_Q8);
@@ -504,6 +494,33 @@ rcu_status rcu_gemm_tc_batched_f16(rcu_device* dev, const void* w, const void* x
         return rcu_fail(dev, RCU_ERR_CUDA, "gemm_tc: cuTensorMapEncodeTiled failed (batched M=%llu N=%llu K=%llu)", (unsigned long long)M,
                         (unsigned long long)N, (unsigned long long)K);
     QuantArgs qa{nullptr, nullptr, nullptr};
-    return bn == 128 ? launch_tc<128, WK_F16>(dev, xmap, wmap, qa, nullptr, y, (int)M, (int)N, (int)K, (int)batch)
-                     : launch_tc<64, WK_F16>(dev, xmap, wmap, qa, nullptr, y, (int)M, (int)N, (int)K, (int)batch);
+    return bn == 128 ? launch_tc<128, WK_F16>(dev, xmap, wmap, qa, GemmEpilogue<__half>{nullptr, nullptr, 1.f}, y, (int)M, (int)N, (int)K, (int)batch)
+                     : launch_tc<64, WK_F16>(dev, xmap, wmap, qa, GemmEpilogue<__half>{nullptr, nullptr, 1.f}, y, (int)M, (int)N, (int)K, (int)batch);
+}
+
+// A Linear with 16-bit operands and a chosen output (rcu_linear): out = x . W^T (+ bias) rounded to the operands' type, or
+// in f32 with resid + alpha * (...).  The activations may be a column window of wider rows (t.x_pitch).
+rcu_status rcu_gemm_tc_linear(rcu_device* dev, const void* w, const void* x, const void* bias, void* y, uint64_t M, uint64_t N, uint64_t K,
+                              const TcLinear& t) {
+    const uint64_t pitch = t.x_pitch ? t.x_pitch : K;
+    if (M < 2 || N < 64 || K < 64 || K % 8 != 0 || N % 8 != 0 || pitch % 8 != 0) return RCU_ERR_UNSUPPORTED;
+    if (M > 0x7fffffffull || N > 0x7fffffffull || K > 0x7fffffffull) return RCU_ERR_UNSUPPORTED;
+    if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(y) | reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(t.resid)) & 15)
+        return RCU_ERR_UNSUPPORTED;
+    DevGuard g(dev->ordinal);
+    if (rcu_gemm_tc2_eligible(dev, M, N, K)) return rcu_gemm_tc2_launch(dev, w, x, bias, y, M, N, K, t);
+    const uint64_t tiles128 = ((M + TM - 1) / TM) * ((N + 127) / 128);
+    const int bn = tiles128 >= (uint64_t)dev->sm_count ? 128 : 64;
+    CUtensorMap xmap, wmap;
+    if (!make_map_f16_sw128(&xmap, x, M, K, TM, 1, pitch, t.bf16) || !make_map_f16_sw128(&wmap, w, N, K, (uint32_t)bn, 1, 0, t.bf16))
+        return rcu_fail(dev, RCU_ERR_CUDA, "gemm_tc: cuTensorMapEncodeTiled failed (M=%llu N=%llu K=%llu)", (unsigned long long)M,
+                        (unsigned long long)N, (unsigned long long)K);
+    const QuantArgs qa{nullptr, nullptr, nullptr};
+#define RCU_TC(OUT_, EPI_)                                                                                                       \
+    (bn == 128 ? launch_tc<128, WK_F16, OUT_>(dev, xmap, wmap, qa, EPI_, y, (int)M, (int)N, (int)K, 1, t.bf16)                   \
+               : launch_tc<64, WK_F16, OUT_>(dev, xmap, wmap, qa, EPI_, y, (int)M, (int)N, (int)K, 1, t.bf16))
+    if (t.out_dt == RCU_F32) return RCU_TC(float, (GemmEpilogue<float>{(const float*)bias, t.resid, t.alpha}));
+    if (t.out_dt == RCU_BF16) return RCU_TC(__nv_bfloat16, (GemmEpilogue<__nv_bfloat16>{(const __nv_bfloat16*)bias, nullptr, 1.f}));
+    return RCU_TC(__half, (GemmEpilogue<__half>{(const __half*)bias, nullptr, 1.f}));
+#undef RCU_TC
 }

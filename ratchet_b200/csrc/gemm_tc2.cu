@@ -77,9 +77,10 @@ __device__ __forceinline__ void umma2_commit_both(uint64_t* bar) {
                  : "memory");
 }
 
+template <class Out>
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(kThreadsTc, 1)
-gemm_tc2_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant__ CUtensorMap wmap, const __half* __restrict__ bias,
-                __half* __restrict__ out, int M, int N, int K, int tiles_m, int n_tiles, int* status) {
+gemm_tc2_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant__ CUtensorMap wmap, const GemmEpilogue<Out> epi,
+                Out* out, int M, int N, int K, int tiles_m, int n_tiles, int* status, uint32_t idesc) {
     extern __shared__ unsigned char smem_dyn[];
     unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_dyn) + 1023) & ~(uintptr_t)1023);
     uint64_t* full = reinterpret_cast<uint64_t*>(smem + kStages2 * kStageBytes2);   // leader's are the ones in use
@@ -135,7 +136,6 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant_
         }
     } else if (warp == 1) {
         if (lane == 0 && rank == 0) {
-            constexpr uint32_t idesc = umma_idesc_f16(2 * TM, kTileN2);
             int it = 0, i = 0;
             bool ok = true;
             for (int t = pair; t < n_tiles && ok; t += n_pairs, ++i) {
@@ -179,18 +179,14 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant_
                 float v[32];
                 tmem_ld_32x32(tmem_base + ((uint32_t)(q * 32) << 16) + (uint32_t)(b * kAccCols + c), v);
                 if (row < M) {
-                    __half* orow = out + (size_t)row * N + n0 + c;
+                    const size_t base = (size_t)row * N + n0 + c;
 #pragma unroll
                     for (int j = 0; j < 32; j += 8) {
                         const int col = n0 + c + j;
                         if (col + 8 <= N) {
-                            __align__(16) __half h[8];
-#pragma unroll
-                            for (int e = 0; e < 8; ++e) h[e] = __float2half_rn(v[j + e] + (bias ? __half2float(bias[col + e]) : 0.f));
-                            *reinterpret_cast<uint4*>(orow + j) = *reinterpret_cast<const uint4*>(h);
+                            epi.store8(out, base + j, v + j, col);
                         } else {
-                            for (int e = 0; e < 8 && col + e < N; ++e)
-                                orow[j + e] = __float2half_rn(v[j + e] + (bias ? __half2float(bias[col + e]) : 0.f));
+                            for (int e = 0; e < 8 && col + e < N; ++e) out[base + j + e] = epi(v[j + e], col + e, base + j + e);
                         }
                     }
                 }
@@ -209,14 +205,14 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant_
     }
 }
 
-bool make_map_f16_sw128_rows(CUtensorMap* map, const void* base, uint64_t rows, uint64_t K, uint32_t box_rows) {
+bool make_map_f16_sw128_rows(CUtensorMap* map, const void* base, uint64_t rows, uint64_t K, uint32_t box_rows, uint64_t pitch, bool bf16) {
     gemvq8::EncodeTiledFn fn = gemvq8::encode_tiled_fn();
     if (!fn) return false;
     cuuint64_t dims[2] = {K, rows};
-    cuuint64_t strides[1] = {K * 2};
+    cuuint64_t strides[1] = {pitch * 2};
     cuuint32_t box[2] = {(cuuint32_t)TK, box_rows};
     cuuint32_t estr[2] = {1, 1};
-    return fn(map, CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+    return fn(map, bf16 ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16 : CU_TENSOR_MAP_DATA_TYPE_FLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
               CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
@@ -231,18 +227,31 @@ bool rcu_gemm_tc2_eligible(rcu_device* dev, uint64_t M, uint64_t N, uint64_t K) 
     return tiles >= (uint64_t)dev->sm_count / 4;
 }
 
-rcu_status rcu_gemm_tc2_launch(rcu_device* dev, const void* w, const void* x, const void* bias, void* y, uint64_t M, uint64_t N, uint64_t K) {
-    CUtensorMap xmap, wmap;
-    if (!make_map_f16_sw128_rows(&xmap, x, M, K, TM) || !make_map_f16_sw128_rows(&wmap, w, N, K, kTileN2 / 2))
-        return rcu_fail(dev, RCU_ERR_CUDA, "gemm_tc2: cuTensorMapEncodeTiled failed (M=%llu N=%llu K=%llu)", (unsigned long long)M,
-                        (unsigned long long)N, (unsigned long long)K);
+namespace {
+template <class Out>
+rcu_status launch_pair(rcu_device* dev, const CUtensorMap& xmap, const CUtensorMap& wmap, const GemmEpilogue<Out>& epi, void* y, uint64_t M, uint64_t N,
+                       uint64_t K, bool bf16) {
     const int tiles_m = (int)((M + 255) / 256), tiles_n = (int)((N + 255) / 256);
     const int n_tiles = tiles_m * tiles_n;
     const int n_pairs = std::min(n_tiles, dev->sm_count / 2);
     const size_t smem = (size_t)kStages2 * kStageBytes2 + 1024 + 256;
-    RCU_CUDA(dev, cudaFuncSetAttribute(gemm_tc2_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    gemm_tc2_kernel<<<2 * n_pairs, kThreadsTc, smem, dev->stream>>>(xmap, wmap, (const __half*)bias, (__half*)y, (int)M, (int)N, (int)K, tiles_m,
-                                                                  n_tiles, dev->d_status);
+    RCU_CUDA(dev, cudaFuncSetAttribute(gemm_tc2_kernel<Out>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    gemm_tc2_kernel<Out><<<2 * n_pairs, kThreadsTc, smem, dev->stream>>>(xmap, wmap, epi, (Out*)y, (int)M, (int)N, (int)K, tiles_m, n_tiles,
+                                                                       dev->d_status, umma_idesc_f16(2 * TM, kTileN2, bf16));
     RCU_LAUNCH_CHECK(dev);
     return RCU_OK;
+}
+}  // namespace
+
+rcu_status rcu_gemm_tc2_launch(rcu_device* dev, const void* w, const void* x, const void* bias, void* y, uint64_t M, uint64_t N, uint64_t K,
+                               const TcLinear& t) {
+    CUtensorMap xmap, wmap;
+    if (!make_map_f16_sw128_rows(&xmap, x, M, K, TM, t.x_pitch ? t.x_pitch : K, t.bf16) ||
+        !make_map_f16_sw128_rows(&wmap, w, N, K, kTileN2 / 2, K, t.bf16))
+        return rcu_fail(dev, RCU_ERR_CUDA, "gemm_tc2: cuTensorMapEncodeTiled failed (M=%llu N=%llu K=%llu)", (unsigned long long)M,
+                        (unsigned long long)N, (unsigned long long)K);
+    if (t.out_dt == RCU_F32) return launch_pair<float>(dev, xmap, wmap, GemmEpilogue<float>{(const float*)bias, t.resid, t.alpha}, y, M, N, K, t.bf16);
+    if (t.out_dt == RCU_BF16)
+        return launch_pair<__nv_bfloat16>(dev, xmap, wmap, GemmEpilogue<__nv_bfloat16>{(const __nv_bfloat16*)bias, nullptr, 1.f}, y, M, N, K, t.bf16);
+    return launch_pair<__half>(dev, xmap, wmap, GemmEpilogue<__half>{(const __half*)bias, nullptr, 1.f}, y, M, N, K, t.bf16);
 }

@@ -31,7 +31,8 @@ namespace {
 
 enum LazyKind {
     K_CONST = 0, K_VIEW, K_BINARY, K_UNARY, K_CAST, K_MATMUL, K_NORM, K_SOFTMAX, K_ROPE, K_CONCAT, K_SELECT,
-    K_PERMUTE, K_SLICE, K_BROADCAST, K_CACHE, K_INDEX_WRITE, K_CONV
+    K_PERMUTE, K_SLICE, K_BROADCAST, K_CACHE, K_INDEX_WRITE, K_CONV,
+    K_LINEAR, K_NORM_ROWS, K_GLU, K_ROTARY, K_LIGHTNING, K_LATENT_APPEND, K_WINDOW_ATTENTION
 };
 
 struct Storage {
@@ -118,9 +119,11 @@ rcu_lazy* new_node(rcu_device* dev, int kind, int32_t dt, uint32_t rank, const u
     return n;
 }
 
-bool supports_inplace(int kind) {
+bool supports_inplace(const rcu_lazy* n) {
+    const int kind = n->kind;
+    if (kind == K_LINEAR) return n->flags[0] != 0;      // srcs[0] is the residual
     // ops/binary.rs:179, ops/unary.rs:268, ops/softmax.rs:196, ops/rope.rs:80, ops/index_write.rs:49
-    return kind == K_BINARY || kind == K_UNARY || kind == K_SOFTMAX || kind == K_ROPE || kind == K_INDEX_WRITE;
+    return kind == K_ROTARY || kind == K_BINARY || kind == K_UNARY || kind == K_SOFTMAX || kind == K_ROPE || kind == K_INDEX_WRITE;
 }
 
 // The op about to overwrite `s`'s buffer must be the only thing that can still read it: `s` has one
@@ -216,6 +219,13 @@ const char* kind_name(int kind) {
         case K_CACHE: return "cache";
         case K_INDEX_WRITE: return "index_write";
         case K_CONV: return "conv";
+        case K_LINEAR: return "linear";
+        case K_NORM_ROWS: return "norm_rows";
+        case K_GLU: return "glu";
+        case K_ROTARY: return "rotary";
+        case K_LIGHTNING: return "lightning";
+        case K_LATENT_APPEND: return "latent_append";
+        case K_WINDOW_ATTENTION: return "window_attention";
         default: return "other";
     }
 }
@@ -277,6 +287,30 @@ rcu_status run_node(rcu_lazy* n) {
             if (n->srcs.size() > 2) bias = S(2);
             return rcu_conv1d(dev, &x, &w, n->srcs.size() > 2 ? &bias : nullptr, n->u[0], n->u[1], &dst);
         }
+        case K_LINEAR: {        // [residual], w, x, [bias]
+            size_t i = 0;
+            rcu_tensor resid, bias;
+            if (n->flags[0]) resid = S(i++);
+            rcu_tensor w = S(i++), x = S(i++);
+            if (n->flags[1]) bias = S(i++);
+            return rcu_linear(dev, &w, &x, n->u[0], n->flags[1] ? &bias : nullptr, n->flags[0] ? &resid : nullptr, n->f[0], &dst);
+        }
+        case K_NORM_ROWS: {
+            rcu_tensor x = S(0), sc = S(1), gate;
+            if (n->srcs.size() > 2) gate = S(2);
+            return rcu_norm_rows(dev, n->op, &x, n->u[0], &sc, n->srcs.size() > 2 ? &gate : nullptr, n->u[1], n->f[0], &dst);
+        }
+        case K_GLU: { rcu_tensor x = S(0); return rcu_glu(dev, n->op, &x, &dst); }
+        case K_ROTARY: { rcu_tensor x = S(0), fr = S(1); return rcu_rotary(dev, &x, n->u[0], &fr, n->f[0], n->u[1], &dst); }
+        case K_LIGHTNING: { rcu_tensor x = S(0), dp = S(1), st = S(2); return rcu_lightning(dev, &x, &dp, &st, n->flags[0], &dst); }
+        case K_LATENT_APPEND: {
+            rcu_tensor x = S(0), sc = S(1), fr = S(2), ring = S(3);
+            return rcu_latent_append(dev, &x, n->u[0], &sc, n->f[0], &fr, n->f[1], n->u[1], &ring, &dst);
+        }
+        case K_WINDOW_ATTENTION: {
+            rcu_tensor q = S(0), kv = S(1), sh = S(2);
+            return rcu_window_attention(dev, &q, &kv, &sh, n->u[0], n->u[1], n->u[2], n->f[0], &dst);
+        }
         default: return rcu_fail(dev, RCU_ERR_UNSUPPORTED, "resolve: node kind %d has no kernel", n->kind);
     }
 }
@@ -323,7 +357,7 @@ rcu_status resolve(rcu_lazy* out) {
         rcu_lazy* s0 = t->srcs[0];
         if (t->kind == K_VIEW) {
             owner[i] = owner[index[s0->id]];
-        } else if (!no_reuse && supports_inplace(t->kind) && sole_owner(s0) && s0->dt == t->dt && s0->numel() == t->numel() &&
+        } else if (!no_reuse && supports_inplace(t) && sole_owner(s0) && s0->dt == t->dt && s0->numel() == t->numel() &&
                    !(s0->resolved() && !s0->storage->owned)) {
             // the op is the sole owner of its first source (tensor.rs:823-824); a borrowed buffer
             // (rcu_lazy_wrap) is never written in place
@@ -717,6 +751,106 @@ rcu_status rcu_lazy_index_write(rcu_lazy* dst, rcu_lazy* src, const uint64_t* st
         LAZY_REQUIRE(dst->dev, start[i] + src->shape[i] <= dst->shape[i], "index_write: block exceeds dst on axis %u", i);
     rcu_lazy* n = new_node(dst->dev, K_INDEX_WRITE, dst->dt, dst->rank, dst->shape, {dst, src});
     for (uint32_t i = 0; i < dst->rank; ++i) n->a[i] = start[i];
+    *out = n;
+    return RCU_OK;
+}
+
+rcu_status rcu_lazy_linear(rcu_lazy* w, rcu_lazy* x, uint32_t x_col, rcu_lazy* bias, rcu_lazy* resid, float alpha, int32_t dst_dt, rcu_lazy** out) {
+    if (!w || !x || !out) return RCU_ERR_INVALID_ARG;
+    LAZY_REQUIRE(w->dev, x->dev == w->dev && (!bias || bias->dev == w->dev) && (!resid || resid->dev == w->dev), "Mixed devices");
+    LAZY_REQUIRE(w->dev, w->rank == 2 && w->dt == x->dt && dt_is_float(w->dt), "linear: w must be a float matrix of the activations' dtype");
+    LAZY_REQUIRE(w->dev, dst_dt == x->dt || dst_dt == RCU_F32, "linear: the output is f32 or has the activations' dtype");
+    LAZY_REQUIRE(w->dev, x_col + w->shape[1] <= x->shape[x->rank - 1], "linear: the columns lie outside the rows");
+    uint64_t shape[RCU_MAX_RANK];
+    for (uint32_t i = 0; i < x->rank; ++i) shape[i] = x->shape[i];
+    shape[x->rank - 1] = w->shape[0];
+    rcu_lazy* n = new_node(w->dev, K_LINEAR, dst_dt, x->rank, shape, {resid, w, x, bias});
+    const bool ok = !resid || (resid->numel() == n->numel() && resid->dt == RCU_F32 && dst_dt == RCU_F32);
+    if (!ok) { release(n); return rcu_fail(w->dev, RCU_ERR_INVALID_ARG, "linear: the residual must be f32 of the output's size"); }
+    n->flags[0] = resid != nullptr;
+    n->flags[1] = bias != nullptr;
+    n->u[0] = x_col;
+    n->f[0] = alpha;
+    *out = n;
+    return RCU_OK;
+}
+
+rcu_status rcu_lazy_norm_rows(int kind, rcu_lazy* x, uint32_t x_col, rcu_lazy* scale, rcu_lazy* gate, uint32_t gate_col, float eps, int32_t dst_dt,
+                              rcu_lazy** out) {
+    if (!x || !scale || !out) return RCU_ERR_INVALID_ARG;
+    LAZY_REQUIRE(x->dev, kind == RCU_LAYER_NORM || kind == RCU_RMS_NORM, "norm_rows: LayerNorm or RMSNorm");
+    LAZY_REQUIRE(x->dev, x->dt == RCU_F32 && dt_is_float(dst_dt), "norm_rows: f32 input, float output");
+    LAZY_REQUIRE(x->dev, x_col + scale->numel() <= x->shape[x->rank - 1], "norm_rows: the columns lie outside the rows");
+    uint64_t shape[RCU_MAX_RANK];
+    for (uint32_t i = 0; i < x->rank; ++i) shape[i] = x->shape[i];
+    shape[x->rank - 1] = scale->numel();
+    rcu_lazy* n = new_node(x->dev, K_NORM_ROWS, dst_dt, x->rank, shape, {x, scale, gate});
+    n->op = kind;
+    n->u[0] = x_col;
+    n->u[1] = gate_col;
+    n->f[0] = eps;
+    *out = n;
+    return RCU_OK;
+}
+
+rcu_status rcu_lazy_glu(int act, rcu_lazy* x, rcu_lazy** out) {
+    if (!x || !out) return RCU_ERR_INVALID_ARG;
+    LAZY_REQUIRE(x->dev, act == RCU_GELU || act == RCU_SILU, "glu: the activation is gelu or silu");
+    LAZY_REQUIRE(x->dev, x->shape[x->rank - 1] % 2 == 0, "glu: rows hold gate and up halves");
+    uint64_t shape[RCU_MAX_RANK];
+    for (uint32_t i = 0; i < x->rank; ++i) shape[i] = x->shape[i];
+    shape[x->rank - 1] /= 2;
+    rcu_lazy* n = new_node(x->dev, K_GLU, x->dt, x->rank, shape, {x});
+    n->op = act;
+    *out = n;
+    return RCU_OK;
+}
+
+rcu_status rcu_lazy_rotary(rcu_lazy* x, uint32_t first, rcu_lazy* freqs, float magnitude, uint32_t position, rcu_lazy** out) {
+    if (!x || !freqs || !out) return RCU_ERR_INVALID_ARG;
+    LAZY_REQUIRE(x->dev, x->rank == 3 && freqs->rank == 2 && first + 2 * freqs->shape[1] <= x->shape[2], "rotary: the rotated features lie outside the head");
+    rcu_lazy* n = new_node(x->dev, K_ROTARY, x->dt, x->rank, x->shape, {x, freqs});
+    n->u[0] = first;
+    n->u[1] = position;
+    n->f[0] = magnitude;
+    *out = n;
+    return RCU_OK;
+}
+
+rcu_status rcu_lazy_lightning(rcu_lazy* x, rcu_lazy* decay_pow, rcu_lazy* state, int silu, rcu_lazy** out) {
+    if (!x || !decay_pow || !state || !out) return RCU_ERR_INVALID_ARG;
+    LAZY_REQUIRE(x->dev, state->rank == 3, "lightning: the state is [heads, dim, vdim]");
+    const uint64_t shape[2] = {x->numel() / x->shape[x->rank - 1], state->shape[0] * state->shape[2]};
+    rcu_lazy* n = new_node(x->dev, K_LIGHTNING, RCU_F32, 2, shape, {x, decay_pow, state});
+    n->flags[0] = silu;
+    *out = n;
+    return RCU_OK;
+}
+
+rcu_status rcu_lazy_latent_append(rcu_lazy* x, uint32_t x_col, rcu_lazy* scale, float eps, rcu_lazy* freqs, float magnitude, uint32_t position,
+                                  rcu_lazy* ring, uint32_t rows, rcu_lazy** out) {
+    if (!x || !scale || !freqs || !ring || !out) return RCU_ERR_INVALID_ARG;
+    LAZY_REQUIRE(x->dev, ring->rank == 2, "latent_append: the ring is [rows, width]");
+    const uint64_t shape[2] = {rows, ring->shape[1]};
+    rcu_lazy* n = new_node(x->dev, K_LATENT_APPEND, ring->dt, 2, shape, {x, scale, freqs, ring});
+    n->u[0] = x_col;
+    n->u[1] = position;
+    n->f[0] = eps;
+    n->f[1] = magnitude;
+    *out = n;
+    return RCU_OK;
+}
+
+rcu_status rcu_lazy_window_attention(rcu_lazy* q, rcu_lazy* kv, rcu_lazy* shared, uint32_t shared_col, uint32_t vdim, uint32_t window, float scale,
+                                     rcu_lazy** out) {
+    if (!q || !kv || !shared || !out) return RCU_ERR_INVALID_ARG;
+    LAZY_REQUIRE(q->dev, q->rank == 3 && kv->rank == 2 && shared->rank == 2, "window_attention: q [tokens, heads, dim], kv and shared rows");
+    const uint64_t shape[2] = {q->shape[0], q->shape[1] * vdim};
+    rcu_lazy* n = new_node(q->dev, K_WINDOW_ATTENTION, q->dt, 2, shape, {q, kv, shared});
+    n->u[0] = shared_col;
+    n->u[1] = vdim;
+    n->u[2] = window;
+    n->f[0] = scale;
     *out = n;
     return RCU_OK;
 }

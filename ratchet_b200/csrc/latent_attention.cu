@@ -1,0 +1,199 @@
+// Latent attention over a block of tokens with a sliding window: what a layer caches per token is one normalised latent
+// and one rotated key part shared by all heads, and a head's keys and values are linear images of the latent.
+//
+//   rcu_latent_append   normalises and rotates the block's latents, keeps the last `ring` of them in the layer's ring
+//                       (row of position p: p mod ring) and lays out the rows the block can see;
+//   rcu_window_attention  softmax attention of the block's queries over those rows, keys and values expanded from the
+//                       latents by one Linear before the call.
+#include "lm_math.cuh"
+
+namespace {
+
+struct AppendArgs {
+    const float* x;            // [T, pitch], latent at column 0 of the pointer, key part behind it
+    long long pitch;
+    const float* scale;
+    const float* freqs;
+    float magnitude, eps;
+    int C, R, pairs, T, L, ring;
+    uint32_t pos;              // position of the block's first token
+};
+
+// rows [0, L - T) of the window come from the ring, the others from the block; one warp per row
+template <class O>
+__global__ void __launch_bounds__(128) latent_window_kernel(const AppendArgs a, const O* __restrict__ ring, O* __restrict__ out) {
+    rcu_kernel_entry();
+    const int lane = threadIdx.x & 31;
+    const int r = blockIdx.x * 4 + (threadIdx.x >> 5);
+    if (r >= a.L) return;
+    const int W = a.C + a.R, old = a.L - a.T;
+    O* orow = out + (size_t)r * W;
+    if (r < old) {
+        const O* src = ring + (size_t)((a.pos - (uint32_t)(old - r)) % (uint32_t)a.ring) * W;
+        for (int j = lane; j < W; j += 32) orow[j] = src[j];
+        return;
+    }
+    const float* x = a.x + (long long)(r - old) * a.pitch;
+    float s = 0.f;
+    for (int j = lane; j < a.C; j += 32) s = fmaf(x[j], x[j], s);
+    const float rstd = 1.0f / sqrtf(warp_sum(s) / (float)a.C + a.eps);
+    for (int j = lane; j < a.C; j += 32) orow[j] = from_f32<O>(x[j] * rstd * a.scale[j]);
+    const float* kr = x + a.C;
+    const uint32_t p = a.pos + (uint32_t)(r - old);
+    for (int i = lane; i < a.pairs; i += 32) {
+        const float2 cs = lm::rotary_angle(a.freqs, a.pairs, i, p, a.magnitude);
+        const float u = kr[2 * i], v = kr[2 * i + 1];
+        orow[a.C + 2 * i] = from_f32<O>(u * cs.x - v * cs.y);
+        orow[a.C + 2 * i + 1] = from_f32<O>(v * cs.x + u * cs.y);
+    }
+    for (int j = 2 * a.pairs + lane; j < a.R; j += 32) orow[a.C + j] = from_f32<O>(kr[j]);
+}
+
+// the block's last min(T, ring) rows into the ring
+template <class O>
+__global__ void __launch_bounds__(128) latent_store_kernel(const O* __restrict__ rows, O* __restrict__ ring, int W, int n, int L, int ring_rows, uint32_t end) {
+    rcu_kernel_entry();
+    const int lane = threadIdx.x & 31;
+    const int i = blockIdx.x * 4 + (threadIdx.x >> 5);
+    if (i >= n) return;
+    const O* src = rows + (size_t)(L - n + i) * W;
+    O* dst = ring + (size_t)((end - (uint32_t)(n - i)) % (uint32_t)ring_rows) * W;
+    for (int j = lane; j < W; j += 32) dst[j] = src[j];
+}
+
+template <class O>
+rcu_status launch_append(rcu_device* dev, const AppendArgs& a, void* ring, void* out) {
+    rcu_launch(dev, latent_window_kernel<O>, (unsigned)((a.L + 3) / 4), 128, 0, a, (const O*)ring, (O*)out);
+    dev->launches++;
+    const int n = a.T < a.ring ? a.T : a.ring;
+    rcu_launch(dev, latent_store_kernel<O>, (unsigned)((n + 3) / 4), 128, 0, (const O*)out, (O*)ring, a.C + a.R, n, a.L, a.ring, a.pos + (uint32_t)a.T);
+    RCU_LAUNCH_CHECK(dev);
+    return RCU_OK;
+}
+
+struct WindowArgs {
+    const void *q, *kv, *shared;
+    void* out;
+    long long shared_pitch;
+    int T, L, H, D, R, E, window;     // D: own key features of a head, R: shared ones (a query has D + R)
+    float scale;
+};
+
+// A warp per (token, head): scores 32 keys at a time, one key per lane, online softmax in f32; the weighted sum of the
+// values runs over lanes = value columns.
+template <class T, int PE>
+__global__ void __launch_bounds__(256) window_attention_kernel(const WindowArgs a) {
+    rcu_kernel_entry();
+    extern __shared__ float q_s[];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int h = blockIdx.y;
+    const int i = blockIdx.x * 8 + warp;
+    if (i >= a.T) return;
+    const int Q = a.D + a.R;
+    float* q = q_s + warp * Q;
+    const T* qg = reinterpret_cast<const T*>(a.q) + ((size_t)i * a.H + h) * Q;
+    for (int d = lane; d < Q; d += 32) q[d] = to_f32<T>(qg[d]);
+    __syncwarp();
+    const size_t kv_pitch = (size_t)a.H * (a.D + a.E);
+    const T* K = reinterpret_cast<const T*>(a.kv) + (size_t)h * a.D;
+    const T* V = reinterpret_cast<const T*>(a.kv) + (size_t)a.H * a.D + (size_t)h * a.E;
+    const T* KS = reinterpret_cast<const T*>(a.shared);
+    const int last = a.L - a.T + i, first = max(0, last - a.window + 1);
+    float m = -INFINITY, l = 0.f, o[PE];
+#pragma unroll
+    for (int j = 0; j < PE; ++j) o[j] = 0.f;
+    for (int j0 = first; j0 <= last; j0 += 32) {
+        const int j = j0 + lane;
+        float s = -INFINITY;
+        if (j <= last) {
+            const T* k = K + j * kv_pitch;
+            const T* ks = KS + j * a.shared_pitch;
+            float acc = 0.f;
+            for (int d = 0; d < a.D; ++d) acc = fmaf(q[d], to_f32<T>(k[d]), acc);
+            for (int d = 0; d < a.R; ++d) acc = fmaf(q[a.D + d], to_f32<T>(ks[d]), acc);
+            s = acc * a.scale;
+        }
+        const float mn = fmaxf(m, warp_max(s));
+        const float corr = expf(m - mn);
+        const float p = expf(s - mn);          // 0 for lanes beyond the last key
+        l = l * corr + warp_sum(p);
+        m = mn;
+#pragma unroll
+        for (int c = 0; c < PE; ++c) o[c] *= corr;
+        const int n = min(32, last - j0 + 1);
+        for (int t = 0; t < n; ++t) {
+            const float pt = __shfl_sync(0xffffffffu, p, t);
+            const T* v = V + (size_t)(j0 + t) * kv_pitch;
+#pragma unroll
+            for (int c = 0; c < PE; ++c) {
+                const int e = lane + 32 * c;
+                if (e < a.E) o[c] = fmaf(pt, to_f32<T>(v[e]), o[c]);
+            }
+        }
+    }
+    T* og = reinterpret_cast<T*>(a.out) + ((size_t)i * a.H + h) * a.E;
+#pragma unroll
+    for (int c = 0; c < PE; ++c) {
+        const int e = lane + 32 * c;
+        if (e < a.E) og[e] = from_f32<T>(o[c] / l);
+    }
+}
+
+template <class T> rcu_status launch_window(rcu_device* dev, const WindowArgs& a) {
+    const dim3 grid((a.T + 7) / 8, a.H);
+    const size_t smem = (size_t)8 * (a.D + a.R) * 4;
+#define RCU_WA(PE_)                                                                                                                              \
+    do {                                                                                                                                         \
+        if (smem > 40 * 1024) RCU_CUDA(dev, cudaFuncSetAttribute(window_attention_kernel<T, PE_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
+        rcu_launch(dev, window_attention_kernel<T, PE_>, grid, 256, smem, a);                                                                    \
+    } while (0)
+    if (a.E <= 64) RCU_WA(2);
+    else if (a.E <= 128) RCU_WA(4);
+    else if (a.E <= 256) RCU_WA(8);
+    else RCU_WA(16);
+#undef RCU_WA
+    RCU_LAUNCH_CHECK(dev);
+    return RCU_OK;
+}
+
+}  // namespace
+
+extern "C" {
+
+rcu_status rcu_latent_append(rcu_device* dev, const rcu_tensor* x, uint32_t x_col, const rcu_tensor* scale, float eps, const rcu_tensor* freqs,
+                             float magnitude, uint32_t position, rcu_tensor* ring, rcu_tensor* dst) {
+    if (!dev) return RCU_ERR_INVALID_ARG;
+    RCU_REQUIRE(dev, t_valid(x) && t_valid(scale) && t_valid(freqs) && t_valid(ring) && t_valid(dst), "latent_append: invalid tensor descriptor");
+    RCU_REQUIRE(dev, x->dt == RCU_F32 && scale->dt == RCU_F32 && freqs->dt == RCU_F32, "latent_append: f32 rows, scale and frequencies");
+    RCU_REQUIRE(dev, ring->rank == 2 && dst->rank == 2 && ring->dt == dst->dt && (ring->dt == RCU_F32 || ring->dt == RCU_BF16) &&
+                         ring->shape[1] == dst->shape[1], "latent_append: ring and dst are f32 or bf16 rows of one width");
+    RCU_REQUIRE(dev, freqs->rank == 2 && freqs->shape[0] == 2, "latent_append: the frequency table is f32 [2, pairs]");
+    const uint64_t W = ring->shape[1], C = t_numel(scale), pitch = x->shape[x->rank - 1], T = t_numel(x) / pitch, L = dst->shape[0];
+    RCU_REQUIRE(dev, C < W && x_col + W <= pitch && 2 * freqs->shape[1] <= W - C, "latent_append: columns do not fit the rows");
+    RCU_REQUIRE(dev, L >= T && L - T <= position && L - T <= ring->shape[0] && L <= 0x7fffffffull, "latent_append: the window reaches before the ring");
+    DevGuard g(dev->ordinal);
+    AppendArgs a{(const float*)x->data + x_col, (long long)pitch, (const float*)scale->data, (const float*)freqs->data, magnitude, eps, (int)C, (int)(W - C),
+                 (int)freqs->shape[1], (int)T, (int)L, (int)ring->shape[0], position};
+    return ring->dt == RCU_F32 ? launch_append<float>(dev, a, ring->data, dst->data) : launch_append<__nv_bfloat16>(dev, a, ring->data, dst->data);
+}
+
+rcu_status rcu_window_attention(rcu_device* dev, const rcu_tensor* q, const rcu_tensor* kv, const rcu_tensor* shared, uint32_t shared_col, uint32_t vdim,
+                                uint32_t window, float scale, rcu_tensor* dst) {
+    if (!dev) return RCU_ERR_INVALID_ARG;
+    RCU_REQUIRE(dev, t_valid(q) && t_valid(kv) && t_valid(shared) && t_valid(dst), "window_attention: invalid tensor descriptor");
+    RCU_REQUIRE(dev, q->rank == 3 && kv->rank == 2 && shared->rank == 2 && q->dt == kv->dt && q->dt == shared->dt && q->dt == dst->dt &&
+                         (q->dt == RCU_F32 || q->dt == RCU_BF16), "window_attention: q [tokens, heads, dim], kv and shared rows, f32 or bf16");
+    const uint64_t T = q->shape[0], H = q->shape[1], L = kv->shape[0];
+    RCU_REQUIRE(dev, vdim > 0 && window > 0 && shared_col <= shared->shape[1] && shared->shape[0] == L && L >= T, "window_attention: bad sizes");
+    const uint64_t R = shared->shape[1] - shared_col;
+    RCU_REQUIRE(dev, q->shape[2] >= R && kv->shape[1] == H * (q->shape[2] - R + vdim), "window_attention: kv rows hold every head's keys, then its values");
+    RCU_REQUIRE(dev, t_numel(dst) == T * H * vdim, "window_attention: dst holds %llu elements, expected %llu", (unsigned long long)t_numel(dst),
+                (unsigned long long)(T * H * vdim));
+    if (vdim > 512 || H > 65535 || L > 0x7fffffffull || q->shape[2] > 4096) return rcu_fail(dev, RCU_ERR_UNSUPPORTED, "window_attention: vdim %u (at most 512)", vdim);
+    DevGuard g(dev->ordinal);
+    WindowArgs a{q->data, kv->data, (const char*)shared->data + (size_t)shared_col * dt_esize(shared->dt), dst->data, (long long)shared->shape[1], (int)T,
+                 (int)L, (int)H, (int)(q->shape[2] - R), (int)R, (int)vdim, (int)(window < L ? window : L), scale};
+    return q->dt == RCU_F32 ? launch_window<float>(dev, a) : launch_window<__nv_bfloat16>(dev, a);
+}
+
+}  // extern "C"

@@ -1,0 +1,249 @@
+// Row operations between the projections of a model that keeps its residual stream, norms and gates in 32 bits while
+// its matrix products take 16-bit operands: norms of f32 rows (or of a column window of them) into any float type with an
+// optional sigmoid gate, the gated activation of a feed-forward, and rotary positions on interleaved pairs with an
+// explicit frequency table.
+#include <cmath>
+
+#include "lm_math.cuh"
+
+namespace {
+
+struct NormArgs {
+    const float* x;
+    long long x_pitch;
+    const float* scale;
+    const void* gate;          // nullable: output *= sigmoid(gate[row * gate_pitch + j])
+    long long gate_pitch;
+    int N;
+    float eps;
+    int layer;                 // 1: LayerNorm (no bias), 0: RMSNorm
+};
+
+template <class G> __device__ __forceinline__ float gate_of(const NormArgs& a, size_t row, int j) {
+    return lm::sigmoid(to_f32<G>(reinterpret_cast<const G*>(a.gate)[row * a.gate_pitch + j]));
+}
+
+// A warp per row, the row in registers (N <= 32 * PER).  The variance is the mean of the squared deviations, taken in
+// a second pass over the registers.
+template <class Out, int PER>
+__global__ void __launch_bounds__(256) norm_rows_warp_kernel(const NormArgs a, Out* __restrict__ out, long long rows) {
+    rcu_kernel_entry();
+    const int lane = threadIdx.x & 31;
+    const long long row = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+    if (row >= rows) return;
+    const float* xr = a.x + row * a.x_pitch;
+    float v[PER];
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+        const int j = lane + 32 * i;
+        v[i] = j < a.N ? xr[j] : 0.f;
+        s += v[i];
+    }
+    const float mean = a.layer ? warp_sum(s) / (float)a.N : 0.f;
+    float q = 0.f;
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+        const int j = lane + 32 * i;
+        v[i] -= mean;
+        if (j < a.N) q = fmaf(v[i], v[i], q);
+    }
+    const float rstd = 1.0f / sqrtf(warp_sum(q) / (float)a.N + a.eps);
+#pragma unroll
+    for (int i = 0; i < PER; ++i) {
+        const int j = lane + 32 * i;
+        if (j < a.N) {
+            float y = v[i] * rstd * a.scale[j];
+            if (a.gate) y *= gate_of<Out>(a, (size_t)row, j);
+            out[(size_t)row * a.N + j] = from_f32<Out>(y);
+        }
+    }
+}
+
+// A CTA per row, the row in shared memory.
+template <class Out>
+__global__ void __launch_bounds__(256) norm_rows_kernel(const NormArgs a, Out* __restrict__ out) {
+    rcu_kernel_entry();
+    extern __shared__ float row_s[];
+    __shared__ float scratch[32];
+    const size_t row = blockIdx.x;
+    const float* xr = a.x + row * a.x_pitch;
+    float s = 0.f;
+    for (int j = threadIdx.x; j < a.N; j += 256) {
+        const float v = xr[j];
+        row_s[j] = v;
+        s += v;
+    }
+    const float mean = a.layer ? lm::block_sum(s, scratch) / (float)a.N : 0.f;
+    float q = 0.f;
+    for (int j = threadIdx.x; j < a.N; j += 256) {
+        const float d = row_s[j] - mean;
+        q = fmaf(d, d, q);
+    }
+    const float rstd = 1.0f / sqrtf(lm::block_sum(q, scratch) / (float)a.N + a.eps);
+    for (int j = threadIdx.x; j < a.N; j += 256) {
+        float y = (row_s[j] - mean) * rstd * a.scale[j];
+        if (a.gate) y *= gate_of<Out>(a, row, j);
+        out[row * a.N + j] = from_f32<Out>(y);
+    }
+}
+
+template <class Out>
+rcu_status launch_norm_rows(rcu_device* dev, const NormArgs& a, void* out, uint64_t rows) {
+    const unsigned warp_grid = (unsigned)((rows + 7) / 8);
+    if (a.N <= 128) rcu_launch(dev, norm_rows_warp_kernel<Out, 4>, warp_grid, 256, 0, a, (Out*)out, (long long)rows);
+    else if (a.N <= 512) rcu_launch(dev, norm_rows_warp_kernel<Out, 16>, warp_grid, 256, 0, a, (Out*)out, (long long)rows);
+    else {
+        const size_t smem = (size_t)a.N * 4;
+        if (smem + 1024 > (size_t)dev->smem_optin) return rcu_fail(dev, RCU_ERR_UNSUPPORTED, "norm_rows: rows of %d do not fit shared memory", a.N);
+        if (smem > 40 * 1024) RCU_CUDA(dev, cudaFuncSetAttribute(norm_rows_kernel<Out>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        rcu_launch(dev, norm_rows_kernel<Out>, (unsigned)rows, 256, smem, a, (Out*)out);
+    }
+    RCU_LAUNCH_CHECK(dev);
+    return RCU_OK;
+}
+
+template <class T, int V>
+__global__ void __launch_bounds__(256) glu_kernel(const T* __restrict__ x, T* __restrict__ out, size_t n, int F, int act) {
+    rcu_kernel_entry();
+    struct alignas(sizeof(T) * V) Vec { T v[V]; };
+    const int fv = F / V;
+    for (size_t i = (size_t)blockIdx.x * 256 + threadIdx.x; i < n; i += (size_t)gridDim.x * 256) {
+        const size_t row = i / fv, j = (i % fv) * V;
+        const Vec g = *reinterpret_cast<const Vec*>(x + row * 2 * F + j), u = *reinterpret_cast<const Vec*>(x + row * 2 * F + F + j);
+        Vec o;
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+            const float z = to_f32<T>(g.v[e]);
+            o.v[e] = from_f32<T>((act == RCU_GELU ? lm::gelu_tanh(z) : lm::silu(z)) * to_f32<T>(u.v[e]));
+        }
+        *reinterpret_cast<Vec*>(out + row * F + j) = o;
+    }
+}
+
+template <class T> rcu_status launch_glu(rcu_device* dev, const void* x, void* out, uint64_t rows, uint64_t F, int act) {
+    constexpr int V = 16 / (int)sizeof(T);
+    const bool vec = F % V == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+    const size_t n = vec ? rows * F / V : rows * F;
+    const unsigned grid = (unsigned)grid_for(n, 256, dev->sm_count * 16);
+    if (vec) rcu_launch(dev, glu_kernel<T, V>, grid, 256, 0, (const T*)x, (T*)out, n, (int)F, act);
+    else rcu_launch(dev, glu_kernel<T, 1>, grid, 256, 0, (const T*)x, (T*)out, n, (int)F, act);
+    RCU_LAUNCH_CHECK(dev);
+    return RCU_OK;
+}
+
+// One CTA per token: the angles of its pairs once in shared memory, then every head.
+template <class T>
+__global__ void __launch_bounds__(128) rotary_kernel(const T* x, const float* __restrict__ freqs, T* out, int H, int D, int first, int pairs,
+                                                     float magnitude, uint32_t position) {
+    rcu_kernel_entry();
+    extern __shared__ float2 cs[];
+    const size_t t = blockIdx.x;
+    for (int i = threadIdx.x; i < pairs; i += blockDim.x) cs[i] = lm::rotary_angle(freqs, pairs, i, position + (uint32_t)t, magnitude);
+    __syncthreads();
+    const T* xr = x + t * (size_t)H * D;
+    T* orow = out + t * (size_t)H * D;
+    for (int j = threadIdx.x; j < H * pairs; j += blockDim.x) {
+        const int h = j / pairs, i = j % pairs;
+        const size_t o = (size_t)h * D + first + 2 * i;
+        const float u = to_f32<T>(xr[o]), v = to_f32<T>(xr[o + 1]);
+        orow[o] = from_f32<T>(u * cs[i].x - v * cs[i].y);
+        orow[o + 1] = from_f32<T>(v * cs[i].x + u * cs[i].y);
+    }
+    if (x != out)
+        for (int j = threadIdx.x; j < H * D; j += blockDim.x) {
+            const int d = j % D;
+            if (d < first || d >= first + 2 * pairs) orow[j] = xr[j];
+        }
+}
+
+}  // namespace
+
+extern "C" {
+
+rcu_status rcu_norm_rows(rcu_device* dev, int kind, const rcu_tensor* x, uint32_t x_col, const rcu_tensor* scale, const rcu_tensor* gate,
+                         uint32_t gate_col, float eps, rcu_tensor* dst) {
+    if (!dev) return RCU_ERR_INVALID_ARG;
+    RCU_REQUIRE(dev, t_valid(x) && t_valid(scale) && t_valid(dst), "norm_rows: invalid tensor descriptor");
+    RCU_REQUIRE(dev, kind == RCU_LAYER_NORM || kind == RCU_RMS_NORM, "norm_rows: LayerNorm or RMSNorm");
+    RCU_REQUIRE(dev, x->dt == RCU_F32 && scale->dt == RCU_F32 && dt_is_float(dst->dt), "norm_rows: f32 input and scale, float output");
+    const uint64_t N = t_numel(scale), pitch = x->shape[x->rank - 1], rows = t_numel(x) / pitch;
+    RCU_REQUIRE(dev, x_col + N <= pitch && N <= 0x7fffffffull && rows <= 0x7fffffffull, "norm_rows: the columns lie outside the rows");
+    RCU_REQUIRE(dev, t_numel(dst) == rows * N, "norm_rows: dst holds %llu elements, expected %llu", (unsigned long long)t_numel(dst), (unsigned long long)(rows * N));
+    uint64_t gp = 0;
+    if (gate) {
+        RCU_REQUIRE(dev, t_valid(gate) && gate->dt == dst->dt, "norm_rows: the gate has the output's dtype");
+        gp = gate->shape[gate->rank - 1];
+        RCU_REQUIRE(dev, gate_col + N <= gp && t_numel(gate) / gp == rows, "norm_rows: the gate's columns lie outside its rows");
+    }
+    DevGuard g(dev->ordinal);
+    NormArgs a{(const float*)x->data + x_col, (long long)pitch, (const float*)scale->data,
+               gate ? (const char*)gate->data + (size_t)gate_col * dt_esize(gate->dt) : nullptr, (long long)gp, (int)N, eps, kind == RCU_LAYER_NORM};
+    switch (dst->dt) {
+        case RCU_F32: return launch_norm_rows<float>(dev, a, dst->data, rows);
+        case RCU_F16: return launch_norm_rows<__half>(dev, a, dst->data, rows);
+        default: return launch_norm_rows<__nv_bfloat16>(dev, a, dst->data, rows);
+    }
+}
+
+rcu_status rcu_glu(rcu_device* dev, int act, const rcu_tensor* x, rcu_tensor* dst) {
+    if (!dev) return RCU_ERR_INVALID_ARG;
+    RCU_REQUIRE(dev, t_valid(x) && t_valid(dst), "glu: invalid tensor descriptor");
+    RCU_REQUIRE(dev, act == RCU_GELU || act == RCU_SILU, "glu: the activation is gelu or silu");
+    RCU_REQUIRE(dev, x->dt == dst->dt && dt_is_float(x->dt), "glu: float tensors of one dtype");
+    const uint64_t F2 = x->shape[x->rank - 1], rows = t_numel(x) / F2;
+    RCU_REQUIRE(dev, F2 % 2 == 0 && t_numel(dst) == rows * (F2 / 2) && F2 <= 0x7fffffffull, "glu: dst must hold half of each row");
+    DevGuard g(dev->ordinal);
+    switch (x->dt) {
+        case RCU_F32: return launch_glu<float>(dev, x->data, dst->data, rows, F2 / 2, act);
+        case RCU_F16: return launch_glu<__half>(dev, x->data, dst->data, rows, F2 / 2, act);
+        default: return launch_glu<__nv_bfloat16>(dev, x->data, dst->data, rows, F2 / 2, act);
+    }
+}
+
+rcu_status rcu_rotary_frequencies(uint32_t dims, double base, double factor, double original, double fast, double slow, float* host_freqs,
+                                  float* magnitude) {
+    if (!host_freqs || !magnitude || dims < 2 || dims % 2 || !(base > 1.0)) return RCU_ERR_INVALID_ARG;
+    const bool yarn = factor > 0.0;
+    if (yarn && !(original > 0.0 && fast > 0.0 && slow > 0.0)) return RCU_ERR_INVALID_ARG;
+    const uint32_t pairs = dims / 2;
+    double lo = 0.0, hi = 0.0;
+    if (yarn) {
+        // index of the pair whose wave turns `t` times over the original length
+        auto pair_at = [&](double t) { return dims * std::log(original / (2.0 * M_PI * t)) / (2.0 * std::log(base)); };
+        lo = std::fmax(std::floor(pair_at(fast)), 0.0);
+        hi = std::fmin(std::ceil(pair_at(slow)), (double)dims - 1.0);
+    }
+    for (uint32_t i = 0; i < pairs; ++i) {
+        double f = std::pow(base, -2.0 * i / dims);
+        if (yarn) {
+            const double ramp = std::fmin(std::fmax((i - lo) / std::fmax(hi - lo, 0.001), 0.0), 1.0);
+            f = f / factor * ramp + f * (1.0 - ramp);
+        }
+        host_freqs[i] = (float)f;
+        host_freqs[pairs + i] = (float)(f - (double)(float)f);
+    }
+    *magnitude = yarn ? (float)(0.1 * std::log(factor) + 1.0) : 1.0f;
+    return RCU_OK;
+}
+
+rcu_status rcu_rotary(rcu_device* dev, const rcu_tensor* x, uint32_t first, const rcu_tensor* freqs, float magnitude, uint32_t position, rcu_tensor* dst) {
+    if (!dev) return RCU_ERR_INVALID_ARG;
+    RCU_REQUIRE(dev, t_valid(x) && t_valid(freqs) && t_valid(dst), "rotary: invalid tensor descriptor");
+    RCU_REQUIRE(dev, x->rank == 3 && t_same_shape(x, dst) && x->dt == dst->dt && dt_is_float(x->dt), "rotary: x and dst are float [tokens, heads, dim]");
+    RCU_REQUIRE(dev, freqs->dt == RCU_F32 && freqs->rank == 2 && freqs->shape[0] == 2, "rotary: the frequency table is f32 [2, pairs]");
+    const uint64_t pairs = freqs->shape[1];
+    RCU_REQUIRE(dev, first + 2 * pairs <= x->shape[2] && pairs <= 4096 && x->shape[0] <= 0x7fffffffull, "rotary: the rotated features lie outside the head");
+    DevGuard g(dev->ordinal);
+#define RCU_ROT(T_)                                                                                                                              \
+    rcu_launch(dev, rotary_kernel<T_>, (unsigned)x->shape[0], 128, pairs * sizeof(float2), (const T_*)x->data, (const float*)freqs->data, (T_*)dst->data, \
+               (int)x->shape[1], (int)x->shape[2], (int)first, (int)pairs, magnitude, position)
+    if (x->dt == RCU_F32) RCU_ROT(float);
+    else if (x->dt == RCU_BF16) RCU_ROT(__nv_bfloat16);
+    else RCU_ROT(__half);
+#undef RCU_ROT
+    RCU_LAUNCH_CHECK(dev);
+    return RCU_OK;
+}
+
+}  // extern "C"

@@ -35,10 +35,10 @@ __device__ __forceinline__ uint64_t umma_desc_sw128(const void* smem_ptr) {
     return d;
 }
 
-// 32-bit instruction descriptor, kind::f16: f16 A and B (both K-major), f32 D, M x N tile.
-__host__ __device__ constexpr uint32_t umma_idesc_f16(int m, int n) {
+// 32-bit instruction descriptor, kind::f16: A and B both f16 or both bf16 (both K-major), f32 D, M x N tile.
+__host__ __device__ constexpr uint32_t umma_idesc_f16(int m, int n, bool bf16 = false) {
     return (1u << 4)                      // D format f32
-           | (0u << 7) | (0u << 10)       // A, B format f16
+           | ((bf16 ? 1u : 0u) << 7) | ((bf16 ? 1u : 0u) << 10)   // A, B format: 0 = f16, 1 = bf16
            | (0u << 15) | (0u << 16)      // A, B K-major
            | ((uint32_t)(n >> 3) << 17) | ((uint32_t)(m >> 4) << 24);
 }
@@ -76,5 +76,44 @@ __device__ __forceinline__ void tmem_ld_32x32(uint32_t taddr, float* v) {
     for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]);
 }
 
+// What the epilogue of a tensor-core GEMM does with an accumulator: Out = f16 / bf16: round(acc + bias);
+// Out = f32: residual + alpha * (acc + bias), the residual stream of a model that keeps it in 32 bits
+// (`resid` may be the output itself: every element is read by the thread that writes it).
+template <class Out> struct GemmEpilogue {
+    const Out* bias;          // per output column, nullable
+    const float* resid;       // f32 output only, nullable
+    float alpha;
+    __device__ __forceinline__ Out operator()(float acc, int col, size_t idx) const {
+        float v = acc + (bias ? to_f32<Out>(bias[col]) : 0.f);
+        if (sizeof(Out) == 4) v = resid ? fmaf(alpha, v, resid[idx]) : alpha * v;
+        return from_f32<Out>(v);
+    }
+    // eight consecutive columns, 16-byte aligned
+    __device__ __forceinline__ void store8(Out* out, size_t idx, const float* acc, int col) const {
+        __align__(16) Out h[8];
+        if (sizeof(Out) == 4 && resid) {
+            __align__(16) float r[8];
+            *reinterpret_cast<float4*>(r) = *reinterpret_cast<const float4*>(resid + idx);
+            *reinterpret_cast<float4*>(r + 4) = *reinterpret_cast<const float4*>(resid + idx + 4);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) h[e] = from_f32<Out>(fmaf(alpha, acc[e] + (bias ? to_f32<Out>(bias[col + e]) : 0.f), r[e]));
+        } else {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) h[e] = (*this)(acc[e], col + e, idx + e);
+        }
+#pragma unroll
+        for (int v = 0; v < (int)sizeof(Out) / 2; ++v) reinterpret_cast<uint4*>(out + idx)[v] = reinterpret_cast<const uint4*>(h)[v];
+    }
+};
 
 }  // namespace tc
+
+// Host-side description of a 16-bit tensor-core Linear beyond its sizes (rcu_linear): operand type, row pitch of the
+// activations in elements (0: K), output type and the f32 epilogue.
+struct TcLinear {
+    bool bf16 = false;
+    uint64_t x_pitch = 0;
+    int out_dt = RCU_F16;
+    const float* resid = nullptr;
+    float alpha = 1.f;
+};

@@ -125,3 +125,51 @@ class Decoder:
         self.dev.h2d(self.token.ptr, np.array([token_id], np.int32))
         self.step_device(argmax=False)
         return self.logits.to_numpy()
+
+
+class StackDecoder:
+    """Fused decode step of a parallel-residual layer stack (``rcu_stack_*``): one token per call over the weights and the
+    ``SequenceState`` tensors the lazy graph uses.  ``runs`` are ``capi.rcu_stack_run`` descriptions in execution order with their
+    states filled in; ``keep`` holds whatever owns the memory they point to."""
+
+    def __init__(self, dev: Device, cfg: "capi.rcu_stack_config", runs: List["capi.rcu_stack_run"], embed_ptr: int, norm_ptr: int, head_ptr: int, keep):
+        self.dev, self.vocab, self._keep = dev, cfg.vocab, keep
+        arr = (capi.rcu_stack_run * len(runs))(*runs)
+        h = C.c_void_p()
+        dev.check(dev._lib.rcu_stack_create(dev.handle, C.byref(cfg), arr, C.c_void_p(embed_ptr), C.c_void_p(norm_ptr), C.c_void_p(head_ptr), C.byref(h)))
+        self._h = h
+        self.token = dev.empty(capi.I32, (1,))
+        self.logits = dev.empty(capi.F32, (1, cfg.vocab))
+
+    def close(self) -> None:
+        if self._h is not None and self.dev.handle:
+            self.dev._lib.rcu_stack_destroy(self._h)
+        self._h = None
+
+    def __del__(self):
+        try:
+            self.close()
+        except Exception:
+            pass
+
+    @property
+    def position(self) -> int:
+        return self.dev._lib.rcu_stack_position(self._h)
+
+    @position.setter
+    def position(self, p: int) -> None:
+        if p != self.position:
+            self.dev.check(self.dev._lib.rcu_stack_set_position(self._h, p))
+
+    @property
+    def kernels_per_step(self) -> int:
+        return self.dev._lib.rcu_stack_kernels_per_step(self._h)
+
+    def step_device(self) -> None:
+        """One step on the device: reads ``token``, writes ``logits``, leaves the arg-max in ``token``.  Asynchronous."""
+        self.dev.check(self.dev._lib.rcu_stack_step(self._h, C.c_void_p(self.token.ptr), C.c_void_p(self.logits.ptr), C.c_void_p(self.token.ptr)))
+
+    def step(self, token_id: int) -> None:
+        """One step for a token id of the host.  Asynchronous: read ``logits`` or ``token`` afterwards."""
+        self.dev.h2d(self.token.ptr, np.array([token_id], np.int32))
+        self.step_device()

@@ -328,3 +328,42 @@ class Device:
         self.check(self._lib.rcu_conv1d(self.handle, self._ref(x), self._ref(w), self._ref(bias), stride, padding,
                                         self._ref(out)))
         return out
+
+    # ------------------------------------------------------------------ ops of models with a 32-bit residual stream
+    def linear(self, w: Buffer, x: Buffer, bias: Optional[Buffer] = None, resid: Optional[Buffer] = None, alpha: float = 1.0, x_col: int = 0,
+               dt: Optional[int] = None, out: Optional[Buffer] = None) -> Buffer:
+        out = out or self.empty(x.dt if dt is None else dt, list(x.shape[:-1]) + [w.shape[0]])
+        self.check(self._lib.rcu_linear(self.handle, self._ref(w), self._ref(x), x_col, self._ref(bias), self._ref(resid), alpha, self._ref(out)))
+        return out
+
+    def norm_rows(self, kind: int, x: Buffer, scale: Buffer, eps: float, dt: int, col: int = 0, gate: Optional[Buffer] = None, gate_col: int = 0):
+        out = self.empty(dt, list(x.shape[:-1]) + [scale.numel])
+        self.check(self._lib.rcu_norm_rows(self.handle, kind, self._ref(x), col, self._ref(scale), self._ref(gate), gate_col, eps, self._ref(out)))
+        return out
+
+    def glu(self, act: str, x: Buffer) -> Buffer:
+        out = self.empty(x.dt, list(x.shape[:-1]) + [x.shape[-1] // 2])
+        self.check(self._lib.rcu_glu(self.handle, capi.UNARY_OPS[act], self._ref(x), self._ref(out)))
+        return out
+
+    def rotary(self, x: Buffer, freqs: Buffer, magnitude: float, position: int, first: int = 0, out: Optional[Buffer] = None) -> Buffer:
+        out = out or self.empty(x.dt, x.shape)
+        self.check(self._lib.rcu_rotary(self.handle, self._ref(x), first, self._ref(freqs), magnitude, position, self._ref(out)))
+        return out
+
+    def lightning(self, x: Buffer, decay_pow: Buffer, state: Buffer, silu: bool) -> Buffer:
+        out = self.empty(capi.F32, (x.numel // x.shape[-1], state.shape[0] * state.shape[2]))
+        self.check(self._lib.rcu_lightning(self.handle, self._ref(x), self._ref(decay_pow), self._ref(state), int(silu), self._ref(out)))
+        return out
+
+    def latent_append(self, x: Buffer, scale: Buffer, eps: float, freqs: Buffer, magnitude: float, position: int, ring: Buffer, rows: int, col: int = 0):
+        out = self.empty(ring.dt, (rows, ring.shape[1]))
+        self.check(self._lib.rcu_latent_append(self.handle, self._ref(x), col, self._ref(scale), eps, self._ref(freqs), magnitude, position,
+                                               self._ref(ring), self._ref(out)))
+        return out
+
+    def window_attention(self, q: Buffer, kv: Buffer, shared: Buffer, shared_col: int, vdim: int, window: int, scale: float) -> Buffer:
+        out = self.empty(q.dt, (q.shape[0], q.shape[1] * vdim))
+        self.check(self._lib.rcu_window_attention(self.handle, self._ref(q), self._ref(kv), self._ref(shared), shared_col, vdim, window, scale,
+                                                  self._ref(out)))
+        return out

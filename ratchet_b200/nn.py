@@ -96,3 +96,53 @@ class KVCache:
     def reset(self) -> None:
         for e in self.layers:
             e.entries = 0
+
+
+# ---------------------------------------------------------------------------------------- models with a 32-bit residual stream
+class StreamNorm:
+    """LayerNorm without bias / RMSNorm of an f32 tensor (or of a column window of its rows) into the operand dtype of the
+    matrix product that follows."""
+
+    def __init__(self, kind: int, weight, eps: float, dt: int):
+        self.kind, self.weight, self.eps, self.dt = kind, weight, eps, dt
+
+    def schedule(self, x, col: int = 0, gate=None, gate_col: int = 0):
+        return x.norm_rows(self.kind, self.weight, self.eps, self.dt, col=col, gate=gate, gate_col=gate_col)
+
+
+class GatedMLP:
+    """x + alpha * W_down (act(W_gate h) * W_up h), gate and up rows stacked in one weight."""
+
+    def __init__(self, gate_up, down, act: str):
+        self.gate_up, self.down, self.act = gate_up, down, act
+
+    def schedule(self, h, resid, alpha: float):
+        return self.down.linear(self.gate_up.linear(h).glu(self.act), resid=resid, alpha=alpha, dt=capi.F32)
+
+
+class RotaryTable:
+    """Frequencies of interleaved rotary pairs (plain or YaRN) on the device, and the factor on cos and sin."""
+
+    def __init__(self, freqs, magnitude: float):
+        self.freqs, self.magnitude = freqs, magnitude
+
+
+class SequenceState:
+    """What one sequence keeps between steps: per layer run one tensor - a recurrent state f32 [heads, dim, vdim] or a ring of
+    latents [rows, latent + rotated] - and the number of tokens seen.  The counterpart of ``KVCache`` for models whose layers
+    keep different things."""
+
+    def __init__(self, runs):
+        self.runs = runs
+        self.position = 0
+        self.stack = None                  # the fused decode step bound to these tensors, once one has been made
+
+    def reset(self) -> None:
+        """Back to an empty sequence.  Recurrent states start at zero; ring rows are read only once written."""
+        for t in self.runs:
+            if t.rank() == 3:
+                n = 4
+                for s in t.shape():
+                    n *= s
+                t.dev.check(t.dev._lib.rcu_memset(t.dev.handle, t.data_ptr(), 0, n))
+        self.position = 0

@@ -221,6 +221,36 @@ class Tensor:
     def index_write(self, src: "Tensor", write_start: Sequence[int]) -> "Tensor":
         return self._new(self.dev._lib.rcu_lazy_index_write, self._h, src._h, _u64(write_start))
 
+    # ------------------------------------------------------------------ ops of models with a 32-bit residual stream
+    def linear(self, x: "Tensor", bias: Optional["Tensor"] = None, resid: Optional["Tensor"] = None, alpha: float = 1.0,
+               x_col: int = 0, dt: Optional[int] = None) -> "Tensor":
+        """resid + alpha * (x[..., x_col:] . self^T + bias), self the [N, K] weight; dt: the activations' dtype or F32."""
+        return self._new(self.dev._lib.rcu_lazy_linear, self._h, x._h, x_col, bias._h if bias else None, resid._h if resid else None, alpha,
+                         x.dt() if dt is None else dt)
+
+    def norm_rows(self, kind: int, scale: "Tensor", eps: float, dt: int, col: int = 0, gate: Optional["Tensor"] = None, gate_col: int = 0):
+        """LayerNorm (no bias) / RMSNorm of columns [col, col + len(scale)), optionally times sigmoid(gate[:, gate_col:])."""
+        return self._new(self.dev._lib.rcu_lazy_norm_rows, kind, self._h, col, scale._h, gate._h if gate else None, gate_col, eps, dt)
+
+    def glu(self, act: str) -> "Tensor":
+        """act(gate) * up of rows that hold gate, then up."""
+        return self._new(self.dev._lib.rcu_lazy_glu, capi.UNARY_OPS[act], self._h)
+
+    def rotary(self, freqs: "Tensor", magnitude: float, position: int, first: int = 0) -> "Tensor":
+        """Interleaved-pair rotation of features [first, first + 2 pairs) of [tokens, heads, dim]."""
+        return self._new(self.dev._lib.rcu_lazy_rotary, self._h, first, freqs._h, magnitude, position)
+
+    def lightning(self, decay_pow: "Tensor", state: "Tensor", silu: bool) -> "Tensor":
+        """Linear attention over q, k, v columns of these rows; `state` is updated in place."""
+        return self._new(self.dev._lib.rcu_lazy_lightning, self._h, decay_pow._h, state._h, int(silu))
+
+    def latent_append(self, scale: "Tensor", eps: float, freqs: "Tensor", magnitude: float, position: int, ring: "Tensor", rows: int, col: int = 0):
+        """Latents and rotated key parts of a block into `ring`; the result is the `rows` rows the block sees."""
+        return self._new(self.dev._lib.rcu_lazy_latent_append, self._h, col, scale._h, eps, freqs._h, magnitude, position, ring._h, rows)
+
+    def window_attention(self, kv: "Tensor", shared: "Tensor", shared_col: int, vdim: int, window: int, scale: float) -> "Tensor":
+        return self._new(self.dev._lib.rcu_lazy_window_attention, self._h, kv._h, shared._h, shared_col, vdim, window, scale)
+
     # ------------------------------------------------------------------ execution
     def resolve(self) -> "Tensor":
         """Tensor::resolve (tensor.rs:861-863). Asynchronous; ``to_numpy`` / ``Device.sync`` wait."""

@@ -61,6 +61,8 @@ pub const RCU_GROUP_NORM: c_int = 2;
 pub const RCU_REDUCE_SUM: c_int = 0;
 pub const RCU_REDUCE_MAX: c_int = 1;
 pub const RCU_REDUCE_MEAN: c_int = 2;
+pub const RCU_MIXER_LIGHTNING: c_int = 0;
+pub const RCU_MIXER_LATENT: c_int = 1;
 pub const RCU_DEBUG_NO_REUSE: u32 = 1;
 pub const RCU_DEBUG_PROFILE: u32 = 2;
 pub const RCU_DEBUG_LOG: u32 = 4;
@@ -130,7 +132,51 @@ pub struct rcu_gguf_tensor_info {
 macro_rules! opaque {
     ($($name:ident),*) => { $(#[repr(C)] pub struct $name { _private: [u8; 0] })* };
 }
-opaque!(rcu_device, rcu_lazy, rcu_comm, rcu_decoder, rcu_gguf);
+opaque!(rcu_device, rcu_lazy, rcu_comm, rcu_decoder, rcu_stack, rcu_gguf);
+
+#[repr(C)]
+#[derive(Clone, Copy, Debug)]
+pub struct rcu_stack_config {
+    pub width: u32,
+    pub vocab: u32,
+    pub n_runs: u32,
+    pub eps: f32,
+    pub residual_mult: f32,
+    pub weight_dt: i32,
+}
+
+#[repr(C)]
+#[derive(Clone, Copy, Debug)]
+pub struct rcu_stack_run {
+    pub mixer: i32,
+    pub heads: u32,
+    pub dim: u32,
+    pub vdim: u32,
+    pub ff: u32,
+    pub q_rank: u32,
+    pub kv_rank: u32,
+    pub rot_dim: u32,
+    pub rot_pairs: u32,
+    pub window: u32,
+    pub ring_rows: u32,
+    pub scale: f32,
+    pub rot_magnitude: f32,
+    pub enter: *const c_void,
+    pub enter_bias: *const c_void,
+    pub norm1: *const c_void,
+    pub norm2: *const c_void,
+    pub mix_in: *const c_void,
+    pub mix_norm: *const c_void,
+    pub kv_norm: *const c_void,
+    pub uq: *const c_void,
+    pub ukv: *const c_void,
+    pub freqs: *const c_void,
+    pub decay: *const c_void,
+    pub out: *const c_void,
+    pub gate_up: *const c_void,
+    pub down: *const c_void,
+    pub state: *mut c_void,
+}
 
 #[link(name = "ratchet_cuda")]
 extern "C" {
@@ -178,6 +224,28 @@ extern "C" {
     pub fn rcu_cache(dev: *mut rcu_device, cache: *mut rcu_tensor, src: *const rcu_tensor, dim: u32, offset: u32, dst: *mut rcu_tensor) -> rcu_status;
     pub fn rcu_index_write(dev: *mut rcu_device, dst: *mut rcu_tensor, src: *const rcu_tensor, start: *const u64) -> rcu_status;
     pub fn rcu_conv1d(dev: *mut rcu_device, x: *const rcu_tensor, w: *const rcu_tensor, bias: *const rcu_tensor, stride: u32, padding: u32, dst: *mut rcu_tensor) -> rcu_status;
+    pub fn rcu_linear(
+        dev: *mut rcu_device, w: *const rcu_tensor, x: *const rcu_tensor, x_col: u32, bias: *const rcu_tensor, resid: *const rcu_tensor, alpha: f32, dst: *mut rcu_tensor,
+    ) -> rcu_status;
+    pub fn rcu_norm_rows(
+        dev: *mut rcu_device, kind: c_int, x: *const rcu_tensor, x_col: u32, scale: *const rcu_tensor, gate: *const rcu_tensor, gate_col: u32, eps: f32, dst: *mut rcu_tensor,
+    ) -> rcu_status;
+    pub fn rcu_glu(dev: *mut rcu_device, act: c_int, x: *const rcu_tensor, dst: *mut rcu_tensor) -> rcu_status;
+    pub fn rcu_rotary_frequencies(
+        dims: u32, base: f64, factor: f64, original: f64, fast: f64, slow: f64, host_freqs: *mut f32, magnitude: *mut f32,
+    ) -> rcu_status;
+    pub fn rcu_rotary(
+        dev: *mut rcu_device, x: *const rcu_tensor, first: u32, freqs: *const rcu_tensor, magnitude: f32, position: u32, dst: *mut rcu_tensor,
+    ) -> rcu_status;
+    pub fn rcu_lightning(
+        dev: *mut rcu_device, x: *const rcu_tensor, decay_pow: *const rcu_tensor, state: *mut rcu_tensor, silu: c_int, dst: *mut rcu_tensor,
+    ) -> rcu_status;
+    pub fn rcu_latent_append(
+        dev: *mut rcu_device, x: *const rcu_tensor, x_col: u32, scale: *const rcu_tensor, eps: f32, freqs: *const rcu_tensor, magnitude: f32, position: u32, ring: *mut rcu_tensor, dst: *mut rcu_tensor,
+    ) -> rcu_status;
+    pub fn rcu_window_attention(
+        dev: *mut rcu_device, q: *const rcu_tensor, kv: *const rcu_tensor, shared: *const rcu_tensor, shared_col: u32, vdim: u32, window: u32, scale: f32, dst: *mut rcu_tensor,
+    ) -> rcu_status;
     pub fn rcu_lazy_from_host(dev: *mut rcu_device, dt: i32, rank: u32, shape: *const u64, host: *const c_void, nbytes: u64, out: *mut *mut rcu_lazy) -> rcu_status;
     pub fn rcu_lazy_zeros(dev: *mut rcu_device, dt: i32, rank: u32, shape: *const u64, out: *mut *mut rcu_lazy) -> rcu_status;
     pub fn rcu_lazy_wrap(dev: *mut rcu_device, t: *const rcu_tensor, out: *mut *mut rcu_lazy) -> rcu_status;
@@ -201,6 +269,25 @@ extern "C" {
     pub fn rcu_lazy_index_select(src: *mut rcu_lazy, ids: *mut rcu_lazy, dim: u32, out: *mut *mut rcu_lazy) -> rcu_status;
     pub fn rcu_lazy_cache(cache: *mut rcu_lazy, src: *mut rcu_lazy, dim: u32, offset: u32, out: *mut *mut rcu_lazy) -> rcu_status;
     pub fn rcu_lazy_index_write(dst: *mut rcu_lazy, src: *mut rcu_lazy, start: *const u64, out: *mut *mut rcu_lazy) -> rcu_status;
+    pub fn rcu_lazy_linear(
+        w: *mut rcu_lazy, x: *mut rcu_lazy, x_col: u32, bias: *mut rcu_lazy, resid: *mut rcu_lazy, alpha: f32, dst_dt: i32, out: *mut *mut rcu_lazy,
+    ) -> rcu_status;
+    pub fn rcu_lazy_norm_rows(
+        kind: c_int, x: *mut rcu_lazy, x_col: u32, scale: *mut rcu_lazy, gate: *mut rcu_lazy, gate_col: u32, eps: f32, dst_dt: i32, out: *mut *mut rcu_lazy,
+    ) -> rcu_status;
+    pub fn rcu_lazy_glu(act: c_int, x: *mut rcu_lazy, out: *mut *mut rcu_lazy) -> rcu_status;
+    pub fn rcu_lazy_rotary(
+        x: *mut rcu_lazy, first: u32, freqs: *mut rcu_lazy, magnitude: f32, position: u32, out: *mut *mut rcu_lazy,
+    ) -> rcu_status;
+    pub fn rcu_lazy_lightning(
+        x: *mut rcu_lazy, decay_pow: *mut rcu_lazy, state: *mut rcu_lazy, silu: c_int, out: *mut *mut rcu_lazy,
+    ) -> rcu_status;
+    pub fn rcu_lazy_latent_append(
+        x: *mut rcu_lazy, x_col: u32, scale: *mut rcu_lazy, eps: f32, freqs: *mut rcu_lazy, magnitude: f32, position: u32, ring: *mut rcu_lazy, rows: u32, out: *mut *mut rcu_lazy,
+    ) -> rcu_status;
+    pub fn rcu_lazy_window_attention(
+        q: *mut rcu_lazy, kv: *mut rcu_lazy, shared: *mut rcu_lazy, shared_col: u32, vdim: u32, window: u32, scale: f32, out: *mut *mut rcu_lazy,
+    ) -> rcu_status;
     pub fn rcu_lazy_id(t: *const rcu_lazy) -> u64;
     pub fn rcu_lazy_execution_order(t: *mut rcu_lazy, ids: *mut u64, capacity: u32, n_nodes: *mut u32) -> rcu_status;
     pub fn rcu_lazy_resolve(t: *mut rcu_lazy) -> rcu_status;
@@ -216,6 +303,14 @@ extern "C" {
     pub fn rcu_decoder_profile_step(dec: *mut rcu_decoder, token_dev: *const i32, logits_dev: *mut c_void, stamps_ns: *mut u64, capacity: u32, n_stamps: *mut u32) -> rcu_status;
     pub fn rcu_attn_decode(dev: *mut rcu_device, qkv: *const c_void, k_cache: *mut c_void, v_cache: *mut c_void, n_heads: u32, n_kv_heads: u32, head_dim: u32, max_cache: u32, rope_dim: u32, rope_base: f32, position: u32, out: *mut c_void) -> rcu_status;
     pub fn rcu_attn_decode_static(dev: *mut rcu_device, qkv: *const c_void, k_cache: *mut c_void, v_cache: *mut c_void, n_heads: u32, n_kv_heads: u32, head_dim: u32, max_cache: u32, rope_dim: u32, rope_base: f32, position: u32, out: *mut c_void) -> rcu_status;
+    pub fn rcu_stack_create(
+        dev: *mut rcu_device, cfg: *const rcu_stack_config, runs: *const rcu_stack_run, embed: *const c_void, final_norm: *const c_void, head: *const c_void, out: *mut *mut rcu_stack,
+    ) -> rcu_status;
+    pub fn rcu_stack_destroy(stack: *mut rcu_stack);
+    pub fn rcu_stack_set_position(stack: *mut rcu_stack, position: u32) -> rcu_status;
+    pub fn rcu_stack_position(stack: *const rcu_stack) -> u32;
+    pub fn rcu_stack_step(stack: *mut rcu_stack, token_dev: *const i32, logits_dev: *mut f32, argmax_dev: *mut i32) -> rcu_status;
+    pub fn rcu_stack_kernels_per_step(stack: *const rcu_stack) -> u32;
     pub fn rcu_comm_create(dev: *mut rcu_device, rank: c_int, world: c_int, slot_bytes: u64, out: *mut *mut rcu_comm) -> rcu_status;
     pub fn rcu_comm_export(comm: *mut rcu_comm, handle64: *mut c_void) -> rcu_status;
     pub fn rcu_comm_import(comm: *mut rcu_comm, peer: c_int, handle64: *const c_void) -> rcu_status;
