@@ -217,11 +217,11 @@ rcu_status rcu_conv1d(rcu_device* dev, const rcu_tensor* x, const rcu_tensor* w,
  * No counterpart in the reference, whose models keep activations in one dtype between ops (ratchet-nn/src/norm.rs:37-69).
  * The residual stream, norms, gates, attention scores and recurrent states are f32; matrix products take bf16 or f16
  * operands (or f32: then everything is true f32). */
-/* dst[M, N] = resid + alpha * (x[:, x_col : x_col + K] . w[N, K]^T + bias): x's last dimension may be wider than K.  w and x
- * have one float dtype; dst has it too (resid NULL, alpha 1) or is F32.  bias [N] in dst's dtype, resid F32 (may be dst);
+/* dst[M, N] = resid + alpha * f(x[:, x_col : x_col + K] . w[N, K]^T + bias): x's last dimension may be wider than K; f is silu on
+ * the first silu_cols columns and the identity on the others.  w and x have one float dtype; dst has it too (resid NULL, alpha 1) or is F32.  bias [N] in dst's dtype, resid F32 (may be dst);
  * both nullable. */
-rcu_status rcu_linear(rcu_device* dev, const rcu_tensor* w, const rcu_tensor* x, uint32_t x_col, const rcu_tensor* bias, const rcu_tensor* resid,
-                      float alpha, rcu_tensor* dst);
+rcu_status rcu_linear(rcu_device* dev, const rcu_tensor* w, const rcu_tensor* x, uint32_t x_col, const rcu_tensor* bias, uint32_t silu_cols,
+                      const rcu_tensor* resid, float alpha, rcu_tensor* dst);
 /* LayerNorm without bias / RMSNorm over columns [x_col, x_col + N) of f32 rows (N = scale's length), statistics in f32 (the
  * variance from the deviations), times sigmoid of columns [gate_col, gate_col + N) of `gate` (nullable, dst's dtype).  dst
  * [rows, N] in any float dtype. */
@@ -240,9 +240,9 @@ rcu_status rcu_rotary_frequencies(uint32_t dims, double base, double factor, dou
  * t at `position` + t, freqs F32 [2, pairs] (value and remainder).  dst may alias x.  (rcu_rope rotates half-split pairs.) */
 rcu_status rcu_rotary(rcu_device* dev, const rcu_tensor* x, uint32_t first, const rcu_tensor* freqs, float magnitude, uint32_t position, rcu_tensor* dst);
 /* Linear attention with a fixed decay per head: S <- d S + k v^T, o = S^T q over the rows of x, whose columns are q [H, D], k
- * [H, D], v [H, E] (further columns are ignored), passed through silu first when `silu` is set.  decay_pow F32 [H, n >= 2]: d^0,
- * d^1, ... (64 or more of them let long blocks run in chunks); state F32 [H, D, E], updated in place; dst F32 [tokens, H * E]. */
-rcu_status rcu_lightning(rcu_device* dev, const rcu_tensor* x, const rcu_tensor* decay_pow, rcu_tensor* state, int silu, rcu_tensor* dst);
+ * [H, D], v [H, E] (further columns are ignored).  decay_pow F32 [H, n >= 2]: d^0, d^1, ... (with 129 of them blocks of bf16
+ * rows run in chunks of 128 tokens); state F32 [H, D, E], updated in place; dst F32 [tokens, H * E]. */
+rcu_status rcu_lightning(rcu_device* dev, const rcu_tensor* x, const rcu_tensor* decay_pow, rcu_tensor* state, rcu_tensor* dst);
 /* Latent cache of a sliding-window layer: columns [x_col, x_col + C) of the f32 rows x are RMS-normed with `scale` [C], the
  * R = ring width - C columns behind them rotated (rcu_rotary); the rows go into `ring` [ring rows, C + R] (position p in row p mod
  * ring rows) and dst [L, C + R] receives the L rows the block sees: L - T older ones from the ring, then the block's T. */
@@ -301,12 +301,13 @@ rcu_status rcu_lazy_index_write(rcu_lazy* dst, rcu_lazy* src, const uint64_t* st
 /* The ops of models with a 32-bit residual stream as nodes (arguments as their eager forms; nullable handles are NULL).
  * rcu_lazy_linear writes into `resid` when it is its sole owner; rcu_lazy_lightning and rcu_lazy_latent_append update their
  * state / ring as a side effect, as rcu_lazy_cache does. */
-rcu_status rcu_lazy_linear(rcu_lazy* w, rcu_lazy* x, uint32_t x_col, rcu_lazy* bias, rcu_lazy* resid, float alpha, int32_t dst_dt, rcu_lazy** out);
+rcu_status rcu_lazy_linear(rcu_lazy* w, rcu_lazy* x, uint32_t x_col, rcu_lazy* bias, uint32_t silu_cols, rcu_lazy* resid, float alpha,
+                           int32_t dst_dt, rcu_lazy** out);
 rcu_status rcu_lazy_norm_rows(int kind, rcu_lazy* x, uint32_t x_col, rcu_lazy* scale, rcu_lazy* gate, uint32_t gate_col, float eps, int32_t dst_dt,
                               rcu_lazy** out);
 rcu_status rcu_lazy_glu(int act, rcu_lazy* x, rcu_lazy** out);
 rcu_status rcu_lazy_rotary(rcu_lazy* x, uint32_t first, rcu_lazy* freqs, float magnitude, uint32_t position, rcu_lazy** out);
-rcu_status rcu_lazy_lightning(rcu_lazy* x, rcu_lazy* decay_pow, rcu_lazy* state, int silu, rcu_lazy** out);
+rcu_status rcu_lazy_lightning(rcu_lazy* x, rcu_lazy* decay_pow, rcu_lazy* state, rcu_lazy** out);
 rcu_status rcu_lazy_latent_append(rcu_lazy* x, uint32_t x_col, rcu_lazy* scale, float eps, rcu_lazy* freqs, float magnitude, uint32_t position,
                                   rcu_lazy* ring, uint32_t rows, rcu_lazy** out);
 rcu_status rcu_lazy_window_attention(rcu_lazy* q, rcu_lazy* kv, rcu_lazy* shared, uint32_t shared_col, uint32_t vdim, uint32_t window, float scale,

@@ -197,9 +197,9 @@ class LightningMixer:
         self.heads, self.dim, self.vdim = heads, dim, vdim
 
     def schedule(self, h, resid, alpha: float, state, position: int):
-        rows = self.proj.linear(h)
-        o = rows.lightning(self.decay_pow, state, True)
-        y = self.norm.schedule(o, gate=rows, gate_col=self.heads * (2 * self.dim + self.vdim))
+        qkv = self.heads * (2 * self.dim + self.vdim)
+        rows = self.proj.linear(h, silu_cols=qkv)
+        y = self.norm.schedule(rows.lightning(self.decay_pow, state), gate=rows, gate_col=qkv)
         return self.out.linear(y, resid=resid, alpha=alpha, dt=capi.F32)
 
 

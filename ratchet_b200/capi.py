@@ -135,12 +135,12 @@ SIGNATURES = {
     "rcu_index_write": (C.c_int, [_DEV, _T, _T, _u64p]),
     "rcu_conv1d": (C.c_int, [_DEV, _T, _T, _T, C.c_uint32, C.c_uint32, _T]),
     # models with a 32-bit residual stream
-    "rcu_linear": (C.c_int, [_DEV, _T, _T, C.c_uint32, _T, _T, C.c_float, _T]),
+    "rcu_linear": (C.c_int, [_DEV, _T, _T, C.c_uint32, _T, C.c_uint32, _T, C.c_float, _T]),
     "rcu_norm_rows": (C.c_int, [_DEV, C.c_int, _T, C.c_uint32, _T, _T, C.c_uint32, C.c_float, _T]),
     "rcu_glu": (C.c_int, [_DEV, C.c_int, _T, _T]),
     "rcu_rotary_frequencies": (C.c_int, [C.c_uint32] + [C.c_double] * 5 + [C.POINTER(C.c_float), C.POINTER(C.c_float)]),
     "rcu_rotary": (C.c_int, [_DEV, _T, C.c_uint32, _T, C.c_float, C.c_uint32, _T]),
-    "rcu_lightning": (C.c_int, [_DEV, _T, _T, _T, C.c_int, _T]),
+    "rcu_lightning": (C.c_int, [_DEV, _T, _T, _T, _T]),
     "rcu_latent_append": (C.c_int, [_DEV, _T, C.c_uint32, _T, C.c_float, _T, C.c_float, C.c_uint32, _T, _T]),
     "rcu_window_attention": (C.c_int, [_DEV, _T, _T, _T, C.c_uint32, C.c_uint32, C.c_uint32, C.c_float, _T]),
     # lazy tensor graph
@@ -167,11 +167,11 @@ SIGNATURES = {
     "rcu_lazy_index_select": (C.c_int, [_LZ, _LZ, C.c_uint32, C.POINTER(_LZ)]),
     "rcu_lazy_cache": (C.c_int, [_LZ, _LZ, C.c_uint32, C.c_uint32, C.POINTER(_LZ)]),
     "rcu_lazy_index_write": (C.c_int, [_LZ, _LZ, _u64p, C.POINTER(_LZ)]),
-    "rcu_lazy_linear": (C.c_int, [_LZ, _LZ, C.c_uint32, _LZ, _LZ, C.c_float, C.c_int32, C.POINTER(_LZ)]),
+    "rcu_lazy_linear": (C.c_int, [_LZ, _LZ, C.c_uint32, _LZ, C.c_uint32, _LZ, C.c_float, C.c_int32, C.POINTER(_LZ)]),
     "rcu_lazy_norm_rows": (C.c_int, [C.c_int, _LZ, C.c_uint32, _LZ, _LZ, C.c_uint32, C.c_float, C.c_int32, C.POINTER(_LZ)]),
     "rcu_lazy_glu": (C.c_int, [C.c_int, _LZ, C.POINTER(_LZ)]),
     "rcu_lazy_rotary": (C.c_int, [_LZ, C.c_uint32, _LZ, C.c_float, C.c_uint32, C.POINTER(_LZ)]),
-    "rcu_lazy_lightning": (C.c_int, [_LZ, _LZ, _LZ, C.c_int, C.POINTER(_LZ)]),
+    "rcu_lazy_lightning": (C.c_int, [_LZ, _LZ, _LZ, C.POINTER(_LZ)]),
     "rcu_lazy_latent_append": (C.c_int, [_LZ, C.c_uint32, _LZ, C.c_float, _LZ, C.c_float, C.c_uint32, _LZ, C.c_uint32, C.POINTER(_LZ)]),
     "rcu_lazy_window_attention": (C.c_int, [_LZ, _LZ, _LZ, C.c_uint32, C.c_uint32, C.c_uint32, C.c_float, C.POINTER(_LZ)]),
     "rcu_lazy_id": (C.c_uint64, [_LZ]),

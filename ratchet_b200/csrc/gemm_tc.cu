@@ -363,7 +363,7 @@ rcu_status launch_tc(rcu_device* dev, const CUtensorMap& xmap, const CUtensorMap
         rcu_status st = rcu_alloc(dev, (uint64_t)splits * M * N * 4, &partial);
         if (st != RCU_OK) return st;
         grid.z = splits;
-        rcu_launch(dev, kern, grid, threads, smem, xmap, wmap, qa, GemmEpilogue<Out>{nullptr, nullptr, 1.f}, (Out*)out, M, N, K, dev->d_status, splits,
+        rcu_launch(dev, kern, grid, threads, smem, xmap, wmap, qa, GemmEpilogue<Out>{nullptr, nullptr, 1.f, 0}, (Out*)out, M, N, K, dev->d_status, splits,
                    (float*)partial, idesc);
         dev->launches++;
         const size_t MN = (size_t)M * N;
@@ -467,7 +467,7 @@ rcu_status rcu_gemm_tc_dispatch(rcu_device* dev, int lhs_dt, const void* w, int 
     if (!maps)
         st = rcu_fail(dev, RCU_ERR_CUDA, "gemm_tc: cuTensorMapEncodeTiled failed (M=%llu N=%llu K=%llu)", (unsigned long long)M,
                       (unsigned long long)N, (unsigned long long)K);
-#define RCU_TC(BN_, WK_) launch_tc<BN_, WK_>(dev, xmap, wmap, qa, GemmEpilogue<__half>{(const __half*)bias, nullptr, 1.f}, y, (int)M, (int)N, (int)K)
+#define RCU_TC(BN_, WK_) launch_tc<BN_, WK_>(dev, xmap, wmap, qa, GemmEpilogue<__half>{(const __half*)bias, nullptr, 1.f, 0}, y, (int)M, (int)N, (int)K)
     if (st == RCU_OK) {
         if (wk == WK_F16) st = bn == 256 ? RCU_TC(256, WK_F16) : bn == 128 ? RCU_TC(128, WK_F16) : RCU_TC(64, WK_F16);
         else if (wk == WK_Q8) st = bn == 128 ? RCU_TC(128, WK_Q8) : RCU_TC(64, WK_Q8);
@@ -494,8 +494,8 @@ rcu_status rcu_gemm_tc_batched_f16(rcu_device* dev, const void* w, const void* x
         return rcu_fail(dev, RCU_ERR_CUDA, "gemm_tc: cuTensorMapEncodeTiled failed (batched M=%llu N=%llu K=%llu)", (unsigned long long)M,
                         (unsigned long long)N, (unsigned long long)K);
     QuantArgs qa{nullptr, nullptr, nullptr};
-    return bn == 128 ? launch_tc<128, WK_F16>(dev, xmap, wmap, qa, GemmEpilogue<__half>{nullptr, nullptr, 1.f}, y, (int)M, (int)N, (int)K, (int)batch)
-                     : launch_tc<64, WK_F16>(dev, xmap, wmap, qa, GemmEpilogue<__half>{nullptr, nullptr, 1.f}, y, (int)M, (int)N, (int)K, (int)batch);
+    return bn == 128 ? launch_tc<128, WK_F16>(dev, xmap, wmap, qa, GemmEpilogue<__half>{nullptr, nullptr, 1.f, 0}, y, (int)M, (int)N, (int)K, (int)batch)
+                     : launch_tc<64, WK_F16>(dev, xmap, wmap, qa, GemmEpilogue<__half>{nullptr, nullptr, 1.f, 0}, y, (int)M, (int)N, (int)K, (int)batch);
 }
 
 // A Linear with 16-bit operands and a chosen output (rcu_linear): out = x . W^T (+ bias) rounded to the operands' type, or
@@ -519,8 +519,8 @@ rcu_status rcu_gemm_tc_linear(rcu_device* dev, const void* w, const void* x, con
 #define RCU_TC(OUT_, EPI_)                                                                                                       \
     (bn == 128 ? launch_tc<128, WK_F16, OUT_>(dev, xmap, wmap, qa, EPI_, y, (int)M, (int)N, (int)K, 1, t.bf16)                   \
                : launch_tc<64, WK_F16, OUT_>(dev, xmap, wmap, qa, EPI_, y, (int)M, (int)N, (int)K, 1, t.bf16))
-    if (t.out_dt == RCU_F32) return RCU_TC(float, (GemmEpilogue<float>{(const float*)bias, t.resid, t.alpha}));
-    if (t.out_dt == RCU_BF16) return RCU_TC(__nv_bfloat16, (GemmEpilogue<__nv_bfloat16>{(const __nv_bfloat16*)bias, nullptr, 1.f}));
-    return RCU_TC(__half, (GemmEpilogue<__half>{(const __half*)bias, nullptr, 1.f}));
+    if (t.out_dt == RCU_F32) return RCU_TC(float, (GemmEpilogue<float>{(const float*)bias, t.resid, t.alpha, t.silu_cols}));
+    if (t.out_dt == RCU_BF16) return RCU_TC(__nv_bfloat16, (GemmEpilogue<__nv_bfloat16>{(const __nv_bfloat16*)bias, nullptr, 1.f, t.silu_cols}));
+    return RCU_TC(__half, (GemmEpilogue<__half>{(const __half*)bias, nullptr, 1.f, t.silu_cols}));
 #undef RCU_TC
 }

@@ -293,7 +293,7 @@ rcu_status run_node(rcu_lazy* n) {
             if (n->flags[0]) resid = S(i++);
             rcu_tensor w = S(i++), x = S(i++);
             if (n->flags[1]) bias = S(i++);
-            return rcu_linear(dev, &w, &x, n->u[0], n->flags[1] ? &bias : nullptr, n->flags[0] ? &resid : nullptr, n->f[0], &dst);
+            return rcu_linear(dev, &w, &x, n->u[0], n->flags[1] ? &bias : nullptr, n->u[1], n->flags[0] ? &resid : nullptr, n->f[0], &dst);
         }
         case K_NORM_ROWS: {
             rcu_tensor x = S(0), sc = S(1), gate;
@@ -302,7 +302,7 @@ rcu_status run_node(rcu_lazy* n) {
         }
         case K_GLU: { rcu_tensor x = S(0); return rcu_glu(dev, n->op, &x, &dst); }
         case K_ROTARY: { rcu_tensor x = S(0), fr = S(1); return rcu_rotary(dev, &x, n->u[0], &fr, n->f[0], n->u[1], &dst); }
-        case K_LIGHTNING: { rcu_tensor x = S(0), dp = S(1), st = S(2); return rcu_lightning(dev, &x, &dp, &st, n->flags[0], &dst); }
+        case K_LIGHTNING: { rcu_tensor x = S(0), dp = S(1), st = S(2); return rcu_lightning(dev, &x, &dp, &st, &dst); }
         case K_LATENT_APPEND: {
             rcu_tensor x = S(0), sc = S(1), fr = S(2), ring = S(3);
             return rcu_latent_append(dev, &x, n->u[0], &sc, n->f[0], &fr, n->f[1], n->u[1], &ring, &dst);
@@ -755,7 +755,7 @@ rcu_status rcu_lazy_index_write(rcu_lazy* dst, rcu_lazy* src, const uint64_t* st
     return RCU_OK;
 }
 
-rcu_status rcu_lazy_linear(rcu_lazy* w, rcu_lazy* x, uint32_t x_col, rcu_lazy* bias, rcu_lazy* resid, float alpha, int32_t dst_dt, rcu_lazy** out) {
+rcu_status rcu_lazy_linear(rcu_lazy* w, rcu_lazy* x, uint32_t x_col, rcu_lazy* bias, uint32_t silu_cols, rcu_lazy* resid, float alpha, int32_t dst_dt, rcu_lazy** out) {
     if (!w || !x || !out) return RCU_ERR_INVALID_ARG;
     LAZY_REQUIRE(w->dev, x->dev == w->dev && (!bias || bias->dev == w->dev) && (!resid || resid->dev == w->dev), "Mixed devices");
     LAZY_REQUIRE(w->dev, w->rank == 2 && w->dt == x->dt && dt_is_float(w->dt), "linear: w must be a float matrix of the activations' dtype");
@@ -770,6 +770,7 @@ rcu_status rcu_lazy_linear(rcu_lazy* w, rcu_lazy* x, uint32_t x_col, rcu_lazy* b
     n->flags[0] = resid != nullptr;
     n->flags[1] = bias != nullptr;
     n->u[0] = x_col;
+    n->u[1] = silu_cols;
     n->f[0] = alpha;
     *out = n;
     return RCU_OK;
@@ -817,12 +818,11 @@ rcu_status rcu_lazy_rotary(rcu_lazy* x, uint32_t first, rcu_lazy* freqs, float m
     return RCU_OK;
 }
 
-rcu_status rcu_lazy_lightning(rcu_lazy* x, rcu_lazy* decay_pow, rcu_lazy* state, int silu, rcu_lazy** out) {
+rcu_status rcu_lazy_lightning(rcu_lazy* x, rcu_lazy* decay_pow, rcu_lazy* state, rcu_lazy** out) {
     if (!x || !decay_pow || !state || !out) return RCU_ERR_INVALID_ARG;
     LAZY_REQUIRE(x->dev, state->rank == 3, "lightning: the state is [heads, dim, vdim]");
     const uint64_t shape[2] = {x->numel() / x->shape[x->rank - 1], state->shape[0] * state->shape[2]};
     rcu_lazy* n = new_node(x->dev, K_LIGHTNING, RCU_F32, 2, shape, {x, decay_pow, state});
-    n->flags[0] = silu;
     *out = n;
     return RCU_OK;
 }

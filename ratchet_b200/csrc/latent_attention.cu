@@ -4,8 +4,8 @@
 //   rcu_latent_append   normalises and rotates the block's latents, keeps the last `ring` of them in the layer's ring
 //                       (row of position p: p mod ring) and lays out the rows the block can see;
 //   rcu_window_attention  softmax attention of the block's queries over those rows, keys and values expanded from the
-//                       latents by one Linear before the call.
-#include "lm_math.cuh"
+//                       latents by one Linear before the call.  bf16 blocks run on the tensor cores, f32 ones in FFMA.
+#include "lm_mma.cuh"
 
 namespace {
 
@@ -156,6 +156,180 @@ template <class T> rcu_status launch_window(rcu_device* dev, const WindowArgs& a
     return RCU_OK;
 }
 
+// Tensor-core form for bf16: CTA = (128 queries, head), a warp per 16 queries; keys and values 64 at a time through two
+// asynchronous stages in shared memory.  Scores, softmax and the output sums are f32; the weights enter the product with the
+// values as bf16 value plus remainder.
+constexpr int kQueries = 128, kKeys = 64;
+
+template <int EP>
+__global__ void __launch_bounds__(256) window_mma_kernel(const WindowArgs a, int vec) {
+    rcu_kernel_entry();
+    using lm::bf16;
+    extern __shared__ __align__(16) bf16 tiles[];
+    const int Q = a.D + a.R, qp = (Q + 15) & ~15, ld = qp + 8;
+    constexpr int ldv = EP + 8;
+    bf16 *qs = tiles, *ks = qs + kQueries * ld, *vs = ks + 2 * kKeys * ld;
+    const int h = blockIdx.y, i0 = blockIdx.x * kQueries;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+    const int nq = min(kQueries, a.T - i0);
+    const long long kvp = (long long)a.H * (a.D + a.E);
+    const bf16* K = reinterpret_cast<const bf16*>(a.kv) + (size_t)h * a.D;
+    const bf16* V = reinterpret_cast<const bf16*>(a.kv) + (size_t)a.H * a.D + (size_t)h * a.E;
+    const bf16* KS = reinterpret_cast<const bf16*>(a.shared);
+    const int base = a.L - a.T + i0;                       // key row of the CTA's first query
+    const int first = max(0, base - a.window + 1), last = base + nq - 1;
+    const int tiles_n = (last - first) / kKeys + 1;
+
+    auto load_keys = [&](int n) {
+        const int j0 = first + n * kKeys, rows = min(kKeys, last + 1 - j0);
+        bf16* kt = ks + (n & 1) * kKeys * ld;
+        if (vec) {
+            lm::load_tile(kt, ld, K + (long long)j0 * kvp, kvp, kKeys, rows, a.D, a.D, true);
+            lm::load_tile(kt + a.D, ld, KS + (long long)j0 * a.shared_pitch, a.shared_pitch, kKeys, rows, a.R, a.R, true);
+        } else {
+            for (int i = threadIdx.x; i < kKeys * Q; i += 256) {
+                const int r = i / Q, c = i - r * Q;
+                const bf16* s = c < a.D ? K + (long long)(j0 + r) * kvp + c : KS + (long long)(j0 + r) * a.shared_pitch + c - a.D;
+                kt[r * ld + c] = r < rows ? *s : __float2bfloat16_rn(0.f);
+            }
+        }
+        lm::load_tile(vs + (n & 1) * kKeys * ldv, ldv, V + (long long)j0 * kvp, kvp, kKeys, rows, a.E, EP, vec);
+        lm::cp_commit();
+    };
+    // columns between the head's features and the next multiple of 16 stay zero
+    for (int i = threadIdx.x; i < (kQueries + 2 * kKeys) * (qp - Q); i += 256) {
+        const int r = i / (qp - Q);
+        (r < kQueries ? qs + r * ld : ks + (r - kQueries) * ld)[Q + i % (qp - Q)] = __float2bfloat16_rn(0.f);
+    }
+    const bf16* qg = reinterpret_cast<const bf16*>(a.q) + ((size_t)i0 * a.H + h) * Q;
+    if (vec) {
+        lm::load_tile(qs, ld, qg, (long long)a.H * Q, kQueries, nq, Q, Q, true);
+    } else {
+        for (int i = threadIdx.x; i < kQueries * Q; i += 256) {
+            const int r = i / Q, c = i - r * Q;
+            qs[r * ld + c] = r < nq ? qg[(size_t)r * a.H * Q + c] : __float2bfloat16_rn(0.f);
+        }
+    }
+    load_keys(0);
+
+    const int r0 = warp * 16, row0 = base + r0 + g, row1 = row0 + 8;      // key rows of this thread's two queries
+    const float sc = a.scale * 1.4426950408889634f;                       // scores in units of log 2
+    float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f, o[EP / 8][4];
+#pragma unroll
+    for (int j = 0; j < EP / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
+
+    for (int n = 0; n < tiles_n; ++n) {
+        if (n + 1 < tiles_n) {
+            load_keys(n + 1);
+            lm::cp_wait<1>();
+        } else {
+            lm::cp_wait<0>();
+        }
+        __syncthreads();
+        const int j0 = first + n * kKeys;
+        // a tile no query of this warp sees is passed over
+        if (r0 < nq && j0 <= base + r0 + 15 && j0 + kKeys - 1 >= base + r0 - a.window + 1) {
+            const bf16* kt = ks + (n & 1) * kKeys * ld;
+            const bf16* vt = vs + (n & 1) * kKeys * ldv;
+            float s[8][4] = {};
+            for (int k0 = 0; k0 < qp; k0 += 16) {
+                uint32_t qa[4];
+                lm::load_a(qa, qs, ld, r0, k0);
+#pragma unroll
+                for (int c = 0; c < 4; ++c) {
+                    uint32_t b[4];
+                    lm::load_b(b, kt, ld, 16 * c, k0);
+                    lm::mma(s[2 * c], qa, b[0], b[1]);
+                    lm::mma(s[2 * c + 1], qa, b[2], b[3]);
+                }
+            }
+            float t0 = -INFINITY, t1 = -INFINITY;
+#pragma unroll
+            for (int c = 0; c < 8; ++c)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int j = j0 + 8 * c + 2 * t + (e & 1), row = e < 2 ? row0 : row1;
+                    const float v = j <= row && j > row - a.window ? s[c][e] * sc : -INFINITY;
+                    s[c][e] = v;
+                    if (e < 2) t0 = fmaxf(t0, v);
+                    else t1 = fmaxf(t1, v);
+                }
+            t0 = fmaxf(t0, __shfl_xor_sync(0xffffffffu, t0, 1));
+            t1 = fmaxf(t1, __shfl_xor_sync(0xffffffffu, t1, 1));
+            t0 = fmaxf(t0, __shfl_xor_sync(0xffffffffu, t0, 2));
+            t1 = fmaxf(t1, __shfl_xor_sync(0xffffffffu, t1, 2));
+            const float n0 = fmaxf(m0, t0), n1 = fmaxf(m1, t1);
+            const float z0 = n0 == -INFINITY ? 0.f : n0, z1 = n1 == -INFINITY ? 0.f : n1;      // no key seen yet: weights of zero
+            const float c0 = exp2f(m0 - z0), c1 = exp2f(m1 - z1);
+            m0 = n0; m1 = n1;
+            l0 *= c0; l1 *= c1;
+#pragma unroll
+            for (int c = 0; c < 8; ++c) {
+                s[c][0] = exp2f(s[c][0] - z0); s[c][1] = exp2f(s[c][1] - z0);
+                s[c][2] = exp2f(s[c][2] - z1); s[c][3] = exp2f(s[c][3] - z1);
+                l0 += s[c][0] + s[c][1];
+                l1 += s[c][2] + s[c][3];
+            }
+#pragma unroll
+            for (int j = 0; j < EP / 8; ++j) { o[j][0] *= c0; o[j][1] *= c0; o[j][2] *= c1; o[j][3] *= c1; }
+#pragma unroll
+            for (int kk = 0; kk < 4; ++kk) {
+                uint32_t ph[4], pl[4];
+                lm::split2(s[2 * kk][0], s[2 * kk][1], ph[0], pl[0]);
+                lm::split2(s[2 * kk][2], s[2 * kk][3], ph[1], pl[1]);
+                lm::split2(s[2 * kk + 1][0], s[2 * kk + 1][1], ph[2], pl[2]);
+                lm::split2(s[2 * kk + 1][2], s[2 * kk + 1][3], ph[3], pl[3]);
+#pragma unroll
+                for (int j = 0; j < EP / 16; ++j) {
+                    uint32_t b[4];
+                    lm::load_b_t(b, vt, ldv, 16 * j, 16 * kk);
+                    lm::mma(o[2 * j], ph, b[0], b[1]);
+                    lm::mma(o[2 * j + 1], ph, b[2], b[3]);
+                    lm::mma(o[2 * j], pl, b[0], b[1]);
+                    lm::mma(o[2 * j + 1], pl, b[2], b[3]);
+                }
+            }
+        }
+        __syncthreads();
+    }
+    l0 += __shfl_xor_sync(0xffffffffu, l0, 1);
+    l1 += __shfl_xor_sync(0xffffffffu, l1, 1);
+    l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
+    l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
+    const float w0 = 1.0f / l0, w1 = 1.0f / l1;
+    bf16* og = reinterpret_cast<bf16*>(a.out) + (size_t)i0 * a.H * a.E + (size_t)h * a.E;
+#pragma unroll
+    for (int j = 0; j < EP / 8; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int r = r0 + g + (e < 2 ? 0 : 8), c = 8 * j + 2 * t + (e & 1);
+            if (r < nq && c < a.E) og[(size_t)r * a.H * a.E + c] = __float2bfloat16_rn(o[j][e] * (e < 2 ? w0 : w1));
+        }
+}
+
+size_t window_mma_smem(int Q, int EP) { return ((size_t)(kQueries + 2 * kKeys) * (((Q + 15) & ~15) + 8) + 2 * (size_t)kKeys * (EP + 8)) * sizeof(lm::bf16); }
+
+rcu_status launch_window_mma(rcu_device* dev, const WindowArgs& a) {
+    const int Q = a.D + a.R, ep = a.E <= 32 ? 32 : a.E <= 64 ? 64 : a.E <= 128 ? 128 : 256;
+    if (a.E > 256 || window_mma_smem(Q, ep) > (size_t)dev->smem_optin) return RCU_ERR_UNSUPPORTED;
+    const size_t smem = window_mma_smem(Q, ep);
+    const int vec = a.D % 8 == 0 && a.R % 8 == 0 && a.E % 8 == 0 && a.shared_pitch % 8 == 0 &&
+                    ((reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.kv) | reinterpret_cast<uintptr_t>(a.shared)) & 15) == 0;
+    const dim3 grid((a.T + kQueries - 1) / kQueries, a.H);
+#define RCU_WM(EP_)                                                                                                          \
+    do {                                                                                                                     \
+        RCU_CUDA(dev, cudaFuncSetAttribute(window_mma_kernel<EP_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
+        rcu_launch(dev, window_mma_kernel<EP_>, grid, 256, smem, a, vec);                                                    \
+    } while (0)
+    if (ep == 32) RCU_WM(32);
+    else if (ep == 64) RCU_WM(64);
+    else if (ep == 128) RCU_WM(128);
+    else RCU_WM(256);
+#undef RCU_WM
+    RCU_LAUNCH_CHECK(dev);
+    return RCU_OK;
+}
+
 }  // namespace
 
 extern "C" {
@@ -193,7 +367,9 @@ rcu_status rcu_window_attention(rcu_device* dev, const rcu_tensor* q, const rcu_
     DevGuard g(dev->ordinal);
     WindowArgs a{q->data, kv->data, (const char*)shared->data + (size_t)shared_col * dt_esize(shared->dt), dst->data, (long long)shared->shape[1], (int)T,
                  (int)L, (int)H, (int)(q->shape[2] - R), (int)R, (int)vdim, (int)(window < L ? window : L), scale};
-    return q->dt == RCU_F32 ? launch_window<float>(dev, a) : launch_window<__nv_bfloat16>(dev, a);
+    if (q->dt == RCU_F32) return launch_window<float>(dev, a);
+    const rcu_status st = launch_window_mma(dev, a);
+    return st == RCU_ERR_UNSUPPORTED ? launch_window<__nv_bfloat16>(dev, a) : st;
 }
 
 }  // extern "C"

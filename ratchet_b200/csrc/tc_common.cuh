@@ -83,8 +83,13 @@ template <class Out> struct GemmEpilogue {
     const Out* bias;          // per output column, nullable
     const float* resid;       // f32 output only, nullable
     float alpha;
+    int silu_cols;            // columns below this pass through silu (after the bias)
+    __device__ __forceinline__ float value(float acc, int col) const {
+        const float v = acc + (bias ? to_f32<Out>(bias[col]) : 0.f);
+        return col < silu_cols ? v / (1.0f + expf(-v)) : v;
+    }
     __device__ __forceinline__ Out operator()(float acc, int col, size_t idx) const {
-        float v = acc + (bias ? to_f32<Out>(bias[col]) : 0.f);
+        float v = value(acc, col);
         if (sizeof(Out) == 4) v = resid ? fmaf(alpha, v, resid[idx]) : alpha * v;
         return from_f32<Out>(v);
     }
@@ -96,7 +101,7 @@ template <class Out> struct GemmEpilogue {
             *reinterpret_cast<float4*>(r) = *reinterpret_cast<const float4*>(resid + idx);
             *reinterpret_cast<float4*>(r + 4) = *reinterpret_cast<const float4*>(resid + idx + 4);
 #pragma unroll
-            for (int e = 0; e < 8; ++e) h[e] = from_f32<Out>(fmaf(alpha, acc[e] + (bias ? to_f32<Out>(bias[col + e]) : 0.f), r[e]));
+            for (int e = 0; e < 8; ++e) h[e] = from_f32<Out>(fmaf(alpha, value(acc[e], col + e), r[e]));
         } else {
 #pragma unroll
             for (int e = 0; e < 8; ++e) h[e] = (*this)(acc[e], col + e, idx + e);
@@ -116,4 +121,5 @@ struct TcLinear {
     int out_dt = RCU_F16;
     const float* resid = nullptr;
     float alpha = 1.f;
+    int silu_cols = 0;
 };

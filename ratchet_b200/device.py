@@ -331,9 +331,10 @@ class Device:
 
     # ------------------------------------------------------------------ ops of models with a 32-bit residual stream
     def linear(self, w: Buffer, x: Buffer, bias: Optional[Buffer] = None, resid: Optional[Buffer] = None, alpha: float = 1.0, x_col: int = 0,
-               dt: Optional[int] = None, out: Optional[Buffer] = None) -> Buffer:
+               silu_cols: int = 0, dt: Optional[int] = None, out: Optional[Buffer] = None) -> Buffer:
         out = out or self.empty(x.dt if dt is None else dt, list(x.shape[:-1]) + [w.shape[0]])
-        self.check(self._lib.rcu_linear(self.handle, self._ref(w), self._ref(x), x_col, self._ref(bias), self._ref(resid), alpha, self._ref(out)))
+        self.check(self._lib.rcu_linear(self.handle, self._ref(w), self._ref(x), x_col, self._ref(bias), silu_cols,
+                                        self._ref(resid), alpha, self._ref(out)))
         return out
 
     def norm_rows(self, kind: int, x: Buffer, scale: Buffer, eps: float, dt: int, col: int = 0, gate: Optional[Buffer] = None, gate_col: int = 0):
@@ -351,9 +352,9 @@ class Device:
         self.check(self._lib.rcu_rotary(self.handle, self._ref(x), first, self._ref(freqs), magnitude, position, self._ref(out)))
         return out
 
-    def lightning(self, x: Buffer, decay_pow: Buffer, state: Buffer, silu: bool) -> Buffer:
+    def lightning(self, x: Buffer, decay_pow: Buffer, state: Buffer) -> Buffer:
         out = self.empty(capi.F32, (x.numel // x.shape[-1], state.shape[0] * state.shape[2]))
-        self.check(self._lib.rcu_lightning(self.handle, self._ref(x), self._ref(decay_pow), self._ref(state), int(silu), self._ref(out)))
+        self.check(self._lib.rcu_lightning(self.handle, self._ref(x), self._ref(decay_pow), self._ref(state), self._ref(out)))
         return out
 
     def latent_append(self, x: Buffer, scale: Buffer, eps: float, freqs: Buffer, magnitude: float, position: int, ring: Buffer, rows: int, col: int = 0):

@@ -26,7 +26,7 @@ from .tensor import Tensor
 DTYPES = {"bfloat16": capi.BF16, "float32": capi.F32}
 REGISTRY: Dict[str, type] = {}
 
-CHUNK = 64                    # tokens of a linear-attention chunk: the decay tables hold this many powers
+CHUNK = 128                   # tokens of a linear-attention chunk: the decay tables hold this many powers
 
 
 def register(architecture: str):

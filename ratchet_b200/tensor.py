@@ -223,9 +223,10 @@ class Tensor:
 
     # ------------------------------------------------------------------ ops of models with a 32-bit residual stream
     def linear(self, x: "Tensor", bias: Optional["Tensor"] = None, resid: Optional["Tensor"] = None, alpha: float = 1.0,
-               x_col: int = 0, dt: Optional[int] = None) -> "Tensor":
-        """resid + alpha * (x[..., x_col:] . self^T + bias), self the [N, K] weight; dt: the activations' dtype or F32."""
-        return self._new(self.dev._lib.rcu_lazy_linear, self._h, x._h, x_col, bias._h if bias else None, resid._h if resid else None, alpha,
+               x_col: int = 0, silu_cols: int = 0, dt: Optional[int] = None) -> "Tensor":
+        """resid + alpha * f(x[..., x_col:] . self^T + bias), self the [N, K] weight, f silu on the first `silu_cols` columns; dt:
+        the activations' dtype or F32."""
+        return self._new(self.dev._lib.rcu_lazy_linear, self._h, x._h, x_col, bias._h if bias else None, silu_cols, resid._h if resid else None, alpha,
                          x.dt() if dt is None else dt)
 
     def norm_rows(self, kind: int, scale: "Tensor", eps: float, dt: int, col: int = 0, gate: Optional["Tensor"] = None, gate_col: int = 0):
@@ -240,9 +241,9 @@ class Tensor:
         """Interleaved-pair rotation of features [first, first + 2 pairs) of [tokens, heads, dim]."""
         return self._new(self.dev._lib.rcu_lazy_rotary, self._h, first, freqs._h, magnitude, position)
 
-    def lightning(self, decay_pow: "Tensor", state: "Tensor", silu: bool) -> "Tensor":
+    def lightning(self, decay_pow: "Tensor", state: "Tensor") -> "Tensor":
         """Linear attention over q, k, v columns of these rows; `state` is updated in place."""
-        return self._new(self.dev._lib.rcu_lazy_lightning, self._h, decay_pow._h, state._h, int(silu))
+        return self._new(self.dev._lib.rcu_lazy_lightning, self._h, decay_pow._h, state._h)
 
     def latent_append(self, scale: "Tensor", eps: float, freqs: "Tensor", magnitude: float, position: int, ring: "Tensor", rows: int, col: int = 0):
         """Latents and rotated key parts of a block into `ring`; the result is the `rows` rows the block sees."""

@@ -225,7 +225,7 @@ extern "C" {
     pub fn rcu_index_write(dev: *mut rcu_device, dst: *mut rcu_tensor, src: *const rcu_tensor, start: *const u64) -> rcu_status;
     pub fn rcu_conv1d(dev: *mut rcu_device, x: *const rcu_tensor, w: *const rcu_tensor, bias: *const rcu_tensor, stride: u32, padding: u32, dst: *mut rcu_tensor) -> rcu_status;
     pub fn rcu_linear(
-        dev: *mut rcu_device, w: *const rcu_tensor, x: *const rcu_tensor, x_col: u32, bias: *const rcu_tensor, resid: *const rcu_tensor, alpha: f32, dst: *mut rcu_tensor,
+        dev: *mut rcu_device, w: *const rcu_tensor, x: *const rcu_tensor, x_col: u32, bias: *const rcu_tensor, silu_cols: u32, resid: *const rcu_tensor, alpha: f32, dst: *mut rcu_tensor,
     ) -> rcu_status;
     pub fn rcu_norm_rows(
         dev: *mut rcu_device, kind: c_int, x: *const rcu_tensor, x_col: u32, scale: *const rcu_tensor, gate: *const rcu_tensor, gate_col: u32, eps: f32, dst: *mut rcu_tensor,
@@ -238,7 +238,7 @@ extern "C" {
         dev: *mut rcu_device, x: *const rcu_tensor, first: u32, freqs: *const rcu_tensor, magnitude: f32, position: u32, dst: *mut rcu_tensor,
     ) -> rcu_status;
     pub fn rcu_lightning(
-        dev: *mut rcu_device, x: *const rcu_tensor, decay_pow: *const rcu_tensor, state: *mut rcu_tensor, silu: c_int, dst: *mut rcu_tensor,
+        dev: *mut rcu_device, x: *const rcu_tensor, decay_pow: *const rcu_tensor, state: *mut rcu_tensor, dst: *mut rcu_tensor,
     ) -> rcu_status;
     pub fn rcu_latent_append(
         dev: *mut rcu_device, x: *const rcu_tensor, x_col: u32, scale: *const rcu_tensor, eps: f32, freqs: *const rcu_tensor, magnitude: f32, position: u32, ring: *mut rcu_tensor, dst: *mut rcu_tensor,
@@ -270,7 +270,7 @@ extern "C" {
     pub fn rcu_lazy_cache(cache: *mut rcu_lazy, src: *mut rcu_lazy, dim: u32, offset: u32, out: *mut *mut rcu_lazy) -> rcu_status;
     pub fn rcu_lazy_index_write(dst: *mut rcu_lazy, src: *mut rcu_lazy, start: *const u64, out: *mut *mut rcu_lazy) -> rcu_status;
     pub fn rcu_lazy_linear(
-        w: *mut rcu_lazy, x: *mut rcu_lazy, x_col: u32, bias: *mut rcu_lazy, resid: *mut rcu_lazy, alpha: f32, dst_dt: i32, out: *mut *mut rcu_lazy,
+        w: *mut rcu_lazy, x: *mut rcu_lazy, x_col: u32, bias: *mut rcu_lazy, silu_cols: u32, resid: *mut rcu_lazy, alpha: f32, dst_dt: i32, out: *mut *mut rcu_lazy,
     ) -> rcu_status;
     pub fn rcu_lazy_norm_rows(
         kind: c_int, x: *mut rcu_lazy, x_col: u32, scale: *mut rcu_lazy, gate: *mut rcu_lazy, gate_col: u32, eps: f32, dst_dt: i32, out: *mut *mut rcu_lazy,
@@ -279,9 +279,7 @@ extern "C" {
     pub fn rcu_lazy_rotary(
         x: *mut rcu_lazy, first: u32, freqs: *mut rcu_lazy, magnitude: f32, position: u32, out: *mut *mut rcu_lazy,
     ) -> rcu_status;
-    pub fn rcu_lazy_lightning(
-        x: *mut rcu_lazy, decay_pow: *mut rcu_lazy, state: *mut rcu_lazy, silu: c_int, out: *mut *mut rcu_lazy,
-    ) -> rcu_status;
+    pub fn rcu_lazy_lightning(x: *mut rcu_lazy, decay_pow: *mut rcu_lazy, state: *mut rcu_lazy, out: *mut *mut rcu_lazy) -> rcu_status;
     pub fn rcu_lazy_latent_append(
         x: *mut rcu_lazy, x_col: u32, scale: *mut rcu_lazy, eps: f32, freqs: *mut rcu_lazy, magnitude: f32, position: u32, ring: *mut rcu_lazy, rows: u32, out: *mut *mut rcu_lazy,
     ) -> rcu_status;
