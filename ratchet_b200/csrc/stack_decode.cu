@@ -8,23 +8,31 @@
 //                   [queries into latent space] -> [attention over latents] -> [merge + values] -> [both output
 //                   projections + residual]
 //
-// Every matrix is streamed once by rows_kernel: a persistent grid of one CTA per SM; a team of 1, 2, 4 or 8 warps owns
-// two rows at a time, keeps the next batch of 16-byte weight loads in flight while it multiplies the current one, and
-// requests its first batch before it waits for the kernel before it (weights are constant, so programmatic dependent
-// launch hides the start-up).  Norms, gates and activations are folded into the staging of the input vector in shared
-// memory (f32) and into the row epilogues; activations stay in f32 between kernels.  Position and token live in device
+// Every matrix is streamed once.  bf16 weights whose rows are whole 64-element blocks take rows_mma_kernel: a persistent
+// grid of one CTA per SM, sixteen rows per unit, a team of 1, 2, 4 or 8 warps sharing a unit's columns.  Each warp keeps a ring
+// of shared-memory slots filled by TMA (16 rows x 128 columns, 128-byte swizzle, mbarrier transaction counts) and fills it
+// before it waits for the kernel before it: weights are constant, so with programmatic dependent launch the first rows
+// travel while that kernel drains.  The products run on the tensor cores as 16 x 16 times 16 x 8 with the input vector as
+// two of the eight columns - its bf16 rounding and the remainder, so that activations keep 16 bits of mantissa - because
+// unpacking bf16 weights for FFMA costs more issue slots than the memory system leaves.  f32 weights and other row lengths
+// take rows_kernel (FFMA, plain loads).  Norms, gates and activations are folded into the staging of the input vector in
+// shared memory and into the row epilogues; activations stay in f32 between kernels.  Position and token live in device
 // memory, so the whole step replays from one CUDA graph.
 #include <algorithm>
 #include <cmath>
 #include <cstdlib>
 
-#include "lm_math.cuh"
+#include "bulk_async.cuh"
+#include "lm_mma.cuh"
 
 namespace {
 
 constexpr int kThreads = 256, kWarps = 8;
-constexpr int kRows = 2;            // rows per unit
-constexpr int kBatch = 4;           // chunks of a row in flight per buffer
+constexpr int kRows = 2;            // rows per unit of rows_kernel
+constexpr int kUnit = 16;           // rows per unit of rows_mma_kernel
+constexpr int kItem = 128;          // columns per ring slot
+constexpr int kSlotBytes = kUnit * kItem * 2;
+constexpr int kMaxSlots = 8;
 constexpr int kSub = 16;            // cached positions staged at a time
 constexpr int kHeads = 8;           // heads per CTA of the latent attention (one warp each)
 constexpr int kMaxSplits = 64;
@@ -46,7 +54,8 @@ struct RowsArgs {
     float *out, *out2;              // piece A rows; activated pairs
     const float *resid, *bias;
     int n_silu, n_sigmoid;          // EPI_MIXER_IN: rows below n_silu pass silu, rows from n_sigmoid on sigmoid
-    int parts, aligned;
+    int parts, slots;               // warps per team; ring slots per warp
+    int* status;
     // latent append, done by the first CTA (C == 0: none)
     const float* low;               // [C + R]
     const float *c_scale, *freqs;
@@ -55,16 +64,6 @@ struct RowsArgs {
     float magnitude;
     const uint32_t* d_pos;
 };
-
-template <class T> __device__ __forceinline__ uint4 load_chunk(const T* row, int k, int K, bool aligned) {
-    constexpr int VEC = 16 / (int)sizeof(T);
-    if (k >= K) return make_uint4(0u, 0u, 0u, 0u);
-    if (aligned) return ld_stream_v4(row + k);
-    __align__(16) T v[VEC];
-#pragma unroll
-    for (int e = 0; e < VEC; ++e) v[e] = k + e < K ? row[k + e] : from_f32<T>(0.f);
-    return *reinterpret_cast<const uint4*>(v);
-}
 
 // normalised latent and rotated key part of the current token into its ring row
 template <class T> __device__ void append_latent(const RowsArgs& a, float* scratch) {
@@ -84,162 +83,305 @@ template <class T> __device__ void append_latent(const RowsArgs& a, float* scrat
     for (int j = 2 * a.n_freq + threadIdx.x; j < a.R; j += kThreads) row[a.C + j] = from_f32<T>(kr[j]);
 }
 
+__host__ __device__ __forceinline__ int padded(int k) { return (k + 127) & ~127; }      // whole ring items
+
+__device__ __forceinline__ float4 load4(const float* p, int n) {       // elements from n on read as zero
+    if (n >= 4 && (reinterpret_cast<uintptr_t>(p) & 15) == 0) return *reinterpret_cast<const float4*>(p);
+    return make_float4(n > 0 ? p[0] : 0.f, n > 1 ? p[1] : 0.f, n > 2 ? p[2] : 0.f, n > 3 ? p[3] : 0.f);
+}
+
+// The input vectors of a product, normalised or gated, four elements at a time: put(piece, j, values); zeros from the end of a
+// vector to its padded length.
+template <class Put> __device__ __forceinline__ void stage_input(const RowsArgs& a, float* scratch, Put put) {
+    constexpr int kKept = 4;                            // quads of x kept in registers between the passes of a norm
+    const int step = kThreads * 4, j0 = threadIdx.x * 4;
+    if (a.pro == PRO_LAYER_NORM || a.pro == PRO_RMS) {
+        float4 v[kKept];
+#pragma unroll
+        for (int i = 0; i < kKept; ++i) v[i] = load4(a.x + j0 + i * step, a.ka - (j0 + i * step));
+        auto quad = [&](int i) { return i < kKept ? v[i] : load4(a.x + j0 + i * step, a.ka - (j0 + i * step)); };
+        const int quads = (padded(a.ka) + step - 1) / step;
+        float mean = 0.f;
+        if (a.pro == PRO_LAYER_NORM) {
+            float s = 0.f;
+#pragma unroll
+            for (int i = 0; i < kKept; ++i) s += (v[i].x + v[i].y) + (v[i].z + v[i].w);
+            for (int i = kKept; i < quads; ++i) {
+                const float4 w = quad(i);
+                s += (w.x + w.y) + (w.z + w.w);
+            }
+            mean = lm::block_sum(s, scratch) / (float)a.ka;
+        }
+        float q = 0.f;
+        auto square = [&](const float4& w, int j) {
+            if (j < a.ka) q = fmaf(w.x - mean, w.x - mean, q);
+            if (j + 1 < a.ka) q = fmaf(w.y - mean, w.y - mean, q);
+            if (j + 2 < a.ka) q = fmaf(w.z - mean, w.z - mean, q);
+            if (j + 3 < a.ka) q = fmaf(w.w - mean, w.w - mean, q);
+        };
+#pragma unroll
+        for (int i = 0; i < kKept; ++i) square(v[i], j0 + i * step);
+        for (int i = kKept; i < quads; ++i) square(quad(i), j0 + i * step);
+        const float rstd = 1.0f / sqrtf(lm::block_sum(q, scratch) / (float)a.ka + a.eps);
+        auto emit = [&](const float4& w, int j) {
+            if (j >= padded(a.ka)) return;
+            const float4 s1 = load4(a.s1 + j, a.ka - j);        // zero beyond the end
+            const float x = (w.x - mean) * rstd, y = (w.y - mean) * rstd, z = (w.z - mean) * rstd, t = (w.w - mean) * rstd;
+            put(0, j, make_float4(x * s1.x, y * s1.y, z * s1.z, t * s1.w));
+            if (a.s2) {
+                const float4 s2 = load4(a.s2 + j, a.ka - j);
+                put(1, j, make_float4(x * s2.x, y * s2.y, z * s2.z, t * s2.w));
+            }
+        };
+#pragma unroll
+        for (int i = 0; i < kKept; ++i) emit(v[i], j0 + i * step);
+        for (int i = kKept; i < quads; ++i) emit(quad(i), j0 + i * step);
+        return;
+    }
+    float rstd = 1.f;
+    if (a.pro == PRO_GATED_RMS) {
+        float q = 0.f;
+#pragma unroll 4
+        for (int j = j0; j < a.ka; j += step) {
+            const float4 v = load4(a.x + j, a.ka - j);
+            q += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+        }
+        rstd = 1.0f / sqrtf(lm::block_sum(q, scratch) / (float)a.ka + a.eps);
+    }
+#pragma unroll 4
+    for (int j = j0; j < padded(a.ka); j += step) {
+        float4 v;
+        if (a.pro == PRO_GATED_RMS) {
+            v = load4(a.x + j, a.ka - j);
+            const float4 w = load4(a.s1 + j, a.ka - j), g = load4(a.gate + j, a.ka - j);
+            v = make_float4(v.x * rstd * w.x * g.x, v.y * rstd * w.y * g.y, v.z * rstd * w.z * g.z, v.w * rstd * w.w * g.w);
+        } else if (a.split) {
+            auto at = [&](int i) { return i >= a.ka ? 0.f : i < a.split ? a.x[i] : a.x2[i - a.split]; };
+            v = make_float4(at(j), at(j + 1), at(j + 2), at(j + 3));
+        } else {
+            v = load4(a.x + j, a.ka - j);
+        }
+        put(0, j, v);
+    }
+#pragma unroll 4
+    for (int j = j0; j < padded(a.kb); j += step) put(1, j, load4(a.x2 + j, a.kb - j));
+}
+
+__device__ __forceinline__ void finish_row(const RowsArgs& a, int row, float v) {
+    if (row >= a.na) return;
+    if (a.epi == EPI_MIXER_IN) {
+        if (row < a.n_silu) v = lm::silu(v);
+        else if (row >= a.n_sigmoid) v = lm::sigmoid(v);
+    } else if (a.epi == EPI_RESIDUAL) {
+        v = fmaf(a.alpha, v, a.resid[row]);
+    } else if (a.epi == EPI_BIAS) {
+        v += a.bias[row];
+    }
+    a.out[row] = v;
+}
+
+// Any type and row length: two rows per unit in FFMA, a team of warps splitting the columns.
 template <class T>
 __global__ void __launch_bounds__(kThreads) rows_kernel(const RowsArgs a) {
-    constexpr int VEC = 16 / (int)sizeof(T), CH = 32 * VEC;
-    extern __shared__ __align__(16) float xs[];        // input A, padded to a multiple of 8; input B behind it
+    rcu_kernel_entry();
+    extern __shared__ __align__(16) float xs[];        // input A, input B
     __shared__ float scratch[32];
     __shared__ float red[kWarps][kRows];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int parts = a.parts, teams = kWarps / parts, team = warp / parts, part = warp % parts;
     const int ua = (a.na + kRows - 1) / kRows, units = ua + (a.dual ? 0 : a.pairs);
-    const int xb = (a.ka + 7) & ~7;
-    const int nca = (a.ka + CH - 1) / CH, ncb = (a.kb + CH - 1) / CH;
-    const int gt = blockIdx.x * teams + team, gteams = gridDim.x * teams;
-
-    // a unit's chunks: piece A's (or B's), in the dual form A's then B's; this warp takes chunks part, part + parts, ...
-    auto chunks_of = [&](int u) { return a.dual ? nca + ncb : (u < ua ? nca : ncb); };
-    auto row_ptr = [&](int u, int r, bool b_piece) -> const T* {
-        if (a.dual || u < ua) {
-            const int row = min(u * kRows + r, a.na - 1);
-            return b_piece ? reinterpret_cast<const T*>(a.wb) + (size_t)row * a.kb : reinterpret_cast<const T*>(a.wa) + (size_t)row * a.ka;
+    const int xb = padded(a.ka);
+    stage_input(a, scratch, [&](int piece, int j, const float4& v) { *reinterpret_cast<float4*>(xs + (piece ? xb : 0) + j) = v; });
+    if (a.C > 0 && blockIdx.x == 0) append_latent<T>(a, scratch);
+    __syncthreads();
+    const T *wa = reinterpret_cast<const T*>(a.wa), *wb = reinterpret_cast<const T*>(a.wb);
+    for (int u = blockIdx.x * teams + team; u < units; u += gridDim.x * teams) {
+        float acc[kRows] = {};
+        auto dot = [&](const T* w0, const T* w1, const float* x, int K) {
+#pragma unroll 8
+            for (int k = part * 32 + lane; k < K; k += parts * 32) {
+                acc[0] = fmaf(to_f32<T>(w0[k]), x[k], acc[0]);
+                acc[1] = fmaf(to_f32<T>(w1[k]), x[k], acc[1]);
+            }
+        };
+        const size_t r0 = (size_t)u * kRows, r1 = min(u * kRows + 1, a.na - 1);
+        if (a.dual || u < ua) dot(wa + r0 * a.ka, wa + r1 * a.ka, xs, a.ka);
+        if (a.dual) dot(wb + r0 * a.kb, wb + r1 * a.kb, xs + xb, a.kb);
+        else if (u >= ua) dot(wb + (size_t)(u - ua) * a.kb, wb + (size_t)(u - ua + a.pairs) * a.kb, xs + xb, a.kb);
+#pragma unroll
+        for (int r = 0; r < kRows; ++r) acc[r] = warp_sum(acc[r]);
+        if (parts > 1) {
+            if (lane == 0) {
+#pragma unroll
+                for (int r = 0; r < kRows; ++r) red[warp][r] = acc[r];
+            }
+            asm volatile("bar.sync %0, %1;" ::"r"(1 + team), "r"(parts * 32) : "memory");
+            if (part == 0) {
+#pragma unroll
+                for (int r = 0; r < kRows; ++r) {
+                    acc[r] = 0.f;
+                    for (int q = 0; q < parts; ++q) acc[r] += red[team * parts + q][r];
+                }
+            }
+            asm volatile("bar.sync %0, %1;" ::"r"(1 + team), "r"(parts * 32) : "memory");
         }
-        return reinterpret_cast<const T*>(a.wb) + (size_t)(u - ua + r * a.pairs) * a.kb;
-    };
-    auto load_batch = [&](int u, int c0, uint4 (&w)[kBatch][kRows]) {
-        const int nc = chunks_of(u);
-#pragma unroll
-        for (int i = 0; i < kBatch; ++i) {
-            const int c = c0 + i * parts;
-            const bool b_piece = a.dual ? c >= nca : u >= ua;
-            const int k = (a.dual && b_piece ? c - nca : c) * CH + lane * VEC, K = b_piece ? a.kb : a.ka;
-#pragma unroll
-            for (int r = 0; r < kRows; ++r)
-                w[i][r] = c < nc ? load_chunk<T>(row_ptr(u, r, b_piece), k, K, a.aligned) : make_uint4(0u, 0u, 0u, 0u);
+        if (part == 0 && lane == 0) {
+            if (a.dual || u < ua) {
+                finish_row(a, u * kRows, acc[0]);
+                finish_row(a, u * kRows + 1, acc[1]);
+            } else {
+                a.out2[u - ua] = lm::gelu_tanh(acc[0]) * acc[1];
+            }
+        }
+    }
+}
+
+// bf16 weights, rows of whole 64-element blocks.  A unit is sixteen rows of piece A (or of both pieces, dual), or eight gate and
+// their eight up rows.  ma / mb: [columns within a block, row, block] maps of the pieces, box 64 x 8 x 2.
+__global__ void __launch_bounds__(kThreads) rows_mma_kernel(const __grid_constant__ CUtensorMap ma, const __grid_constant__ CUtensorMap mb,
+                                                            const __grid_constant__ RowsArgs a) {
+    extern __shared__ unsigned char smem_dyn[];        // rings (1024-byte aligned), then the inputs in fragment order
+    __shared__ float scratch[32];
+    __shared__ float red[2][kWarps][kUnit];
+    __shared__ __align__(8) uint64_t full[kWarps][kMaxSlots];
+    __shared__ volatile int abort_flag;
+    unsigned char* rings = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_dyn) + 1023) & ~(uintptr_t)1023);
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int slots = a.slots, parts = a.parts, teams = kWarps / parts, team = warp / parts, part = warp % parts;
+    unsigned char* ring = rings + (size_t)warp * slots * kSlotBytes;
+    // Input element k as columns 0 (rounding) and 1 (remainder) of a 16 x 8 operand: lane 4 n + (k % 8) / 2 of block k / 16 holds it
+    uint32_t* xf = reinterpret_cast<uint32_t*>(rings + (size_t)kWarps * slots * kSlotBytes);
+    const int xb = padded(a.ka);                        // one word per element
+    const int ua = (a.na + kUnit - 1) / kUnit, units = ua + (a.dual ? 0 : (a.pairs + kUnit / 2 - 1) / (kUnit / 2));
+    const int ia = (a.ka + kItem - 1) / kItem, ib = (a.kb + kItem - 1) / kItem;      // items of a piece
+    const int gt = blockIdx.x * teams + team, gteams = gridDim.x * teams;
+    auto items_of = [&](int u) { return a.dual ? ia + ib : (u < ua ? ia : ib); };
+    int pu = gt, pi = part, pslot = 0;                  // next item to request: unit, item, slot
+    auto request = [&]() {
+        const bool pair = !a.dual && pu >= ua, b = pair || (a.dual && pi >= ia);
+        const CUtensorMap* map = b ? &mb : &ma;
+        const int block = 2 * (a.dual && b ? pi - ia : pi), row = pair ? (pu - ua) * (kUnit / 2) : pu * kUnit;
+        unsigned char* dst = ring + pslot * kSlotBytes;
+        uint64_t* bar = &full[warp][pslot];
+        if (pi < items_of(pu)) {
+            gemvq8::mbar_expect_tx(bar, kSlotBytes);
+            gemvq8::tma_load_3d(dst, map, 0, row, block, bar);
+            gemvq8::tma_load_3d(dst + kSlotBytes / 2, map, 0, pair ? row + a.pairs : row + kUnit / 2, block, bar);
+        } else {
+            gemvq8::mbar_arrive(bar);                   // a warp with no item in a unit passes through it with an empty slot
+        }
+        if (++pslot == slots) pslot = 0;
+        pi += parts;
+        if (pi >= items_of(pu)) {
+            pu += gteams;
+            pi = part;
         }
     };
 
     asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
-    uint4 cur[kBatch][kRows];
-    int u = gt, c0 = part;
-    if (u < units) load_batch(u, c0, cur);
+    if (threadIdx.x == 0) abort_flag = 0;
+    if (lane == 0) {
+        for (int i = 0; i < slots; ++i) gemvq8::mbar_init(&full[warp][i], 1);
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+        for (int i = 0; i < slots && pu < units; ++i) request();
+    }
+    __syncwarp();
     asm volatile("griddepcontrol.wait;" ::: "memory");
 
-    // ---- stage the input
-    if (a.pro == PRO_LAYER_NORM || a.pro == PRO_RMS) {
-        float s = 0.f;
-        for (int j = threadIdx.x; j < a.ka; j += kThreads) {
-            const float v = a.x[j];
-            xs[j] = v;
-            s += v;
-        }
-        const float mean = a.pro == PRO_LAYER_NORM ? lm::block_sum(s, scratch) / (float)a.ka : 0.f;
-        float q = 0.f;
-        for (int j = threadIdx.x; j < a.ka; j += kThreads) {
-            const float d = xs[j] - mean;
-            q = fmaf(d, d, q);
-        }
-        const float rstd = 1.0f / sqrtf(lm::block_sum(q, scratch) / (float)a.ka + a.eps);
-        for (int j = threadIdx.x; j < a.ka; j += kThreads) {
-            const float d = (xs[j] - mean) * rstd;
-            xs[j] = d * a.s1[j];
-            if (a.s2) xs[xb + j] = d * a.s2[j];
-        }
-    } else {
-        float rstd = 1.f;
-        if (a.pro == PRO_GATED_RMS) {
-            float q = 0.f;
-            for (int j = threadIdx.x; j < a.ka; j += kThreads) q = fmaf(a.x[j], a.x[j], q);
-            rstd = 1.0f / sqrtf(lm::block_sum(q, scratch) / (float)a.ka + a.eps);
-        }
-        for (int j = threadIdx.x; j < a.ka; j += kThreads) {
-            if (a.pro == PRO_GATED_RMS) xs[j] = a.x[j] * rstd * a.s1[j] * a.gate[j];
-            else xs[j] = a.split && j >= a.split ? a.x2[j - a.split] : a.x[j];
-        }
-        for (int j = threadIdx.x; j < a.kb; j += kThreads) xs[xb + j] = a.x2[j];
-    }
-    for (int j = a.ka + threadIdx.x; j < xb; j += kThreads) xs[j] = 0.f;
-    for (int j = a.kb + threadIdx.x; j < ((a.kb + 7) & ~7); j += kThreads) xs[xb + j] = 0.f;
-    if (a.C > 0 && blockIdx.x == 0) append_latent<T>(a, scratch);
+    stage_input(a, scratch, [&](int piece, int j, const float4& v) {
+        uint32_t h0, l0, h1, l1;
+        lm::split2(v.x, v.y, h0, l0);
+        lm::split2(v.z, v.w, h1, l1);
+        uint32_t* f = xf + (piece ? xb : 0) + (j >> 4) * 16 + ((j & 7) >> 1) * 2 + ((j >> 3) & 1);
+        f[0] = h0; f[2] = h1;                           // column 0, lanes t and t + 1
+        f[8] = l0; f[10] = l1;                          // column 1
+    });
+    if (a.C > 0 && blockIdx.x == 0) append_latent<__nv_bfloat16>(a, scratch);
     __syncthreads();
 
-    // ---- rows
-    float acc[kRows] = {};
-    while (u < units) {
-        const int nc = chunks_of(u);
-        int nu = u, n0 = c0 + kBatch * parts;
-        const bool last = n0 >= nc;
-        if (last) { nu = u + gteams; n0 = part; }
-        uint4 next[kBatch][kRows];
-        if (nu < units) load_batch(nu, n0, next);
+    const int row = lane & 7;
+    const uint32_t frag = lm::smem_addr(ring) + ((lane >> 3) & 1) * (kSlotBytes / 2) + row * 128;
+    uint32_t sw[4];                                     // swizzled place of this lane's 16 bytes in each 16-column step of a block
 #pragma unroll
-        for (int i = 0; i < kBatch; ++i) {
-            const int c = c0 + i * parts;
-            if (c >= nc) break;
-            const bool b_piece = a.dual ? c >= nca : u >= ua;
-            const int k = (a.dual && b_piece ? c - nca : c) * CH + lane * VEC;
-            if (k < (b_piece ? a.kb : a.ka)) {
-                const float* xv = xs + (b_piece ? xb : 0) + k;
-                float f[VEC];
+    for (int i = 0; i < 4; ++i) sw[i] = (uint32_t)(((2 * i + (lane >> 4)) ^ row) << 4);
+    bool ok = true;
+    int slot = 0, parity = 0;
+    uint32_t phase = 0;
+    for (int u = gt; u < units; u += gteams, parity ^= 1) {
+        const int n = items_of(u);
+        float c0[4] = {}, c1[4] = {};
+        int i = part;
+        do {
+            // once a wait has given up, the warp only keeps its team's barriers company
+            ok = ok && gemvq8::mbar_wait_spin(&full[warp][slot], phase, &abort_flag, a.status);
+            if (ok && i < n) {
+                const bool b = a.dual ? i >= ia : u >= ua;
+                const uint2* xv = reinterpret_cast<const uint2*>(xf + (b ? xb : 0) + (a.dual && b ? i - ia : i) * kItem) + lane;
+                const uint32_t base = frag + slot * kSlotBytes;
 #pragma unroll
-                for (int e = 0; e < VEC; e += 4) *reinterpret_cast<float4*>(f + e) = *reinterpret_cast<const float4*>(xv + e);
-#pragma unroll
-                for (int r = 0; r < kRows; ++r) {
-                    const T* wv = reinterpret_cast<const T*>(&cur[i][r]);
-#pragma unroll
-                    for (int e = 0; e < VEC; ++e) acc[r] = fmaf(to_f32<T>(wv[e]), f[e], acc[r]);
+                for (int s = 0; s < kItem / 16; ++s) {
+                    uint32_t w[4];
+                    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+                                 : "=r"(w[0]), "=r"(w[1]), "=r"(w[2]), "=r"(w[3])
+                                 : "r"(base + (s >> 2) * 1024 + sw[s & 3]));
+                    uint2 x = make_uint2(0u, 0u);
+                    if (lane < 8) x = xv[s * 8];
+                    if (s & 1) lm::mma(c1, w, x.x, x.y);
+                    else lm::mma(c0, w, x.x, x.y);
+                }
+            }
+            __syncwarp();                               // every lane has read the slot
+            if (lane == 0 && ok && pu < units) request();
+            if (ok && ++slot == slots) { slot = 0; phase ^= 1; }
+            i += parts;
+        } while (i < n);
+        // lanes 4 g: columns 0 and 1 of rows g and g + 8
+        float lo = (c0[0] + c1[0]) + (c0[1] + c1[1]), hi = (c0[2] + c1[2]) + (c0[3] + c1[3]);
+        int g = lane >> 2;
+        bool mine = (lane & 3) == 0;
+        if (parts > 1) {
+            if (mine) {
+                red[parity][warp][g] = lo;
+                red[parity][warp][g + 8] = hi;
+            }
+            asm volatile("bar.sync %0, %1;" ::"r"(1 + team), "r"(parts * 32) : "memory");
+            mine = part == 0 && lane < 8;
+            g = lane;
+            if (mine) {
+                lo = hi = 0.f;
+                for (int q = 0; q < parts; ++q) {
+                    lo += red[parity][team * parts + q][g];
+                    hi += red[parity][team * parts + q][g + 8];
                 }
             }
         }
-        if (last) {
-#pragma unroll
-            for (int r = 0; r < kRows; ++r) acc[r] = warp_sum(acc[r]);
-            if (parts > 1) {
-                if (lane == 0) {
-#pragma unroll
-                    for (int r = 0; r < kRows; ++r) red[warp][r] = acc[r];
-                }
-                asm volatile("bar.sync %0, %1;" ::"r"(1 + team), "r"(parts * 32) : "memory");
-                if (part == 0) {
-#pragma unroll
-                    for (int r = 0; r < kRows; ++r) {
-                        acc[r] = 0.f;
-                        for (int q = 0; q < parts; ++q) acc[r] += red[team * parts + q][r];
-                    }
-                }
-                asm volatile("bar.sync %0, %1;" ::"r"(1 + team), "r"(parts * 32) : "memory");
+        if (mine) {
+            if (a.dual || u < ua) {
+                finish_row(a, u * kUnit + g, lo);
+                finish_row(a, u * kUnit + g + 8, hi);
+            } else {
+                const int p = (u - ua) * (kUnit / 2) + g;
+                if (p < a.pairs) a.out2[p] = lm::gelu_tanh(lo) * hi;
             }
-            if (part == 0 && lane == 0) {
-                if (a.dual || u < ua) {
-#pragma unroll
-                    for (int r = 0; r < kRows; ++r) {
-                        const int row = u * kRows + r;
-                        if (row >= a.na) break;
-                        float v = acc[r];
-                        if (a.epi == EPI_MIXER_IN) {
-                            if (row < a.n_silu) v = lm::silu(v);
-                            else if (row >= a.n_sigmoid) v = lm::sigmoid(v);
-                        } else if (a.epi == EPI_RESIDUAL) {
-                            v = fmaf(a.alpha, v, a.resid[row]);
-                        } else if (a.epi == EPI_BIAS) {
-                            v += a.bias[row];
-                        }
-                        a.out[row] = v;
-                    }
-                } else {
-                    a.out2[u - ua] = lm::gelu_tanh(acc[0]) * acc[1];
-                }
-            }
-#pragma unroll
-            for (int r = 0; r < kRows; ++r) acc[r] = 0.f;
         }
-        u = nu;
-        c0 = n0;
-#pragma unroll
-        for (int i = 0; i < kBatch; ++i)
-#pragma unroll
-            for (int r = 0; r < kRows; ++r) cur[i][r] = next[i][r];
     }
+    if (!ok) {
+        // A wait gave up (the status word says so).  Before leaving, give this warp's copies in flight another chance to land.
+        for (int i = 0; i < slots; ++i)
+            for (int t = 0; t < (1 << 16) && !gemvq8::mbar_test_wait(&full[warp][i], i < slot ? phase ^ 1 : phase); ++t) {}
+    }
+}
+
+// [64 columns, rows, K / 64 blocks] view of a row-major bf16 matrix
+bool make_block_map(CUtensorMap* map, const void* base, uint64_t rows, uint64_t K) {
+    gemvq8::EncodeTiledFn fn = gemvq8::encode_tiled_fn();
+    if (!fn) return false;
+    cuuint64_t dims[3] = {64, rows, K / 64};
+    cuuint64_t strides[2] = {K * 2, 128};
+    cuuint32_t box[3] = {64, kUnit / 2, kItem / 64};
+    cuuint32_t estr[3] = {1, 1, 1};
+    return fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+              CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
 // x0 = x = embedding row of the token; an id outside the table is clamped and flagged
@@ -273,11 +415,19 @@ __global__ void __launch_bounds__(kThreads) lightning_step_kernel(const float* _
     float* S = state + (size_t)h * D * E;
     float o = 0.f;
     if (e < E) {
-#pragma unroll 4
-        for (int d = g; d < D; d += kWarps) {
-            const float s = fmaf(dec, S[(size_t)d * E + e], k[d] * v);
-            S[(size_t)d * E + e] = s;
-            o = fmaf(q[d], s, o);
+        constexpr int kAhead = 16;            // rows requested before the first of them is written back
+        for (int d0 = g; d0 < D; d0 += kWarps * kAhead) {
+            float s[kAhead];
+#pragma unroll
+            for (int i = 0; i < kAhead; ++i) s[i] = d0 + i * kWarps < D ? S[(size_t)(d0 + i * kWarps) * E + e] : 0.f;
+#pragma unroll
+            for (int i = 0; i < kAhead; ++i) {
+                const int d = d0 + i * kWarps;
+                if (d >= D) break;
+                s[i] = fmaf(dec, s[i], k[d] * v);
+                S[(size_t)d * E + e] = s[i];
+                o = fmaf(q[d], s[i], o);
+            }
         }
     }
     part[g][lane] = o;
@@ -326,44 +476,84 @@ __global__ void __launch_bounds__(kThreads) absorb_kernel(const float* __restric
     }
 }
 
+// Eight consecutive elements of a row in shared memory as floats (16 bytes of bf16, 32 of f32).
+__device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
+    *reinterpret_cast<float4*>(v) = *reinterpret_cast<const float4*>(p);
+    *reinterpret_cast<float4*>(v + 4) = *reinterpret_cast<const float4*>(p + 4);
+}
+__device__ __forceinline__ void load8(const __nv_bfloat16* p, float (&v)[8]) {
+    const uint4 r = *reinterpret_cast<const uint4*>(p);
+    const uint32_t w[4] = {r.x, r.y, r.z, r.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        v[2 * i] = __uint_as_float(w[i] << 16);
+        v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+    }
+}
+
+// row pitch of the partial results: C sums, the maximum and the sum of the weights, in whole 16 bytes
+__host__ __device__ __forceinline__ int partial_pitch(int C) { return ((C + 3) & ~3) + 4; }
+
 // Attention of one token over the cached latents: CTA = (run of positions, eight heads), a warp per head.  Positions are
-// staged kSub at a time in shared memory and shared by the heads; each warp keeps an online softmax and its share of the
-// weighted latents.  partial[split][head]: C sums, then the maximum and the sum of the weights.
-template <class T, int PC>
+// staged kSub at a time in shared memory (rows padded with zeros to a multiple of eight elements) and shared by the heads; a
+// lane owns eight consecutive features of every 256.  Each warp keeps an online softmax and its share of the weighted
+// latents.  partial[split][head]: C sums, then the maximum and the sum of the weights.  PW: 256-feature groups of a row.
+template <class T, int PW>
 __global__ void __launch_bounds__(kThreads) latent_step_kernel(const float* __restrict__ qa, const T* __restrict__ ring, int ring_rows, int window,
                                                                const uint32_t* d_pos, float* __restrict__ partial, int H, int C, int R) {
     rcu_kernel_entry();
-    extern __shared__ __align__(16) float q_s[];         // [kHeads][C + R], then the staged rows
-    const int W = C + R, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    T* rows = reinterpret_cast<T*>(q_s + (size_t)kHeads * W);
+    extern __shared__ __align__(16) float q_s[];         // [kHeads][WP], then the staged rows [kSub][WP]
+    const int W = C + R, WP = (W + 7) & ~7, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    T* rows = reinterpret_cast<T*>(q_s + (size_t)kHeads * WP);
     const int h0 = blockIdx.y * kHeads, h = h0 + warp;
     const int pos = (int)*d_pos, first = max(0, pos - window + 1), n = pos - first + 1;
     const int per = (n + gridDim.x - 1) / gridDim.x;
     const int begin = first + min(n, (int)blockIdx.x * per), end = first + min(n, ((int)blockIdx.x + 1) * per);
-    for (int j = threadIdx.x; j < min(kHeads, H - h0) * W; j += kThreads) q_s[j] = qa[(size_t)h0 * W + j];
-    const float* q = q_s + (size_t)warp * W;
-    float m = -INFINITY, l = 0.f, o[PC];
+    constexpr int VEC = 16 / (int)sizeof(T);
+    const bool vec = W % VEC == 0;
+    if (h < H)
+        for (int c = lane; c < WP; c += 32) q_s[warp * WP + c] = c < W ? qa[(size_t)h * W + c] : 0.f;
+    for (int i = threadIdx.x; i < kSub * (WP - W); i += kThreads) rows[(i / (WP - W)) * WP + W + i % (WP - W)] = from_f32<T>(0.f);
+    __syncwarp();
+    float q[PW][8], o[PW][8];
 #pragma unroll
-    for (int c = 0; c < PC; ++c) o[c] = 0.f;
+    for (int g = 0; g < PW; ++g) {
+        const int c = g * 256 + lane * 8;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) q[g][e] = o[g][e] = 0.f;
+        if (c < WP && h < H) load8(q_s + warp * WP + c, q[g]);
+    }
+    float m = -INFINITY, l = 0.f;
     for (int p0 = begin; p0 < end; p0 += kSub) {
         const int np = min(kSub, end - p0);
         __syncthreads();
-        for (int j = threadIdx.x; j < np * W; j += kThreads) {
-            const int r = j / W;
-            rows[j] = ring[(size_t)((p0 + r) % ring_rows) * W + (j - r * W)];
+        for (int r = warp; r < np; r += kWarps) {
+            const T* src = ring + (size_t)((p0 + r) % ring_rows) * W;
+            if (vec)
+                for (int c = lane * VEC; c < W; c += 32 * VEC) *reinterpret_cast<uint4*>(rows + r * WP + c) = *reinterpret_cast<const uint4*>(src + c);
+            else
+                for (int c = lane; c < W; c += 32) rows[r * WP + c] = src[c];
         }
         __syncthreads();
         if (h >= H) continue;
         float s[kSub];
-#pragma unroll
-        for (int r = 0; r < kSub; ++r) s[r] = 0.f;
-        for (int c = lane; c < W; c += 32) {
-            const float qv = q[c];
-#pragma unroll
-            for (int r = 0; r < kSub; ++r)
-                if (r < np) s[r] = fmaf(qv, to_f32<T>(rows[r * W + c]), s[r]);
-        }
         float mt = -INFINITY;
+#pragma unroll
+        for (int r = 0; r < kSub; ++r) {
+            s[r] = 0.f;
+            if (r < np) {
+#pragma unroll
+                for (int g = 0; g < PW; ++g) {
+                    const int c = g * 256 + lane * 8;
+                    if (c < WP) {
+                        float v[8];
+                        load8(rows + r * WP + c, v);
+#pragma unroll
+                        for (int e = 0; e < 8; ++e) s[r] = fmaf(q[g][e], v[e], s[r]);
+                    }
+                }
+            }
+        }
 #pragma unroll
         for (int r = 0; r < kSub; ++r) {
             s[r] = r < np ? warp_sum(s[r]) : -INFINITY;
@@ -372,65 +562,101 @@ __global__ void __launch_bounds__(kThreads) latent_step_kernel(const float* __re
         const float mn = fmaxf(m, mt), corr = expf(m - mn);
         l *= corr;
 #pragma unroll
-        for (int c = 0; c < PC; ++c) o[c] *= corr;
+        for (int g = 0; g < PW; ++g)
 #pragma unroll
-        for (int r = 0; r < kSub; ++r) {
-            s[r] = expf(s[r] - mn);
-            l += s[r];
-        }
+            for (int e = 0; e < 8; ++e) o[g][e] *= corr;
         m = mn;
 #pragma unroll
         for (int r = 0; r < kSub; ++r) {
             if (r >= np) break;
+            const float p = expf(s[r] - mn);
+            l += p;
 #pragma unroll
-            for (int c = 0; c < PC; ++c)
-                if (lane + 32 * c < C) o[c] = fmaf(s[r], to_f32<T>(rows[r * W + lane + 32 * c]), o[c]);
+            for (int g = 0; g < PW; ++g) {
+                const int c = g * 256 + lane * 8;
+                if (c < C) {
+                    float v[8];
+                    load8(rows + r * WP + c, v);
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) o[g][e] = fmaf(p, v[e], o[g][e]);
+                }
+            }
         }
     }
     if (h >= H) return;
-    float* dst = partial + ((size_t)blockIdx.x * H + h) * (C + 2);
+    float* dst = partial + ((size_t)blockIdx.x * H + h) * partial_pitch(C);
 #pragma unroll
-    for (int c = 0; c < PC; ++c)
-        if (lane + 32 * c < C) dst[lane + 32 * c] = o[c];
+    for (int g = 0; g < PW; ++g)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+            const int c = g * 256 + lane * 8 + e;
+            if (c < C) dst[c] = o[g][e];
+        }
     if (lane == 0) {
-        dst[C] = m;
-        dst[C + 1] = l;
+        dst[partial_pitch(C) - 2] = m;
+        dst[partial_pitch(C) - 1] = l;
     }
 }
 
 // Merge of a head's partial results and its values: out[h] = W_uv[h] . (weighted latent).  CTA = (head, run of value rows).
+// Groups of threads merge different splits, four features per thread and load.
 template <class T>
 __global__ void __launch_bounds__(kThreads) latent_values_kernel(const float* __restrict__ partial, int splits, const T* __restrict__ uv, float* __restrict__ out,
                                                                  int H, int C, int E, int rows_per) {
     rcu_kernel_entry();
-    extern __shared__ float c_s[];
+    extern __shared__ __align__(16) float c_s[];        // [groups][quads * 4], the sum in group 0
     __shared__ float wgt[kMaxSplits];
     const int h = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const float* ph = partial + (size_t)h * (C + 2);
-    const size_t stride = (size_t)H * (C + 2);
+    const int pitch = partial_pitch(C), quads = (C + 3) / 4, groups = max(1, kThreads / quads);
+    const float* ph = partial + (size_t)h * pitch;
+    const size_t stride = (size_t)H * pitch;
     if (warp == 0) {
-        float m0 = lane < splits ? ph[lane * stride + C] : -INFINITY, m1 = lane + 32 < splits ? ph[(lane + 32) * stride + C] : -INFINITY;
+        const float m0 = lane < splits ? ph[lane * stride + pitch - 2] : -INFINITY, m1 = lane + 32 < splits ? ph[(lane + 32) * stride + pitch - 2] : -INFINITY;
+        const float l0 = lane < splits ? ph[lane * stride + pitch - 1] : 0.f, l1 = lane + 32 < splits ? ph[(lane + 32) * stride + pitch - 1] : 0.f;
         const float M = warp_max(fmaxf(m0, m1));
         const float w0 = lane < splits ? expf(m0 - M) : 0.f, w1 = lane + 32 < splits ? expf(m1 - M) : 0.f;
-        float l = (lane < splits ? w0 * ph[lane * stride + C + 1] : 0.f) + (lane + 32 < splits ? w1 * ph[(lane + 32) * stride + C + 1] : 0.f);
-        l = warp_sum(l);
+        const float l = warp_sum(w0 * l0 + w1 * l1);
         wgt[lane] = w0 / l;
         wgt[lane + 32] = w1 / l;
     }
     __syncthreads();
-    for (int c = threadIdx.x; c < C; c += kThreads) {
-        float s = 0.f;
+    for (int i = threadIdx.x; i < groups * quads; i += kThreads) {
+        const int g = i / quads, c = (i - g * quads) * 4;
+        float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll 8
-        for (int i = 0; i < splits; ++i) s = fmaf(wgt[i], ph[i * stride + c], s);
+        for (int j = g; j < splits; j += groups) {
+            const float4 v = *reinterpret_cast<const float4*>(ph + j * stride + c);
+            s.x = fmaf(wgt[j], v.x, s.x);
+            s.y = fmaf(wgt[j], v.y, s.y);
+            s.z = fmaf(wgt[j], v.z, s.z);
+            s.w = fmaf(wgt[j], v.w, s.w);
+        }
+        *reinterpret_cast<float4*>(c_s + (size_t)g * quads * 4 + c) = s;
+    }
+    __syncthreads();
+    for (int c = threadIdx.x; c < C; c += kThreads) {
+        float s = c_s[c];
+        for (int g = 1; g < groups; ++g) s += c_s[(size_t)g * quads * 4 + c];
         c_s[c] = s;
     }
     __syncthreads();
     const int e1 = min(E, ((int)blockIdx.y + 1) * rows_per);
+    constexpr int VEC = 16 / (int)sizeof(T);
+    const bool vec = C % VEC == 0 && (reinterpret_cast<uintptr_t>(uv) & 15) == 0;
     for (int e = blockIdx.y * rows_per + warp; e < e1; e += kWarps) {
         const T* w = uv + ((size_t)h * E + e) * C;
         float acc = 0.f;
+        if (vec) {
 #pragma unroll 4
-        for (int c = lane; c < C; c += 32) acc = fmaf(to_f32<T>(w[c]), c_s[c], acc);
+            for (int c = lane * VEC; c < C; c += 32 * VEC) {
+                const uint4 raw = *reinterpret_cast<const uint4*>(w + c);
+                const T* wv = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) acc = fmaf(to_f32<T>(wv[i]), c_s[c + i], acc);
+            }
+        } else {
+            for (int c = lane; c < C; c += 32) acc = fmaf(to_f32<T>(w[c]), c_s[c], acc);
+        }
         acc = warp_sum(acc);
         if (lane == 0) out[(size_t)h * E + e] = acc;
     }
@@ -444,8 +670,11 @@ __global__ void __launch_bounds__(1024) argmax_next_kernel(const float* __restri
     if (out) {
         float best = -INFINITY;
         int idx = 0x7fffffff;
-        for (int i = threadIdx.x; i < n; i += 1024)
-            if (logits[i] > best || idx == 0x7fffffff) { best = logits[i]; idx = i; }
+#pragma unroll 8
+        for (int i = threadIdx.x; i < n; i += 1024) {
+            const float v = logits[i];
+            if (v > best || idx == 0x7fffffff) { best = v; idx = i; }
+        }
 #pragma unroll
         for (int pass = 0; pass < 2; ++pass) {
 #pragma unroll
@@ -494,38 +723,57 @@ namespace {
 
 int latent_splits(const rcu_stack_run& r) { return (int)std::min<uint32_t>(kMaxSplits, std::max<uint32_t>(1, (std::min(r.window, r.ring_rows) + kSub - 1) / kSub)); }
 
-// warps per team: fewest warp steps over the whole grid
-int plan_parts(int grid, int units, int nc) {
+// Warps per team: fewest warp steps over the whole grid.  Ending a unit (reduction, epilogue) costs about an item's time,
+// and meeting the team's other warps another.
+int plan_parts(int grid, int units, int items) {
     int best = 1;
     long long best_cost = -1;
     for (int parts = 1; parts <= kWarps; parts *= 2) {
         const long long teams = (long long)grid * (kWarps / parts), rounds = (units + teams - 1) / teams;
-        const long long cost = rounds * ((((nc + parts - 1) / parts) + kBatch - 1) / kBatch * kBatch);
+        const long long cost = rounds * ((items + parts - 1) / parts + (parts > 1 ? 2 : 1));
         if (best_cost < 0 || cost < best_cost) { best = parts; best_cost = cost; }
     }
     return best;
 }
 
 template <class T> rcu_status launch_rows(rcu_device* dev, RowsArgs a) {
-    constexpr int VEC = 16 / (int)sizeof(T), CH = 32 * VEC;
-    const int units = (a.na + kRows - 1) / kRows + (a.dual ? 0 : a.pairs);
-    const int nca = (a.ka + CH - 1) / CH, ncb = (a.kb + CH - 1) / CH;
-    a.parts = plan_parts(dev->sm_count, units, a.dual ? nca + ncb : std::max(nca, ncb));
+    a.status = dev->d_status;
     const bool has_b = a.kb > 0 && a.wb;
-    a.aligned = a.ka % VEC == 0 && (!has_b || a.kb % VEC == 0) && ((reinterpret_cast<uintptr_t>(a.wa) | reinterpret_cast<uintptr_t>(a.wb)) & 15) == 0;
-    const int teams = kWarps / a.parts;
-    const int grid = std::max(1, std::min(dev->sm_count, (units + teams - 1) / teams));
-    const size_t smem = ((size_t)((a.ka + 7) & ~7) + (size_t)((a.kb + 7) & ~7)) * 4;
-    if (smem + 1024 > (size_t)dev->smem_optin) return rcu_fail(dev, RCU_ERR_UNSUPPORTED, "stack: input vectors of %d + %d do not fit shared memory", a.ka, a.kb);
-    RCU_CUDA(dev, cudaFuncSetAttribute(rows_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)std::max(smem, (size_t)(64 * 1024))));
-    RCU_CUDA(dev, rcu_launch(dev, rows_kernel<T>, grid, kThreads, smem, a));
+    const size_t inputs = ((size_t)padded(a.ka) + (size_t)padded(a.kb)) * 4, per_slot = (size_t)kWarps * kSlotBytes;
+    const size_t most = (size_t)dev->smem_optin - 4096;
+    // ring slots: half an SM's shared memory in all where that leaves each warp two, so that the next kernel's CTA fits beside this one
+    const size_t half = 110 * 1024;
+    int slots = inputs + 1024 < half ? (int)((half - 1024 - inputs) / per_slot) : 0;
+    if (slots < 2) slots = inputs + 1024 + 3 * per_slot <= most ? 3 : 0;
+    a.slots = std::min(slots, kMaxSlots);
+    const bool blocks = sizeof(T) == 2 && a.ka % 64 == 0 && (!has_b || a.kb % 64 == 0) && a.slots > 0 &&
+                        ((reinterpret_cast<uintptr_t>(a.wa) | reinterpret_cast<uintptr_t>(a.wb)) & 15) == 0;
+    if (blocks) {
+        const int units = (a.na + kUnit - 1) / kUnit + (a.dual ? 0 : (a.pairs + kUnit / 2 - 1) / (kUnit / 2));
+        const int ia = (a.ka + kItem - 1) / kItem, ib = has_b ? (a.kb + kItem - 1) / kItem : 0;
+        a.parts = plan_parts(dev->sm_count, units, a.dual ? ia + ib : std::max(ia, ib));
+        const int teams = kWarps / a.parts, grid = std::max(1, std::min(dev->sm_count, (units + teams - 1) / teams));
+        CUtensorMap ma, mb;
+        if (!make_block_map(&ma, a.wa, a.na, a.ka) || !make_block_map(&mb, has_b ? a.wb : a.wa, has_b ? (a.dual ? a.na : 2 * a.pairs) : a.na, has_b ? a.kb : a.ka))
+            return rcu_fail(dev, RCU_ERR_CUDA, "stack: cuTensorMapEncodeTiled failed (%d x %d)", a.na, a.ka);
+        RCU_CUDA(dev, cudaFuncSetAttribute(rows_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)most));
+        RCU_CUDA(dev, rcu_launch(dev, rows_mma_kernel, grid, kThreads, 1024 + a.slots * per_slot + inputs, ma, mb, a));
+    } else {
+        const int units = (a.na + kRows - 1) / kRows + (a.dual ? 0 : a.pairs), nca = (a.ka + 255) / 256, ncb = (a.kb + 255) / 256;
+        a.parts = plan_parts(dev->sm_count, units, a.dual ? nca + ncb : std::max(nca, ncb));
+        const int teams = kWarps / a.parts, grid = std::max(1, std::min(4 * dev->sm_count, (units + teams - 1) / teams));
+        if (inputs > most) return rcu_fail(dev, RCU_ERR_UNSUPPORTED, "stack: input vectors of %d + %d do not fit shared memory", a.ka, a.kb);
+        RCU_CUDA(dev, cudaFuncSetAttribute(rows_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)most));
+        RCU_CUDA(dev, rcu_launch(dev, rows_kernel<T>, grid, kThreads, inputs, a));
+    }
     RCU_LAUNCH_CHECK(dev);
     return RCU_OK;
 }
 
 template <class T> rcu_status launch_latent_step(rcu_device* dev, const rcu_stack* s, const rcu_stack_run& r) {
     const int H = (int)r.heads, C = (int)r.kv_rank, R = (int)r.rot_dim, splits = latent_splits(r);
-    const size_t smem = (size_t)kHeads * (C + R) * 4 + (size_t)kSub * (C + R) * sizeof(T);
+    const int WP = (C + R + 7) & ~7;
+    const size_t smem = (size_t)kHeads * WP * 4 + (size_t)kSub * WP * sizeof(T);
     const dim3 grid(splits, (H + kHeads - 1) / kHeads);
 #define RCU_LS(PC_)                                                                                                                              \
     do {                                                                                                                                         \
@@ -533,10 +781,13 @@ template <class T> rcu_status launch_latent_step(rcu_device* dev, const rcu_stac
         RCU_CUDA(dev, rcu_launch(dev, latent_step_kernel<T, PC_>, grid, kThreads, smem, s->qa, (const T*)r.state, (int)r.ring_rows, (int)r.window, s->d_pos, \
                                  s->partial, H, C, R));                                                                                          \
     } while (0)
-    if (C <= 128) RCU_LS(4);
-    else if (C <= 256) RCU_LS(8);
-    else if (C <= 512) RCU_LS(16);
-    else RCU_LS(32);
+    switch ((WP + 255) / 256) {
+        case 1: RCU_LS(1); break;
+        case 2: RCU_LS(2); break;
+        case 3: RCU_LS(3); break;
+        case 4: RCU_LS(4); break;
+        default: RCU_LS(5); break;
+    }
 #undef RCU_LS
     RCU_LAUNCH_CHECK(dev);
     return RCU_OK;
@@ -594,8 +845,8 @@ template <class T> rcu_status run_step(rcu_stack* s, const int32_t* token, float
                                      s->d_pos, s->qa, D, R, C, r.scale));
             RCU_LAUNCH_CHECK(dev);
             STACK_TRY(launch_latent_step<T>(dev, s, r));
-            const int per = 16;
-            RCU_CUDA(dev, rcu_launch(dev, latent_values_kernel<T>, dim3(H, (E + per - 1) / per), kThreads, (size_t)C * 4, s->partial, latent_splits(r),
+            const int per = 32, quads = (C + 3) / 4, groups = std::max(1, kThreads / quads);
+            RCU_CUDA(dev, rcu_launch(dev, latent_values_kernel<T>, dim3(H, (E + per - 1) / per), kThreads, (size_t)groups * quads * 16, s->partial, latent_splits(r),
                                      (const T*)r.ukv + (size_t)H * D * C, s->y, H, C, E, per));
             RCU_LAUNCH_CHECK(dev);
             out.pro = PRO_CONCAT; out.x = s->y;
@@ -637,11 +888,11 @@ rcu_status rcu_stack_create(rcu_device* dev, const rcu_stack_config* cfg, const 
             RCU_REQUIRE(dev, r.q_rank && r.kv_rank && r.kv_norm && r.uq && r.ukv && (r.rot_pairs == 0 || r.freqs) && 2 * r.rot_pairs <= r.rot_dim,
                         "stack: run %u lacks a weight or a size", i);
             RCU_REQUIRE(dev, r.window > 0 && r.ring_rows > 0, "stack: run %u has no window", i);
-            if (r.kv_rank > 1024) return rcu_fail(dev, RCU_ERR_UNSUPPORTED, "stack: latents of %u (at most 1024)", r.kv_rank);
+            if (r.kv_rank + r.rot_dim > 1280) return rcu_fail(dev, RCU_ERR_UNSUPPORTED, "stack: cached rows of %u (at most 1280)", r.kv_rank + r.rot_dim);
             mix = std::max(mix, (size_t)r.q_rank + r.kv_rank + r.rot_dim);
             q = std::max(q, (size_t)r.heads * (r.dim + r.rot_dim));
             qa = std::max(qa, (size_t)r.heads * (r.kv_rank + r.rot_dim));
-            partial = std::max(partial, (size_t)latent_splits(r) * r.heads * (r.kv_rank + 2));
+            partial = std::max(partial, (size_t)latent_splits(r) * r.heads * partial_pitch((int)r.kv_rank));
         }
         act = std::max(act, (size_t)r.ff);
         y = std::max(y, (size_t)r.heads * r.vdim);

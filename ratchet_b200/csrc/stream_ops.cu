@@ -60,6 +60,53 @@ __global__ void __launch_bounds__(256) norm_rows_warp_kernel(const NormArgs a, O
     }
 }
 
+// A CTA per row of at most 256 * 4 * QUADS elements that starts on 16 bytes: the row in registers, four elements per load.
+template <class Out, int QUADS>
+__global__ void __launch_bounds__(256) norm_rows_quad_kernel(const NormArgs a, Out* __restrict__ out) {
+    rcu_kernel_entry();
+    __shared__ float scratch[32];
+    const size_t row = blockIdx.x;
+    const float* xr = a.x + row * a.x_pitch;
+    float v[QUADS][4];
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < QUADS; ++i) {
+        const int j = (threadIdx.x + i * 256) * 4;
+        float4 q = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (j < a.N) q = *reinterpret_cast<const float4*>(xr + j);
+        v[i][0] = q.x; v[i][1] = q.y; v[i][2] = q.z; v[i][3] = q.w;
+        s += (q.x + q.y) + (q.z + q.w);
+    }
+    const float mean = a.layer ? lm::block_sum(s, scratch) / (float)a.N : 0.f;
+    float q = 0.f;
+#pragma unroll
+    for (int i = 0; i < QUADS; ++i)
+        if ((threadIdx.x + i * 256) * 4 < a.N)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                v[i][e] -= mean;
+                q = fmaf(v[i][e], v[i][e], q);
+            }
+    const float rstd = 1.0f / sqrtf(lm::block_sum(q, scratch) / (float)a.N + a.eps);
+    struct alignas(sizeof(Out) * 4) Quad { Out v[4]; };
+#pragma unroll
+    for (int i = 0; i < QUADS; ++i) {
+        const int j = (threadIdx.x + i * 256) * 4;
+        if (j >= a.N) continue;
+        const float4 g = *reinterpret_cast<const float4*>(a.scale + j);
+        float y[4] = {v[i][0] * rstd * g.x, v[i][1] * rstd * g.y, v[i][2] * rstd * g.z, v[i][3] * rstd * g.w};
+        if (a.gate) {
+            const Quad t = *reinterpret_cast<const Quad*>(reinterpret_cast<const Out*>(a.gate) + row * a.gate_pitch + j);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) y[e] *= lm::sigmoid(to_f32<Out>(t.v[e]));
+        }
+        Quad o;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o.v[e] = from_f32<Out>(y[e]);
+        *reinterpret_cast<Quad*>(out + row * a.N + j) = o;
+    }
+}
+
 // A CTA per row, the row in shared memory.
 template <class Out>
 __global__ void __launch_bounds__(256) norm_rows_kernel(const NormArgs a, Out* __restrict__ out) {
@@ -93,7 +140,14 @@ rcu_status launch_norm_rows(rcu_device* dev, const NormArgs& a, void* out, uint6
     const unsigned warp_grid = (unsigned)((rows + 7) / 8);
     if (a.N <= 128) rcu_launch(dev, norm_rows_warp_kernel<Out, 4>, warp_grid, 256, 0, a, (Out*)out, (long long)rows);
     else if (a.N <= 512) rcu_launch(dev, norm_rows_warp_kernel<Out, 16>, warp_grid, 256, 0, a, (Out*)out, (long long)rows);
-    else {
+    else if (a.N % 4 == 0 && a.N <= 8192 && a.x_pitch % 4 == 0 && a.gate_pitch % 4 == 0 &&
+             ((reinterpret_cast<uintptr_t>(a.x) | reinterpret_cast<uintptr_t>(a.scale) | reinterpret_cast<uintptr_t>(out)) & 15) == 0 &&
+             (reinterpret_cast<uintptr_t>(a.gate) & (4 * sizeof(Out) - 1)) == 0) {
+        if (a.N <= 1024) rcu_launch(dev, norm_rows_quad_kernel<Out, 1>, (unsigned)rows, 256, 0, a, (Out*)out);
+        else if (a.N <= 2048) rcu_launch(dev, norm_rows_quad_kernel<Out, 2>, (unsigned)rows, 256, 0, a, (Out*)out);
+        else if (a.N <= 4096) rcu_launch(dev, norm_rows_quad_kernel<Out, 4>, (unsigned)rows, 256, 0, a, (Out*)out);
+        else rcu_launch(dev, norm_rows_quad_kernel<Out, 8>, (unsigned)rows, 256, 0, a, (Out*)out);
+    } else {
         const size_t smem = (size_t)a.N * 4;
         if (smem + 1024 > (size_t)dev->smem_optin) return rcu_fail(dev, RCU_ERR_UNSUPPORTED, "norm_rows: rows of %d do not fit shared memory", a.N);
         if (smem > 40 * 1024) RCU_CUDA(dev, cudaFuncSetAttribute(norm_rows_kernel<Out>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
