@@ -12,7 +12,7 @@
 // grid of one CTA per SM, sixteen rows per unit, a team of 1, 2, 4 or 8 warps sharing a unit's columns.  Each warp keeps a ring
 // of shared-memory slots filled by TMA (16 rows x 128 columns, 128-byte swizzle, mbarrier transaction counts) and fills it
 // before it waits for the kernel before it: weights are constant, so with programmatic dependent launch the first rows
-// travel while that kernel drains.  The products run on the tensor cores as 16 x 16 times 16 x 8 with the input vector as
+// travel as soon as that kernel leaves an SM.  The products run on the tensor cores as 16 x 16 times 16 x 8 with the input vector as
 // two of the eight columns - its bf16 rounding and the remainder, so that activations keep 16 bits of mantissa - because
 // unpacking bf16 weights for FFMA costs more issue slots than the memory system leaves.  f32 weights and other row lengths
 // take rows_kernel (FFMA, plain loads).  Norms, gates and activations are folded into the staging of the input vector in
@@ -90,10 +90,25 @@ __device__ __forceinline__ float4 load4(const float* p, int n) {       // elemen
     return make_float4(n > 0 ? p[0] : 0.f, n > 1 ? p[1] : 0.f, n > 2 ? p[2] : 0.f, n > 3 ? p[3] : 0.f);
 }
 
+constexpr int kKept = 4;                // quads of a vector that a thread keeps in registers
+
+// The norm scales of a product's input, requested before the wait for the kernel before it (they are constant).
+struct StagedScales {
+    float4 s1[kKept], s2[kKept];
+    __device__ __forceinline__ void request(const RowsArgs& a) {
+        if (a.pro == PRO_CONCAT) return;
+#pragma unroll
+        for (int i = 0; i < kKept; ++i) {
+            const int j = (threadIdx.x + i * kThreads) * 4;
+            s1[i] = load4(a.s1 + j, a.ka - j);          // zero beyond the end
+            if (a.s2) s2[i] = load4(a.s2 + j, a.ka - j);
+        }
+    }
+};
+
 // The input vectors of a product, normalised or gated, four elements at a time: put(piece, j, values); zeros from the end of a
 // vector to its padded length.
-template <class Put> __device__ __forceinline__ void stage_input(const RowsArgs& a, float* scratch, Put put) {
-    constexpr int kKept = 4;                            // quads of x kept in registers between the passes of a norm
+template <class Put> __device__ __forceinline__ void stage_input(const RowsArgs& a, const StagedScales& sc, float* scratch, Put put) {
     const int step = kThreads * 4, j0 = threadIdx.x * 4;
     if (a.pro == PRO_LAYER_NORM || a.pro == PRO_RMS) {
         float4 v[kKept];
@@ -123,45 +138,49 @@ template <class Put> __device__ __forceinline__ void stage_input(const RowsArgs&
         for (int i = 0; i < kKept; ++i) square(v[i], j0 + i * step);
         for (int i = kKept; i < quads; ++i) square(quad(i), j0 + i * step);
         const float rstd = 1.0f / sqrtf(lm::block_sum(q, scratch) / (float)a.ka + a.eps);
-        auto emit = [&](const float4& w, int j) {
+        auto emit = [&](const float4& w, int j, const float4& s1, const float4& s2) {
             if (j >= padded(a.ka)) return;
-            const float4 s1 = load4(a.s1 + j, a.ka - j);        // zero beyond the end
             const float x = (w.x - mean) * rstd, y = (w.y - mean) * rstd, z = (w.z - mean) * rstd, t = (w.w - mean) * rstd;
             put(0, j, make_float4(x * s1.x, y * s1.y, z * s1.z, t * s1.w));
-            if (a.s2) {
-                const float4 s2 = load4(a.s2 + j, a.ka - j);
-                put(1, j, make_float4(x * s2.x, y * s2.y, z * s2.z, t * s2.w));
-            }
+            if (a.s2) put(1, j, make_float4(x * s2.x, y * s2.y, z * s2.z, t * s2.w));
         };
 #pragma unroll
-        for (int i = 0; i < kKept; ++i) emit(v[i], j0 + i * step);
-        for (int i = kKept; i < quads; ++i) emit(quad(i), j0 + i * step);
-        return;
+        for (int i = 0; i < kKept; ++i) emit(v[i], j0 + i * step, sc.s1[i], sc.s2[i]);
+        for (int i = kKept; i < quads; ++i) {
+            const int j = j0 + i * step;
+            emit(quad(i), j, load4(a.s1 + j, a.ka - j), a.s2 ? load4(a.s2 + j, a.ka - j) : make_float4(0.f, 0.f, 0.f, 0.f));
+        }
+        return;                                         // both pieces come from the norm
     }
-    float rstd = 1.f;
     if (a.pro == PRO_GATED_RMS) {
+        float4 v[kKept];
         float q = 0.f;
-#pragma unroll 4
-        for (int j = j0; j < a.ka; j += step) {
-            const float4 v = load4(a.x + j, a.ka - j);
-            q += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+        auto square = [&](const float4& w) { q += (w.x * w.x + w.y * w.y) + (w.z * w.z + w.w * w.w); };
+#pragma unroll
+        for (int i = 0; i < kKept; ++i) {
+            v[i] = load4(a.x + j0 + i * step, a.ka - (j0 + i * step));
+            square(v[i]);
         }
-        rstd = 1.0f / sqrtf(lm::block_sum(q, scratch) / (float)a.ka + a.eps);
-    }
+        for (int j = j0 + kKept * step; j < a.ka; j += step) square(load4(a.x + j, a.ka - j));
+        const float rstd = 1.0f / sqrtf(lm::block_sum(q, scratch) / (float)a.ka + a.eps);
+        auto emit = [&](const float4& w, int j, const float4& s) {
+            if (j >= padded(a.ka)) return;
+            const float4 g = load4(a.gate + j, a.ka - j);
+            put(0, j, make_float4(w.x * rstd * s.x * g.x, w.y * rstd * s.y * g.y, w.z * rstd * s.z * g.z, w.w * rstd * s.w * g.w));
+        };
+#pragma unroll
+        for (int i = 0; i < kKept; ++i) emit(v[i], j0 + i * step, sc.s1[i]);
+        for (int j = j0 + kKept * step; j < padded(a.ka); j += step) emit(load4(a.x + j, a.ka - j), j, load4(a.s1 + j, a.ka - j));
+    } else {
 #pragma unroll 4
-    for (int j = j0; j < padded(a.ka); j += step) {
-        float4 v;
-        if (a.pro == PRO_GATED_RMS) {
-            v = load4(a.x + j, a.ka - j);
-            const float4 w = load4(a.s1 + j, a.ka - j), g = load4(a.gate + j, a.ka - j);
-            v = make_float4(v.x * rstd * w.x * g.x, v.y * rstd * w.y * g.y, v.z * rstd * w.z * g.z, v.w * rstd * w.w * g.w);
-        } else if (a.split) {
-            auto at = [&](int i) { return i >= a.ka ? 0.f : i < a.split ? a.x[i] : a.x2[i - a.split]; };
-            v = make_float4(at(j), at(j + 1), at(j + 2), at(j + 3));
-        } else {
-            v = load4(a.x + j, a.ka - j);
+        for (int j = j0; j < padded(a.ka); j += step) {
+            if (a.split) {
+                auto at = [&](int i) { return i >= a.ka ? 0.f : i < a.split ? a.x[i] : a.x2[i - a.split]; };
+                put(0, j, make_float4(at(j), at(j + 1), at(j + 2), at(j + 3)));
+            } else {
+                put(0, j, load4(a.x + j, a.ka - j));
+            }
         }
-        put(0, j, v);
     }
 #pragma unroll 4
     for (int j = j0; j < padded(a.kb); j += step) put(1, j, load4(a.x2 + j, a.kb - j));
@@ -191,11 +210,13 @@ __global__ void __launch_bounds__(kThreads) rows_kernel(const RowsArgs a) {
     const int parts = a.parts, teams = kWarps / parts, team = warp / parts, part = warp % parts;
     const int ua = (a.na + kRows - 1) / kRows, units = ua + (a.dual ? 0 : a.pairs);
     const int xb = padded(a.ka);
-    stage_input(a, scratch, [&](int piece, int j, const float4& v) { *reinterpret_cast<float4*>(xs + (piece ? xb : 0) + j) = v; });
+    StagedScales sc;
+    sc.request(a);
+    stage_input(a, sc, scratch, [&](int piece, int j, const float4& v) { *reinterpret_cast<float4*>(xs + (piece ? xb : 0) + j) = v; });
     if (a.C > 0 && blockIdx.x == 0) append_latent<T>(a, scratch);
     __syncthreads();
     const T *wa = reinterpret_cast<const T*>(a.wa), *wb = reinterpret_cast<const T*>(a.wb);
-    for (int u = blockIdx.x * teams + team; u < units; u += gridDim.x * teams) {
+    for (int u = team * gridDim.x + blockIdx.x; u < units; u += gridDim.x * teams) {
         float acc[kRows] = {};
         auto dot = [&](const T* w0, const T* w1, const float* x, int K) {
 #pragma unroll 8
@@ -254,7 +275,7 @@ __global__ void __launch_bounds__(kThreads) rows_mma_kernel(const __grid_constan
     const int xb = padded(a.ka);                        // one word per element
     const int ua = (a.na + kUnit - 1) / kUnit, units = ua + (a.dual ? 0 : (a.pairs + kUnit / 2 - 1) / (kUnit / 2));
     const int ia = (a.ka + kItem - 1) / kItem, ib = (a.kb + kItem - 1) / kItem;      // items of a piece
-    const int gt = blockIdx.x * teams + team, gteams = gridDim.x * teams;
+    const int gt = team * gridDim.x + blockIdx.x, gteams = gridDim.x * teams;      // a last, partial round of units spreads over the SMs
     auto items_of = [&](int u) { return a.dual ? ia + ib : (u < ua ? ia : ib); };
     int pu = gt, pi = part, pslot = 0;                  // next item to request: unit, item, slot
     auto request = [&]() {
@@ -286,9 +307,11 @@ __global__ void __launch_bounds__(kThreads) rows_mma_kernel(const __grid_constan
         for (int i = 0; i < slots && pu < units; ++i) request();
     }
     __syncwarp();
+    StagedScales sc;
+    sc.request(a);
     asm volatile("griddepcontrol.wait;" ::: "memory");
 
-    stage_input(a, scratch, [&](int piece, int j, const float4& v) {
+    stage_input(a, sc, scratch, [&](int piece, int j, const float4& v) {
         uint32_t h0, l0, h1, l1;
         lm::split2(v.x, v.y, h0, l0);
         lm::split2(v.z, v.w, h1, l1);
@@ -476,19 +499,9 @@ __global__ void __launch_bounds__(kThreads) absorb_kernel(const float* __restric
     }
 }
 
-// Eight consecutive elements of a row in shared memory as floats (16 bytes of bf16, 32 of f32).
 __device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
     *reinterpret_cast<float4*>(v) = *reinterpret_cast<const float4*>(p);
     *reinterpret_cast<float4*>(v + 4) = *reinterpret_cast<const float4*>(p + 4);
-}
-__device__ __forceinline__ void load8(const __nv_bfloat16* p, float (&v)[8]) {
-    const uint4 r = *reinterpret_cast<const uint4*>(p);
-    const uint32_t w[4] = {r.x, r.y, r.z, r.w};
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-        v[2 * i] = __uint_as_float(w[i] << 16);
-        v[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
-    }
 }
 
 // row pitch of the partial results: C sums, the maximum and the sum of the weights, in whole 16 bytes
@@ -598,16 +611,165 @@ __global__ void __launch_bounds__(kThreads) latent_step_kernel(const float* __re
     }
 }
 
+// The same for bf16 rings, on the tensor cores: CTA = (run of positions, sixteen heads).  Per sixteen positions: scores as
+// [heads, features] . [features, positions], the features split over the warps and summed in shared memory; online softmax, a
+// thread per (head, position); the weighted latents as [heads, positions] . [positions, features], each warp owning a run
+// of features.  Queries and weights enter as bf16 value plus remainder.
+constexpr int kMmaHeads = 16;
+template <int PC>
+__global__ void __launch_bounds__(kThreads) latent_step_mma_kernel(const float* __restrict__ qa, const lm::bf16* __restrict__ ring, int ring_rows, int window,
+                                                                   const uint32_t* d_pos, float* __restrict__ partial, int H, int C, int R) {
+    rcu_kernel_entry();
+    using lm::bf16;
+    extern __shared__ __align__(16) bf16 tiles[];        // queries (value, remainder), staged rows
+    __shared__ float part[kWarps][kMmaHeads][kSub + 1];
+    __shared__ __align__(16) bf16 ph[kMmaHeads][kSub + 8], pl[kMmaHeads][kSub + 8];
+    __shared__ float corr_s[kMmaHeads];
+    const int W = C + R, wp = (W + 15) & ~15, ld = wp + 8;
+    bf16 *qh = tiles, *ql = qh + kMmaHeads * ld, *rows = ql + kMmaHeads * ld;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
+    const int h0 = blockIdx.y * kMmaHeads;
+    const int pos = (int)*d_pos, first = max(0, pos - window + 1), n = pos - first + 1;
+    const int per = (n + gridDim.x - 1) / gridDim.x;
+    const int begin = first + min(n, (int)blockIdx.x * per), end = first + min(n, ((int)blockIdx.x + 1) * per);
+    auto stage = [&](int p0) {
+        const int np = min(kSub, end - p0), octets = wp / 8;
+        if (W % 8 == 0) {
+#pragma unroll 6
+            for (int i = threadIdx.x; i < kSub * octets; i += kThreads) {
+                const int r = i / octets, c = (i - r * octets) * 8;
+                const bool in = r < np && c < W;
+                lm::cp_async16(rows + r * ld + c, ring + (in ? (size_t)((p0 + r) % ring_rows) * W + c : 0), in);
+            }
+            lm::cp_commit();
+        } else {
+            for (int i = threadIdx.x; i < kSub * wp; i += kThreads) {
+                const int r = i / wp, c = i - r * wp;
+                rows[r * ld + c] = r < np && c < W ? ring[(size_t)((p0 + r) % ring_rows) * W + c] : __float2bfloat16_rn(0.f);
+            }
+        }
+    };
+    if (begin < end) stage(begin);
+    const int quads = wp / 4;
+#pragma unroll 8
+    for (int i = threadIdx.x; i < kMmaHeads * quads; i += kThreads) {
+        const int r = i / quads, c = (i - r * quads) * 4;
+        const float4 v = h0 + r < H ? load4(qa + (size_t)(h0 + r) * W + c, W - c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        uint2 hi, lo;
+        lm::split2(v.x, v.y, hi.x, lo.x);
+        lm::split2(v.z, v.w, hi.y, lo.y);
+        *reinterpret_cast<uint2*>(qh + r * ld + c) = hi;
+        *reinterpret_cast<uint2*>(ql + r * ld + c) = lo;
+    }
+    const int sh = threadIdx.x >> 4, sp = threadIdx.x & 15;              // this thread's (head, position) of the softmax
+    float m = -INFINITY, l = 0.f, o[PC][2][4];
+#pragma unroll
+    for (int c = 0; c < PC; ++c)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o[c][0][e] = o[c][1][e] = 0.f;
+    for (int p0 = begin; p0 < end; p0 += kSub) {
+        if (p0 != begin) {
+            __syncthreads();
+            stage(p0);
+        }
+        lm::cp_wait<0>();
+        __syncthreads();
+        float s0[4] = {}, s1[4] = {};
+        for (int k0 = warp * 16; k0 < wp; k0 += kWarps * 16) {
+            uint32_t ah[4], al[4], b[4];
+            lm::load_a(ah, qh, ld, 0, k0);
+            lm::load_a(al, ql, ld, 0, k0);
+            lm::load_b(b, rows, ld, 0, k0);
+            lm::mma(s0, ah, b[0], b[1]);
+            lm::mma(s1, ah, b[2], b[3]);
+            lm::mma(s0, al, b[0], b[1]);
+            lm::mma(s1, al, b[2], b[3]);
+        }
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            part[warp][g + (e >> 1) * 8][2 * t + (e & 1)] = s0[e];
+            part[warp][g + (e >> 1) * 8][8 + 2 * t + (e & 1)] = s1[e];
+        }
+        __syncthreads();
+        float s = 0.f;
+#pragma unroll
+        for (int w = 0; w < kWarps; ++w) s += part[w][sh][sp];
+        if (p0 + sp >= end) s = -INFINITY;
+        float mt = s;
+#pragma unroll
+        for (int x = 8; x > 0; x >>= 1) mt = fmaxf(mt, __shfl_xor_sync(0xffffffffu, mt, x));
+        const float mn = fmaxf(m, mt), corr = expf(m - mn), p = expf(s - mn);
+        float ps = p;
+#pragma unroll
+        for (int x = 8; x > 0; x >>= 1) ps += __shfl_xor_sync(0xffffffffu, ps, x);
+        l = l * corr + ps;
+        m = mn;
+        const bf16 hi = __float2bfloat16_rn(p);
+        ph[sh][sp] = hi;
+        pl[sh][sp] = __float2bfloat16_rn(p - __bfloat162float(hi));
+        if (sp == 0) corr_s[sh] = corr;
+        __syncthreads();
+        uint32_t ah[4], al[4];
+        lm::load_a(ah, &ph[0][0], kSub + 8, 0, 0);
+        lm::load_a(al, &pl[0][0], kSub + 8, 0, 0);
+        const float c0 = corr_s[g], c1 = corr_s[g + 8];
+#pragma unroll
+        for (int c = 0; c < PC; ++c) {
+            const int col = (warp + c * kWarps) * 16;
+            if (col >= wp) break;
+            uint32_t b[4];
+            lm::load_b_t(b, rows, ld, col, 0);
+#pragma unroll
+            for (int x = 0; x < 2; ++x) {
+                o[c][x][0] *= c0; o[c][x][1] *= c0;
+                o[c][x][2] *= c1; o[c][x][3] *= c1;
+                lm::mma(o[c][x], ah, b[2 * x], b[2 * x + 1]);
+                lm::mma(o[c][x], al, b[2 * x], b[2 * x + 1]);
+            }
+        }
+    }
+    const int pitch = partial_pitch(C);
+    float* dst = partial + ((size_t)blockIdx.x * H + h0) * pitch;
+#pragma unroll
+    for (int c = 0; c < PC; ++c)
+#pragma unroll
+        for (int x = 0; x < 2; ++x)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int col = (warp + c * kWarps) * 16 + 8 * x + 2 * t + (e & 1), r = g + (e >> 1) * 8;
+                if (col < C && h0 + r < H) dst[(size_t)r * pitch + col] = o[c][x][e];
+            }
+    if (sp == 0 && h0 + sh < H) {
+        dst[(size_t)sh * pitch + pitch - 2] = m;
+        dst[(size_t)sh * pitch + pitch - 1] = l;
+    }
+}
+
 // Merge of a head's partial results and its values: out[h] = W_uv[h] . (weighted latent).  CTA = (head, run of value rows).
 // Groups of threads merge different splits, four features per thread and load.
 template <class T>
 __global__ void __launch_bounds__(kThreads) latent_values_kernel(const float* __restrict__ partial, int splits, const T* __restrict__ uv, float* __restrict__ out,
                                                                  int H, int C, int E, int rows_per) {
-    rcu_kernel_entry();
     extern __shared__ __align__(16) float c_s[];        // [groups][quads * 4], the sum in group 0
     __shared__ float wgt[kMaxSplits];
     const int h = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int pitch = partial_pitch(C), quads = (C + 3) / 4, groups = max(1, kThreads / quads);
+    // the warp's first two rows of up to 1024 features are requested before the wait (weights are constant)
+    constexpr int VEC = 16 / (int)sizeof(T), kEarly = 1024 / (32 * VEC);
+    const bool vec = C % VEC == 0 && C <= 1024 && (reinterpret_cast<uintptr_t>(uv) & 15) == 0;
+    const int e0 = blockIdx.y * rows_per + warp, e1 = min(E, ((int)blockIdx.y + 1) * rows_per);
+    uint4 early[2][kEarly];
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+    if (vec) {
+#pragma unroll
+        for (int r = 0; r < 2; ++r)
+#pragma unroll
+            for (int i = 0; i < kEarly; ++i) {
+                const int e = e0 + r * kWarps, c = (lane + 32 * i) * VEC;
+                if (e < e1 && c < C) early[r][i] = ld_stream_v4(uv + ((size_t)h * E + e) * C + c);
+            }
+    }
+    asm volatile("griddepcontrol.wait;" ::: "memory");
     const float* ph = partial + (size_t)h * pitch;
     const size_t stride = (size_t)H * pitch;
     if (warp == 0) {
@@ -623,7 +785,7 @@ __global__ void __launch_bounds__(kThreads) latent_values_kernel(const float* __
     for (int i = threadIdx.x; i < groups * quads; i += kThreads) {
         const int g = i / quads, c = (i - g * quads) * 4;
         float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 8
+#pragma unroll 16
         for (int j = g; j < splits; j += groups) {
             const float4 v = *reinterpret_cast<const float4*>(ph + j * stride + c);
             s.x = fmaf(wgt[j], v.x, s.x);
@@ -640,19 +802,21 @@ __global__ void __launch_bounds__(kThreads) latent_values_kernel(const float* __
         c_s[c] = s;
     }
     __syncthreads();
-    const int e1 = min(E, ((int)blockIdx.y + 1) * rows_per);
-    constexpr int VEC = 16 / (int)sizeof(T);
-    const bool vec = C % VEC == 0 && (reinterpret_cast<uintptr_t>(uv) & 15) == 0;
-    for (int e = blockIdx.y * rows_per + warp; e < e1; e += kWarps) {
+    for (int r = 0; e0 + r * kWarps < e1; ++r) {
+        const int e = e0 + r * kWarps;
         const T* w = uv + ((size_t)h * E + e) * C;
         float acc = 0.f;
         if (vec) {
-#pragma unroll 4
-            for (int c = lane * VEC; c < C; c += 32 * VEC) {
-                const uint4 raw = *reinterpret_cast<const uint4*>(w + c);
-                const T* wv = reinterpret_cast<const T*>(&raw);
 #pragma unroll
-                for (int i = 0; i < VEC; ++i) acc = fmaf(to_f32<T>(wv[i]), c_s[c + i], acc);
+            for (int i = 0; i < kEarly; ++i) {
+                const int c = (lane + 32 * i) * VEC;
+                if (c < C) {
+                    uint4 raw = r == 0 ? early[0][i] : early[1][i];
+                    if (r > 1) raw = ld_stream_v4(w + c);
+                    const T* wv = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+                    for (int x = 0; x < VEC; ++x) acc = fmaf(to_f32<T>(wv[x]), c_s[c + x], acc);
+                }
             }
         } else {
             for (int c = lane; c < C; c += 32) acc = fmaf(to_f32<T>(w[c]), c_s[c], acc);
@@ -723,15 +887,18 @@ namespace {
 
 int latent_splits(const rcu_stack_run& r) { return (int)std::min<uint32_t>(kMaxSplits, std::max<uint32_t>(1, (std::min(r.window, r.ring_rows) + kSub - 1) / kSub)); }
 
-// Warps per team: fewest warp steps over the whole grid.  Ending a unit (reduction, epilogue) costs about an item's time,
-// and meeting the team's other warps another.
+// Warps per team.  A CTA's time is bound below by the memory system (its units' items, one after the other) and by the longest
+// chain of items a warp works through, an item taking a warp about twice as long as the memory system; ending a unit
+// (reduction, epilogue) counts as an item, and meeting the team's other warps as another.
 int plan_parts(int grid, int units, int items) {
     int best = 1;
-    long long best_cost = -1;
+    double best_cost = -1.0;
+    const double stream = (double)((units + grid - 1) / grid) * items;
     for (int parts = 1; parts <= kWarps; parts *= 2) {
         const long long teams = (long long)grid * (kWarps / parts), rounds = (units + teams - 1) / teams;
-        const long long cost = rounds * ((items + parts - 1) / parts + (parts > 1 ? 2 : 1));
-        if (best_cost < 0 || cost < best_cost) { best = parts; best_cost = cost; }
+        const double chain = 2.0 * rounds * ((items + parts - 1) / parts + (parts > 1 ? 2 : 1));
+        const double cost = std::max(stream, chain) + 0.25 * chain;
+        if (best_cost < 0.0 || cost < best_cost) { best = parts; best_cost = cost; }
     }
     return best;
 }
@@ -741,18 +908,16 @@ template <class T> rcu_status launch_rows(rcu_device* dev, RowsArgs a) {
     const bool has_b = a.kb > 0 && a.wb;
     const size_t inputs = ((size_t)padded(a.ka) + (size_t)padded(a.kb)) * 4, per_slot = (size_t)kWarps * kSlotBytes;
     const size_t most = (size_t)dev->smem_optin - 4096;
-    // ring slots: half an SM's shared memory in all where that leaves each warp two, so that the next kernel's CTA fits beside this one
-    const size_t half = 110 * 1024;
-    int slots = inputs + 1024 < half ? (int)((half - 1024 - inputs) / per_slot) : 0;
-    if (slots < 2) slots = inputs + 1024 + 3 * per_slot <= most ? 3 : 0;
-    a.slots = std::min(slots, kMaxSlots);
-    const bool blocks = sizeof(T) == 2 && a.ka % 64 == 0 && (!has_b || a.kb % 64 == 0) && a.slots > 0 &&
+    // Rings as deep as shared memory allows: bytes in flight are worth more than room for the next kernel's CTA (measured with
+    // rings held to half an SM: 414 us per token against 376 at width 2048).
+    a.slots = inputs + 1024 < most ? (int)std::min<size_t>(kMaxSlots, (most - 1024 - inputs) / per_slot) : 0;
+    const bool blocks = sizeof(T) == 2 && a.ka % 64 == 0 && (!has_b || a.kb % 64 == 0) && a.slots >= 2 &&
                         ((reinterpret_cast<uintptr_t>(a.wa) | reinterpret_cast<uintptr_t>(a.wb)) & 15) == 0;
     if (blocks) {
         const int units = (a.na + kUnit - 1) / kUnit + (a.dual ? 0 : (a.pairs + kUnit / 2 - 1) / (kUnit / 2));
         const int ia = (a.ka + kItem - 1) / kItem, ib = has_b ? (a.kb + kItem - 1) / kItem : 0;
         a.parts = plan_parts(dev->sm_count, units, a.dual ? ia + ib : std::max(ia, ib));
-        const int teams = kWarps / a.parts, grid = std::max(1, std::min(dev->sm_count, (units + teams - 1) / teams));
+        const int grid = std::max(1, std::min(dev->sm_count, units));
         CUtensorMap ma, mb;
         if (!make_block_map(&ma, a.wa, a.na, a.ka) || !make_block_map(&mb, has_b ? a.wb : a.wa, has_b ? (a.dual ? a.na : 2 * a.pairs) : a.na, has_b ? a.kb : a.ka))
             return rcu_fail(dev, RCU_ERR_CUDA, "stack: cuTensorMapEncodeTiled failed (%d x %d)", a.na, a.ka);
@@ -770,23 +935,31 @@ template <class T> rcu_status launch_rows(rcu_device* dev, RowsArgs a) {
     return RCU_OK;
 }
 
-template <class T> rcu_status launch_latent_step(rcu_device* dev, const rcu_stack* s, const rcu_stack_run& r) {
+rcu_status launch_latent_step(rcu_device* dev, const rcu_stack* s, const rcu_stack_run& r, int dt) {
     const int H = (int)r.heads, C = (int)r.kv_rank, R = (int)r.rot_dim, splits = latent_splits(r);
-    const int WP = (C + R + 7) & ~7;
-    const size_t smem = (size_t)kHeads * WP * 4 + (size_t)kSub * WP * sizeof(T);
-    const dim3 grid(splits, (H + kHeads - 1) / kHeads);
-#define RCU_LS(PC_)                                                                                                                              \
+#define RCU_LS(KERN_, GRID_, T_)                                                                                                                 \
     do {                                                                                                                                         \
-        RCU_CUDA(dev, cudaFuncSetAttribute(latent_step_kernel<T, PC_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)std::max(smem, (size_t)(48 * 1024)))); \
-        RCU_CUDA(dev, rcu_launch(dev, latent_step_kernel<T, PC_>, grid, kThreads, smem, s->qa, (const T*)r.state, (int)r.ring_rows, (int)r.window, s->d_pos, \
-                                 s->partial, H, C, R));                                                                                          \
+        RCU_CUDA(dev, cudaFuncSetAttribute(KERN_, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)std::max(smem, (size_t)(48 * 1024))));       \
+        RCU_CUDA(dev, rcu_launch(dev, KERN_, GRID_, kThreads, smem, s->qa, (const T_*)r.state, (int)r.ring_rows, (int)r.window, s->d_pos, s->partial, H, C, R)); \
     } while (0)
-    switch ((WP + 255) / 256) {
-        case 1: RCU_LS(1); break;
-        case 2: RCU_LS(2); break;
-        case 3: RCU_LS(3); break;
-        case 4: RCU_LS(4); break;
-        default: RCU_LS(5); break;
+    if (dt == RCU_BF16) {
+        const int wp = (C + R + 15) & ~15;
+        const size_t smem = (size_t)(2 * kMmaHeads + kSub) * (wp + 8) * sizeof(lm::bf16);
+        const dim3 grid(splits, (H + kMmaHeads - 1) / kMmaHeads);
+        if (wp <= 256) RCU_LS(latent_step_mma_kernel<2>, grid, lm::bf16);
+        else if (wp <= 640) RCU_LS(latent_step_mma_kernel<5>, grid, lm::bf16);
+        else RCU_LS(latent_step_mma_kernel<10>, grid, lm::bf16);
+    } else {
+        const int WP = (C + R + 7) & ~7;
+        const size_t smem = (size_t)kHeads * WP * 4 + (size_t)kSub * WP * sizeof(float);
+        const dim3 grid(splits, (H + kHeads - 1) / kHeads);
+        switch ((WP + 255) / 256) {
+            case 1: RCU_LS((latent_step_kernel<float, 1>), grid, float); break;
+            case 2: RCU_LS((latent_step_kernel<float, 2>), grid, float); break;
+            case 3: RCU_LS((latent_step_kernel<float, 3>), grid, float); break;
+            case 4: RCU_LS((latent_step_kernel<float, 4>), grid, float); break;
+            default: RCU_LS((latent_step_kernel<float, 5>), grid, float); break;
+        }
     }
 #undef RCU_LS
     RCU_LAUNCH_CHECK(dev);
@@ -844,8 +1017,8 @@ template <class T> rcu_status run_step(rcu_stack* s, const int32_t* token, float
             RCU_CUDA(dev, rcu_launch(dev, absorb_kernel<T>, dim3(H, (C + 31) / 32), kThreads, 0, s->q, (const T*)r.ukv, (const float*)r.freqs, nf, r.rot_magnitude,
                                      s->d_pos, s->qa, D, R, C, r.scale));
             RCU_LAUNCH_CHECK(dev);
-            STACK_TRY(launch_latent_step<T>(dev, s, r));
-            const int per = 32, quads = (C + 3) / 4, groups = std::max(1, kThreads / quads);
+            STACK_TRY(launch_latent_step(dev, s, r, c.weight_dt));
+            const int per = 2 * kWarps, quads = (C + 3) / 4, groups = std::max(1, kThreads / quads);
             RCU_CUDA(dev, rcu_launch(dev, latent_values_kernel<T>, dim3(H, (E + per - 1) / per), kThreads, (size_t)groups * quads * 16, s->partial, latent_splits(r),
                                      (const T*)r.ukv + (size_t)H * D * C, s->y, H, C, E, per));
             RCU_LAUNCH_CHECK(dev);
