@@ -94,7 +94,8 @@ template <class T> rcu_status launch_recurrent(rcu_device* dev, const LightningA
     if (per <= 4) rcu_launch(dev, lightning_recurrent_kernel<T, 4>, grid, 256, 0, a);
     else if (per <= 8) rcu_launch(dev, lightning_recurrent_kernel<T, 8>, grid, 256, 0, a);
     else if (per <= 16) rcu_launch(dev, lightning_recurrent_kernel<T, 16>, grid, 256, 0, a);
-    else rcu_launch(dev, lightning_recurrent_kernel<T, 32>, grid, 256, 0, a);
+    else if (per <= 32) rcu_launch(dev, lightning_recurrent_kernel<T, 32>, grid, 256, 0, a);
+    else rcu_launch(dev, lightning_recurrent_kernel<T, 64>, grid, 256, 0, a);
     RCU_LAUNCH_CHECK(dev);
     return RCU_OK;
 }
@@ -332,7 +333,7 @@ extern "C" rcu_status rcu_lightning(rcu_device* dev, const rcu_tensor* x, const 
     RCU_REQUIRE(dev, decay_pow->dt == RCU_F32 && decay_pow->rank == 2 && decay_pow->shape[0] == H && decay_pow->shape[1] >= 2,
                 "lightning: decay powers are f32 [heads, >= 2]");
     RCU_REQUIRE(dev, 2 * H * D + H * E <= pitch && t_numel(dst) == T * H * E, "lightning: rows or output do not fit heads x (dim, dim, vdim)");
-    if (D > 256 || H > 65535 || E > 65535 * 32ull || T > 0x7fffffffull) return rcu_fail(dev, RCU_ERR_UNSUPPORTED, "lightning: dim %llu (at most 256)", (unsigned long long)D);
+    if (D > 512 || H > 65535 || E > 65535 * 32ull || T > 0x7fffffffull) return rcu_fail(dev, RCU_ERR_UNSUPPORTED, "lightning: dim %llu (at most 512)", (unsigned long long)D);
     DevGuard g(dev->ordinal);
     LightningArgs a{x->data, (long long)pitch, (const float*)decay_pow->data, (int)decay_pow->shape[1], (float*)state->data, (float*)dst->data,
                     (int)T, (int)H, (int)D, (int)E};

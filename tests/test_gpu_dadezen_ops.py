@@ -135,7 +135,7 @@ def powers(decay, n=129):
 
 @pytest.mark.parametrize("dt", [F32, BF16])
 @pytest.mark.parametrize("H,D,E,decay", [(1, 1, 1, (0.5,)), (3, 24, 40, (0.02, 0.9, 0.999)), (2, 9, 13, (1.0, 0.97)), (2, 64, 64, (0.6, 0.99)),
-                                         (2, 128, 128, (0.93, 0.9995)), (1, 200, 72, (0.98,)), (2, 32, 136, (0.0, 0.9))])
+                                         (2, 128, 128, (0.93, 0.9995)), (1, 200, 72, (0.98,)), (1, 300, 20, (0.9,)), (2, 32, 136, (0.0, 0.9))])
 def test_linear_attention_in_portions(dev, dt, H, D, E, decay):
     g = rng(H * D + E)
     T = 300
