@@ -10,6 +10,8 @@
 //   chunk_out    o_i = d^(i+1) S_n^T q_i + sum_(j <= i) d^(i-j) (q_i . k_j) v_j.
 // The operands that must keep f32 accuracy (decayed keys, states, decayed scores) enter the bf16 products as value plus
 // remainder, two products each.
+#include <algorithm>
+
 #include "lm_mma.cuh"
 
 namespace {
@@ -116,6 +118,15 @@ struct ChunkArgs {
     int T, H, D, E, vec;
 };
 
+// two neighbouring elements of a row of n (e is even, and so is the row's offset where n is)
+__device__ __forceinline__ void store2(float* row, int e, int n, float x, float y) {
+    if (n % 2 == 0 && e < n) *reinterpret_cast<float2*>(row + e) = make_float2(x, y);
+    else {
+        if (e < n) row[e] = x;
+        if (e + 1 < n) row[e + 1] = y;
+    }
+}
+
 __global__ void __launch_bounds__(128) chunk_kv_kernel(const ChunkArgs a) {
     rcu_kernel_entry();
     extern __shared__ __align__(16) lm::bf16 tiles[];
@@ -129,18 +140,24 @@ __global__ void __launch_bounds__(128) chunk_kv_kernel(const ChunkArgs a) {
     lm::load_tile(vs, kLdT, v, a.pitch, kChunk, rows, min(kTile, a.E - e0), kTile, a.vec);
     const float* pw = a.decay_pow + (size_t)h * a.n_pow;
     const int kc = min(kTile, a.D - d0);
-    for (int i = threadIdx.x; i < kChunk * (kTile / 8); i += 128) {
-        const int r = i / (kTile / 8), c = (i % (kTile / 8)) * 8;
-        __align__(16) lm::bf16 in[8];
+    constexpr int kVecs = kChunk * (kTile / 8) / 128;          // 16-byte pieces of the key tile per thread, all requested first
+    __align__(16) lm::bf16 in[kVecs][8];
+#pragma unroll
+    for (int v = 0; v < kVecs; ++v) {
+        const int i = threadIdx.x + v * 128, r = i / (kTile / 8), c = (i % (kTile / 8)) * 8;
         const lm::bf16* s = k + (long long)r * a.pitch + c;
-        if (a.vec) *reinterpret_cast<uint4*>(in) = r < rows && c < kc ? *reinterpret_cast<const uint4*>(s) : make_uint4(0u, 0u, 0u, 0u);
+        if (a.vec) *reinterpret_cast<uint4*>(in[v]) = r < rows && c < kc ? *reinterpret_cast<const uint4*>(s) : make_uint4(0u, 0u, 0u, 0u);
         else
 #pragma unroll
-            for (int e = 0; e < 8; ++e) in[e] = r < rows && c + e < kc ? s[e] : __float2bfloat16_rn(0.f);
+            for (int e = 0; e < 8; ++e) in[v][e] = r < rows && c + e < kc ? s[e] : __float2bfloat16_rn(0.f);
+    }
+#pragma unroll
+    for (int v = 0; v < kVecs; ++v) {
+        const int i = threadIdx.x + v * 128, r = i / (kTile / 8), c = (i % (kTile / 8)) * 8;
         const float w = r < rows ? pw[rows - 1 - r] : 0.f;
         __align__(16) uint32_t hi[4], lo[4];
 #pragma unroll
-        for (int e = 0; e < 4; ++e) lm::split2(w * __bfloat162float(in[2 * e]), w * __bfloat162float(in[2 * e + 1]), hi[e], lo[e]);
+        for (int e = 0; e < 4; ++e) lm::split2(w * __bfloat162float(in[v][2 * e]), w * __bfloat162float(in[v][2 * e + 1]), hi[e], lo[e]);
         *reinterpret_cast<uint4*>(kh + r * kLdT + c) = *reinterpret_cast<const uint4*>(hi);
         *reinterpret_cast<uint4*>(kl + r * kLdT + c) = *reinterpret_cast<const uint4*>(lo);
     }
@@ -171,33 +188,45 @@ __global__ void __launch_bounds__(128) chunk_kv_kernel(const ChunkArgs a) {
 #pragma unroll
         for (int j = 0; j < 4; ++j)
 #pragma unroll
-            for (int q = 0; q < 4; ++q) {
-                const int d = d0 + wd + 16 * m + (lane >> 2) + (q >> 1) * 8, e = e0 + we + 8 * j + (lane & 3) * 2 + (q & 1);
-                if (d < a.D && e < a.E) U[(size_t)d * a.E + e] = acc[m][j][q];
+            for (int q = 0; q < 4; q += 2) {
+                const int d = d0 + wd + 16 * m + (lane >> 2) + (q >> 1) * 8, e = e0 + we + 8 * j + (lane & 3) * 2;
+                if (d < a.D) store2(U + (size_t)d * a.E, e, a.E, acc[m][j][q], acc[m][j][q + 1]);
             }
 }
 
+// V neighbouring state elements of one head per thread
+template <int V>
 __global__ void __launch_bounds__(256) chunk_scan_kernel(const ChunkArgs a, int chunks) {
     rcu_kernel_entry();
-    const size_t per = (size_t)a.H * a.D * a.E, i = (size_t)blockIdx.x * 256 + threadIdx.x;
+    struct alignas(4 * V) Words { uint32_t w[V]; };
+    struct alignas(4 * V) Floats { float f[V]; };
+    const size_t per = (size_t)a.H * a.D * a.E / V, i = (size_t)blockIdx.x * 256 + threadIdx.x;
     if (i >= per) return;
-    const float* pw = a.decay_pow + (i / ((size_t)a.D * a.E)) * a.n_pow;
+    const float* pw = a.decay_pow + (i * V / ((size_t)a.D * a.E)) * a.n_pow;
     const float dc = pw[kChunk], dl = pw[a.T - (chunks - 1) * kChunk];
-    float s = a.state[i];
+    Words* scratch = reinterpret_cast<Words*>(a.scratch) + i;
+    Floats s = reinterpret_cast<const Floats*>(a.state)[i];
     constexpr int kAhead = 8;                  // chunks requested before the first of them is folded in
     for (int n0 = 0; n0 < chunks; n0 += kAhead) {
-        float u[kAhead];
+        Words u[kAhead];
 #pragma unroll
-        for (int j = 0; j < kAhead; ++j) u[j] = n0 + j < chunks ? __uint_as_float(a.scratch[(size_t)(n0 + j) * per + i]) : 0.f;
+        for (int j = 0; j < kAhead; ++j)
+            if (n0 + j < chunks) u[j] = scratch[(size_t)(n0 + j) * per];
 #pragma unroll
         for (int j = 0; j < kAhead; ++j) {
             if (n0 + j >= chunks) break;
-            const lm::bf16 hi = __float2bfloat16_rn(s);
-            a.scratch[(size_t)(n0 + j) * per + i] = lm::pack(__float2bfloat16_rn(s - __bfloat162float(hi)), hi);
-            s = fmaf(n0 + j == chunks - 1 ? dl : dc, s, u[j]);
+            const float d = n0 + j == chunks - 1 ? dl : dc;
+            Words o;
+#pragma unroll
+            for (int v = 0; v < V; ++v) {
+                const lm::bf16 hi = __float2bfloat16_rn(s.f[v]);
+                o.w[v] = lm::pack(__float2bfloat16_rn(s.f[v] - __bfloat162float(hi)), hi);
+                s.f[v] = fmaf(d, s.f[v], __uint_as_float(u[j].w[v]));
+            }
+            scratch[(size_t)(n0 + j) * per] = o;
         }
     }
-    a.state[i] = s;
+    reinterpret_cast<Floats*>(a.state)[i] = s;
 }
 
 __global__ void __launch_bounds__(256) chunk_out_kernel(const ChunkArgs a) {
@@ -205,30 +234,38 @@ __global__ void __launch_bounds__(256) chunk_out_kernel(const ChunkArgs a) {
     extern __shared__ __align__(16) lm::bf16 tiles[];
     __shared__ float pw[kChunk + 1];
     const int dp = (a.D + 15) & ~15, ld = dp + 8;
-    lm::bf16 *qs = tiles, *ks = qs + kChunk * ld, *vs = ks + kChunk * ld, *sh = vs + kChunk * kLdT, *sl = sh + dp * kLdT;
+    // the state's tiles, then - in the same place - the chunk's keys and values: two CTAs fit an SM
+    lm::bf16 *qs = tiles, *sh = qs + kChunk * ld, *sl = sh + dp * kLdT, *ks = qs + kChunk * ld, *vs = ks + kChunk * ld;
     const int n = blockIdx.x, h = blockIdx.y, e0 = blockIdx.z * kTile;
     const int rows = min(kChunk, a.T - n * kChunk), ec = min(kTile, a.E - e0);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
     const lm::bf16* q = a.x + (long long)n * kChunk * a.pitch + (size_t)h * a.D;
     lm::load_tile(qs, ld, q, a.pitch, kChunk, rows, a.D, dp, a.vec);
-    lm::load_tile(ks, ld, q + (size_t)a.H * a.D, a.pitch, kChunk, rows, a.D, dp, a.vec);
-    lm::load_tile(vs, kLdT, a.x + (long long)n * kChunk * a.pitch + 2 * (size_t)a.H * a.D + (size_t)h * a.E + e0, a.pitch, kChunk, rows, ec, kTile, a.vec);
     lm::cp_commit();
     const uint32_t* S = a.scratch + ((size_t)n * a.H + h) * a.D * a.E + e0;
-    for (int i = threadIdx.x; i < dp * (kTile / 2); i += 256) {
-        const int d = i / (kTile / 2), c = (i % (kTile / 2)) * 2;
-        const uint32_t s0 = d < a.D && c < ec ? S[(size_t)d * a.E + c] : 0u, s1 = d < a.D && c + 1 < ec ? S[(size_t)d * a.E + c + 1] : 0u;
-        *reinterpret_cast<uint32_t*>(sh + d * kLdT + c) = (s0 >> 16) | (s1 & 0xffff0000u);
-        *reinterpret_cast<uint32_t*>(sl + d * kLdT + c) = (s0 & 0xffffu) | (s1 << 16);
+    if (a.E % 4 == 0) {
+#pragma unroll 8
+        for (int i = threadIdx.x; i < dp * (kTile / 4); i += 256) {
+            const int d = i / (kTile / 4), c = (i % (kTile / 4)) * 4;
+            const uint4 w = d < a.D && c < ec ? *reinterpret_cast<const uint4*>(S + (size_t)d * a.E + c) : make_uint4(0u, 0u, 0u, 0u);
+            *reinterpret_cast<uint2*>(sh + d * kLdT + c) = make_uint2((w.x >> 16) | (w.y & 0xffff0000u), (w.z >> 16) | (w.w & 0xffff0000u));
+            *reinterpret_cast<uint2*>(sl + d * kLdT + c) = make_uint2((w.x & 0xffffu) | (w.y << 16), (w.z & 0xffffu) | (w.w << 16));
+        }
+    } else {
+        for (int i = threadIdx.x; i < dp * kTile; i += 256) {
+            const int d = i / kTile, c = i % kTile;
+            const uint32_t w = d < a.D && c < ec ? S[(size_t)d * a.E + c] : 0u;
+            sh[d * kLdT + c] = __ushort_as_bfloat16((unsigned short)(w >> 16));
+            sl[d * kLdT + c] = __ushort_as_bfloat16((unsigned short)w);
+        }
     }
     for (int i = threadIdx.x; i <= kChunk; i += 256) pw[i] = a.decay_pow[(size_t)h * a.n_pow + i];
     lm::cp_wait<0>();
     __syncthreads();
     const int r0 = warp * 16;
-    if (r0 >= rows) return;
     float o[8][4] = {};
     // what the tokens before the chunk left in the state
-    for (int k0 = 0; k0 < dp; k0 += 16) {
+    for (int k0 = 0; k0 < dp && r0 < rows; k0 += 16) {
         uint32_t qa[4];
         lm::load_a(qa, qs, ld, r0, k0);
 #pragma unroll
@@ -242,6 +279,13 @@ __global__ void __launch_bounds__(256) chunk_out_kernel(const ChunkArgs a) {
             lm::mma(o[2 * j + 1], qa, bl[2], bl[3]);
         }
     }
+    __syncthreads();
+    lm::load_tile(ks, ld, q + (size_t)a.H * a.D, a.pitch, kChunk, rows, a.D, dp, a.vec);
+    lm::load_tile(vs, kLdT, a.x + (long long)n * kChunk * a.pitch + 2 * (size_t)a.H * a.D + (size_t)h * a.E + e0, a.pitch, kChunk, rows, ec, kTile, a.vec);
+    lm::cp_commit();
+    lm::cp_wait<0>();
+    __syncthreads();
+    if (r0 >= rows) return;
     const int i0 = r0 + g, i1 = i0 + 8;
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
@@ -290,15 +334,22 @@ __global__ void __launch_bounds__(256) chunk_out_kernel(const ChunkArgs a) {
 #pragma unroll
     for (int j = 0; j < 8; ++j)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const int i = e < 2 ? i0 : i1, c = 8 * j + 2 * t + (e & 1);
-            if (i < rows && c < ec) out[(size_t)i * a.H * a.E + c] = o[j][e];
+        for (int e = 0; e < 4; e += 2) {
+            const int i = e < 2 ? i0 : i1, c = 8 * j + 2 * t;
+            if (i >= rows) continue;
+            float* row = out + (size_t)i * a.H * a.E;
+            if (a.E % 2 == 0) {
+                store2(row, c, ec, o[j][e], o[j][e + 1]);
+            } else {
+                if (c < ec) row[c] = o[j][e];
+                if (c + 1 < ec) row[c + 1] = o[j][e + 1];
+            }
         }
 }
 
 size_t chunk_out_smem(int D) {
     const size_t dp = (D + 15) & ~15;
-    return (2 * kChunk * (dp + 8) + kChunk * kLdT + 2 * dp * kLdT) * sizeof(lm::bf16);
+    return (kChunk * (dp + 8) + std::max(kChunk * (dp + 8) + kChunk * kLdT, 2 * dp * kLdT)) * sizeof(lm::bf16);
 }
 
 rcu_status launch_chunks(rcu_device* dev, const LightningArgs& l) {
@@ -313,7 +364,10 @@ rcu_status launch_chunks(rcu_device* dev, const LightningArgs& l) {
     RCU_CUDA(dev, cudaFuncSetAttribute(chunk_kv_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_kv));
     RCU_CUDA(dev, cudaFuncSetAttribute(chunk_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem_out));
     rcu_launch(dev, chunk_kv_kernel, dim3(chunks, l.H, td * te), 128, smem_kv, a);
-    rcu_launch(dev, chunk_scan_kernel, (unsigned)(((size_t)l.H * l.D * l.E + 255) / 256), 256, 0, a, chunks);
+    const size_t elems = (size_t)l.H * l.D * l.E;
+    if ((size_t)l.D * l.E % 4 == 0 && (reinterpret_cast<uintptr_t>(l.state) & 15) == 0)
+        rcu_launch(dev, chunk_scan_kernel<4>, (unsigned)((elems / 4 + 255) / 256), 256, 0, a, chunks);
+    else rcu_launch(dev, chunk_scan_kernel<1>, (unsigned)((elems + 255) / 256), 256, 0, a, chunks);
     rcu_launch(dev, chunk_out_kernel, dim3(chunks, l.H, te), 256, smem_out, a);
     rcu_free(dev, scratch);                    // the pool reuses blocks in stream order
     dev->launches += 2;

@@ -45,9 +45,10 @@ __device__ __forceinline__ uint32_t pack(bf16 lo, bf16 hi) {
 }
 // two f32 values as packed bf16 pairs: their roundings and the roundings of what those left over
 __device__ __forceinline__ void split2(float x, float y, uint32_t& value, uint32_t& rest) {
-    const bf16 xh = __float2bfloat16_rn(x), yh = __float2bfloat16_rn(y);
-    value = pack(xh, yh);
-    rest = pack(__float2bfloat16_rn(x - __bfloat162float(xh)), __float2bfloat16_rn(y - __bfloat162float(yh)));
+    const __nv_bfloat162 v = __floats2bfloat162_rn(x, y);
+    value = *reinterpret_cast<const uint32_t*>(&v);
+    const __nv_bfloat162 r = __floats2bfloat162_rn(x - __uint_as_float(value << 16), y - __uint_as_float(value & 0xffff0000u));
+    rest = *reinterpret_cast<const uint32_t*>(&r);
 }
 
 __device__ __forceinline__ void cp_async16(void* dst, const void* src, bool valid) {
