@@ -4,8 +4,10 @@
 //   rcu_latent_append   normalises and rotates the block's latents, keeps the last `ring` of them in the layer's ring
 //                       (row of position p: p mod ring) and lays out the rows the block can see;
 //   rcu_window_attention  softmax attention of the block's queries over those rows, keys and values expanded from the
-//                       latents by one Linear before the call.  bf16 blocks run on the tensor cores, f32 ones in FFMA.
+//                       latents by one Linear before the call.  bf16 blocks run on the tensor cores (256 tokens and more: window_tc.cu,
+//                       fewer, or sizes it does not take: below), f32 ones in FFMA.
 #include "lm_mma.cuh"
+#include "window.cuh"
 
 namespace {
 
@@ -70,14 +72,6 @@ rcu_status launch_append(rcu_device* dev, const AppendArgs& a, void* ring, void*
     RCU_LAUNCH_CHECK(dev);
     return RCU_OK;
 }
-
-struct WindowArgs {
-    const void *q, *kv, *shared;
-    void* out;
-    long long shared_pitch;
-    int T, L, H, D, R, E, window;     // D: own key features of a head, R: shared ones (a query has D + R)
-    float scale;
-};
 
 // A warp per (token, head): scores 32 keys at a time, one key per lane, online softmax in f32; the weighted sum of the
 // values runs over lanes = value columns.
@@ -368,7 +362,8 @@ rcu_status rcu_window_attention(rcu_device* dev, const rcu_tensor* q, const rcu_
     WindowArgs a{q->data, kv->data, (const char*)shared->data + (size_t)shared_col * dt_esize(shared->dt), dst->data, (long long)shared->shape[1], (int)T,
                  (int)L, (int)H, (int)(q->shape[2] - R), (int)R, (int)vdim, (int)(window < L ? window : L), scale};
     if (q->dt == RCU_F32) return launch_window<float>(dev, a);
-    const rcu_status st = launch_window_mma(dev, a);
+    rcu_status st = rcu_window_tc(dev, a);
+    if (st == RCU_ERR_UNSUPPORTED) st = launch_window_mma(dev, a);
     return st == RCU_ERR_UNSUPPORTED ? launch_window<__nv_bfloat16>(dev, a) : st;
 }
 

@@ -76,6 +76,35 @@ __device__ __forceinline__ void tmem_ld_32x32(uint32_t taddr, float* v) {
     for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]);
 }
 
+// 32 registers per thread -> 32 lanes x 32 columns of tensor memory
+__device__ __forceinline__ void tmem_st_32x32(uint32_t taddr, const uint32_t* r) {
+    asm volatile(
+        "tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], "
+        "{%1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16, "
+        "%17, %18, %19, %20, %21, %22, %23, %24, %25, %26, %27, %28, %29, %30, %31, %32};" ::"r"(taddr),
+        "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]),
+        "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]), "r"(r[16]), "r"(r[17]), "r"(r[18]), "r"(r[19]), "r"(r[20]), "r"(r[21]), "r"(r[22]),
+        "r"(r[23]), "r"(r[24]), "r"(r[25]), "r"(r[26]), "r"(r[27]), "r"(r[28]), "r"(r[29]), "r"(r[30]), "r"(r[31])
+        : "memory");
+    asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
+}
+// The same product with the A operand in tensor memory (a row per lane, two 16-bit elements of K per column)
+__device__ __forceinline__ void umma_f16_ta(uint32_t tmem_d, uint32_t tmem_a, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
+    asm volatile(
+        "{\n\t.reg .pred p;\n\t"
+        "setp.ne.b32 p, %4, 0;\n\t"
+        "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t}"
+        ::"r"(tmem_d), "r"(tmem_a), "l"(bdesc), "r"(idesc), "r"(accumulate)
+        : "memory");
+}
+// Descriptor of a 128-byte-swizzled operand stored with its M / N dimension contiguous: 64 elements per 128-byte line, one line
+// per k, 8-line groups 1024 bytes apart (SBO), 64-element blocks `block_bytes` apart (LBO).  The instruction descriptor then
+// has the operand's transpose bit set (bit 16 for B).
+__device__ __forceinline__ uint64_t umma_desc_sw128_mn(const void* smem_ptr, uint32_t block_bytes) {
+    const uint32_t addr = smem_u32(smem_ptr);
+    return (uint64_t)((addr & 0x3FFFF) >> 4) | (uint64_t)(block_bytes >> 4) << 16 | (uint64_t)(1024 >> 4) << 32 | (uint64_t)1 << 46 | (uint64_t)2 << 61;
+}
+
 // What the epilogue of a tensor-core GEMM does with an accumulator: Out = f16 / bf16: round(acc + bias);
 // Out = f32: residual + alpha * (acc + bias), the residual stream of a model that keeps it in 32 bits
 // (`resid` may be the output itself: every element is read by the thread that writes it).

@@ -201,7 +201,7 @@ def test_latent_ring_and_window(dev, dt, H, D, R, E, C, window):
 def test_window_edges_show_a_single_loud_key(dev, dt, window):
     """One key scores far above all others and its value is unique: queries up to window - 1 rows later return that value, the
     query `window` rows later does not."""
-    T, H, D, R, E, at = 400, 2, 16, 8, 16, 150
+    T, H, D, R, E, at = 640, 2, 16, 8, 16, 350
     g = rng(window)
     q = np.abs(g.standard_normal((T, H, D + R))) + 0.5
     k = 0.05 * g.standard_normal((T, H * D + H * E))
