@@ -36,10 +36,20 @@ __global__ void __launch_bounds__(128) latent_window_kernel(const AppendArgs a, 
         return;
     }
     const float* x = a.x + (long long)(r - old) * a.pitch;
+    constexpr int kKept = 16;              // elements per lane kept in registers between the two passes
+    float v[kKept];
     float s = 0.f;
-    for (int j = lane; j < a.C; j += 32) s = fmaf(x[j], x[j], s);
+#pragma unroll
+    for (int i = 0; i < kKept; ++i) {
+        v[i] = lane + 32 * i < a.C ? x[lane + 32 * i] : 0.f;
+        s = fmaf(v[i], v[i], s);
+    }
+    for (int j = lane + 32 * kKept; j < a.C; j += 32) s = fmaf(x[j], x[j], s);
     const float rstd = 1.0f / sqrtf(warp_sum(s) / (float)a.C + a.eps);
-    for (int j = lane; j < a.C; j += 32) orow[j] = from_f32<O>(x[j] * rstd * a.scale[j]);
+#pragma unroll
+    for (int i = 0; i < kKept; ++i)
+        if (lane + 32 * i < a.C) orow[lane + 32 * i] = from_f32<O>(v[i] * rstd * a.scale[lane + 32 * i]);
+    for (int j = lane + 32 * kKept; j < a.C; j += 32) orow[j] = from_f32<O>(x[j] * rstd * a.scale[j]);
     const float* kr = x + a.C;
     const uint32_t p = a.pos + (uint32_t)(r - old);
     for (int i = lane; i < a.pairs; i += 32) {
@@ -60,6 +70,7 @@ __global__ void __launch_bounds__(128) latent_store_kernel(const O* __restrict__
     if (i >= n) return;
     const O* src = rows + (size_t)(L - n + i) * W;
     O* dst = ring + (size_t)((end - (uint32_t)(n - i)) % (uint32_t)ring_rows) * W;
+#pragma unroll 8
     for (int j = lane; j < W; j += 32) dst[j] = src[j];
 }
 

@@ -1,4 +1,4 @@
-// Windowed attention of a long bf16 block on the 5th-generation tensor cores (tcgen05); the contract is that of
+// Windowed attention of a long bf16 block on the 5th-generation tensor cores (tcgen05), behind the interface of
 // rcu_window_attention (latent_attention.cu), which sends blocks of at least 256 tokens here.
 //
 // CTA = 256 queries of one head, in two tiles of 128 that take turns: while the softmax warps of one tile work, the tensor core

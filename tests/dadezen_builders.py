@@ -102,7 +102,7 @@ CONFIGS = {
                              latent(2, 32, 16, 16, 40, 56, 5, 0.15, base=500.0, ff=48), lightning(2, 16, 16, (0.75, 0.97))], loop=(1, 3, 2)),
     "odd": config(45, 53, [latent(3, 5, 6, 7, 19, 21, 11, 0.3, dims=4, scaling=YARN), lightning(1, 9, 13, (0.95,), ff=31),
                            latent(1, 8, 2, 9, 10, 12, 1, 0.5, ff=17)], loop=(0, 1, 3), mult=1.0),
-    "plain": config(64, 70, [lightning(4, 32, 32, (0.5, 0.8, 0.99, 1.0), ff=96), latent(4, 32, 32, 32, 64, 96, 70, 0.125, scaling=YARN, ff=96)], mult=0.4),
+    "plain": config(64, 70, [lightning(4, 32, 32, (0.5, 0.8, 0.99, 1.0), ff=96), latent(3, 40, 24, 48, 64, 96, 70, 0.11, scaling=YARN, ff=96)], mult=0.4),
     "wide": config(160, 130, [latent(3, 128, 64, 128, 96, 144, 130, 0.07, base=50000.0, dims=64, scaling=YARN, ff=200),
                               lightning(2, 128, 128, (0.9, 0.99), ff=256)], loop=(1, 2, 2)),
 }
