@@ -217,16 +217,29 @@ rcu_status rcu_conv1d(rcu_device* dev, const rcu_tensor* x, const rcu_tensor* w,
  * No counterpart in the reference, whose models keep activations in one dtype between ops (ratchet-nn/src/norm.rs:37-69).
  * The residual stream, norms, gates, attention scores and recurrent states are f32; matrix products take bf16 or f16
  * operands (or f32: then everything is true f32). */
-/* dst[M, N] = resid + alpha * f(x[:, x_col : x_col + K] . w[N, K]^T + bias): x's last dimension may be wider than K; f is silu on
- * the first silu_cols columns and the identity on the others.  w and x have one float dtype; dst has it too (resid NULL, alpha 1) or is F32.  bias [N] in dst's dtype, resid F32 (may be dst);
- * both nullable. */
-rcu_status rcu_linear(rcu_device* dev, const rcu_tensor* w, const rcu_tensor* x, uint32_t x_col, const rcu_tensor* bias, uint32_t silu_cols,
-                      const rcu_tensor* resid, float alpha, rcu_tensor* dst);
-/* LayerNorm without bias / RMSNorm over columns [x_col, x_col + N) of f32 rows (N = scale's length), statistics in f32 (the
- * variance from the deviations), times sigmoid of columns [gate_col, gate_col + N) of `gate` (nullable, dst's dtype).  dst
- * [rows, N] in any float dtype. */
-rcu_status rcu_norm_rows(rcu_device* dev, int kind, const rcu_tensor* x, uint32_t x_col, const rcu_tensor* scale, const rcu_tensor* gate,
-                         uint32_t gate_col, float eps, rcu_tensor* dst);
+typedef enum {
+    RCU_ACT_NONE = 0,
+    RCU_ACT_SILU = 1,
+    RCU_ACT_RELU_SQUARED = 2,   /* max(z, 0)^2 */
+    RCU_ACT_SOFTCAP = 3         /* p tanh(z / p), p = act_param > 0 */
+} rcu_linear_act;
+/* dst[M, N] = resid + alpha * f(x[:, x_col : x_col + K] . w[N, K]^T + bias): x's last dimension may be wider than K; f is `act`
+ * (rcu_linear_act) on the first act_cols columns and the identity on the others.  w and x have one float dtype; dst has it too
+ * (resid NULL, alpha 1) or is F32.  bias [N] in dst's dtype, resid F32 (may be dst); both nullable. */
+rcu_status rcu_linear(rcu_device* dev, const rcu_tensor* w, const rcu_tensor* x, uint32_t x_col, const rcu_tensor* bias, int act,
+                      uint32_t act_cols, float act_param, const rcu_tensor* resid, float alpha, rcu_tensor* dst);
+/* LayerNorm / RMSNorm over columns [x_col, x_col + N) of f32 rows (N = scale's length), statistics in f32 (the variance from the
+ * deviations), plus `shift` F32 [N] (nullable), times sigmoid of columns [gate_col, gate_col + N) of `gate` (nullable, dst's
+ * dtype).  dst [rows, N] in any float dtype. */
+rcu_status rcu_norm_rows(rcu_device* dev, int kind, const rcu_tensor* x, uint32_t x_col, const rcu_tensor* scale, const rcu_tensor* shift,
+                         const rcu_tensor* gate, uint32_t gate_col, float eps, rcu_tensor* dst);
+/* A residual stream as rows of W f32 values, followed - when `copy_dt` is BF16 - by the same values rounded to bf16 as operands of the
+ * next matrix product ((W + 1) / 2 more words; rcu_linear reads them through a bf16 view of the rows at column 2 W).
+ * rcu_stream_rows makes such rows from x [T, W] (F32 or BF16); rcu_post_norm adds a normalised sublayer output to them:
+ * dst = x + LayerNorm(y) * scale + shift, y F32 [T, W].  dst may be x. */
+rcu_status rcu_stream_rows(rcu_device* dev, const rcu_tensor* x, int32_t copy_dt, rcu_tensor* dst);
+rcu_status rcu_post_norm(rcu_device* dev, const rcu_tensor* x, const rcu_tensor* y, const rcu_tensor* scale, const rcu_tensor* shift, float eps,
+                         rcu_tensor* dst);
 /* Gated feed-forward activation: x [.., 2F] holds gate then up, dst [.., F] = act(gate) * up; act is RCU_GELU (tanh form) or
  * RCU_SILU, evaluated in f32. */
 rcu_status rcu_glu(rcu_device* dev, int act, const rcu_tensor* x, rcu_tensor* dst);
@@ -239,6 +252,18 @@ rcu_status rcu_rotary_frequencies(uint32_t dims, double base, double factor, dou
 /* Rotation of interleaved pairs (first + 2i, first + 2i + 1) of every head by position * freqs[i]: x [tokens, heads, dim], token
  * t at `position` + t, freqs F32 [2, pairs] (value and remainder).  dst may alias x.  (rcu_rope rotates half-split pairs.) */
 rcu_status rcu_rotary(rcu_device* dev, const rcu_tensor* x, uint32_t first, const rcu_tensor* freqs, float magnitude, uint32_t position, rcu_tensor* dst);
+/* cos and sin (times magnitude) of the pairs' angles at positions position .. position + T - 1, evaluated in double: dst F32 [T, 2 pairs],
+ * (cos, sin) of a pair side by side. */
+rcu_status rcu_rotary_angles(rcu_device* dev, const rcu_tensor* freqs, float magnitude, uint32_t position, rcu_tensor* dst);
+/* RMSNorm of every head (scale F32 [dim], shared by the heads) of columns [x_col, x_col + heads * dim) of the rows x, then the rotation of
+ * its leading interleaved pairs by `angles` (rcu_rotary_angles): dst [T, heads, dim] in x's dtype (F32 or BF16). */
+rcu_status rcu_norm_rotary(rcu_device* dev, const rcu_tensor* x, uint32_t x_col, const rcu_tensor* scale, float eps, const rcu_tensor* angles, rcu_tensor* dst);
+/* Keys and values of a block into a cache of kv_heads heads: columns of x from x_col on hold every head's keys, then its values; keys are
+ * normed and rotated as in rcu_norm_rotary.  `ring` [ring rows, kv_heads * (dim + vdim)] keeps position p in row p mod ring rows;
+ * dst [L, kv_heads * (dim + vdim)] receives the L rows the block sees: L - T older ones from the ring, then the block's T.  The block's
+ * last `keep` rows go into the ring.  angles [T, 2 pairs] as above, dim = scale's length. */
+rcu_status rcu_kv_append(rcu_device* dev, const rcu_tensor* x, uint32_t x_col, uint32_t kv_heads, const rcu_tensor* scale, float eps, const rcu_tensor* angles,
+                         uint32_t position, uint32_t keep, rcu_tensor* ring, rcu_tensor* dst);
 /* Linear attention with a fixed decay per head: S <- d S + k v^T, o = S^T q over the rows of x, whose columns are q [H, D], k
  * [H, D], v [H, E] (further columns are ignored).  decay_pow F32 [H, n >= 2]: d^0, d^1, ... (with 129 of them blocks of bf16
  * rows run in chunks of 128 tokens); state F32 [H, D, E], updated in place; dst F32 [tokens, H * E]. */
@@ -253,6 +278,14 @@ rcu_status rcu_latent_append(rcu_device* dev, const rcu_tensor* x, uint32_t x_co
  * L - T + i of the keys and sees itself and the window - 1 rows before it.  dst [T, H * vdim]. */
 rcu_status rcu_window_attention(rcu_device* dev, const rcu_tensor* q, const rcu_tensor* kv, const rcu_tensor* shared, uint32_t shared_col, uint32_t vdim,
                                 uint32_t window, float scale, rcu_tensor* dst);
+
+/* Softmax attention of grouped heads: q [T, H, dim], kv [L, kv_heads * (dim + vdim)] as rcu_kv_append lays it out; query head h reads
+ * key / value head h / (H / kv_heads).  Query i is row L - T + i of the keys and sees itself and, of the rows before it,
+ *   chunk > 0: those whose position lies in the same run of `chunk` positions (row 0 is position `position`);
+ *   else       the window - 1 nearest (window 0: all).
+ * sink F32 [H] (nullable): exp(sink[h]) joins the denominator.  dst [T, H * vdim]. */
+rcu_status rcu_grouped_attention(rcu_device* dev, const rcu_tensor* q, const rcu_tensor* kv, const rcu_tensor* sink, uint32_t kv_heads, uint32_t vdim,
+                                 uint32_t window, uint32_t chunk, uint32_t position, float scale, rcu_tensor* dst);
 
 /* ------------------------------------------------------------------ lazy tensor graph (tensor.rs)
  * rcu_lazy is ratchet-core's `Tensor` (tensor.rs:45-47): a reference-counted node of a lazy DAG.
@@ -299,12 +332,22 @@ rcu_status rcu_lazy_cache(rcu_lazy* cache, rcu_lazy* src, uint32_t dim, uint32_t
 rcu_status rcu_lazy_index_write(rcu_lazy* dst, rcu_lazy* src, const uint64_t* start, rcu_lazy** out);
 
 /* The ops of models with a 32-bit residual stream as nodes (arguments as their eager forms; nullable handles are NULL).
- * rcu_lazy_linear writes into `resid` when it is its sole owner; rcu_lazy_lightning and rcu_lazy_latent_append update their
- * state / ring as a side effect, as rcu_lazy_cache does. */
-rcu_status rcu_lazy_linear(rcu_lazy* w, rcu_lazy* x, uint32_t x_col, rcu_lazy* bias, uint32_t silu_cols, rcu_lazy* resid, float alpha,
-                           int32_t dst_dt, rcu_lazy** out);
-rcu_status rcu_lazy_norm_rows(int kind, rcu_lazy* x, uint32_t x_col, rcu_lazy* scale, rcu_lazy* gate, uint32_t gate_col, float eps, int32_t dst_dt,
-                              rcu_lazy** out);
+ * rcu_lazy_linear writes into `resid` and rcu_lazy_post_norm into x when they are its sole owner; rcu_lazy_lightning,
+ * rcu_lazy_latent_append and rcu_lazy_kv_append update their state / ring as a side effect, as rcu_lazy_cache does. */
+rcu_status rcu_lazy_linear(rcu_lazy* w, rcu_lazy* x, uint32_t x_col, rcu_lazy* bias, int act, uint32_t act_cols, float act_param,
+                           rcu_lazy* resid, float alpha, int32_t dst_dt, rcu_lazy** out);
+rcu_status rcu_lazy_norm_rows(int kind, rcu_lazy* x, uint32_t x_col, rcu_lazy* scale, rcu_lazy* shift, rcu_lazy* gate, uint32_t gate_col, float eps,
+                              int32_t dst_dt, rcu_lazy** out);
+rcu_status rcu_lazy_stream_rows(rcu_lazy* x, int32_t copy_dt, rcu_lazy** out);
+rcu_status rcu_lazy_post_norm(rcu_lazy* x, rcu_lazy* y, rcu_lazy* scale, rcu_lazy* shift, float eps, rcu_lazy** out);
+/* x's bytes as elements of `dt`: the last dimension scales with the element size.  A view: no kernel, no copy. */
+rcu_status rcu_lazy_bitcast(rcu_lazy* x, int32_t dt, rcu_lazy** out);
+rcu_status rcu_lazy_rotary_angles(rcu_lazy* freqs, float magnitude, uint32_t position, uint32_t tokens, rcu_lazy** out);
+rcu_status rcu_lazy_norm_rotary(rcu_lazy* x, uint32_t x_col, uint32_t heads, rcu_lazy* scale, float eps, rcu_lazy* angles, rcu_lazy** out);
+rcu_status rcu_lazy_kv_append(rcu_lazy* x, uint32_t x_col, uint32_t kv_heads, rcu_lazy* scale, float eps, rcu_lazy* angles, uint32_t position,
+                              uint32_t keep, rcu_lazy* ring, uint32_t rows, rcu_lazy** out);
+rcu_status rcu_lazy_grouped_attention(rcu_lazy* q, rcu_lazy* kv, rcu_lazy* sink, uint32_t kv_heads, uint32_t vdim, uint32_t window, uint32_t chunk,
+                                      uint32_t position, float scale, rcu_lazy** out);
 rcu_status rcu_lazy_glu(int act, rcu_lazy* x, rcu_lazy** out);
 rcu_status rcu_lazy_rotary(rcu_lazy* x, uint32_t first, rcu_lazy* freqs, float magnitude, uint32_t position, rcu_lazy** out);
 rcu_status rcu_lazy_lightning(rcu_lazy* x, rcu_lazy* decay_pow, rcu_lazy* state, rcu_lazy** out);
@@ -416,39 +459,53 @@ rcu_status rcu_attn_decode_static(rcu_device* dev, const void* qkv, void* k_cach
                                   float rope_base, uint32_t position, void* out);
 
 /* ------------------------------------------------------------------ fused decode step of a layer stack
- * The batch-1 step of models built from parallel-residual layers x <- x + m (mixer(norm1 x) + ff(norm2 x)) (LayerNorm without bias,
- * gelu-gated feed-forward) whose mixers are linear attention (rcu_lightning) or latent attention with a sliding window
- * (rcu_latent_append, rcu_window_attention): three or six kernels per layer run, replayed from a CUDA graph.  No counterpart in
- * the reference.  Runs are listed in execution order; a layer that is run several times appears once per run, each with a state of
+ * The batch-1 step of two kinds of layer stacks, replayed from a CUDA graph:
+ *   RCU_LAYER_PARALLEL   x <- x + m (mixer(norm1 x) + ff(norm2 x)), LayerNorm without bias, gelu-gated feed-forward;
+ *   RCU_LAYER_POST_NORM  x <- x + norm1(mixer x), then x <- x + norm2(ff x), norms with scale and shift (a factor per channel behind
+ *                        a norm is part of both), feed-forward down . max(up . x, 0)^2.
+ * Mixers: linear attention (rcu_lightning), latent attention with a sliding window (rcu_latent_append, rcu_window_attention), or
+ * attention of grouped heads with a window or chunks and an optional sink (rcu_kv_append, rcu_grouped_attention).  No counterpart
+ * in the reference.  Runs are listed in execution order; a layer that is run several times appears once per run, each with a state of
  * its own.  Weights are weight_dt (BF16 or F32), norm scales, biases, decays and frequencies F32, activations f32.  All
  * pointers are device memory owned by the caller and must outlive the stack. */
 typedef struct rcu_stack rcu_stack;
-typedef enum { RCU_MIXER_LIGHTNING = 0, RCU_MIXER_LATENT = 1 } rcu_mixer_kind;
+typedef enum { RCU_MIXER_LIGHTNING = 0, RCU_MIXER_LATENT = 1, RCU_MIXER_GROUPED = 2 } rcu_mixer_kind;
+typedef enum { RCU_LAYER_PARALLEL = 0, RCU_LAYER_POST_NORM = 1 } rcu_layer_kind;
 typedef struct {
     uint32_t width, vocab, n_runs;
-    float eps, residual_mult;
+    float eps, residual_mult;     /* residual_mult: parallel layers */
+    float logit_softcap;          /* > 0: logits <- cap tanh(logits / cap) */
     int32_t weight_dt;
+    int32_t layer;                /* rcu_layer_kind */
+    const void* final_shift;      /* F32 [width], nullable: added behind the final norm's scale */
 } rcu_stack_config;
 typedef struct {
     int32_t mixer;           /* rcu_mixer_kind */
     uint32_t heads, dim, vdim, ff;   /* ff 0: no feed-forward */
-    uint32_t q_rank, kv_rank, rot_dim, rot_pairs, window, ring_rows;   /* latent mixer */
+    uint32_t q_rank, kv_rank, rot_dim, rot_pairs, window, ring_rows;   /* latent mixer; the last three: grouped too (window 0: none) */
+    uint32_t kv_heads, chunk;        /* grouped mixer; chunk > 0 instead of a window */
     float scale, rot_magnitude;
     const void* enter;       /* nullable [width, 2 width]: x <- enter . [x; embedding output] + enter_bias before this run */
     const void* enter_bias;  /* F32 [width] */
     const void* norm1;       /* F32 [width] */
     const void* norm2;
-    const void* mix_in;      /* lightning: q, k, v, gate rows; latent: query-latent, latent, rotated-key rows */
-    const void* mix_norm;    /* F32: lightning [heads * vdim], latent [q_rank] */
-    const void* kv_norm;     /* F32 [kv_rank] */
+    const void* norm1_shift; /* F32 [width]: post-norm layers */
+    const void* norm2_shift;
+    const void* mix_in;      /* lightning: q, k, v, gate rows; latent: query-latent, latent, rotated-key rows; grouped: q, k, v rows */
+    const void* mix_bias;    /* F32, grouped: bias of the q, k, v rows (nullable) */
+    const void* mix_norm;    /* F32: lightning [heads * vdim], latent [q_rank], grouped: query norm [dim] */
+    const void* kv_norm;     /* F32: latent [kv_rank], grouped: key norm [dim] */
+    const void* sink;        /* F32 [heads], grouped, nullable */
     const void* uq;          /* [heads * (dim + rot_dim), q_rank] */
     const void* ukv;         /* key rows [heads * dim, kv_rank], then value rows [heads * vdim, kv_rank] */
     const void* freqs;       /* F32 [2, rot_pairs] */
     const void* decay;       /* F32 [heads] */
     const void* out;         /* [width, heads * vdim] */
-    const void* gate_up;     /* [2 ff, width]: gate rows, then up rows */
+    const void* out_bias;    /* F32 [width], grouped, nullable */
+    const void* gate_up;     /* [2 ff, width]: gate rows, then up rows; post-norm layers: up [ff, width] */
     const void* down;        /* [width, ff] */
-    void* state;             /* lightning: F32 [heads, dim, vdim]; latent: ring [ring_rows, kv_rank + rot_dim] in weight_dt */
+    void* state;             /* lightning: F32 [heads, dim, vdim]; latent: ring [ring_rows, kv_rank + rot_dim], grouped: ring
+                              * [ring_rows, kv_heads * (dim + vdim)], in weight_dt */
 } rcu_stack_run;
 rcu_status rcu_stack_create(rcu_device* dev, const rcu_stack_config* cfg, const rcu_stack_run* runs, const void* embed, const void* final_norm,
                             const void* head, rcu_stack** out);

@@ -5,8 +5,9 @@ scheduled through the lazy ``Tensor`` API exactly as the reference schedules the
 * the Phi-2 MLP block inside its parallel-residual layer (phi2/mlp.rs:13-15, phi2/model.rs:78-89),
 * the Whisper encoder (whisper/{encoder,residual_block,mha,mlp}.rs);
 
-and one decoder the reference does not have, Dadezen: parallel layers over linear attention and windowed latent
-attention, with a loop of layers that runs several times.
+and two decoders the reference does not have: Dadezen - parallel layers over linear attention and windowed latent
+attention, with a loop of layers that runs several times - and Mefesun - norms on the sublayers' outputs, grouped heads
+that attend inside chunks of positions, layers that share weights.
 
 They only call ``Tensor`` builder methods, as ``Module::schedule`` does in the reference; no device
 code lives here.
@@ -16,7 +17,7 @@ from __future__ import annotations
 from typing import List, Optional
 
 from . import capi
-from .nn import GatedMLP, RotaryTable, SequenceState, StreamNorm
+from .nn import GatedMLP, PostNorm, RotaryTable, SequenceState, SquaredReluMLP, StreamNorm
 from .nn import KVCache, KVEntry, LayerNorm, Linear, RMSNorm, RotaryEmbedding, Embedding
 
 
@@ -198,7 +199,7 @@ class LightningMixer:
 
     def schedule(self, h, resid, alpha: float, state, position: int):
         qkv = self.heads * (2 * self.dim + self.vdim)
-        rows = self.proj.linear(h, silu_cols=qkv)
+        rows = self.proj.linear(h, act="silu", act_cols=qkv)
         y = self.norm.schedule(rows.lightning(self.decay_pow, state), gate=rows, gate_col=qkv)
         return self.out.linear(y, resid=resid, alpha=alpha, dt=capi.F32)
 
@@ -267,3 +268,66 @@ class Dadezen:
         if want is None:
             return x
         return self.head.linear(self.norm.schedule(x.index_select(want, 0)), dt=capi.F32)
+
+
+# ---------------------------------------------------------------------------------------- Mefesun
+class GroupedMixer:
+    """Softmax attention of grouped heads inside chunks of positions (or a window, or over everything), with a norm per head, rotation and
+    a sink.  ``qkv`` stacks the query, key and value rows (``qkv_bias`` in the operands' dtype for a block's product, ``qkv_bias_f32``
+    for the fused step, which adds it in f32), ``out`` maps to an f32 sublayer output."""
+
+    def __init__(self, qkv, qkv_bias, qkv_bias_f32, q_norm, k_norm, rot: RotaryTable, sink, out, out_bias, eps: float, heads: int, kv_heads: int, dim: int,
+                 vdim: int, scale: float, window: int = 0, chunk: int = 0):
+        self.qkv, self.qkv_bias, self.qkv_bias_f32, self.q_norm, self.k_norm = qkv, qkv_bias, qkv_bias_f32, q_norm, k_norm
+        self.rot, self.sink, self.out, self.out_bias = rot, sink, out, out_bias
+        self.eps, self.heads, self.kv_heads, self.dim, self.vdim, self.scale, self.window, self.chunk = eps, heads, kv_heads, dim, vdim, scale, window, chunk
+
+    def seen_before(self, position: int) -> int:
+        """Cached positions that a token at `position` sees."""
+        if self.chunk:
+            return position % self.chunk
+        return min(position, self.window - 1) if self.window else position
+
+    def schedule(self, h, col: int, angles, ring, position: int):
+        tokens = h.shape()[0]
+        rows = self.qkv.linear(h, bias=self.qkv_bias, x_col=col)
+        q = rows.norm_rotary(self.heads, self.q_norm, self.eps, angles)
+        old = self.seen_before(position)
+        keep = min(tokens, self.seen_before(position + tokens))         # rows that later tokens can see
+        kv = rows.kv_append(self.kv_heads, self.k_norm, self.eps, angles, position, keep, ring, old + tokens, col=self.heads * self.dim)
+        o = q.grouped_attention(kv, self.kv_heads, self.vdim, self.scale, self.sink, self.window, self.chunk, position - old)
+        return self.out.linear(o, bias=self.out_bias, dt=capi.F32)
+
+
+class PostNormLayer:
+    """x <- x + norm1(mixer x), x <- x + norm2(mlp x) on stream rows; no mlp: the mixer alone."""
+
+    def __init__(self, norm1: PostNorm, mixer: GroupedMixer, norm2: Optional[PostNorm], mlp: Optional[SquaredReluMLP]):
+        self.norm1, self.mixer, self.norm2, self.mlp = norm1, mixer, norm2, mlp
+
+    def schedule(self, x, angles, state, position: int):
+        x = self.norm1.schedule(x, self.mixer.schedule(*self.norm1.operand(x), angles, state, position))
+        return x if self.mlp is None else self.norm2.schedule(x, self.mlp.schedule(*self.norm2.operand(x)))
+
+
+class Mefesun:
+    """``order``: the layer of every run (layers that share weights appear more than once)."""
+
+    def __init__(self, embedding: Embedding, layers: List[PostNormLayer], order: List[int], norm: StreamNorm, head, dt: int, softcap: Optional[float]):
+        self.embedding, self.layers, self.order, self.norm, self.head, self.dt, self.softcap = embedding, layers, order, norm, head, dt, softcap
+
+    def schedule(self, ids, state: SequenceState, want=None, streams: Optional[list] = None):
+        """As ``Dadezen.schedule``; ``streams`` receives stream rows (their first `width` columns are the residual stream)."""
+        x = self.embedding.schedule(ids).stream_rows(self.dt)
+        angles = {}                                  # once per frequency table: every layer turns by the same angles
+        for k, i in enumerate(self.order):
+            rot = self.layers[i].mixer.rot
+            if rot not in angles:
+                angles[rot] = rot.freqs.rotary_angles(rot.magnitude, state.position, ids.shape()[0])
+            x = self.layers[i].schedule(x, angles[rot], state.runs[k], state.position)
+            if streams is not None:
+                streams.append(x)
+        if want is None:
+            return x
+        h = self.norm.schedule(x.index_select(want, 0))
+        return self.head.linear(h, dt=capi.F32, act="softcap" if self.softcap else None, act_param=self.softcap or 0.0)

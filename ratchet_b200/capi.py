@@ -34,7 +34,9 @@ UNARY_OPS = {"gelu": 0, "tanh": 1, "exp": 2, "log": 3, "sin": 4, "cos": 5, "abs"
 LAYER_NORM, RMS_NORM, GROUP_NORM = 0, 1, 2
 DEBUG_NO_REUSE, DEBUG_PROFILE, DEBUG_LOG = 1, 2, 4
 REDUCE_SUM, REDUCE_MAX, REDUCE_MEAN = 0, 1, 2
-MIXER_LIGHTNING, MIXER_LATENT = 0, 1
+MIXER_LIGHTNING, MIXER_LATENT, MIXER_GROUPED = 0, 1, 2
+LAYER_PARALLEL, LAYER_POST_NORM = 0, 1
+LINEAR_ACTS = {None: 0, "silu": 1, "relu_squared": 2, "softcap": 3}
 
 
 class RatchetCudaError(RuntimeError):
@@ -71,15 +73,16 @@ class rcu_decoder_layer(C.Structure):
 
 class rcu_stack_config(C.Structure):
     _fields_ = [("width", C.c_uint32), ("vocab", C.c_uint32), ("n_runs", C.c_uint32), ("eps", C.c_float), ("residual_mult", C.c_float),
-                ("weight_dt", C.c_int32)]
+                ("logit_softcap", C.c_float), ("weight_dt", C.c_int32), ("layer", C.c_int32), ("final_shift", C.c_void_p)]
 
 
 class rcu_stack_run(C.Structure):
     _fields_ = ([("mixer", C.c_int32)] +
-                [(n, C.c_uint32) for n in ("heads", "dim", "vdim", "ff", "q_rank", "kv_rank", "rot_dim", "rot_pairs", "window", "ring_rows")] +
+                [(n, C.c_uint32) for n in ("heads", "dim", "vdim", "ff", "q_rank", "kv_rank", "rot_dim", "rot_pairs", "window", "ring_rows", "kv_heads",
+                                           "chunk")] +
                 [("scale", C.c_float), ("rot_magnitude", C.c_float)] +
-                [(n, C.c_void_p) for n in ("enter", "enter_bias", "norm1", "norm2", "mix_in", "mix_norm", "kv_norm", "uq", "ukv", "freqs", "decay",
-                                           "out", "gate_up", "down", "state")])
+                [(n, C.c_void_p) for n in ("enter", "enter_bias", "norm1", "norm2", "norm1_shift", "norm2_shift", "mix_in", "mix_bias", "mix_norm",
+                                           "kv_norm", "sink", "uq", "ukv", "freqs", "decay", "out", "out_bias", "gate_up", "down", "state")])
 
 
 _T = C.POINTER(rcu_tensor)
@@ -135,8 +138,14 @@ SIGNATURES = {
     "rcu_index_write": (C.c_int, [_DEV, _T, _T, _u64p]),
     "rcu_conv1d": (C.c_int, [_DEV, _T, _T, _T, C.c_uint32, C.c_uint32, _T]),
     # models with a 32-bit residual stream
-    "rcu_linear": (C.c_int, [_DEV, _T, _T, C.c_uint32, _T, C.c_uint32, _T, C.c_float, _T]),
-    "rcu_norm_rows": (C.c_int, [_DEV, C.c_int, _T, C.c_uint32, _T, _T, C.c_uint32, C.c_float, _T]),
+    "rcu_linear": (C.c_int, [_DEV, _T, _T, C.c_uint32, _T, C.c_int, C.c_uint32, C.c_float, _T, C.c_float, _T]),
+    "rcu_norm_rows": (C.c_int, [_DEV, C.c_int, _T, C.c_uint32, _T, _T, _T, C.c_uint32, C.c_float, _T]),
+    "rcu_stream_rows": (C.c_int, [_DEV, _T, C.c_int32, _T]),
+    "rcu_post_norm": (C.c_int, [_DEV, _T, _T, _T, _T, C.c_float, _T]),
+    "rcu_rotary_angles": (C.c_int, [_DEV, _T, C.c_float, C.c_uint32, _T]),
+    "rcu_norm_rotary": (C.c_int, [_DEV, _T, C.c_uint32, _T, C.c_float, _T, _T]),
+    "rcu_kv_append": (C.c_int, [_DEV, _T, C.c_uint32, C.c_uint32, _T, C.c_float, _T, C.c_uint32, C.c_uint32, _T, _T]),
+    "rcu_grouped_attention": (C.c_int, [_DEV, _T, _T, _T] + [C.c_uint32] * 5 + [C.c_float, _T]),
     "rcu_glu": (C.c_int, [_DEV, C.c_int, _T, _T]),
     "rcu_rotary_frequencies": (C.c_int, [C.c_uint32] + [C.c_double] * 5 + [C.POINTER(C.c_float), C.POINTER(C.c_float)]),
     "rcu_rotary": (C.c_int, [_DEV, _T, C.c_uint32, _T, C.c_float, C.c_uint32, _T]),
@@ -167,8 +176,15 @@ SIGNATURES = {
     "rcu_lazy_index_select": (C.c_int, [_LZ, _LZ, C.c_uint32, C.POINTER(_LZ)]),
     "rcu_lazy_cache": (C.c_int, [_LZ, _LZ, C.c_uint32, C.c_uint32, C.POINTER(_LZ)]),
     "rcu_lazy_index_write": (C.c_int, [_LZ, _LZ, _u64p, C.POINTER(_LZ)]),
-    "rcu_lazy_linear": (C.c_int, [_LZ, _LZ, C.c_uint32, _LZ, C.c_uint32, _LZ, C.c_float, C.c_int32, C.POINTER(_LZ)]),
-    "rcu_lazy_norm_rows": (C.c_int, [C.c_int, _LZ, C.c_uint32, _LZ, _LZ, C.c_uint32, C.c_float, C.c_int32, C.POINTER(_LZ)]),
+    "rcu_lazy_linear": (C.c_int, [_LZ, _LZ, C.c_uint32, _LZ, C.c_int, C.c_uint32, C.c_float, _LZ, C.c_float, C.c_int32, C.POINTER(_LZ)]),
+    "rcu_lazy_norm_rows": (C.c_int, [C.c_int, _LZ, C.c_uint32, _LZ, _LZ, _LZ, C.c_uint32, C.c_float, C.c_int32, C.POINTER(_LZ)]),
+    "rcu_lazy_stream_rows": (C.c_int, [_LZ, C.c_int32, C.POINTER(_LZ)]),
+    "rcu_lazy_post_norm": (C.c_int, [_LZ, _LZ, _LZ, _LZ, C.c_float, C.POINTER(_LZ)]),
+    "rcu_lazy_bitcast": (C.c_int, [_LZ, C.c_int32, C.POINTER(_LZ)]),
+    "rcu_lazy_rotary_angles": (C.c_int, [_LZ, C.c_float, C.c_uint32, C.c_uint32, C.POINTER(_LZ)]),
+    "rcu_lazy_norm_rotary": (C.c_int, [_LZ, C.c_uint32, C.c_uint32, _LZ, C.c_float, _LZ, C.POINTER(_LZ)]),
+    "rcu_lazy_kv_append": (C.c_int, [_LZ, C.c_uint32, C.c_uint32, _LZ, C.c_float, _LZ, C.c_uint32, C.c_uint32, _LZ, C.c_uint32, C.POINTER(_LZ)]),
+    "rcu_lazy_grouped_attention": (C.c_int, [_LZ, _LZ, _LZ] + [C.c_uint32] * 5 + [C.c_float, C.POINTER(_LZ)]),
     "rcu_lazy_glu": (C.c_int, [C.c_int, _LZ, C.POINTER(_LZ)]),
     "rcu_lazy_rotary": (C.c_int, [_LZ, C.c_uint32, _LZ, C.c_float, C.c_uint32, C.POINTER(_LZ)]),
     "rcu_lazy_lightning": (C.c_int, [_LZ, _LZ, _LZ, C.POINTER(_LZ)]),

@@ -191,6 +191,19 @@ __device__ __forceinline__ unsigned long long rcu_wait_limit(const int* status) 
     return *reinterpret_cast<const volatile unsigned long long*>(status + 2);
 }
 
+// Activation of a Linear's leading columns (rcu_linear), evaluated in f32.
+struct LinearAct {
+    int cols = 0;             // columns below this are activated
+    int kind = RCU_ACT_NONE;
+    float param = 0.f;
+    __device__ __forceinline__ float operator()(float v) const {
+        if (kind == RCU_ACT_SILU) return v / (1.0f + expf(-v));
+        if (kind == RCU_ACT_RELU_SQUARED) return v > 0.f ? v * v : 0.f;
+        if (kind == RCU_ACT_SOFTCAP) return param * tanhf(v / param);
+        return v;
+    }
+};
+
 // streaming 16-byte load that does not allocate in L1 (weights are read exactly once)
 __device__ __forceinline__ uint4 ld_stream_v4(const void* p) {
     uint4 r;

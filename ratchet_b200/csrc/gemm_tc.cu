@@ -519,8 +519,8 @@ rcu_status rcu_gemm_tc_linear(rcu_device* dev, const void* w, const void* x, con
 #define RCU_TC(OUT_, EPI_)                                                                                                       \
     (bn == 128 ? launch_tc<128, WK_F16, OUT_>(dev, xmap, wmap, qa, EPI_, y, (int)M, (int)N, (int)K, 1, t.bf16)                   \
                : launch_tc<64, WK_F16, OUT_>(dev, xmap, wmap, qa, EPI_, y, (int)M, (int)N, (int)K, 1, t.bf16))
-    if (t.out_dt == RCU_F32) return RCU_TC(float, (GemmEpilogue<float>{(const float*)bias, t.resid, t.alpha, t.silu_cols}));
-    if (t.out_dt == RCU_BF16) return RCU_TC(__nv_bfloat16, (GemmEpilogue<__nv_bfloat16>{(const __nv_bfloat16*)bias, nullptr, 1.f, t.silu_cols}));
-    return RCU_TC(__half, (GemmEpilogue<__half>{(const __half*)bias, nullptr, 1.f, t.silu_cols}));
+    if (t.out_dt == RCU_F32) return RCU_TC(float, (GemmEpilogue<float>{(const float*)bias, t.resid, t.alpha, t.act}));
+    if (t.out_dt == RCU_BF16) return RCU_TC(__nv_bfloat16, (GemmEpilogue<__nv_bfloat16>{(const __nv_bfloat16*)bias, nullptr, 1.f, t.act}));
+    return RCU_TC(__half, (GemmEpilogue<__half>{(const __half*)bias, nullptr, 1.f, t.act}));
 #undef RCU_TC
 }

@@ -250,8 +250,8 @@ rcu_status rcu_gemm_tc2_launch(rcu_device* dev, const void* w, const void* x, co
         !make_map_f16_sw128_rows(&wmap, w, N, K, kTileN2 / 2, K, t.bf16))
         return rcu_fail(dev, RCU_ERR_CUDA, "gemm_tc2: cuTensorMapEncodeTiled failed (M=%llu N=%llu K=%llu)", (unsigned long long)M,
                         (unsigned long long)N, (unsigned long long)K);
-    if (t.out_dt == RCU_F32) return launch_pair<float>(dev, xmap, wmap, GemmEpilogue<float>{(const float*)bias, t.resid, t.alpha, t.silu_cols}, y, M, N, K, t.bf16);
+    if (t.out_dt == RCU_F32) return launch_pair<float>(dev, xmap, wmap, GemmEpilogue<float>{(const float*)bias, t.resid, t.alpha, t.act}, y, M, N, K, t.bf16);
     if (t.out_dt == RCU_BF16)
-        return launch_pair<__nv_bfloat16>(dev, xmap, wmap, GemmEpilogue<__nv_bfloat16>{(const __nv_bfloat16*)bias, nullptr, 1.f, t.silu_cols}, y, M, N, K, t.bf16);
-    return launch_pair<__half>(dev, xmap, wmap, GemmEpilogue<__half>{(const __half*)bias, nullptr, 1.f, t.silu_cols}, y, M, N, K, t.bf16);
+        return launch_pair<__nv_bfloat16>(dev, xmap, wmap, GemmEpilogue<__nv_bfloat16>{(const __nv_bfloat16*)bias, nullptr, 1.f, t.act}, y, M, N, K, t.bf16);
+    return launch_pair<__half>(dev, xmap, wmap, GemmEpilogue<__half>{(const __half*)bias, nullptr, 1.f, t.act}, y, M, N, K, t.bf16);
 }

@@ -32,7 +32,8 @@ namespace {
 enum LazyKind {
     K_CONST = 0, K_VIEW, K_BINARY, K_UNARY, K_CAST, K_MATMUL, K_NORM, K_SOFTMAX, K_ROPE, K_CONCAT, K_SELECT,
     K_PERMUTE, K_SLICE, K_BROADCAST, K_CACHE, K_INDEX_WRITE, K_CONV,
-    K_LINEAR, K_NORM_ROWS, K_GLU, K_ROTARY, K_LIGHTNING, K_LATENT_APPEND, K_WINDOW_ATTENTION
+    K_LINEAR, K_NORM_ROWS, K_GLU, K_ROTARY, K_LIGHTNING, K_LATENT_APPEND, K_WINDOW_ATTENTION,
+    K_STREAM_ROWS, K_POST_NORM, K_ROTARY_ANGLES, K_NORM_ROTARY, K_KV_APPEND, K_GROUPED_ATTENTION
 };
 
 struct Storage {
@@ -64,7 +65,7 @@ struct rcu_lazy {
     // op parameters
     int op = 0;                    // binary / unary op, norm kind
     int flags[3] = {0, 0, 0};      // matmul transposes
-    uint32_t u[4] = {0, 0, 0, 0};  // dim / offset / stride / padding / groups / perm
+    uint32_t u[6] = {0, 0, 0, 0, 0, 0};  // dim / offset / stride / padding / groups / perm
     uint64_t a[RCU_MAX_RANK] = {0, 0, 0, 0}, b[RCU_MAX_RANK] = {0, 0, 0, 0};   // slice start/stop, index_write start
     float f[2] = {0.f, 0.f};       // eps, rope base
     std::shared_ptr<Storage> storage;
@@ -123,7 +124,7 @@ bool supports_inplace(const rcu_lazy* n) {
     const int kind = n->kind;
     if (kind == K_LINEAR) return n->flags[0] != 0;      // srcs[0] is the residual
     // ops/binary.rs:179, ops/unary.rs:268, ops/softmax.rs:196, ops/rope.rs:80, ops/index_write.rs:49
-    return kind == K_ROTARY || kind == K_BINARY || kind == K_UNARY || kind == K_SOFTMAX || kind == K_ROPE || kind == K_INDEX_WRITE;
+    return kind == K_ROTARY || kind == K_POST_NORM || kind == K_BINARY || kind == K_UNARY || kind == K_SOFTMAX || kind == K_ROPE || kind == K_INDEX_WRITE;
 }
 
 // The op about to overwrite `s`'s buffer must be the only thing that can still read it: `s` has one
@@ -226,6 +227,12 @@ const char* kind_name(int kind) {
         case K_LIGHTNING: return "lightning";
         case K_LATENT_APPEND: return "latent_append";
         case K_WINDOW_ATTENTION: return "window_attention";
+        case K_STREAM_ROWS: return "stream_rows";
+        case K_POST_NORM: return "post_norm";
+        case K_ROTARY_ANGLES: return "rotary_angles";
+        case K_NORM_ROTARY: return "norm_rotary";
+        case K_KV_APPEND: return "kv_append";
+        case K_GROUPED_ATTENTION: return "grouped_attention";
         default: return "other";
     }
 }
@@ -293,12 +300,14 @@ rcu_status run_node(rcu_lazy* n) {
             if (n->flags[0]) resid = S(i++);
             rcu_tensor w = S(i++), x = S(i++);
             if (n->flags[1]) bias = S(i++);
-            return rcu_linear(dev, &w, &x, n->u[0], n->flags[1] ? &bias : nullptr, n->u[1], n->flags[0] ? &resid : nullptr, n->f[0], &dst);
+            return rcu_linear(dev, &w, &x, n->u[0], n->flags[1] ? &bias : nullptr, n->op, n->u[1], n->f[1], n->flags[0] ? &resid : nullptr, n->f[0], &dst);
         }
-        case K_NORM_ROWS: {
-            rcu_tensor x = S(0), sc = S(1), gate;
-            if (n->srcs.size() > 2) gate = S(2);
-            return rcu_norm_rows(dev, n->op, &x, n->u[0], &sc, n->srcs.size() > 2 ? &gate : nullptr, n->u[1], n->f[0], &dst);
+        case K_NORM_ROWS: {     // x, scale, [shift], [gate]
+            size_t i = 2;
+            rcu_tensor x = S(0), sc = S(1), shift, gate;
+            if (n->flags[0]) shift = S(i++);
+            if (n->flags[1]) gate = S(i++);
+            return rcu_norm_rows(dev, n->op, &x, n->u[0], &sc, n->flags[0] ? &shift : nullptr, n->flags[1] ? &gate : nullptr, n->u[1], n->f[0], &dst);
         }
         case K_GLU: { rcu_tensor x = S(0); return rcu_glu(dev, n->op, &x, &dst); }
         case K_ROTARY: { rcu_tensor x = S(0), fr = S(1); return rcu_rotary(dev, &x, n->u[0], &fr, n->f[0], n->u[1], &dst); }
@@ -310,6 +319,19 @@ rcu_status run_node(rcu_lazy* n) {
         case K_WINDOW_ATTENTION: {
             rcu_tensor q = S(0), kv = S(1), sh = S(2);
             return rcu_window_attention(dev, &q, &kv, &sh, n->u[0], n->u[1], n->u[2], n->f[0], &dst);
+        }
+        case K_STREAM_ROWS: { rcu_tensor x = S(0); return rcu_stream_rows(dev, &x, n->op, &dst); }
+        case K_POST_NORM: { rcu_tensor x = S(0), y = S(1), sc = S(2), sh = S(3); return rcu_post_norm(dev, &x, &y, &sc, &sh, n->f[0], &dst); }
+        case K_ROTARY_ANGLES: { rcu_tensor fr = S(0); return rcu_rotary_angles(dev, &fr, n->f[0], n->u[0], &dst); }
+        case K_NORM_ROTARY: { rcu_tensor x = S(0), sc = S(1), an = S(2); return rcu_norm_rotary(dev, &x, n->u[0], &sc, n->f[0], &an, &dst); }
+        case K_KV_APPEND: {
+            rcu_tensor x = S(0), sc = S(1), an = S(2), ring = S(3);
+            return rcu_kv_append(dev, &x, n->u[0], n->u[1], &sc, n->f[0], &an, n->u[2], n->u[3], &ring, &dst);
+        }
+        case K_GROUPED_ATTENTION: {
+            rcu_tensor q = S(0), kv = S(1), sink;
+            if (n->srcs.size() > 2) sink = S(2);
+            return rcu_grouped_attention(dev, &q, &kv, n->srcs.size() > 2 ? &sink : nullptr, n->u[0], n->u[1], n->u[2], n->u[3], n->u[4], n->f[0], &dst);
         }
         default: return rcu_fail(dev, RCU_ERR_UNSUPPORTED, "resolve: node kind %d has no kernel", n->kind);
     }
@@ -755,7 +777,8 @@ rcu_status rcu_lazy_index_write(rcu_lazy* dst, rcu_lazy* src, const uint64_t* st
     return RCU_OK;
 }
 
-rcu_status rcu_lazy_linear(rcu_lazy* w, rcu_lazy* x, uint32_t x_col, rcu_lazy* bias, uint32_t silu_cols, rcu_lazy* resid, float alpha, int32_t dst_dt, rcu_lazy** out) {
+rcu_status rcu_lazy_linear(rcu_lazy* w, rcu_lazy* x, uint32_t x_col, rcu_lazy* bias, int act, uint32_t act_cols, float act_param, rcu_lazy* resid, float alpha,
+                           int32_t dst_dt, rcu_lazy** out) {
     if (!w || !x || !out) return RCU_ERR_INVALID_ARG;
     LAZY_REQUIRE(w->dev, x->dev == w->dev && (!bias || bias->dev == w->dev) && (!resid || resid->dev == w->dev), "Mixed devices");
     LAZY_REQUIRE(w->dev, w->rank == 2 && w->dt == x->dt && dt_is_float(w->dt), "linear: w must be a float matrix of the activations' dtype");
@@ -770,14 +793,16 @@ rcu_status rcu_lazy_linear(rcu_lazy* w, rcu_lazy* x, uint32_t x_col, rcu_lazy* b
     n->flags[0] = resid != nullptr;
     n->flags[1] = bias != nullptr;
     n->u[0] = x_col;
-    n->u[1] = silu_cols;
+    n->u[1] = act_cols;
+    n->op = act;
     n->f[0] = alpha;
+    n->f[1] = act_param;
     *out = n;
     return RCU_OK;
 }
 
-rcu_status rcu_lazy_norm_rows(int kind, rcu_lazy* x, uint32_t x_col, rcu_lazy* scale, rcu_lazy* gate, uint32_t gate_col, float eps, int32_t dst_dt,
-                              rcu_lazy** out) {
+rcu_status rcu_lazy_norm_rows(int kind, rcu_lazy* x, uint32_t x_col, rcu_lazy* scale, rcu_lazy* shift, rcu_lazy* gate, uint32_t gate_col, float eps,
+                              int32_t dst_dt, rcu_lazy** out) {
     if (!x || !scale || !out) return RCU_ERR_INVALID_ARG;
     LAZY_REQUIRE(x->dev, kind == RCU_LAYER_NORM || kind == RCU_RMS_NORM, "norm_rows: LayerNorm or RMSNorm");
     LAZY_REQUIRE(x->dev, x->dt == RCU_F32 && dt_is_float(dst_dt), "norm_rows: f32 input, float output");
@@ -785,8 +810,10 @@ rcu_status rcu_lazy_norm_rows(int kind, rcu_lazy* x, uint32_t x_col, rcu_lazy* s
     uint64_t shape[RCU_MAX_RANK];
     for (uint32_t i = 0; i < x->rank; ++i) shape[i] = x->shape[i];
     shape[x->rank - 1] = scale->numel();
-    rcu_lazy* n = new_node(x->dev, K_NORM_ROWS, dst_dt, x->rank, shape, {x, scale, gate});
+    rcu_lazy* n = new_node(x->dev, K_NORM_ROWS, dst_dt, x->rank, shape, {x, scale, shift, gate});
     n->op = kind;
+    n->flags[0] = shift != nullptr;
+    n->flags[1] = gate != nullptr;
     n->u[0] = x_col;
     n->u[1] = gate_col;
     n->f[0] = eps;
@@ -850,6 +877,94 @@ rcu_status rcu_lazy_window_attention(rcu_lazy* q, rcu_lazy* kv, rcu_lazy* shared
     n->u[0] = shared_col;
     n->u[1] = vdim;
     n->u[2] = window;
+    n->f[0] = scale;
+    *out = n;
+    return RCU_OK;
+}
+
+rcu_status rcu_lazy_stream_rows(rcu_lazy* x, int32_t copy_dt, rcu_lazy** out) {
+    if (!x || !out) return RCU_ERR_INVALID_ARG;
+    LAZY_REQUIRE(x->dev, x->rank == 2 && (x->dt == RCU_F32 || x->dt == RCU_BF16), "stream_rows: x is f32 or bf16 [tokens, width]");
+    LAZY_REQUIRE(x->dev, copy_dt == RCU_F32 || copy_dt == RCU_BF16, "stream_rows: the copy is bf16, or f32 for none");
+    const uint64_t W = x->shape[1], shape[2] = {x->shape[0], copy_dt == RCU_BF16 ? W + (W + 1) / 2 : W};
+    rcu_lazy* n = new_node(x->dev, K_STREAM_ROWS, RCU_F32, 2, shape, {x});
+    n->op = copy_dt;
+    *out = n;
+    return RCU_OK;
+}
+
+rcu_status rcu_lazy_post_norm(rcu_lazy* x, rcu_lazy* y, rcu_lazy* scale, rcu_lazy* shift, float eps, rcu_lazy** out) {
+    if (!x || !y || !scale || !shift || !out) return RCU_ERR_INVALID_ARG;
+    LAZY_REQUIRE(x->dev, x->rank == 2 && y->rank == 2 && x->dt == RCU_F32 && y->dt == RCU_F32 && x->shape[0] == y->shape[0] && y->shape[1] == scale->numel(),
+                 "post_norm: x is f32 stream rows, y f32 [tokens, width]");
+    rcu_lazy* n = new_node(x->dev, K_POST_NORM, RCU_F32, 2, x->shape, {x, y, scale, shift});
+    n->f[0] = eps;
+    *out = n;
+    return RCU_OK;
+}
+
+rcu_status rcu_lazy_bitcast(rcu_lazy* x, int32_t dt, rcu_lazy** out) {
+    if (!x || !out) return RCU_ERR_INVALID_ARG;
+    LAZY_REQUIRE(x->dev, !dt_is_quant(x->dt) && !dt_is_quant(dt) && dt >= 0, "bitcast: quantised tensors have no elements to reinterpret");
+    const uint64_t last = x->shape[x->rank - 1] * dt_esize(x->dt);
+    LAZY_REQUIRE(x->dev, last % dt_esize(dt) == 0, "bitcast: rows of %llu bytes", (unsigned long long)last);
+    uint64_t shape[RCU_MAX_RANK];
+    for (uint32_t i = 0; i < x->rank; ++i) shape[i] = x->shape[i];
+    shape[x->rank - 1] = last / dt_esize(dt);
+    rcu_lazy* n = new_node(x->dev, K_VIEW, dt, x->rank, shape, {x});
+    n->storage = x->storage;
+    *out = n;
+    return RCU_OK;
+}
+
+rcu_status rcu_lazy_rotary_angles(rcu_lazy* freqs, float magnitude, uint32_t position, uint32_t tokens, rcu_lazy** out) {
+    if (!freqs || !out) return RCU_ERR_INVALID_ARG;
+    LAZY_REQUIRE(freqs->dev, freqs->rank == 2 && freqs->shape[0] == 2 && tokens > 0, "rotary_angles: the frequency table is f32 [2, pairs]");
+    const uint64_t shape[2] = {tokens, 2 * freqs->shape[1]};
+    rcu_lazy* n = new_node(freqs->dev, K_ROTARY_ANGLES, RCU_F32, 2, shape, {freqs});
+    n->u[0] = position;
+    n->f[0] = magnitude;
+    *out = n;
+    return RCU_OK;
+}
+
+rcu_status rcu_lazy_norm_rotary(rcu_lazy* x, uint32_t x_col, uint32_t heads, rcu_lazy* scale, float eps, rcu_lazy* angles, rcu_lazy** out) {
+    if (!x || !scale || !angles || !out) return RCU_ERR_INVALID_ARG;
+    LAZY_REQUIRE(x->dev, x->rank == 2 && x_col + heads * scale->numel() <= x->shape[1], "norm_rotary: the heads lie outside the rows");
+    const uint64_t shape[3] = {x->shape[0], heads, scale->numel()};
+    rcu_lazy* n = new_node(x->dev, K_NORM_ROTARY, x->dt, 3, shape, {x, scale, angles});
+    n->u[0] = x_col;
+    n->f[0] = eps;
+    *out = n;
+    return RCU_OK;
+}
+
+rcu_status rcu_lazy_kv_append(rcu_lazy* x, uint32_t x_col, uint32_t kv_heads, rcu_lazy* scale, float eps, rcu_lazy* angles, uint32_t position, uint32_t keep,
+                              rcu_lazy* ring, uint32_t rows, rcu_lazy** out) {
+    if (!x || !scale || !angles || !ring || !out) return RCU_ERR_INVALID_ARG;
+    LAZY_REQUIRE(x->dev, ring->rank == 2, "kv_append: the ring is [rows, width]");
+    const uint64_t shape[2] = {rows, ring->shape[1]};
+    rcu_lazy* n = new_node(x->dev, K_KV_APPEND, ring->dt, 2, shape, {x, scale, angles, ring});
+    n->u[0] = x_col;
+    n->u[1] = kv_heads;
+    n->u[2] = position;
+    n->u[3] = keep;
+    n->f[0] = eps;
+    *out = n;
+    return RCU_OK;
+}
+
+rcu_status rcu_lazy_grouped_attention(rcu_lazy* q, rcu_lazy* kv, rcu_lazy* sink, uint32_t kv_heads, uint32_t vdim, uint32_t window, uint32_t chunk,
+                                      uint32_t position, float scale, rcu_lazy** out) {
+    if (!q || !kv || !out) return RCU_ERR_INVALID_ARG;
+    LAZY_REQUIRE(q->dev, q->rank == 3 && kv->rank == 2, "grouped_attention: q [tokens, heads, dim] and kv rows");
+    const uint64_t shape[2] = {q->shape[0], q->shape[1] * vdim};
+    rcu_lazy* n = new_node(q->dev, K_GROUPED_ATTENTION, q->dt, 2, shape, {q, kv, sink});
+    n->u[0] = kv_heads;
+    n->u[1] = vdim;
+    n->u[2] = window;
+    n->u[3] = chunk;
+    n->u[4] = position;
     n->f[0] = scale;
     *out = n;
     return RCU_OK;

@@ -6,6 +6,7 @@
 //   rcu_window_attention  softmax attention of the block's queries over those rows, keys and values expanded from the
 //                       latents by one Linear before the call.  bf16 blocks run on the tensor cores (256 tokens and more: window_tc.cu,
 //                       fewer, or sizes it does not take: below), f32 ones in FFMA.
+// The attention kernels also serve grouped heads with chunked masks and sinks (grouped_attention.cu).
 #include "lm_mma.cuh"
 #include "window.cuh"
 
@@ -91,7 +92,7 @@ __global__ void __launch_bounds__(256) window_attention_kernel(const WindowArgs 
     rcu_kernel_entry();
     extern __shared__ float q_s[];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int h = blockIdx.y;
+    const int h = blockIdx.y, hk = h / (a.H / a.G);
     const int i = blockIdx.x * 8 + warp;
     if (i >= a.T) return;
     const int Q = a.D + a.R;
@@ -99,11 +100,11 @@ __global__ void __launch_bounds__(256) window_attention_kernel(const WindowArgs 
     const T* qg = reinterpret_cast<const T*>(a.q) + ((size_t)i * a.H + h) * Q;
     for (int d = lane; d < Q; d += 32) q[d] = to_f32<T>(qg[d]);
     __syncwarp();
-    const size_t kv_pitch = (size_t)a.H * (a.D + a.E);
-    const T* K = reinterpret_cast<const T*>(a.kv) + (size_t)h * a.D;
-    const T* V = reinterpret_cast<const T*>(a.kv) + (size_t)a.H * a.D + (size_t)h * a.E;
+    const size_t kv_pitch = (size_t)a.G * (a.D + a.E);
+    const T* K = reinterpret_cast<const T*>(a.kv) + (size_t)hk * a.D;
+    const T* V = reinterpret_cast<const T*>(a.kv) + (size_t)a.G * a.D + (size_t)hk * a.E;
     const T* KS = reinterpret_cast<const T*>(a.shared);
-    const int last = a.L - a.T + i, first = max(0, last - a.window + 1);
+    const int last = a.L - a.T + i, first = a.see.first(last);
     float m = -INFINITY, l = 0.f, o[PE];
 #pragma unroll
     for (int j = 0; j < PE; ++j) o[j] = 0.f;
@@ -136,6 +137,7 @@ __global__ void __launch_bounds__(256) window_attention_kernel(const WindowArgs 
             }
         }
     }
+    if (a.sink) l += expf(a.sink[h] - m);
     T* og = reinterpret_cast<T*>(a.out) + ((size_t)i * a.H + h) * a.E;
 #pragma unroll
     for (int c = 0; c < PE; ++c) {
@@ -174,15 +176,15 @@ __global__ void __launch_bounds__(256) window_mma_kernel(const WindowArgs a, int
     const int Q = a.D + a.R, qp = (Q + 15) & ~15, ld = qp + 8;
     constexpr int ldv = EP + 8;
     bf16 *qs = tiles, *ks = qs + kQueries * ld, *vs = ks + 2 * kKeys * ld;
-    const int h = blockIdx.y, i0 = blockIdx.x * kQueries;
+    const int h = blockIdx.y, hk = h / (a.H / a.G), i0 = blockIdx.x * kQueries;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
     const int nq = min(kQueries, a.T - i0);
-    const long long kvp = (long long)a.H * (a.D + a.E);
-    const bf16* K = reinterpret_cast<const bf16*>(a.kv) + (size_t)h * a.D;
-    const bf16* V = reinterpret_cast<const bf16*>(a.kv) + (size_t)a.H * a.D + (size_t)h * a.E;
+    const long long kvp = (long long)a.G * (a.D + a.E);
+    const bf16* K = reinterpret_cast<const bf16*>(a.kv) + (size_t)hk * a.D;
+    const bf16* V = reinterpret_cast<const bf16*>(a.kv) + (size_t)a.G * a.D + (size_t)hk * a.E;
     const bf16* KS = reinterpret_cast<const bf16*>(a.shared);
     const int base = a.L - a.T + i0;                       // key row of the CTA's first query
-    const int first = max(0, base - a.window + 1), last = base + nq - 1;
+    const int first = a.see.first(base), last = base + nq - 1;
     const int tiles_n = (last - first) / kKeys + 1;
 
     auto load_keys = [&](int n) {
@@ -218,6 +220,7 @@ __global__ void __launch_bounds__(256) window_mma_kernel(const WindowArgs a, int
     load_keys(0);
 
     const int r0 = warp * 16, row0 = base + r0 + g, row1 = row0 + 8;      // key rows of this thread's two queries
+    const int low0 = a.see.first(row0), low1 = a.see.first(row1), low = a.see.first(base + r0);
     const float sc = a.scale * 1.4426950408889634f;                       // scores in units of log 2
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f, o[EP / 8][4];
 #pragma unroll
@@ -233,7 +236,7 @@ __global__ void __launch_bounds__(256) window_mma_kernel(const WindowArgs a, int
         __syncthreads();
         const int j0 = first + n * kKeys;
         // a tile no query of this warp sees is passed over
-        if (r0 < nq && j0 <= base + r0 + 15 && j0 + kKeys - 1 >= base + r0 - a.window + 1) {
+        if (r0 < nq && j0 <= base + r0 + 15 && j0 + kKeys - 1 >= low) {
             const bf16* kt = ks + (n & 1) * kKeys * ld;
             const bf16* vt = vs + (n & 1) * kKeys * ldv;
             float s[8][4] = {};
@@ -253,8 +256,8 @@ __global__ void __launch_bounds__(256) window_mma_kernel(const WindowArgs a, int
             for (int c = 0; c < 8; ++c)
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
-                    const int j = j0 + 8 * c + 2 * t + (e & 1), row = e < 2 ? row0 : row1;
-                    const float v = j <= row && j > row - a.window ? s[c][e] * sc : -INFINITY;
+                    const int j = j0 + 8 * c + 2 * t + (e & 1);
+                    const float v = j <= (e < 2 ? row0 : row1) && j >= (e < 2 ? low0 : low1) ? s[c][e] * sc : -INFINITY;
                     s[c][e] = v;
                     if (e < 2) t0 = fmaxf(t0, v);
                     else t1 = fmaxf(t1, v);
@@ -301,6 +304,11 @@ __global__ void __launch_bounds__(256) window_mma_kernel(const WindowArgs a, int
     l1 += __shfl_xor_sync(0xffffffffu, l1, 1);
     l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
     l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
+    if (a.sink) {
+        const float sink = a.sink[h] * 1.4426950408889634f;
+        l0 += exp2f(sink - m0);
+        l1 += exp2f(sink - m1);
+    }
     const float w0 = 1.0f / l0, w1 = 1.0f / l1;
     bf16* og = reinterpret_cast<bf16*>(a.out) + (size_t)i0 * a.H * a.E + (size_t)h * a.E;
 #pragma unroll
@@ -337,6 +345,13 @@ rcu_status launch_window_mma(rcu_device* dev, const WindowArgs& a) {
 
 }  // namespace
 
+rcu_status rcu_attend(rcu_device* dev, int dt, const WindowArgs& a) {
+    if (dt == RCU_F32) return launch_window<float>(dev, a);
+    rcu_status st = rcu_window_tc(dev, a);
+    if (st == RCU_ERR_UNSUPPORTED) st = launch_window_mma(dev, a);
+    return st == RCU_ERR_UNSUPPORTED ? launch_window<__nv_bfloat16>(dev, a) : st;
+}
+
 extern "C" {
 
 rcu_status rcu_latent_append(rcu_device* dev, const rcu_tensor* x, uint32_t x_col, const rcu_tensor* scale, float eps, const rcu_tensor* freqs,
@@ -371,11 +386,8 @@ rcu_status rcu_window_attention(rcu_device* dev, const rcu_tensor* q, const rcu_
     if (vdim > 512 || H > 65535 || L > 0x7fffffffull || q->shape[2] > 4096) return rcu_fail(dev, RCU_ERR_UNSUPPORTED, "window_attention: vdim %u (at most 512)", vdim);
     DevGuard g(dev->ordinal);
     WindowArgs a{q->data, kv->data, (const char*)shared->data + (size_t)shared_col * dt_esize(shared->dt), dst->data, (long long)shared->shape[1], (int)T,
-                 (int)L, (int)H, (int)(q->shape[2] - R), (int)R, (int)vdim, (int)(window < L ? window : L), scale};
-    if (q->dt == RCU_F32) return launch_window<float>(dev, a);
-    rcu_status st = rcu_window_tc(dev, a);
-    if (st == RCU_ERR_UNSUPPORTED) st = launch_window_mma(dev, a);
-    return st == RCU_ERR_UNSUPPORTED ? launch_window<__nv_bfloat16>(dev, a) : st;
+                 (int)L, (int)H, (int)H, (int)(q->shape[2] - R), (int)R, (int)vdim, Visible{(int)(window < L ? window : L), 0, 0}, scale, nullptr};
+    return rcu_attend(dev, q->dt, a);
 }
 
 }  // extern "C"

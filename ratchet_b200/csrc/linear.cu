@@ -1,5 +1,6 @@
 // Linear with a chosen output type: out[M, N] = x[M, K] . W[N, K]^T (+ bias), rounded to the operands' type or kept in
-// f32 as resid + alpha * (...), with the first silu_cols columns passed through silu.  It is what a model with a 32-bit residual stream and 16-bit projections needs beside
+// f32 as resid + alpha * (...), with an activation on the leading columns.  It is what a model with a 32-bit residual stream and
+// 16-bit projections needs beside
 // rcu_matmul, whose output has the activations' type (ops/matmul/mod.rs:484-495).
 //
 //   16-bit operands, shapes the tensor maps take: the tcgen05 kernels of gemm_tc2.cu / gemm_tc.cu;
@@ -100,9 +101,9 @@ linear_simt_kernel(const T* __restrict__ W, const T* __restrict__ x, long long x
 }
 
 template <class T, class Out>
-rcu_status launch_plain(rcu_device* dev, const void* w, const void* x, uint64_t pitch, const void* bias, const float* resid, float alpha, int silu_cols, void* y,
+rcu_status launch_plain(rcu_device* dev, const void* w, const void* x, uint64_t pitch, const void* bias, const float* resid, float alpha, const LinearAct& act, void* y,
                         uint64_t M, uint64_t N, uint64_t K) {
-    const GemmEpilogue<Out> epi{(const Out*)bias, resid, alpha, silu_cols};
+    const GemmEpilogue<Out> epi{(const Out*)bias, resid, alpha, act};
     if (M <= (uint64_t)kSkinny) {
         constexpr uint64_t VEC = 16 / sizeof(T);
         const int aligned = K % VEC == 0 && pitch % VEC == 0 && ((reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(x)) & 15) == 0;
@@ -120,7 +121,7 @@ rcu_status launch_plain(rcu_device* dev, const void* w, const void* x, uint64_t 
 }  // namespace
 
 extern "C" rcu_status rcu_linear(rcu_device* dev, const rcu_tensor* w, const rcu_tensor* x, uint32_t x_col, const rcu_tensor* bias,
-                                 uint32_t silu_cols, const rcu_tensor* resid, float alpha, rcu_tensor* dst) {
+                                 int act, uint32_t act_cols, float act_param, const rcu_tensor* resid, float alpha, rcu_tensor* dst) {
     if (!dev) return RCU_ERR_INVALID_ARG;
     RCU_REQUIRE(dev, t_valid(w) && t_valid(x) && t_valid(dst), "linear: invalid tensor descriptor");
     RCU_REQUIRE(dev, w->rank == 2 && w->dt == x->dt && dt_is_float(w->dt), "linear: w must be a float matrix of the activations' dtype");
@@ -132,7 +133,10 @@ extern "C" rcu_status rcu_linear(rcu_device* dev, const rcu_tensor* w, const rcu
     RCU_REQUIRE(dev, dst->dt == RCU_F32 || (!resid && alpha == 1.0f), "linear: a residual or a factor needs an f32 output");
     RCU_REQUIRE(dev, !resid || (resid->dt == RCU_F32 && t_numel(resid) == M * N), "linear: the residual must be f32 of the output's size");
     RCU_REQUIRE(dev, M <= 0x7fffffffull && N <= 0x7fffffffull && K <= 0x7fffffffull, "linear: dimension exceeds 2^31");
-    RCU_REQUIRE(dev, silu_cols <= N, "linear: %u activated of %llu columns", silu_cols, (unsigned long long)N);
+    RCU_REQUIRE(dev, act >= RCU_ACT_NONE && act <= RCU_ACT_SOFTCAP && (act != RCU_ACT_SOFTCAP || act_param > 0.f), "linear: unknown activation %d", act);
+    RCU_REQUIRE(dev, act_cols <= N, "linear: %u activated of %llu columns", act_cols, (unsigned long long)N);
+    LinearAct fn;
+    if (act != RCU_ACT_NONE) { fn.cols = (int)act_cols; fn.kind = act; fn.param = act_param; }
     DevGuard g(dev->ordinal);
     const void* xp = (const char*)x->data + (size_t)x_col * dt_esize(x->dt);
     const void* bp = bias ? bias->data : nullptr;
@@ -144,11 +148,11 @@ extern "C" rcu_status rcu_linear(rcu_device* dev, const rcu_tensor* w, const rcu
         t.out_dt = dst->dt;
         t.resid = rp;
         t.alpha = alpha;
-        t.silu_cols = (int)silu_cols;
+        t.act = fn;
         const rcu_status st = rcu_gemm_tc_linear(dev, w->data, xp, bp, dst->data, M, N, K, t);
         if (st != RCU_ERR_UNSUPPORTED) return st;
     }
-#define RCU_LIN(T_, O_) return launch_plain<T_, O_>(dev, w->data, xp, pitch, bp, rp, alpha, (int)silu_cols, dst->data, M, N, K)
+#define RCU_LIN(T_, O_) return launch_plain<T_, O_>(dev, w->data, xp, pitch, bp, rp, alpha, fn, dst->data, M, N, K)
     if (x->dt == RCU_F32) RCU_LIN(float, float);
     if (x->dt == RCU_BF16) { if (dst->dt == RCU_F32) RCU_LIN(__nv_bfloat16, float); RCU_LIN(__nv_bfloat16, __nv_bfloat16); }
     if (dst->dt == RCU_F32) RCU_LIN(__half, float);

@@ -1,12 +1,19 @@
-// Fused decode step for a stack of parallel-residual layers whose mixers are linear attention with a state or latent
-// attention with a sliding window, with stretches of layers that may be entered several times (each run of a layer has
-// a state of its own).  The batch-1 counterpart of the lazy graph that runs prompts, over the same weights and states:
+// Fused decode step for a stack of layers whose mixers are linear attention with a state, latent attention with a sliding
+// window or attention of grouped heads, with stretches of layers that may be entered several times (each run of a layer has
+// a state of its own).  The batch-1 counterpart of the lazy graph that runs prompts, over the same weights and states.
+// Parallel-residual layers (norm before the sublayers, which share their input and are added together):
 //
 //   lightning run:  [norms + mixer projections + gated feed-forward inputs] -> [state update] -> [gated RMSNorm + both
 //                   output projections + residual]
 //   latent run:     [norms + low-rank projections + gated feed-forward inputs] -> [query expansion; latent append] ->
 //                   [queries into latent space] -> [attention over latents] -> [merge + values] -> [both output
 //                   projections + residual]
+//
+// Layers with a norm on each sublayer's output (grouped_step.cuh has the attention kernels):
+//
+//   grouped run:    [q, k, v rows] -> [head norms, rotation, append, attention, merge] -> [output rows] -> [up rows, squared relu] ->
+//                   [down rows], where the first and fourth begin by adding the normed output of the sublayer before to the
+//                   residual stream - every CTA for itself, the first one stores the sum for those that follow.
 //
 // Every matrix is streamed once.  bf16 weights whose rows are whole 64-element blocks take rows_mma_kernel: a persistent
 // grid of one CTA per SM, sixteen rows per unit, a team of 1, 2, 4 or 8 warps sharing a unit's columns.  Each warp keeps a ring
@@ -23,6 +30,7 @@
 #include <cstdlib>
 
 #include "bulk_async.cuh"
+#include "grouped_step.cuh"
 #include "lm_mma.cuh"
 
 namespace {
@@ -37,8 +45,8 @@ constexpr int kSub = 16;            // cached positions staged at a time
 constexpr int kHeads = 8;           // heads per CTA of the latent attention (one warp each)
 constexpr int kMaxSplits = 64;
 
-enum { PRO_LAYER_NORM = 0, PRO_RMS, PRO_CONCAT, PRO_GATED_RMS };
-enum { EPI_STORE = 0, EPI_MIXER_IN, EPI_RESIDUAL, EPI_BIAS };
+enum { PRO_LAYER_NORM = 0, PRO_RMS, PRO_CONCAT, PRO_GATED_RMS, PRO_POST_NORM };
+enum { EPI_STORE = 0, EPI_MIXER_IN, EPI_RESIDUAL, EPI_BIAS, EPI_RELU_SQUARED, EPI_SOFTCAP };
 
 struct RowsArgs {
     // weights: piece A rows [na, ka]; piece B: `pairs` gate rows followed by `pairs` up rows [2 pairs, kb] (not dual), or
@@ -47,8 +55,10 @@ struct RowsArgs {
     int na, ka, pairs, kb, dual;
     int pro, epi;
     int split;                      // PRO_CONCAT: input A is x[0, split) followed by x2 (0: all of it is x, input B is x2)
-    const float *x, *x2;            // input (x2: second input of PRO_CONCAT / PRO_GATED_RMS)
-    const float *s1, *s2;           // norm scales
+    const float *x, *x2;            // input (x2: second input of PRO_CONCAT / PRO_GATED_RMS; sublayer output of PRO_POST_NORM)
+    const float *s1, *s2;           // norm scales (PRO_POST_NORM: of the sublayer norm, of a LayerNorm of the sum or null)
+    const float *b1, *b2;           // their shifts (nullable)
+    float* x_out;                   // PRO_POST_NORM: the first CTA stores the sum here (nullable)
     const float* gate;              // PRO_GATED_RMS
     float eps, alpha;
     float *out, *out2;              // piece A rows; activated pairs
@@ -97,19 +107,95 @@ struct StagedScales {
     float4 s1[kKept], s2[kKept];
     __device__ __forceinline__ void request(const RowsArgs& a) {
         if (a.pro == PRO_CONCAT) return;
+        const float* second = a.pro == PRO_POST_NORM ? a.b1 : a.s2;
 #pragma unroll
         for (int i = 0; i < kKept; ++i) {
             const int j = (threadIdx.x + i * kThreads) * 4;
             s1[i] = load4(a.s1 + j, a.ka - j);          // zero beyond the end
-            if (a.s2) s2[i] = load4(a.s2 + j, a.ka - j);
+            if (second) s2[i] = load4(second + j, a.ka - j);
         }
     }
 };
+
+// x + LayerNorm(x2) * s1 + b1, and - with s2 - LayerNorm(that) * s2 + b2
+template <class Put> __device__ __forceinline__ void stage_post_norm(const RowsArgs& a, const StagedScales& sc, float* scratch, Put put) {
+    const int step = kThreads * 4, j0 = threadIdx.x * 4, quads = (padded(a.ka) + step - 1) / step;
+    float4 y[kKept], x[kKept];
+#pragma unroll
+    for (int i = 0; i < kKept; ++i) {
+        const int j = j0 + i * step;
+        y[i] = load4(a.x2 + j, a.ka - j);
+        x[i] = load4(a.x + j, a.ka - j);
+    }
+    auto total = [](const float4& w) { return (w.x + w.y) + (w.z + w.w); };
+    auto square = [&](float q, const float4& w, int j, float mean) {
+        if (j < a.ka) q = fmaf(w.x - mean, w.x - mean, q);
+        if (j + 1 < a.ka) q = fmaf(w.y - mean, w.y - mean, q);
+        if (j + 2 < a.ka) q = fmaf(w.z - mean, w.z - mean, q);
+        if (j + 3 < a.ka) q = fmaf(w.w - mean, w.w - mean, q);
+        return q;
+    };
+    float s = 0.f, q = 0.f;
+#pragma unroll
+    for (int i = 0; i < kKept; ++i) s += total(y[i]);
+    for (int i = kKept; i < quads; ++i) s += total(load4(a.x2 + j0 + i * step, a.ka - (j0 + i * step)));
+    const float mean = lm::block_sum(s, scratch) / (float)a.ka;
+#pragma unroll
+    for (int i = 0; i < kKept; ++i) q = square(q, y[i], j0 + i * step, mean);
+    for (int i = kKept; i < quads; ++i) q = square(q, load4(a.x2 + j0 + i * step, a.ka - (j0 + i * step)), j0 + i * step, mean);
+    const float rstd = 1.0f / sqrtf(lm::block_sum(q, scratch) / (float)a.ka + a.eps);
+    auto sum = [&](const float4& x, const float4& y, const float4& g, const float4& b) {
+        return make_float4(x.x + fmaf((y.x - mean) * rstd, g.x, b.x), x.y + fmaf((y.y - mean) * rstd, g.y, b.y), x.z + fmaf((y.z - mean) * rstd, g.z, b.z),
+                           x.w + fmaf((y.w - mean) * rstd, g.w, b.w));
+    };
+    auto late = [&](int j) { return sum(load4(a.x + j, a.ka - j), load4(a.x2 + j, a.ka - j), load4(a.s1 + j, a.ka - j), load4(a.b1 + j, a.ka - j)); };
+#pragma unroll
+    for (int i = 0; i < kKept; ++i) x[i] = sum(x[i], y[i], sc.s1[i], sc.s2[i]);       // zero beyond the end: scale and shift are
+    if (a.x_out && blockIdx.x == 0) {
+        auto store = [&](const float4& w, int j) {
+            if (j < a.ka) a.x_out[j] = w.x;
+            if (j + 1 < a.ka) a.x_out[j + 1] = w.y;
+            if (j + 2 < a.ka) a.x_out[j + 2] = w.z;
+            if (j + 3 < a.ka) a.x_out[j + 3] = w.w;
+        };
+#pragma unroll
+        for (int i = 0; i < kKept; ++i) store(x[i], j0 + i * step);
+        for (int i = kKept; i < quads; ++i) store(late(j0 + i * step), j0 + i * step);
+    }
+    float mean2 = 0.f, rstd2 = 1.f;
+    if (a.s2) {
+        s = q = 0.f;
+#pragma unroll
+        for (int i = 0; i < kKept; ++i) s += total(x[i]);
+        for (int i = kKept; i < quads; ++i) s += total(late(j0 + i * step));
+        mean2 = lm::block_sum(s, scratch) / (float)a.ka;
+#pragma unroll
+        for (int i = 0; i < kKept; ++i) q = square(q, x[i], j0 + i * step, mean2);
+        for (int i = kKept; i < quads; ++i) q = square(q, late(j0 + i * step), j0 + i * step, mean2);
+        rstd2 = 1.0f / sqrtf(lm::block_sum(q, scratch) / (float)a.ka + a.eps);
+    }
+    auto emit = [&](float4 w, int j) {
+        if (j >= padded(a.ka)) return;
+        if (a.s2) {
+            const float4 g = load4(a.s2 + j, a.ka - j), b = a.b2 ? load4(a.b2 + j, a.ka - j) : make_float4(0.f, 0.f, 0.f, 0.f);
+            w = make_float4(fmaf((w.x - mean2) * rstd2, g.x, b.x), fmaf((w.y - mean2) * rstd2, g.y, b.y), fmaf((w.z - mean2) * rstd2, g.z, b.z),
+                            fmaf((w.w - mean2) * rstd2, g.w, b.w));
+        }
+        put(0, j, w);
+    };
+#pragma unroll
+    for (int i = 0; i < kKept; ++i) emit(x[i], j0 + i * step);
+    for (int i = kKept; i < quads; ++i) emit(late(j0 + i * step), j0 + i * step);
+}
 
 // The input vectors of a product, normalised or gated, four elements at a time: put(piece, j, values); zeros from the end of a
 // vector to its padded length.
 template <class Put> __device__ __forceinline__ void stage_input(const RowsArgs& a, const StagedScales& sc, float* scratch, Put put) {
     const int step = kThreads * 4, j0 = threadIdx.x * 4;
+    if (a.pro == PRO_POST_NORM) {
+        stage_post_norm(a, sc, scratch, put);
+        return;
+    }
     if (a.pro == PRO_LAYER_NORM || a.pro == PRO_RMS) {
         float4 v[kKept];
 #pragma unroll
@@ -141,7 +227,8 @@ template <class Put> __device__ __forceinline__ void stage_input(const RowsArgs&
         auto emit = [&](const float4& w, int j, const float4& s1, const float4& s2) {
             if (j >= padded(a.ka)) return;
             const float x = (w.x - mean) * rstd, y = (w.y - mean) * rstd, z = (w.z - mean) * rstd, t = (w.w - mean) * rstd;
-            put(0, j, make_float4(x * s1.x, y * s1.y, z * s1.z, t * s1.w));
+            const float4 b = a.b1 ? load4(a.b1 + j, a.ka - j) : make_float4(0.f, 0.f, 0.f, 0.f);
+            put(0, j, make_float4(fmaf(x, s1.x, b.x), fmaf(y, s1.y, b.y), fmaf(z, s1.z, b.z), fmaf(t, s1.w, b.w)));
             if (a.s2) put(1, j, make_float4(x * s2.x, y * s2.y, z * s2.z, t * s2.w));
         };
 #pragma unroll
@@ -195,6 +282,10 @@ __device__ __forceinline__ void finish_row(const RowsArgs& a, int row, float v) 
         v = fmaf(a.alpha, v, a.resid[row]);
     } else if (a.epi == EPI_BIAS) {
         v += a.bias[row];
+    } else if (a.epi == EPI_RELU_SQUARED) {
+        v = v > 0.f ? v * v : 0.f;
+    } else if (a.epi == EPI_SOFTCAP) {
+        v = a.alpha * tanhf(v / a.alpha);
     }
     a.out[row] = v;
 }
@@ -407,17 +498,31 @@ bool make_block_map(CUtensorMap* map, const void* base, uint64_t rows, uint64_t 
               CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-// x0 = x = embedding row of the token; an id outside the table is clamped and flagged
+// (cos, sin) of the step's position for one frequency table
+struct AngleTable {
+    const float* freqs;
+    float2* out;
+    int pairs;
+    float magnitude;
+};
+
+// x0 = x = embedding row of the token; an id outside the table is clamped and flagged.  The last n_angles CTAs fill an angle table each.
 template <class T>
 __global__ void __launch_bounds__(kThreads) embed_kernel(const int32_t* token, const T* __restrict__ table, int vocab, int width, float* x0, float* x,
-                                                         int* status) {
+                                                         const AngleTable* __restrict__ angles, int n_angles, const uint32_t* d_pos, int* status) {
     rcu_kernel_entry();
+    const int rows = (int)gridDim.x - n_angles;
+    if ((int)blockIdx.x >= rows) {
+        const AngleTable t = angles[blockIdx.x - rows];
+        for (int i = threadIdx.x; i < t.pairs; i += kThreads) t.out[i] = lm::rotary_angle(t.freqs, t.pairs, i, *d_pos, t.magnitude);
+        return;
+    }
     int t = *token;
     if (t < 0 || t >= vocab) {
         if (threadIdx.x == 0 && blockIdx.x == 0) atomicOr(status, RCU_DEVFLAG_BOUNDS);
         t = t < 0 ? 0 : vocab - 1;
     }
-    for (int j = blockIdx.x * kThreads + threadIdx.x; j < width; j += gridDim.x * kThreads) {
+    for (int j = blockIdx.x * kThreads + threadIdx.x; j < width; j += rows * kThreads) {
         const float v = to_f32<T>(table[(size_t)t * width + j]);
         x0[j] = v;
         x[j] = v;
@@ -873,7 +978,10 @@ struct rcu_stack {
     const void *embed, *head;
     const float* final_norm;
     float* pool = nullptr;              // every f32 vector below
-    float *x0, *xa, *xb, *mix, *act, *y, *q, *qa, *partial, *logits;
+    float *x0, *xa, *xb, *mix, *act, *y, *sub, *q, *qa, *partial, *logits;
+    float *angle_pool, *angle_tables, *arrived;      // (cos, sin) pairs; AngleTable[n_angles]; counters of the grouped attention
+    std::vector<float2*> run_angles;                 // per run: its pairs (null: no grouped mixer)
+    int n_angles = 0;
     uint32_t* d_pos = nullptr;
     uint32_t position = 0, kernels_per_step = 0;
     uint64_t steps = 0;
@@ -886,6 +994,15 @@ struct rcu_stack {
 namespace {
 
 int latent_splits(const rcu_stack_run& r) { return (int)std::min<uint32_t>(kMaxSplits, std::max<uint32_t>(1, (std::min(r.window, r.ring_rows) + kSub - 1) / kSub)); }
+
+uint64_t grouped_seen(const rcu_stack_run& r) {      // rows a token can see at most
+    const uint64_t most = r.chunk ? r.chunk : r.window ? r.window : r.ring_rows;
+    return std::min<uint64_t>(most, r.ring_rows);
+}
+int grouped_splits(const rcu_device* dev, const rcu_stack_run& r, int dt) {
+    const int per = gstep::takes_mma(dt, (int)r.dim, (int)r.vdim, r.state) ? gstep::kMmaHeads : gstep::kFmaHeads;
+    return gstep::splits(dev->sm_count, (int)r.kv_heads * gstep::head_groups((int)r.heads, (int)r.kv_heads, per), grouped_seen(r));
+}
 
 // Warps per team.  A CTA's time is bound below by the memory system (its units' items, one after the other) and by the longest
 // chain of items a warp works through, an item taking a warp about twice as long as the memory system; ending a unit
@@ -977,9 +1094,50 @@ template <class T> rcu_status run_step(rcu_stack* s, const int32_t* token, float
     const rcu_stack_config& c = s->cfg;
     const int W = (int)c.width;
     float *x = s->xa, *other = s->xb;
-    RCU_CUDA(dev, rcu_launch(dev, embed_kernel<T>, (W + kThreads - 1) / kThreads, kThreads, 0, token, (const T*)s->embed, (int)c.vocab, W, s->x0, x, dev->d_status));
+    RCU_CUDA(dev, rcu_launch(dev, embed_kernel<T>, (W + kThreads - 1) / kThreads + s->n_angles, kThreads, 0, token, (const T*)s->embed, (int)c.vocab, W, s->x0, x,
+                             (const AngleTable*)s->angle_tables, s->n_angles, s->d_pos, dev->d_status));
     RCU_LAUNCH_CHECK(dev);
-    for (const rcu_stack_run& r : s->runs) {
+    const float *after = nullptr, *after_shift = nullptr;      // post-norm layers: the norm that awaits the last sublayer's output
+    // the residual stream as a product's input; with a sublayer output waiting, the sum goes to the other stream buffer
+    auto stream_input = [&](RowsArgs& a) {
+        a.ka = W;
+        a.x = x;
+        a.eps = c.eps;
+        a.pro = PRO_CONCAT;
+        if (after) {
+            a.pro = PRO_POST_NORM; a.x2 = s->sub; a.s1 = after; a.b1 = after_shift; a.x_out = other;
+            std::swap(x, other);
+        }
+    };
+    for (size_t k = 0; k < s->runs.size(); ++k) {
+        const rcu_stack_run& r = s->runs[k];
+        if (c.layer == RCU_LAYER_POST_NORM) {
+            const int H = (int)r.heads, G = (int)r.kv_heads, D = (int)r.dim, E = (int)r.vdim;
+            RowsArgs in = {};
+            stream_input(in);
+            in.wa = r.mix_in; in.na = (H + G) * D + G * E; in.epi = r.mix_bias ? EPI_BIAS : EPI_STORE; in.bias = (const float*)r.mix_bias; in.out = s->mix;
+            STACK_TRY(launch_rows<T>(dev, in));
+            const gstep::Args at{s->mix, (const float*)r.mix_norm, (const float*)r.kv_norm, s->run_angles[k], (const float*)r.sink, r.state, s->d_pos, s->y, s->partial,
+                                 (uint32_t*)s->arrived, H, G, D, E, (int)r.rot_pairs, (int)r.ring_rows,
+                                 r.window ? (int)std::min<uint32_t>(r.window, 1u << 30) : 1 << 30, (int)std::min<uint32_t>(r.chunk, 1u << 30), c.eps, r.scale};
+            STACK_TRY(gstep::launch(dev, c.weight_dt, at, grouped_splits(dev, r, c.weight_dt)));
+            RowsArgs o = {};
+            o.wa = r.out; o.na = W; o.ka = H * E; o.pro = PRO_CONCAT; o.x = s->y; o.out = s->sub;
+            o.epi = r.out_bias ? EPI_BIAS : EPI_STORE; o.bias = (const float*)r.out_bias;
+            STACK_TRY(launch_rows<T>(dev, o));
+            after = (const float*)r.norm1; after_shift = (const float*)r.norm1_shift;
+            if (r.ff) {
+                RowsArgs up = {};
+                stream_input(up);
+                up.wa = r.gate_up; up.na = (int)r.ff; up.epi = EPI_RELU_SQUARED; up.out = s->act;
+                STACK_TRY(launch_rows<T>(dev, up));
+                RowsArgs down = {};
+                down.wa = r.down; down.na = W; down.ka = (int)r.ff; down.pro = PRO_CONCAT; down.x = s->act; down.out = s->sub;
+                STACK_TRY(launch_rows<T>(dev, down));
+                after = (const float*)r.norm2; after_shift = (const float*)r.norm2_shift;
+            }
+            continue;
+        }
         if (r.enter) {                          // x <- W_enter [x; x0] + step
             RowsArgs a = {};
             a.wa = r.enter; a.na = W; a.ka = 2 * W;
@@ -1027,7 +1185,15 @@ template <class T> rcu_status run_step(rcu_stack* s, const int32_t* token, float
         STACK_TRY(launch_rows<T>(dev, out));
     }
     RowsArgs head = {};
-    head.wa = s->head; head.na = (int)c.vocab; head.ka = W; head.pro = PRO_LAYER_NORM; head.x = x; head.s1 = s->final_norm; head.eps = c.eps; head.out = logits;
+    if (after) {
+        stream_input(head);
+        head.x_out = nullptr;
+        head.s2 = s->final_norm; head.b2 = (const float*)c.final_shift;
+    } else {
+        head.ka = W; head.pro = PRO_LAYER_NORM; head.x = x; head.s1 = s->final_norm; head.b1 = (const float*)c.final_shift; head.eps = c.eps;
+    }
+    head.wa = s->head; head.na = (int)c.vocab; head.out = logits;
+    if (c.logit_softcap > 0.f) { head.epi = EPI_SOFTCAP; head.alpha = c.logit_softcap; }
     STACK_TRY(launch_rows<T>(dev, head));
     RCU_CUDA(dev, rcu_launch(dev, argmax_next_kernel, 1, 1024, 0, logits, (int)c.vocab, argmax, s->d_pos));
     RCU_LAUNCH_CHECK(dev);
@@ -1047,15 +1213,38 @@ rcu_status rcu_stack_create(rcu_device* dev, const rcu_stack_config* cfg, const 
     if (!dev || !cfg || !runs || !embed || !final_norm || !head || !out) return RCU_ERR_INVALID_ARG;
     RCU_REQUIRE(dev, cfg->weight_dt == RCU_BF16 || cfg->weight_dt == RCU_F32, "stack: weights are bf16 or f32");
     RCU_REQUIRE(dev, cfg->width > 0 && cfg->vocab > 0 && cfg->n_runs > 0, "stack: empty model");
-    size_t mix = 0, act = 1, y = 0, q = 1, qa = 1, partial = 1;
+    RCU_REQUIRE(dev, cfg->layer == RCU_LAYER_PARALLEL || cfg->layer == RCU_LAYER_POST_NORM, "stack: unknown kind of layer %d", cfg->layer);
+    const bool post = cfg->layer == RCU_LAYER_POST_NORM;
+    size_t mix = 0, act = 1, y = 0, q = 1, qa = 1, partial = 1, arrived = 1, pairs = 1;
+    std::vector<int> table_of(cfg->n_runs, -1);
+    std::vector<uint32_t> table_run;                 // the run each angle table comes from
     for (uint32_t i = 0; i < cfg->n_runs; ++i) {
         const rcu_stack_run& r = runs[i];
+        if (post != (r.mixer == RCU_MIXER_GROUPED))
+            return rcu_fail(dev, RCU_ERR_UNSUPPORTED, "stack: run %u: post-norm layers take grouped heads, parallel ones the other mixers", i);
         RCU_REQUIRE(dev, r.norm1 && r.mix_in && r.mix_norm && r.out && r.state && r.heads && r.dim && r.vdim, "stack: run %u lacks a weight or a size", i);
         RCU_REQUIRE(dev, r.ff == 0 || (r.norm2 && r.gate_up && r.down), "stack: run %u lacks a feed-forward weight", i);
         RCU_REQUIRE(dev, r.heads <= 65535, "stack: run %u has too many heads", i);
+        RCU_REQUIRE(dev, !post || (r.norm1_shift && (r.ff == 0 || r.norm2_shift) && !r.enter), "stack: run %u lacks a norm's shift, or enters a pass", i);
         if (r.mixer == RCU_MIXER_LIGHTNING) {
             RCU_REQUIRE(dev, r.decay, "stack: run %u has no decay", i);
             mix = std::max(mix, (size_t)r.heads * 2 * (r.dim + r.vdim));
+        } else if (r.mixer == RCU_MIXER_GROUPED) {
+            RCU_REQUIRE(dev, r.kv_heads && r.heads % r.kv_heads == 0 && r.kv_norm && (r.rot_pairs == 0 || r.freqs) && 2 * r.rot_pairs <= r.dim && r.ring_rows,
+                        "stack: run %u lacks a weight or a size", i);
+            if (r.dim > 1024 || r.vdim > 512) return rcu_fail(dev, RCU_ERR_UNSUPPORTED, "stack: run %u: heads of %u and %u (at most 1024 and 512)", i, r.dim, r.vdim);
+            mix = std::max(mix, (size_t)(r.heads + r.kv_heads) * r.dim + (size_t)r.kv_heads * r.vdim);
+            partial = std::max(partial, (size_t)grouped_splits(dev, r, cfg->weight_dt) * r.heads * gstep::pitch_of((int)r.vdim));
+            arrived = std::max(arrived, (size_t)r.heads);
+            for (size_t t = 0; t < table_run.size() && table_of[i] < 0; ++t) {
+                const rcu_stack_run& o = runs[table_run[t]];
+                if (o.freqs == r.freqs && o.rot_pairs == r.rot_pairs && o.rot_magnitude == r.rot_magnitude) table_of[i] = (int)t;
+            }
+            if (table_of[i] < 0) {
+                table_of[i] = (int)table_run.size();
+                table_run.push_back(i);
+            }
+            pairs = std::max(pairs, (size_t)r.rot_pairs);
         } else {
             RCU_REQUIRE(dev, r.mixer == RCU_MIXER_LATENT, "stack: run %u has an unknown mixer", i);
             RCU_REQUIRE(dev, r.q_rank && r.kv_rank && r.kv_norm && r.uq && r.ukv && (r.rot_pairs == 0 || r.freqs) && 2 * r.rot_pairs <= r.rot_dim,
@@ -1076,8 +1265,9 @@ rcu_status rcu_stack_create(rcu_device* dev, const rcu_stack_config* cfg, const 
     s->cfg = *cfg;
     s->runs.assign(runs, runs + cfg->n_runs);
     s->embed = embed; s->head = head; s->final_norm = (const float*)final_norm;
-    const size_t sizes[] = {cfg->width, cfg->width, cfg->width, mix, act, y, q, qa, partial};
-    float** ptrs[] = {&s->x0, &s->xa, &s->xb, &s->mix, &s->act, &s->y, &s->q, &s->qa, &s->partial};
+    const size_t n_tables = table_run.size();
+    const size_t sizes[] = {cfg->width, cfg->width, cfg->width, mix, act, y, cfg->width, q, qa, partial, 2 * pairs * n_tables, n_tables * (sizeof(AngleTable) / 4), arrived};
+    float** ptrs[] = {&s->x0, &s->xa, &s->xb, &s->mix, &s->act, &s->y, &s->sub, &s->q, &s->qa, &s->partial, &s->angle_pool, &s->angle_tables, &s->arrived};
     size_t total = 64;
     for (size_t n : sizes) total += (n + 63) & ~(size_t)63;
     void* p = nullptr;
@@ -1090,7 +1280,17 @@ rcu_status rcu_stack_create(rcu_device* dev, const rcu_stack_config* cfg, const 
         *ptrs[i] = at;
         at += (sizes[i] + 63) & ~(size_t)63;
     }
-    st = rcu_stack_set_position(s, 0);
+    std::vector<AngleTable> tables;
+    for (size_t t = 0; t < n_tables; ++t) {
+        const rcu_stack_run& r = runs[table_run[t]];
+        tables.push_back(AngleTable{(const float*)r.freqs, (float2*)s->angle_pool + t * pairs, (int)r.rot_pairs, r.rot_magnitude});
+    }
+    for (uint32_t i = 0; i < cfg->n_runs; ++i) s->run_angles.push_back(table_of[i] < 0 ? nullptr : tables[table_of[i]].out);
+    s->n_angles = (int)n_tables;
+    if (n_tables) st = rcu_h2d(dev, s->angle_tables, tables.data(), n_tables * sizeof(AngleTable));
+    if (st == RCU_OK) st = rcu_memset(dev, s->arrived, 0, arrived * 4);
+    if (st == RCU_OK) st = rcu_sync(dev);             // the tables' host copy ends with this call
+    if (st == RCU_OK) st = rcu_stack_set_position(s, 0);
     if (st != RCU_OK) { rcu_free(dev, p); delete s; return st; }
     *out = s;
     return RCU_OK;
@@ -1121,7 +1321,10 @@ rcu_status rcu_stack_step(rcu_stack* s, const int32_t* token_dev, float* logits_
     if (!s || !token_dev || !logits_dev) return RCU_ERR_INVALID_ARG;
     rcu_device* dev = s->dev;
     for (const rcu_stack_run& r : s->runs)
-        RCU_REQUIRE(dev, r.mixer != RCU_MIXER_LATENT || r.ring_rows >= r.window || s->position < r.ring_rows, "stack: the latent cache is full (%u rows)", r.ring_rows);
+    {
+        const uint64_t seen = r.mixer == RCU_MIXER_GROUPED && r.chunk ? r.chunk : r.mixer == RCU_MIXER_GROUPED && !r.window ? ~0ull : r.window;
+        RCU_REQUIRE(dev, r.mixer == RCU_MIXER_LIGHTNING || r.ring_rows >= seen || s->position < r.ring_rows, "stack: the cache is full (%u rows)", r.ring_rows);
+    }
     DevGuard g(dev->ordinal);
     const bool use_graph = std::getenv("RCU_NO_GRAPH") == nullptr && dev->stream != nullptr;
     if (!use_graph || s->steps == 0) {      // the first step sets kernel attributes and counts the launches

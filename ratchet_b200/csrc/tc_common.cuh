@@ -112,10 +112,10 @@ template <class Out> struct GemmEpilogue {
     const Out* bias;          // per output column, nullable
     const float* resid;       // f32 output only, nullable
     float alpha;
-    int silu_cols;            // columns below this pass through silu (after the bias)
+    LinearAct act;            // after the bias
     __device__ __forceinline__ float value(float acc, int col) const {
         const float v = acc + (bias ? to_f32<Out>(bias[col]) : 0.f);
-        return col < silu_cols ? v / (1.0f + expf(-v)) : v;
+        return col < act.cols ? act(v) : v;
     }
     __device__ __forceinline__ Out operator()(float acc, int col, size_t idx) const {
         float v = value(acc, col);
@@ -150,5 +150,5 @@ struct TcLinear {
     int out_dt = RCU_F16;
     const float* resid = nullptr;
     float alpha = 1.f;
-    int silu_cols = 0;
+    LinearAct act = {};
 };

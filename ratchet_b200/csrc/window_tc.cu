@@ -1,5 +1,5 @@
-// Windowed attention of a long bf16 block on the 5th-generation tensor cores (tcgen05), behind the interface of
-// rcu_window_attention (latent_attention.cu), which sends blocks of at least 256 tokens here.
+// Masked attention of a long bf16 block on the 5th-generation tensor cores (tcgen05), behind the interfaces of
+// rcu_window_attention and rcu_grouped_attention (rcu_attend in latent_attention.cu sends blocks of at least 256 tokens here).
 //
 // CTA = 256 queries of one head, in two tiles of 128 that take turns: while the softmax warps of one tile work, the tensor core
 // runs the other tile's products.
@@ -27,8 +27,10 @@ constexpr int kBlockQ = kTileQ * 128, kBlockK = kTileK * 128;       // bytes of 
 
 struct TcArgs {
     __nv_bfloat16* out;
-    int T, L, H, D, R, E, window;
+    int T, L, H, G, D, R, E;
+    Visible see;
     float scale;
+    const float* sink;
     int* status;
 };
 
@@ -52,12 +54,12 @@ window_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_constant
     __shared__ volatile int abort_flag;
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int h = blockIdx.y, i0 = blockIdx.x * 2 * kTileQ;
+    const int h = blockIdx.y, hk = h / (a.H / a.G), i0 = blockIdx.x * 2 * kTileQ;
     const int base = a.L - a.T + i0, nq = min(2 * kTileQ, a.T - i0);    // key row of the CTA's first query; its queries
-    const int first = max(0, base - a.window + 1);
+    const int first = a.see.first(base);
     const int tiles = (base + nq - 1 - first) / kTileK + 1;
     // key tiles [lo, hi) that some query of tile w sees
-    auto lo_of = [&](int w) { return (max(0, base + w * kTileQ - a.window + 1) - first) / kTileK; };
+    auto lo_of = [&](int w) { return (a.see.first(base + w * kTileQ) - first) / kTileK; };
     auto hi_of = [&](int w) { return w * kTileQ < nq ? (min(base + (w + 1) * kTileQ, base + nq) - 1 - first) / kTileK + 1 : 0; };
 
     if (threadIdx.x == 0) {
@@ -94,11 +96,11 @@ window_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_constant
                 const int s = n & 1, j0 = first + n * kTileK;
                 if (n >= 2 && !mbar_wait(&k_empty[s], ((n >> 1) - 1) & 1, &abort_flag, a.status)) break;
                 mbar_expect_tx(&k_full[s], nb * kBlockK);
-                for (int b = 0; b < nd; ++b) tma_load_3d(ks + (s * nb + b) * kBlockK, &kmap, b * 64, h, j0, &k_full[s]);
+                for (int b = 0; b < nd; ++b) tma_load_3d(ks + (s * nb + b) * kBlockK, &kmap, b * 64, hk, j0, &k_full[s]);
                 for (int b = nd; b < nb; ++b) tma_load_2d(ks + (s * nb + b) * kBlockK, &krmap, (b - nd) * 64, j0, &k_full[s]);
                 if (n >= 2 && !mbar_wait(&v_empty[s], ((n >> 1) - 1) & 1, &abort_flag, a.status)) break;
                 mbar_expect_tx(&v_full[s], eb * kBlockK);
-                for (int b = 0; b < eb; ++b) tma_load_3d(vs + (s * eb + b) * kBlockK, &vmap, b * 64, h, j0, &v_full[s]);
+                for (int b = 0; b < eb; ++b) tma_load_3d(vs + (s * eb + b) * kBlockK, &vmap, b * 64, hk, j0, &v_full[s]);
             }
         }
     } else if (warp == 1) {
@@ -150,6 +152,7 @@ window_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_constant
         const int lo = lo_of(w), hi = hi_of(w);
         const uint32_t t = tmem + (uint32_t)w * 256 + ((uint32_t)(quarter * 32) << 16);
         const int row0 = base + w * kTileQ + quarter * 32, row1 = row0 + 31;   // the warp's key rows
+        const int low = a.see.first(row), low1 = a.see.first(row1);
         const float sc = a.scale * 1.4426950408889634f;                       // scores in units of log 2
         const int ocols = (a.E + 31) & ~31;
         float m = -INFINITY, l = 0.f;
@@ -163,7 +166,7 @@ window_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_constant
             tmem_ld_32x32(t + 32, s + 32);
             const int j0 = first + n * kTileK;
             float top = -INFINITY;
-            if (j0 + kTileK - 1 <= row0 && j0 > row1 - a.window) {
+            if (j0 + kTileK - 1 <= row0 && j0 >= low1) {
 #pragma unroll
                 for (int j = 0; j < 64; ++j) {
                     s[j] *= sc;
@@ -172,7 +175,7 @@ window_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_constant
             } else {
 #pragma unroll
                 for (int j = 0; j < 64; ++j) {
-                    s[j] = j0 + j <= row && j0 + j > row - a.window ? s[j] * sc : -INFINITY;
+                    s[j] = j0 + j <= row && j0 + j >= low ? s[j] * sc : -INFINITY;
                     top = fmaxf(top, s[j]);
                 }
             }
@@ -213,6 +216,7 @@ window_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_constant
             ok = __all_sync(0xffffffffu, mbar_wait(&pv_done[w], (hi - lo - 1) & 1, &abort_flag, a.status));
             tc_fence_after();
             if (ok) {
+                if (a.sink) l += ex2(a.sink[h] * 1.4426950408889634f - m);
                 const float inv = 1.0f / l;
                 __nv_bfloat16* out = a.out + ((size_t)(i0 + r) * a.H + h) * a.E;
                 for (int c = 0; c < ocols; c += 32) {
@@ -265,20 +269,24 @@ bool make_row_map(CUtensorMap* map, const void* base, uint64_t cols, uint64_t ro
 
 rcu_status rcu_window_tc(rcu_device* dev, const WindowArgs& a) {
     const int Q = a.D + a.R, nb = (a.D + 63) / 64 + (a.R + 63) / 64, eb = (a.E + 63) / 64;
-    if (a.T < 256 || a.D < 8 || a.R < 8 || a.D % 8 || a.R % 8 || a.E % 8 || a.E > 128 || nb > 4 || a.shared_pitch % 8) return RCU_ERR_UNSUPPORTED;
+    if (a.T < 256 || a.D < 8 || a.D % 8 || a.R % 8 || a.E % 8 || a.E > 128 || nb > 4 || a.shared_pitch % 8) return RCU_ERR_UNSUPPORTED;
     if ((reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.kv) | reinterpret_cast<uintptr_t>(a.shared) | reinterpret_cast<uintptr_t>(a.out)) & 15)
         return RCU_ERR_UNSUPPORTED;
     const size_t smem = 1024 + (size_t)2 * nb * kBlockQ + (size_t)2 * (nb + eb) * kBlockK;
     if (smem + 512 > (size_t)dev->smem_optin) return RCU_ERR_UNSUPPORTED;
     const __nv_bfloat16 *q = (const __nv_bfloat16*)a.q, *kv = (const __nv_bfloat16*)a.kv;
-    const uint64_t kvp = (uint64_t)a.H * (a.D + a.E), qp = (uint64_t)a.H * Q;
+    const uint64_t kvp = (uint64_t)a.G * (a.D + a.E), qp = (uint64_t)a.H * Q;
     CUtensorMap qm, qr, km, kr, vm;
-    if (!make_head_map(&qm, q, a.D, a.H, a.T, Q, qp, kTileQ) || !make_head_map(&qr, q + a.D, a.R, a.H, a.T, Q, qp, kTileQ) ||
-        !make_head_map(&km, kv, a.D, a.H, a.L, a.D, kvp, kTileK) || !make_row_map(&kr, a.shared, a.R, a.L, a.shared_pitch, kTileK) ||
-        !make_head_map(&vm, kv + (size_t)a.H * a.D, a.E, a.H, a.L, a.E, kvp, kTileK))
+    if (!make_head_map(&qm, q, a.D, a.H, a.T, Q, qp, kTileQ) || !make_head_map(&km, kv, a.D, a.G, a.L, a.D, kvp, kTileK) ||
+        !make_head_map(&vm, kv + (size_t)a.G * a.D, a.E, a.G, a.L, a.E, kvp, kTileK))
+        return rcu_fail(dev, RCU_ERR_CUDA, "window_attention: cuTensorMapEncodeTiled failed (T=%d L=%d H=%d)", a.T, a.L, a.H);
+    if (a.R == 0) {
+        qr = qm;              // no shared features: never read
+        kr = km;
+    } else if (!make_head_map(&qr, q + a.D, a.R, a.H, a.T, Q, qp, kTileQ) || !make_row_map(&kr, a.shared, a.R, a.L, a.shared_pitch, kTileK))
         return rcu_fail(dev, RCU_ERR_CUDA, "window_attention: cuTensorMapEncodeTiled failed (T=%d L=%d H=%d)", a.T, a.L, a.H);
     RCU_CUDA(dev, cudaFuncSetAttribute(window_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    const TcArgs t{(__nv_bfloat16*)a.out, a.T, a.L, a.H, a.D, a.R, a.E, a.window, a.scale, dev->d_status};
+    const TcArgs t{(__nv_bfloat16*)a.out, a.T, a.L, a.H, a.G, a.D, a.R, a.E, a.see, a.scale, a.sink, dev->d_status};
     const dim3 grid((a.T + 2 * kTileQ - 1) / (2 * kTileQ), a.H);
     RCU_CUDA(dev, rcu_launch(dev, window_tc_kernel, grid, kThreadsW, smem, qm, qr, km, kr, vm, t));
     RCU_LAUNCH_CHECK(dev);

@@ -331,15 +331,52 @@ class Device:
 
     # ------------------------------------------------------------------ ops of models with a 32-bit residual stream
     def linear(self, w: Buffer, x: Buffer, bias: Optional[Buffer] = None, resid: Optional[Buffer] = None, alpha: float = 1.0, x_col: int = 0,
-               silu_cols: int = 0, dt: Optional[int] = None, out: Optional[Buffer] = None) -> Buffer:
+               act: Optional[str] = None, act_cols: Optional[int] = None, act_param: float = 0.0, dt: Optional[int] = None,
+               out: Optional[Buffer] = None) -> Buffer:
         out = out or self.empty(x.dt if dt is None else dt, list(x.shape[:-1]) + [w.shape[0]])
-        self.check(self._lib.rcu_linear(self.handle, self._ref(w), self._ref(x), x_col, self._ref(bias), silu_cols,
-                                        self._ref(resid), alpha, self._ref(out)))
+        self.check(self._lib.rcu_linear(self.handle, self._ref(w), self._ref(x), x_col, self._ref(bias), capi.LINEAR_ACTS[act],
+                                        w.shape[0] if act_cols is None else act_cols, act_param, self._ref(resid), alpha, self._ref(out)))
         return out
 
-    def norm_rows(self, kind: int, x: Buffer, scale: Buffer, eps: float, dt: int, col: int = 0, gate: Optional[Buffer] = None, gate_col: int = 0):
+    def norm_rows(self, kind: int, x: Buffer, scale: Buffer, eps: float, dt: int, col: int = 0, gate: Optional[Buffer] = None, gate_col: int = 0,
+                  shift: Optional[Buffer] = None):
         out = self.empty(dt, list(x.shape[:-1]) + [scale.numel])
-        self.check(self._lib.rcu_norm_rows(self.handle, kind, self._ref(x), col, self._ref(scale), self._ref(gate), gate_col, eps, self._ref(out)))
+        self.check(self._lib.rcu_norm_rows(self.handle, kind, self._ref(x), col, self._ref(scale), self._ref(shift), self._ref(gate), gate_col, eps,
+                                           self._ref(out)))
+        return out
+
+    def stream_rows(self, x: Buffer, copy_dt: int) -> Buffer:
+        w = x.shape[1]
+        out = self.empty(capi.F32, (x.shape[0], w + (w + 1) // 2 if copy_dt == capi.BF16 else w))
+        self.check(self._lib.rcu_stream_rows(self.handle, self._ref(x), copy_dt, self._ref(out)))
+        return out
+
+    def post_norm(self, x: Buffer, y: Buffer, scale: Buffer, shift: Buffer, eps: float, out: Optional[Buffer] = None) -> Buffer:
+        out = out or self.empty(capi.F32, x.shape)
+        self.check(self._lib.rcu_post_norm(self.handle, self._ref(x), self._ref(y), self._ref(scale), self._ref(shift), eps, self._ref(out)))
+        return out
+
+    def rotary_angles(self, freqs: Buffer, magnitude: float, position: int, tokens: int) -> Buffer:
+        out = self.empty(capi.F32, (tokens, 2 * freqs.shape[1]))
+        self.check(self._lib.rcu_rotary_angles(self.handle, self._ref(freqs), magnitude, position, self._ref(out)))
+        return out
+
+    def norm_rotary(self, x: Buffer, heads: int, scale: Buffer, eps: float, angles: Buffer, col: int = 0) -> Buffer:
+        out = self.empty(x.dt, (x.shape[0], heads, scale.numel))
+        self.check(self._lib.rcu_norm_rotary(self.handle, self._ref(x), col, self._ref(scale), eps, self._ref(angles), self._ref(out)))
+        return out
+
+    def kv_append(self, x: Buffer, kv_heads: int, scale: Buffer, eps: float, angles: Buffer, position: int, keep: int, ring: Buffer, rows: int, col: int = 0):
+        out = self.empty(ring.dt, (rows, ring.shape[1]))
+        self.check(self._lib.rcu_kv_append(self.handle, self._ref(x), col, kv_heads, self._ref(scale), eps, self._ref(angles), position, keep,
+                                           self._ref(ring), self._ref(out)))
+        return out
+
+    def grouped_attention(self, q: Buffer, kv: Buffer, kv_heads: int, vdim: int, scale: float, sink: Optional[Buffer] = None, window: int = 0, chunk: int = 0,
+                          position: int = 0) -> Buffer:
+        out = self.empty(q.dt, (q.shape[0], q.shape[1] * vdim))
+        self.check(self._lib.rcu_grouped_attention(self.handle, self._ref(q), self._ref(kv), self._ref(sink), kv_heads, vdim, window, chunk, position, scale,
+                                                   self._ref(out)))
         return out
 
     def glu(self, act: str, x: Buffer) -> Buffer:

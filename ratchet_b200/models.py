@@ -15,11 +15,11 @@ from typing import Dict, List, Optional, Sequence, Tuple
 import numpy as np
 
 from . import capi
-from .callers import Dadezen, LatentMixer, LightningMixer, LoopEntry, ParallelLayer
+from .callers import Dadezen, GroupedMixer, LatentMixer, LightningMixer, LoopEntry, Mefesun, ParallelLayer, PostNormLayer
 from .capi import ERR_INVALID_ARG, ERR_UNSUPPORTED, RatchetCudaError
 from .decoder import StackDecoder
 from .device import Device
-from .nn import Embedding, GatedMLP, RotaryTable, SequenceState, StreamNorm
+from .nn import Embedding, GatedMLP, PostNorm, RotaryTable, SequenceState, SquaredReluMLP, StreamNorm
 from .safetensors import SafetensorsFile
 from .tensor import Tensor
 
@@ -132,7 +132,60 @@ class DadezenConfig:
                 [(i, None) for i in range(stop, n)])
 
 
-# ---------------------------------------------------------------------------------------- Dadezen
+@dataclass(frozen=True)
+class GroupedConfig:
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    rot: RotaryConfig
+    scale: float
+    chunk: int                # 0: every earlier position is seen
+
+
+@dataclass(frozen=True)
+class MefesunConfig:
+    width: int
+    vocab: int
+    eps: float
+    softcap: Optional[float]
+    layers: Tuple[LayerConfig, ...]
+    weights_of: Tuple[int, ...]          # per layer: the layer whose tensors it uses (itself, unless they are shared)
+
+    @staticmethod
+    def read(c: dict) -> "MefesunConfig":
+        layers, shared = [], []
+        for i, e in enumerate(c["layers"]):
+            m = e["mixer"]
+            if e["type"] != "attention":
+                raise RatchetCudaError(ERR_UNSUPPORTED, f"layer {i}: mixer {e['type']!r}")
+            mask = m.get("mask")
+            mixer = GroupedConfig(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), RotaryConfig.read(m["rot"]), float(m["scale"]),
+                                  int(mask["size"]) if mask else 0)
+            if mixer.kv_heads < 1 or mixer.heads % mixer.kv_heads or mixer.rot.dims > mixer.dim or mixer.chunk < (1 if mask else 0):
+                raise RatchetCudaError(ERR_INVALID_ARG, f"layer {i}: {mixer}")
+            mlp = e.get("mlp")
+            if mlp and mlp.get("kind", "dense") != "dense":
+                raise RatchetCudaError(ERR_UNSUPPORTED, f"layer {i}: feed-forward {mlp['kind']!r}")
+            layers.append(LayerConfig(mixer, bool(mlp)))
+            shared.append(e.get("weights_of"))
+        order = []
+        for i in range(len(layers)):
+            j, steps = i, 0
+            while shared[j] is not None:
+                j, steps = int(shared[j]), steps + 1
+                if not 0 <= j < len(layers) or steps > len(layers):
+                    raise RatchetCudaError(ERR_INVALID_ARG, f"layer {i}: weights of layer {j}")
+            if layers[j] != layers[i]:
+                raise RatchetCudaError(ERR_INVALID_ARG, f"layer {i} uses the weights of layer {j}, whose sizes are others")
+            order.append(j)
+        cap = c.get("logit_softcap")
+        if cap is not None and not float(cap) > 0:
+            raise RatchetCudaError(ERR_INVALID_ARG, f"logit_softcap {cap}")
+        return MefesunConfig(int(c["width"]), int(c["vocab"]), float(c["norm"]["eps"]), None if cap is None else float(cap), tuple(layers), tuple(order))
+
+
+# ---------------------------------------------------------------------------------------- models
 class _Weights:
     """Device tensors from a safetensors file: matrices in the model's dtype, rows of several matrices stacked into one;
     vectors (norm scales, biases) in f32."""
@@ -153,21 +206,52 @@ class _Weights:
                 parts.append(self.file.f32(n))
         return Tensor.from_data(parts[0] if len(parts) == 1 else np.concatenate(parts), device=self.dev, dt=self.dt)
 
-    def vector(self, name: str) -> Tensor:
-        return self.const(self.file.f32(name).reshape(-1))
+    def vector(self, *names: str, dt: int = capi.F32) -> Tensor:
+        v = np.concatenate([self.file.f32(n).reshape(-1) for n in names])
+        return Tensor.from_data(capi.to_bf16(v), device=self.dev, dt=dt) if dt == capi.BF16 else self.const(v)
 
     def const(self, a: np.ndarray) -> Tensor:
         return Tensor.from_data(np.ascontiguousarray(a, np.float32), device=self.dev)
 
 
-@register("Dadezen")
-class DadezenModel:
-    def __init__(self, config: dict, file: SafetensorsFile, dev: Device, dtype: str = "bfloat16"):
+class DecoderModel:
+    """What the served decoders share: ``graph`` (a caller with ``schedule(ids, state, want, streams)``) runs blocks of tokens,
+    ``_stack(state)`` makes the fused step over a state's tensors, which runs single ones."""
+
+    def __init__(self, cfg, dev: Device, dtype: str):
         if dtype not in DTYPES:
             raise RatchetCudaError(ERR_UNSUPPORTED, f"dtype {dtype!r} (bfloat16 or float32)")
-        self.dev, self.dt, self.cfg = dev, DTYPES[dtype], DadezenConfig.read(config)
+        self.dev, self.dt, self.cfg, self.vocab = dev, DTYPES[dtype], cfg, cfg.vocab
+
+    @staticmethod
+    def _check(file: SafetensorsFile, name: str, shape) -> None:
+        if file.shape(name) != tuple(shape):
+            raise RatchetCudaError(ERR_INVALID_ARG, f"{name} is {file.shape(name)}, expected {tuple(shape)}")
+
+    def prefill(self, tokens: Sequence[int], state: SequenceState, want: Sequence[int] = (), streams: Optional[list] = None) -> np.ndarray:
+        ids = Tensor.from_data(np.asarray(tokens, np.int32), device=self.dev)
+        places = Tensor.from_data(np.asarray(want, np.int32), device=self.dev) if len(want) else None
+        out = self.graph.schedule(ids, state, places, streams).resolve()
+        state.position += len(tokens)
+        return out.to_numpy() if places is not None else np.empty((0, self.vocab), np.float32)
+
+    def decode(self, state: SequenceState, token: Optional[int] = None):
+        if state.stack is None:
+            state.stack = self._stack(state)
+        state.stack.position = state.position
+        if token is None:
+            state.stack.step_device()
+        else:
+            state.stack.step(token)
+        state.position += 1
+        return state.stack.logits, state.stack.token
+
+
+@register("Dadezen")
+class DadezenModel(DecoderModel):
+    def __init__(self, config: dict, file: SafetensorsFile, dev: Device, dtype: str = "bfloat16"):
+        super().__init__(DadezenConfig.read(config), dev, dtype)
         c, w = self.cfg, _Weights(file, dev, self.dt)
-        self.vocab = c.vocab
         self._check(file, "embed", (c.vocab, c.width))
         self._check(file, "head", (c.vocab, c.width))
         layers = [self._layer(w, i, lc) for i, lc in enumerate(c.layers)]
@@ -179,11 +263,6 @@ class DadezenModel:
             entry = LoopEntry(w.matrix("loop.in"), self._steps)
         norm = StreamNorm(capi.LAYER_NORM, w.vector("final.norm"), c.eps, self.dt)
         self.graph = Dadezen(Embedding(w.matrix("embed")), layers, c.runs(), c.loop[0] if c.loop else None, entry, norm, w.matrix("head"))
-
-    @staticmethod
-    def _check(file: SafetensorsFile, name: str, shape) -> None:
-        if file.shape(name) != tuple(shape):
-            raise RatchetCudaError(ERR_INVALID_ARG, f"{name} is {file.shape(name)}, expected {tuple(shape)}")
 
     def _layer(self, w: _Weights, i: int, lc: LayerConfig) -> ParallelLayer:
         c, m, p, f = self.cfg, lc.mixer, f"l{i}.", w.file
@@ -234,25 +313,7 @@ class DadezenModel:
                 tensors.append(Tensor.zeros((rows, mixer.ukv.shape()[1] + m.rot_dim), self.dt, self.dev))
         return SequenceState(tensors)
 
-    # ------------------------------------------------------------------ steps
-    def prefill(self, tokens: Sequence[int], state: SequenceState, want: Sequence[int] = (), streams: Optional[list] = None) -> np.ndarray:
-        ids = Tensor.from_data(np.asarray(tokens, np.int32), device=self.dev)
-        places = Tensor.from_data(np.asarray(want, np.int32), device=self.dev) if len(want) else None
-        out = self.graph.schedule(ids, state, places, streams).resolve()
-        state.position += len(tokens)
-        return out.to_numpy() if places is not None else np.empty((0, self.vocab), np.float32)
-
-    def decode(self, state: SequenceState, token: Optional[int] = None):
-        if state.stack is None:
-            state.stack = self._stack(state)
-        state.stack.position = state.position
-        if token is None:
-            state.stack.step_device()
-        else:
-            state.stack.step(token)
-        state.position += 1
-        return state.stack.logits, state.stack.token
-
+    # ------------------------------------------------------------------ single tokens
     def _stack(self, state: SequenceState) -> StackDecoder:
         c, g = self.cfg, self.graph
         runs = []
@@ -275,5 +336,82 @@ class DadezenModel:
             if t is not None and i == g.first:
                 r.enter, r.enter_bias = g.entry.w.data_ptr(), self._steps[t].data_ptr()
             runs.append(r)
-        cfg = capi.rcu_stack_config(c.width, c.vocab, len(runs), c.eps, c.residual_mult, self.dt)
+        cfg = capi.rcu_stack_config(c.width, c.vocab, len(runs), c.eps, c.residual_mult, 0.0, self.dt, capi.LAYER_PARALLEL, None)
+        return StackDecoder(self.dev, cfg, runs, g.embedding.weight.data_ptr(), g.norm.weight.data_ptr(), g.head.data_ptr(), (g, state.runs))
+
+
+@register("Mefesun")
+class MefesunModel(DecoderModel):
+    def __init__(self, config: dict, file: SafetensorsFile, dev: Device, dtype: str = "bfloat16"):
+        super().__init__(MefesunConfig.read(config), dev, dtype)
+        c, w = self.cfg, _Weights(file, dev, self.dt)
+        self._check(file, "embed", (c.vocab, c.width))
+        self._rotary: Dict[RotaryConfig, RotaryTable] = {}
+        layers = [self._layer(w, i, lc) if c.weights_of[i] == i else None for i, lc in enumerate(c.layers)]
+        embed = w.matrix("embed")
+        norm = StreamNorm(capi.LAYER_NORM, w.vector("final.norm"), c.eps, self.dt, shift=w.vector("final.norm.b"))
+        self.graph = Mefesun(Embedding(embed), layers, list(c.weights_of), norm, embed, self.dt, c.softcap)
+
+    def _rot(self, w: _Weights, r: RotaryConfig) -> RotaryTable:
+        if r not in self._rotary:
+            table, magnitude = capi.rotary_frequencies(r.dims, r.base, r.factor, r.original, r.fast, r.slow)
+            self._rotary[r] = RotaryTable(w.const(table), magnitude)
+        return self._rotary[r]
+
+    def _layer(self, w: _Weights, i: int, lc: LayerConfig) -> PostNormLayer:
+        c, m, p, f = self.cfg, lc.mixer, f"l{i}.", w.file
+        H, G, D, E = m.heads, m.kv_heads, m.dim, m.vdim
+        x = p + "mix."
+        for n, rows in (("q", H * D), ("k", G * D), ("v", G * E)):
+            self._check(f, x + n, (rows, c.width))
+            self._check(f, x + n + ".b", (rows,))
+        for n, shape in (("o", (c.width, H * E)), ("o.b", (c.width,)), ("q.norm", (D,)), ("k.norm", (D,)), ("sink", (H,))):
+            self._check(f, x + n, shape)
+
+        def norm(k: str) -> PostNorm:
+            for n in (f"norm{k}", f"norm{k}.b", f"ls{k}"):
+                self._check(f, p + n, (c.width,))
+            ls = f.f32(f"{p}ls{k}")
+            return PostNorm(w.const(f.f32(f"{p}norm{k}") * ls), w.const(f.f32(f"{p}norm{k}.b") * ls), c.eps, self.dt)
+
+        biases = (x + "q.b", x + "k.b", x + "v.b")
+        mixer = GroupedMixer(w.matrix(x + "q", x + "k", x + "v"), w.vector(*biases, dt=self.dt), w.vector(*biases), w.vector(x + "q.norm"), w.vector(x + "k.norm"),
+                             self._rot(w, m.rot), w.vector(x + "sink"), w.matrix(x + "o"), w.vector(x + "o.b"), c.eps, H, G, D, E, m.scale, chunk=m.chunk)
+        norm2 = mlp = None
+        if lc.mlp:
+            ff = f.shape(p + "mlp.up")[0]
+            self._check(f, p + "mlp.up", (ff, c.width))
+            self._check(f, p + "mlp.down", (c.width, ff))
+            norm2, mlp = norm("2"), SquaredReluMLP(w.matrix(p + "mlp.up"), w.matrix(p + "mlp.down"))
+        return PostNormLayer(norm("1"), mixer, norm2, mlp)
+
+    def new_state(self, max_tokens: Optional[int] = None) -> SequenceState:
+        """A ring of keys and values per layer run: the chunk's positions, no more than the sequence's."""
+        tensors = []
+        for lc in self.cfg.layers:
+            m = lc.mixer
+            sizes = [n for n in (m.chunk, max_tokens) if n]
+            if not sizes:
+                raise RatchetCudaError(ERR_INVALID_ARG, "a layer that sees every position needs the most tokens a sequence may hold")
+            tensors.append(Tensor.zeros((min(sizes), m.kv_heads * (m.dim + m.vdim)), self.dt, self.dev))
+        return SequenceState(tensors)
+
+    def _stack(self, state: SequenceState) -> StackDecoder:
+        c, g = self.cfg, self.graph
+        runs = []
+        for k, i in enumerate(g.order):
+            layer, r = g.layers[i], capi.rcu_stack_run()
+            mx = layer.mixer
+            r.mixer, r.heads, r.kv_heads, r.dim, r.vdim = capi.MIXER_GROUPED, mx.heads, mx.kv_heads, mx.dim, mx.vdim
+            r.rot_pairs, r.rot_magnitude, r.freqs = mx.rot.freqs.shape()[1], mx.rot.magnitude, mx.rot.freqs.data_ptr()
+            r.window, r.chunk, r.scale, r.ring_rows, r.state = mx.window, mx.chunk, mx.scale, state.runs[k].shape()[0], state.runs[k].data_ptr()
+            r.mix_in, r.mix_bias, r.mix_norm, r.kv_norm = mx.qkv.data_ptr(), mx.qkv_bias_f32.data_ptr(), mx.q_norm.data_ptr(), mx.k_norm.data_ptr()
+            r.sink, r.out, r.out_bias = mx.sink.data_ptr(), mx.out.data_ptr(), mx.out_bias.data_ptr()
+            r.norm1, r.norm1_shift = layer.norm1.scale.data_ptr(), layer.norm1.shift.data_ptr()
+            if layer.mlp is not None:
+                r.ff = layer.mlp.down.shape()[1]
+                r.norm2, r.norm2_shift = layer.norm2.scale.data_ptr(), layer.norm2.shift.data_ptr()
+                r.gate_up, r.down = layer.mlp.up.data_ptr(), layer.mlp.down.data_ptr()
+            runs.append(r)
+        cfg = capi.rcu_stack_config(c.width, c.vocab, len(runs), c.eps, 0.0, c.softcap or 0.0, self.dt, capi.LAYER_POST_NORM, g.norm.shift.data_ptr())
         return StackDecoder(self.dev, cfg, runs, g.embedding.weight.data_ptr(), g.norm.weight.data_ptr(), g.head.data_ptr(), (g, state.runs))

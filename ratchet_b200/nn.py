@@ -100,14 +100,29 @@ class KVCache:
 
 # ---------------------------------------------------------------------------------------- models with a 32-bit residual stream
 class StreamNorm:
-    """LayerNorm without bias / RMSNorm of an f32 tensor (or of a column window of its rows) into the operand dtype of the
-    matrix product that follows."""
+    """LayerNorm / RMSNorm of an f32 tensor (or of a column window of its rows) into the operand dtype of the matrix product that
+    follows."""
 
-    def __init__(self, kind: int, weight, eps: float, dt: int):
-        self.kind, self.weight, self.eps, self.dt = kind, weight, eps, dt
+    def __init__(self, kind: int, weight, eps: float, dt: int, shift=None):
+        self.kind, self.weight, self.eps, self.dt, self.shift = kind, weight, eps, dt, shift
 
     def schedule(self, x, col: int = 0, gate=None, gate_col: int = 0):
-        return x.norm_rows(self.kind, self.weight, self.eps, self.dt, col=col, gate=gate, gate_col=gate_col)
+        return x.norm_rows(self.kind, self.weight, self.eps, self.dt, col=col, gate=gate, gate_col=gate_col, shift=self.shift)
+
+
+class PostNorm:
+    """x + LayerNorm(y) * scale + shift for a sublayer output y: x are stream rows, f32 values followed by their copy in the operand
+    dtype `dt` (f32: no copy).  A factor per channel behind the norm is folded into scale and shift."""
+
+    def __init__(self, scale, shift, eps: float, dt: int):
+        self.scale, self.shift, self.eps, self.dt = scale, shift, eps, dt
+
+    def schedule(self, x, y):
+        return x.post_norm(y, self.scale, self.shift, self.eps)
+
+    def operand(self, x):
+        """(tensor, first column) of the stream as the operand of a matrix product."""
+        return (x, 0) if self.dt == capi.F32 else (x.bitcast(self.dt), 2 * self.scale.shape()[0])
 
 
 class GatedMLP:
@@ -120,6 +135,16 @@ class GatedMLP:
         return self.down.linear(self.gate_up.linear(h).glu(self.act), resid=resid, alpha=alpha, dt=capi.F32)
 
 
+class SquaredReluMLP:
+    """W_down max(W_up h, 0)^2 as an f32 sublayer output; h at column `col` of wider rows."""
+
+    def __init__(self, up, down):
+        self.up, self.down = up, down
+
+    def schedule(self, h, col: int = 0):
+        return self.down.linear(self.up.linear(h, x_col=col, act="relu_squared"), dt=capi.F32)
+
+
 class RotaryTable:
     """Frequencies of interleaved rotary pairs (plain or YaRN) on the device, and the factor on cos and sin."""
 
@@ -128,8 +153,8 @@ class RotaryTable:
 
 
 class SequenceState:
-    """What one sequence keeps between steps: per layer run one tensor - a recurrent state f32 [heads, dim, vdim] or a ring of
-    latents [rows, latent + rotated] - and the number of tokens seen.  The counterpart of ``KVCache`` for models whose layers
+    """What one sequence keeps between steps: per layer run one tensor - a recurrent state f32 [heads, dim, vdim], a ring of
+    latents [rows, latent + rotated] or a ring of keys and values [rows, kv_heads * (dim + vdim)] - and the number of tokens seen.  The counterpart of ``KVCache`` for models whose layers
     keep different things."""
 
     def __init__(self, runs):

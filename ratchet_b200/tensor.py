@@ -223,15 +223,28 @@ class Tensor:
 
     # ------------------------------------------------------------------ ops of models with a 32-bit residual stream
     def linear(self, x: "Tensor", bias: Optional["Tensor"] = None, resid: Optional["Tensor"] = None, alpha: float = 1.0,
-               x_col: int = 0, silu_cols: int = 0, dt: Optional[int] = None) -> "Tensor":
-        """resid + alpha * f(x[..., x_col:] . self^T + bias), self the [N, K] weight, f silu on the first `silu_cols` columns; dt:
-        the activations' dtype or F32."""
-        return self._new(self.dev._lib.rcu_lazy_linear, self._h, x._h, x_col, bias._h if bias else None, silu_cols, resid._h if resid else None, alpha,
-                         x.dt() if dt is None else dt)
+               x_col: int = 0, act: Optional[str] = None, act_cols: Optional[int] = None, act_param: float = 0.0, dt: Optional[int] = None) -> "Tensor":
+        """resid + alpha * f(x[..., x_col:] . self^T + bias), self the [N, K] weight, f `act` (silu, relu_squared, softcap) on the first
+        `act_cols` columns (None: all); dt: the activations' dtype or F32."""
+        return self._new(self.dev._lib.rcu_lazy_linear, self._h, x._h, x_col, bias._h if bias else None, capi.LINEAR_ACTS[act],
+                         self.shape()[0] if act_cols is None else act_cols, act_param, resid._h if resid else None, alpha, x.dt() if dt is None else dt)
 
-    def norm_rows(self, kind: int, scale: "Tensor", eps: float, dt: int, col: int = 0, gate: Optional["Tensor"] = None, gate_col: int = 0):
-        """LayerNorm (no bias) / RMSNorm of columns [col, col + len(scale)), optionally times sigmoid(gate[:, gate_col:])."""
-        return self._new(self.dev._lib.rcu_lazy_norm_rows, kind, self._h, col, scale._h, gate._h if gate else None, gate_col, eps, dt)
+    def norm_rows(self, kind: int, scale: "Tensor", eps: float, dt: int, col: int = 0, gate: Optional["Tensor"] = None, gate_col: int = 0,
+                  shift: Optional["Tensor"] = None):
+        """LayerNorm / RMSNorm of columns [col, col + len(scale)), plus `shift`, optionally times sigmoid(gate[:, gate_col:])."""
+        return self._new(self.dev._lib.rcu_lazy_norm_rows, kind, self._h, col, scale._h, shift._h if shift else None, gate._h if gate else None, gate_col, eps, dt)
+
+    def stream_rows(self, copy_dt: int) -> "Tensor":
+        """Rows of a residual stream: f32 values, followed by their bf16 roundings when `copy_dt` is BF16."""
+        return self._new(self.dev._lib.rcu_lazy_stream_rows, self._h, copy_dt)
+
+    def post_norm(self, y: "Tensor", scale: "Tensor", shift: "Tensor", eps: float) -> "Tensor":
+        """These stream rows + LayerNorm(y) * scale + shift."""
+        return self._new(self.dev._lib.rcu_lazy_post_norm, self._h, y._h, scale._h, shift._h, eps)
+
+    def bitcast(self, dt: int) -> "Tensor":
+        """The same bytes as elements of `dt` (a view)."""
+        return self._new(self.dev._lib.rcu_lazy_bitcast, self._h, dt)
 
     def glu(self, act: str) -> "Tensor":
         """act(gate) * up of rows that hold gate, then up."""
@@ -251,6 +264,24 @@ class Tensor:
 
     def window_attention(self, kv: "Tensor", shared: "Tensor", shared_col: int, vdim: int, window: int, scale: float) -> "Tensor":
         return self._new(self.dev._lib.rcu_lazy_window_attention, self._h, kv._h, shared._h, shared_col, vdim, window, scale)
+
+    def rotary_angles(self, magnitude: float, position: int, tokens: int) -> "Tensor":
+        """[tokens, 2 pairs]: cos and sin, times `magnitude`, of this frequency table's angles from `position` on."""
+        return self._new(self.dev._lib.rcu_lazy_rotary_angles, self._h, magnitude, position, tokens)
+
+    def norm_rotary(self, heads: int, scale: "Tensor", eps: float, angles: "Tensor", col: int = 0) -> "Tensor":
+        """RMSNorm of each head of columns [col, col + heads * len(scale)), then the rotation by `angles`: [tokens, heads, dim]."""
+        return self._new(self.dev._lib.rcu_lazy_norm_rotary, self._h, col, heads, scale._h, eps, angles._h)
+
+    def kv_append(self, kv_heads: int, scale: "Tensor", eps: float, angles: "Tensor", position: int, keep: int, ring: "Tensor", rows: int, col: int = 0):
+        """Keys (normed, rotated) and values of a block, its last `keep` rows into `ring`; the result is the `rows` rows the block sees."""
+        return self._new(self.dev._lib.rcu_lazy_kv_append, self._h, col, kv_heads, scale._h, eps, angles._h, position, keep, ring._h, rows)
+
+    def grouped_attention(self, kv: "Tensor", kv_heads: int, vdim: int, scale: float, sink: Optional["Tensor"] = None, window: int = 0, chunk: int = 0,
+                          position: int = 0) -> "Tensor":
+        """Softmax attention of these queries [tokens, heads, dim] over kv rows, the first of which is `position`: a sliding window, runs
+        of `chunk` positions, or everything before."""
+        return self._new(self.dev._lib.rcu_lazy_grouped_attention, self._h, kv._h, sink._h if sink else None, kv_heads, vdim, window, chunk, position, scale)
 
     # ------------------------------------------------------------------ execution
     def resolve(self) -> "Tensor":

@@ -63,6 +63,13 @@ pub const RCU_REDUCE_MAX: c_int = 1;
 pub const RCU_REDUCE_MEAN: c_int = 2;
 pub const RCU_MIXER_LIGHTNING: c_int = 0;
 pub const RCU_MIXER_LATENT: c_int = 1;
+pub const RCU_MIXER_GROUPED: c_int = 2;
+pub const RCU_LAYER_PARALLEL: c_int = 0;
+pub const RCU_LAYER_POST_NORM: c_int = 1;
+pub const RCU_ACT_NONE: c_int = 0;
+pub const RCU_ACT_SILU: c_int = 1;
+pub const RCU_ACT_RELU_SQUARED: c_int = 2;
+pub const RCU_ACT_SOFTCAP: c_int = 3;
 pub const RCU_DEBUG_NO_REUSE: u32 = 1;
 pub const RCU_DEBUG_PROFILE: u32 = 2;
 pub const RCU_DEBUG_LOG: u32 = 4;
@@ -142,7 +149,10 @@ pub struct rcu_stack_config {
     pub n_runs: u32,
     pub eps: f32,
     pub residual_mult: f32,
+    pub logit_softcap: f32,
     pub weight_dt: i32,
+    pub layer: i32,
+    pub final_shift: *const c_void,
 }
 
 #[repr(C)]
@@ -159,20 +169,27 @@ pub struct rcu_stack_run {
     pub rot_pairs: u32,
     pub window: u32,
     pub ring_rows: u32,
+    pub kv_heads: u32,
+    pub chunk: u32,
     pub scale: f32,
     pub rot_magnitude: f32,
     pub enter: *const c_void,
     pub enter_bias: *const c_void,
     pub norm1: *const c_void,
     pub norm2: *const c_void,
+    pub norm1_shift: *const c_void,
+    pub norm2_shift: *const c_void,
     pub mix_in: *const c_void,
+    pub mix_bias: *const c_void,
     pub mix_norm: *const c_void,
     pub kv_norm: *const c_void,
+    pub sink: *const c_void,
     pub uq: *const c_void,
     pub ukv: *const c_void,
     pub freqs: *const c_void,
     pub decay: *const c_void,
     pub out: *const c_void,
+    pub out_bias: *const c_void,
     pub gate_up: *const c_void,
     pub down: *const c_void,
     pub state: *mut c_void,
@@ -225,17 +242,26 @@ extern "C" {
     pub fn rcu_index_write(dev: *mut rcu_device, dst: *mut rcu_tensor, src: *const rcu_tensor, start: *const u64) -> rcu_status;
     pub fn rcu_conv1d(dev: *mut rcu_device, x: *const rcu_tensor, w: *const rcu_tensor, bias: *const rcu_tensor, stride: u32, padding: u32, dst: *mut rcu_tensor) -> rcu_status;
     pub fn rcu_linear(
-        dev: *mut rcu_device, w: *const rcu_tensor, x: *const rcu_tensor, x_col: u32, bias: *const rcu_tensor, silu_cols: u32, resid: *const rcu_tensor, alpha: f32, dst: *mut rcu_tensor,
+        dev: *mut rcu_device, w: *const rcu_tensor, x: *const rcu_tensor, x_col: u32, bias: *const rcu_tensor, act: c_int, act_cols: u32, act_param: f32,
+        resid: *const rcu_tensor, alpha: f32, dst: *mut rcu_tensor,
     ) -> rcu_status;
     pub fn rcu_norm_rows(
-        dev: *mut rcu_device, kind: c_int, x: *const rcu_tensor, x_col: u32, scale: *const rcu_tensor, gate: *const rcu_tensor, gate_col: u32, eps: f32, dst: *mut rcu_tensor,
+        dev: *mut rcu_device, kind: c_int, x: *const rcu_tensor, x_col: u32, scale: *const rcu_tensor, shift: *const rcu_tensor, gate: *const rcu_tensor, gate_col: u32, eps: f32,
+        dst: *mut rcu_tensor,
     ) -> rcu_status;
+    pub fn rcu_stream_rows(dev: *mut rcu_device, x: *const rcu_tensor, copy_dt: i32, dst: *mut rcu_tensor) -> rcu_status;
+    pub fn rcu_post_norm(dev: *mut rcu_device, x: *const rcu_tensor, y: *const rcu_tensor, scale: *const rcu_tensor, shift: *const rcu_tensor, eps: f32, dst: *mut rcu_tensor) -> rcu_status;
     pub fn rcu_glu(dev: *mut rcu_device, act: c_int, x: *const rcu_tensor, dst: *mut rcu_tensor) -> rcu_status;
     pub fn rcu_rotary_frequencies(
         dims: u32, base: f64, factor: f64, original: f64, fast: f64, slow: f64, host_freqs: *mut f32, magnitude: *mut f32,
     ) -> rcu_status;
     pub fn rcu_rotary(
         dev: *mut rcu_device, x: *const rcu_tensor, first: u32, freqs: *const rcu_tensor, magnitude: f32, position: u32, dst: *mut rcu_tensor,
+    ) -> rcu_status;
+    pub fn rcu_rotary_angles(dev: *mut rcu_device, freqs: *const rcu_tensor, magnitude: f32, position: u32, dst: *mut rcu_tensor) -> rcu_status;
+    pub fn rcu_norm_rotary(dev: *mut rcu_device, x: *const rcu_tensor, x_col: u32, scale: *const rcu_tensor, eps: f32, angles: *const rcu_tensor, dst: *mut rcu_tensor) -> rcu_status;
+    pub fn rcu_kv_append(
+        dev: *mut rcu_device, x: *const rcu_tensor, x_col: u32, kv_heads: u32, scale: *const rcu_tensor, eps: f32, angles: *const rcu_tensor, position: u32, keep: u32, ring: *mut rcu_tensor, dst: *mut rcu_tensor,
     ) -> rcu_status;
     pub fn rcu_lightning(
         dev: *mut rcu_device, x: *const rcu_tensor, decay_pow: *const rcu_tensor, state: *mut rcu_tensor, dst: *mut rcu_tensor,
@@ -245,6 +271,9 @@ extern "C" {
     ) -> rcu_status;
     pub fn rcu_window_attention(
         dev: *mut rcu_device, q: *const rcu_tensor, kv: *const rcu_tensor, shared: *const rcu_tensor, shared_col: u32, vdim: u32, window: u32, scale: f32, dst: *mut rcu_tensor,
+    ) -> rcu_status;
+    pub fn rcu_grouped_attention(
+        dev: *mut rcu_device, q: *const rcu_tensor, kv: *const rcu_tensor, sink: *const rcu_tensor, kv_heads: u32, vdim: u32, window: u32, chunk: u32, position: u32, scale: f32, dst: *mut rcu_tensor,
     ) -> rcu_status;
     pub fn rcu_lazy_from_host(dev: *mut rcu_device, dt: i32, rank: u32, shape: *const u64, host: *const c_void, nbytes: u64, out: *mut *mut rcu_lazy) -> rcu_status;
     pub fn rcu_lazy_zeros(dev: *mut rcu_device, dt: i32, rank: u32, shape: *const u64, out: *mut *mut rcu_lazy) -> rcu_status;
@@ -270,10 +299,22 @@ extern "C" {
     pub fn rcu_lazy_cache(cache: *mut rcu_lazy, src: *mut rcu_lazy, dim: u32, offset: u32, out: *mut *mut rcu_lazy) -> rcu_status;
     pub fn rcu_lazy_index_write(dst: *mut rcu_lazy, src: *mut rcu_lazy, start: *const u64, out: *mut *mut rcu_lazy) -> rcu_status;
     pub fn rcu_lazy_linear(
-        w: *mut rcu_lazy, x: *mut rcu_lazy, x_col: u32, bias: *mut rcu_lazy, silu_cols: u32, resid: *mut rcu_lazy, alpha: f32, dst_dt: i32, out: *mut *mut rcu_lazy,
+        w: *mut rcu_lazy, x: *mut rcu_lazy, x_col: u32, bias: *mut rcu_lazy, act: c_int, act_cols: u32, act_param: f32, resid: *mut rcu_lazy, alpha: f32, dst_dt: i32, out: *mut *mut rcu_lazy,
     ) -> rcu_status;
     pub fn rcu_lazy_norm_rows(
-        kind: c_int, x: *mut rcu_lazy, x_col: u32, scale: *mut rcu_lazy, gate: *mut rcu_lazy, gate_col: u32, eps: f32, dst_dt: i32, out: *mut *mut rcu_lazy,
+        kind: c_int, x: *mut rcu_lazy, x_col: u32, scale: *mut rcu_lazy, shift: *mut rcu_lazy, gate: *mut rcu_lazy, gate_col: u32, eps: f32, dst_dt: i32,
+        out: *mut *mut rcu_lazy,
+    ) -> rcu_status;
+    pub fn rcu_lazy_stream_rows(x: *mut rcu_lazy, copy_dt: i32, out: *mut *mut rcu_lazy) -> rcu_status;
+    pub fn rcu_lazy_post_norm(x: *mut rcu_lazy, y: *mut rcu_lazy, scale: *mut rcu_lazy, shift: *mut rcu_lazy, eps: f32, out: *mut *mut rcu_lazy) -> rcu_status;
+    pub fn rcu_lazy_bitcast(x: *mut rcu_lazy, dt: i32, out: *mut *mut rcu_lazy) -> rcu_status;
+    pub fn rcu_lazy_rotary_angles(freqs: *mut rcu_lazy, magnitude: f32, position: u32, tokens: u32, out: *mut *mut rcu_lazy) -> rcu_status;
+    pub fn rcu_lazy_norm_rotary(x: *mut rcu_lazy, x_col: u32, heads: u32, scale: *mut rcu_lazy, eps: f32, angles: *mut rcu_lazy, out: *mut *mut rcu_lazy) -> rcu_status;
+    pub fn rcu_lazy_kv_append(
+        x: *mut rcu_lazy, x_col: u32, kv_heads: u32, scale: *mut rcu_lazy, eps: f32, angles: *mut rcu_lazy, position: u32, keep: u32, ring: *mut rcu_lazy, rows: u32, out: *mut *mut rcu_lazy,
+    ) -> rcu_status;
+    pub fn rcu_lazy_grouped_attention(
+        q: *mut rcu_lazy, kv: *mut rcu_lazy, sink: *mut rcu_lazy, kv_heads: u32, vdim: u32, window: u32, chunk: u32, position: u32, scale: f32, out: *mut *mut rcu_lazy,
     ) -> rcu_status;
     pub fn rcu_lazy_glu(act: c_int, x: *mut rcu_lazy, out: *mut *mut rcu_lazy) -> rcu_status;
     pub fn rcu_lazy_rotary(

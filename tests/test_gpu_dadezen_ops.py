@@ -69,9 +69,9 @@ def test_linear_output_types_and_epilogue(dev, dt, M, N, K):
     z = xv[:, :K] @ wv.T + bv
     n = N // 2
     z[:, :n] = dz.silu(z[:, :n])
-    out = dev.linear(w, x, bias=b, resid=r, alpha=0.3, silu_cols=n, dt=F32)
+    out = dev.linear(w, x, bias=b, resid=r, alpha=0.3, act="silu", act_cols=n, dt=F32)
     assert err(get(out), rv + 0.3 * z) < 3e-6
-    dev.linear(w, x, bias=b, resid=r, alpha=0.3, silu_cols=n, dt=F32, out=r)          # into the residual itself
+    dev.linear(w, x, bias=b, resid=r, alpha=0.3, act="silu", act_cols=n, dt=F32, out=r)          # into the residual itself
     assert np.array_equal(get(r), get(out))
 
 
@@ -80,7 +80,7 @@ def test_linear_refuses_what_it_cannot_do(dev):
     w, _ = put(dev, np.ones((8, 8)), BF16)
     x, _ = put(dev, np.ones((2, 8)), BF16)
     r, _ = put(dev, np.ones((2, 8)), F32)
-    for bad in (lambda: dev.linear(w, x, x_col=1), lambda: dev.linear(w, x, resid=r), lambda: dev.linear(w, r), lambda: dev.linear(w, x, silu_cols=9)):
+    for bad in (lambda: dev.linear(w, x, x_col=1), lambda: dev.linear(w, x, resid=r), lambda: dev.linear(w, r), lambda: dev.linear(w, x, act="silu", act_cols=9)):
         with pytest.raises(RatchetCudaError):
             bad()
 
