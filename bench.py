@@ -906,8 +906,9 @@ def main():
                          "8192 rows = 134 MB of weights, still larger than L2, small enough for an ncu capture")
     ap.add_argument("--no-extras", action="store_true", help="skip the GEMV sweep and the Phi-3 decode leg")
     ap.add_argument("--legs", default="all", help="comma list of the extra legs to run at N=1: sweep, prefill, phi2, whisper, decode (default all)")
-    ap.add_argument("--serve", action="store_true", help="instead: prefill and decode throughput of the Dadezen decoder beside Phi-3 layers of equal size")
+    ap.add_argument("--serve", action="store_true", help="instead: prefill and decode throughput of the Mefesun and Dadezen decoders beside Phi-3 layers of equal size")
     ap.add_argument("--serve-sizes", default="", help="with --serve: comma list of w1024, w2048, w4096 (default all)")
+    ap.add_argument("--serve-models", default="", help="with --serve: comma list of mefesun, dadezen (default both)")
     ap.add_argument("--serve-only-new", action="store_true", help="with --serve: leave the Phi-3 layers out")
     args = ap.parse_args()
     if args.serve:

@@ -1,8 +1,9 @@
-"""`python bench.py --serve`: prefill and decode throughput of the Dadezen decoder at layer sizes of real models (random bf16
-weights, half of the layers linear attention, half windowed latent attention), beside Phi-3's layers at the same width, feed-forward
-and depth (f16 prefill through the lazy graph, Q8_0 decode through the fused step).
+"""`python bench.py --serve`: prefill and decode throughput of the Mefesun decoder (grouped heads of 128, four query heads per key head,
+chunks as long as the window) and the Dadezen decoder (half of the layers linear attention, half windowed latent attention) at
+layer sizes of real models with random bf16 weights, beside Phi-3's layers at the same width, feed-forward and depth (f16 prefill
+through the lazy graph, Q8_0 decode through the fused step).
 
-One JSON line: per size the tokens per second, the share of the measured roofline (weights and states once per decoded token
+One JSON line: per size and model the tokens per second, the share of the measured roofline (weights and states once per decoded token
 over the copy bandwidth; matrix-product flops of a prompt over the sustained tensor throughput) and, per op of the lazy graph, its
 time and the share of its own roofline."""
 from __future__ import annotations
@@ -33,28 +34,64 @@ def dadezen_config(c):
     return {"architecture": "Dadezen", "width": c["width"], "vocab": c["vocab"], "norm": {"eps": 1e-5}, "residual_mult": 0.5, "layers": pair * n}
 
 
+def mefesun_config(c):
+    d = c["width"]
+    layer = {"type": "attention", "mixer": {"heads": d // 128, "kv_heads": max(d // 512, 1), "dim": 128, "vdim": 128, "mask": {"size": c["window"]}, "scale": 128 ** -0.5,
+                                            "rot": {"base": 10000.0, "dims": 128,
+                                                    "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}},
+             "mlp": {"kind": "dense", "ff": c["ff"]}}
+    return {"architecture": "Mefesun", "width": d, "vocab": c["vocab"], "norm": {"eps": 1e-5}, "logit_softcap": 30.0, "layers": [layer] * c["layers"]}
+
+
+def mefesun_shapes(config):
+    d = config["width"]
+    S = {"embed": (config["vocab"], d), "final.norm": (d,), "final.norm.b": (d,)}
+    for i, e in enumerate(config["layers"]):
+        m, ff, p, x = e["mixer"], e["mlp"]["ff"], f"l{i}.", f"l{i}.mix."
+        H, G, D, E = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        for n, rows in (("q", H * D), ("k", G * D), ("v", G * E)):
+            S[x + n], S[x + n + ".b"] = (rows, d), (rows,)
+        S.update({x + "o": (d, H * E), x + "o.b": (d,), x + "q.norm": (D,), x + "k.norm": (D,), x + "sink": (H,), p + "mlp.up": (ff, d), p + "mlp.down": (d, ff)})
+        for k in "12":
+            S[f"{p}norm{k}"] = S[f"{p}norm{k}.b"] = S[f"{p}ls{k}"] = (d,)
+    return S
+
+
+def mefesun_work(c):
+    """As dadezen_work."""
+    m, d, ff, n, T = mefesun_config(c)["layers"][0]["mixer"], c["width"], c["ff"], c["layers"], c["prompt"]
+    H, G, D, E, W = m["heads"], m["kv_heads"], m["dim"], m["vdim"], min(c["window"], c["prompt"])
+    weights = n * (d * (H * D + G * (D + E)) + H * E * d + 2 * d * ff) + d * c["vocab"]
+    seen = T // W * (W * (W + 1) // 2) + (T % W) * (T % W + 1) // 2
+    return 2 * weights + n * W * G * (D + E) * 2, {"linear": 2 * T * (weights - d * c["vocab"]), "grouped_attention": n * 2 * seen * H * (D + E)}
+
+
+def dadezen_shapes(config):
+    d, S = config["width"], {}
+    S["embed"] = S["head"] = (config["vocab"], d)
+    S["final.norm"] = (d,)
+    for i, e in enumerate(config["layers"]):
+        m, x, ff = e["mixer"], f"l{i}.mix.", e["mlp"]["ff"]
+        H, D, E = m["heads"], m["dim"], m["vdim"]
+        S[f"l{i}.norm1"] = S[f"l{i}.norm2"] = (d,)
+        S[f"l{i}.mlp.gate"] = S[f"l{i}.mlp.up"] = (ff, d)
+        S[f"l{i}.mlp.down"] = (d, ff)
+        S[x + "o"] = (d, H * E)
+        if e["type"] == "lightning":
+            S.update({x + "q": (H * D, d), x + "k": (H * D, d), x + "v": (H * E, d), x + "g": (H * E, d), x + "norm": (H * E,)})
+        else:
+            Q, C, R = m["q_rank"], m["kv_rank"], m["rot_dim"]
+            S.update({x + "dq": (Q, d), x + "dq.norm": (Q,), x + "uq": (H * (D + R), Q), x + "dkv": (C + R, d), x + "dkv.norm": (C,), x + "uk": (H * D, C),
+                      x + "uv": (H * E, C)})
+    return S
+
+
 class RandomFile:
     """A weights file of random values (the loader's file interface)."""
 
-    def __init__(self, config):
+    def __init__(self, shapes):
         from ratchet_b200 import capi
-        self.shapes, d = {}, config["width"]
-        S = self.shapes
-        S["embed"] = S["head"] = (config["vocab"], d)
-        S["final.norm"] = (d,)
-        for i, e in enumerate(config["layers"]):
-            m, x, ff = e["mixer"], f"l{i}.mix.", e["mlp"]["ff"]
-            H, D, E = m["heads"], m["dim"], m["vdim"]
-            S[f"l{i}.norm1"] = S[f"l{i}.norm2"] = (d,)
-            S[f"l{i}.mlp.gate"] = S[f"l{i}.mlp.up"] = (ff, d)
-            S[f"l{i}.mlp.down"] = (d, ff)
-            S[x + "o"] = (d, H * E)
-            if e["type"] == "lightning":
-                S.update({x + "q": (H * D, d), x + "k": (H * D, d), x + "v": (H * E, d), x + "g": (H * E, d), x + "norm": (H * E,)})
-            else:
-                Q, C, R = m["q_rank"], m["kv_rank"], m["rot_dim"]
-                S.update({x + "dq": (Q, d), x + "dq.norm": (Q,), x + "uq": (H * (D + R), Q), x + "dkv": (C + R, d), x + "dkv.norm": (C,), x + "uk": (H * D, C),
-                          x + "uv": (H * E, C)})
+        self.shapes = shapes
         g = np.random.Generator(np.random.PCG64(3))
         self._pool = capi.to_bf16(g.standard_normal(1 << 22, dtype=np.float32) * np.float32(0.02))
         self._capi = capi
@@ -117,12 +154,16 @@ def op_table(dev, fn):
     return rows
 
 
-def dadezen_leg(dev, torch, stream, c, peaks, steps):
-    from ratchet_b200 import Tensor, capi
-    from ratchet_b200.models import DadezenModel
-    cfg = dadezen_config(c)
-    m = DadezenModel(cfg, RandomFile(cfg), dev)
-    decode_bytes, flops = dadezen_work(c)
+NEW_MODELS = {"mefesun": (mefesun_config, mefesun_shapes, mefesun_work), "dadezen": (dadezen_config, dadezen_shapes, dadezen_work)}
+
+
+def new_model_leg(dev, torch, stream, name, c, peaks, steps):
+    from ratchet_b200 import Tensor
+    from ratchet_b200.models import REGISTRY
+    config, shapes, work = NEW_MODELS[name]
+    cfg = config(c)
+    m = REGISTRY[cfg["architecture"]](cfg, RandomFile(shapes(cfg)), dev)
+    decode_bytes, flops = work(c)
     T = c["prompt"]
     ids = Tensor.from_data(np.random.Generator(np.random.PCG64(1)).integers(0, c["vocab"], T).astype(np.int32), device=dev)
     want = Tensor.from_data(np.array([T - 1], np.int32), device=dev)
@@ -130,8 +171,11 @@ def dadezen_leg(dev, torch, stream, c, peaks, steps):
     forward = lambda: m.graph.schedule(ids, st, want).resolve()
     prefill = event_ms(torch, stream, forward, 5)
     ops = op_table(dev, forward)
-    st.position = T
-    m.decode(st, 5)                                     # the window is full: every step attends over all of it
+    # timed steps attend over a whole window, or the last hundred positions of a chunk
+    if name == "mefesun":
+        steps = min(steps, 100)
+    st.position = T if name == "dadezen" else T - 1 - steps - 8
+    m.decode(st, 5)
     decode = event_ms(torch, stream, lambda: m.decode(st), steps)
     gbs, tflops, sustained = peaks
     total = sum(flops.values())
@@ -213,15 +257,19 @@ def run_serve(args, measured, clock_sampler):
     sampler = clock_sampler(0)
     sampler.start()
     sizes = args.serve_sizes.split(",") if args.serve_sizes else list(SIZES)
+    models = args.serve_models.split(",") if args.serve_models else list(NEW_MODELS)
     out = {}
     for name in sizes:
         c = SIZES[name]
-        out[name] = {"dadezen": dadezen_leg(dev, torch, stream, c, peaks, args.steps), "config": c}
+        out[name] = {"config": c}
+        for model in models:
+            out[name][model] = new_model_leg(dev, torch, stream, model, c, peaks, args.steps)
+            dev.check(dev._lib.rcu_pool_trim(dev.handle))
         if not args.serve_only_new:
             out[name]["phi3_same_size"] = phi3_leg(dev, torch, stream, c, peaks, args.steps)
         dev.check(dev._lib.rcu_pool_trim(dev.handle))
-    last = out[sizes[-1]]["dadezen"]
-    print(json.dumps({"metric": "dadezen_decode_tokens_per_s", "value": last["decode_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": args.steps,
+    last = out[sizes[-1]][models[0]]
+    print(json.dumps({"metric": models[0] + "_decode_tokens_per_s", "value": last["decode_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": args.steps,
                       "warmup": 3, "ms_per_step": last["decode_us"] / 1e3, "higher_is_better": True, "dtype": "bf16", "data": "synthetic",
                       "peaks": {"hbm_gbs": peaks[0], "bf16_tflops": peaks[1], "bf16_tflops_sustained": peaks[2], "kind": "measured" if measured else "fallback"},
                       "clocks": sampler.stop(), "sizes": out}))
