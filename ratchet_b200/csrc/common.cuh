@@ -13,6 +13,7 @@
 #include <mutex>
 #include <string>
 #include <unordered_map>
+#include <utility>
 #include <vector>
 
 #include "../../include/ratchet_cuda.h"
@@ -88,21 +89,36 @@ __device__ __forceinline__ void rcu_kernel_entry() {
 __device__ __forceinline__ void rcu_kernel_entry_wait_only() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
 
 // kern<<<grid, block, smem, dev->stream>>>(args...) as a programmatic dependent of the kernel before it
-// (RCU_NO_PDL in the environment launches it plainly).  The kernel must call rcu_kernel_entry() first.
+// (RCU_NO_PDL in the environment launches it plainly).  The kernel must call rcu_kernel_entry() first.  cluster_x > 0: clusters of
+// that many CTAs along x.
 template <class... P, class... A>
-inline cudaError_t rcu_launch(rcu_device* dev, void (*kern)(P...), dim3 grid, dim3 block, size_t smem, A&&... args) {
+inline cudaError_t rcu_launch_cluster(rcu_device* dev, void (*kern)(P...), dim3 grid, dim3 block, size_t smem, int cluster_x, A&&... args) {
     static const bool pdl = std::getenv("RCU_NO_PDL") == nullptr;
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = grid;
     cfg.blockDim = block;
     cfg.dynamicSmemBytes = smem;
     cfg.stream = dev->stream;
-    cudaLaunchAttribute attr[1];
-    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attr[0].val.programmaticStreamSerializationAllowed = 1;
+    cudaLaunchAttribute attr[2];
+    unsigned n = 0;
+    if (pdl) {
+        attr[n].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+        attr[n++].val.programmaticStreamSerializationAllowed = 1;
+    }
+    if (cluster_x > 0) {
+        attr[n].id = cudaLaunchAttributeClusterDimension;
+        attr[n].val.clusterDim.x = (unsigned)cluster_x;
+        attr[n].val.clusterDim.y = attr[n].val.clusterDim.z = 1;
+        ++n;
+    }
     cfg.attrs = attr;
-    cfg.numAttrs = pdl ? 1 : 0;
+    cfg.numAttrs = n;
     return cudaLaunchKernelEx(&cfg, kern, static_cast<P>(args)...);
+}
+
+template <class... P, class... A>
+inline cudaError_t rcu_launch(rcu_device* dev, void (*kern)(P...), dim3 grid, dim3 block, size_t smem, A&&... args) {
+    return rcu_launch_cluster(dev, kern, grid, block, smem, 0, std::forward<A>(args)...);
 }
 
 struct DevGuard {

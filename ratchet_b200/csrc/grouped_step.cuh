@@ -2,12 +2,18 @@
 // fused decode step (stack_decode.cu).
 //
 // The visible positions are cut into tiles of 16 that CTAs and warps take in turn.  Every CTA norms and rotates the queries of its
-// heads; the one whose tile holds the current position first norms, rotates and stores the token's key and its value.  CTAs leave
-// partial results (maximum, sum of weights, weighted values); the last of a kv head's CTAs to finish merges them and adds the sink.
+// heads; the one whose tile holds the current position first norms, rotates and stores the token's key and its value.  The partial
+// results of a kv head's CTAs (maximum, sum of weights, weighted values) are merged, and the sink added, through distributed shared
+// memory when the CTAs form one cluster of up to eight; more of them leave their parts in global memory, where the last to finish
+// merges them.
 //   grouped_step_mma_kernel   bf16 rings on the tensor cores: up to 16 query heads of a kv head against 16 positions, operands
 //                             straight from global memory in registers, queries and weights as bf16 value plus remainder;
 //   grouped_step_kernel       any type and size in FFMA.
 #pragma once
+#include <cooperative_groups.h>
+
+#include <algorithm>
+
 #include "lm_mma.cuh"
 #include "window.cuh"
 
@@ -18,6 +24,7 @@ constexpr int kTile = 16;             // positions per tile
 constexpr int kMmaHeads = 16;         // query heads per CTA of the tensor-core kernel
 constexpr int kFmaHeads = 8;          // of the other (one warp each)
 constexpr int kMaxSplits = 64;
+constexpr int kCluster = 8;           // CTAs of a kv head that merge through distributed shared memory
 
 struct Args {
     const float* mix;                 // the token's query heads [H, D], key heads [G, D], value heads [G, E]
@@ -117,51 +124,63 @@ __device__ __forceinline__ void merge(const Args& a, int h0, int nh, int active,
 
 // NB: blocks of 32 key features, EB: blocks of 64 value features (D and E multiples of 8).  The products' inner index may run over the
 // features in any order as long as both operands agree: a lane takes eight consecutive features of a key row in one load and feeds
-// them to two products; value columns are dealt to the product's columns eight apart in the same way.
-template <int NB, int EB>
+// them to two products; value columns are dealt to the product's columns eight apart in the same way.  CL: the CTAs of blockIdx.y are
+// one cluster.
+template <int NB, int EB, bool CL>
 __global__ void __launch_bounds__(kThreads) grouped_step_mma_kernel(const Args a) {
-    rcu_kernel_entry();
     using lm::bf16;
     extern __shared__ __align__(16) unsigned char smem[];
-    constexpr int ldq = NB * 32 + 8;
+    constexpr int ldq = NB * 32 + 8, KP = NB / 2;                         // KP: pairs of features per lane
     bf16 *qh = reinterpret_cast<bf16*>(smem), *ql = qh + kMmaHeads * ldq;
-    float* acc_s = reinterpret_cast<float*>(ql + kMmaHeads * ldq);        // [warps][nh][E]
+    float* acc_s = reinterpret_cast<float*>(ql + kMmaHeads * ldq);        // [warps][nh][E]; the CTA's sums end up in the first [nh][E]
     __shared__ float m_s[kWarps][kMmaHeads], l_s[kWarps][kMmaHeads], weights[kMaxSplits * 16];
+    __shared__ float cta_m[kMmaHeads], cta_l[kMmaHeads];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, gr = lane >> 2, t = lane & 3;
     const int per = a.H / a.G, groups = head_groups(a.H, a.G, kMmaHeads);
     const int g = blockIdx.y / groups, hg = (blockIdx.y - g * groups) * kMmaHeads;
     const int h0 = g * per + hg, nh = min(kMmaHeads, per - hg);
+    asm volatile("griddepcontrol.launch_dependents;" ::: "memory");
+    // constants first: the norms' scales, and zeros for what no head fills
+    float2 qs[KP], ks[KP];
+#pragma unroll
+    for (int i = 0; i < KP; ++i) {
+        const int d = 2 * (lane + 32 * i);
+        qs[i] = d < a.D ? *reinterpret_cast<const float2*>(a.q_scale + d) : make_float2(0.f, 0.f);
+        ks[i] = d < a.D ? *reinterpret_cast<const float2*>(a.k_scale + d) : make_float2(0.f, 0.f);
+    }
+    for (int h = warp; h < kMmaHeads; h += kWarps)
+        for (int d = lane; d < ldq; d += 32)
+            if (h >= nh || d >= a.D) qh[h * ldq + d] = ql[h * ldq + d] = __float2bfloat16_rn(0.f);
+    asm volatile("griddepcontrol.wait;" ::: "memory");
+
     const uint32_t pos = *a.d_pos;
+    // the token's heads this warp prepares (two query heads; the last warp also the key and the value) and the angles, all in flight at once
+    float2 xq[2][KP], xk[KP], cs[KP];
+    const float* key = a.mix + (size_t)(a.H + g) * a.D;
+#pragma unroll
+    for (int i = 0; i < KP; ++i) {
+        const int d = 2 * (lane + 32 * i);
+        cs[i] = lane + 32 * i < a.pairs ? a.angles[lane + 32 * i] : make_float2(1.f, 0.f);
+#pragma unroll
+        for (int x = 0; x < 2; ++x)
+            xq[x][i] = d < a.D && warp + x * kWarps < nh ? *reinterpret_cast<const float2*>(a.mix + (size_t)(h0 + warp + x * kWarps) * a.D + d) : make_float2(0.f, 0.f);
+        xk[i] = d < a.D && warp == kWarps - 1 ? *reinterpret_cast<const float2*>(key + d) : make_float2(0.f, 0.f);
+    }
     const Visible see{a.window, a.chunk, 0};
     const int low = see.first((int)pos), n = (int)pos - low + 1, tiles = (n + kTile - 1) / kTile;
     const int active = min((int)gridDim.x, tiles);
-    if ((int)blockIdx.x >= active) return;
-    for (int h = warp; h < kMmaHeads; h += kWarps) {
-        bf16 *oh = qh + h * ldq, *ol = ql + h * ldq;
-        for (int d = lane; d < ldq; d += 32)
-            if (h >= nh || d >= a.D) oh[d] = ol[d] = __float2bfloat16_rn(0.f);
-        if (h < nh)
-            current_head(a, a.mix + (size_t)(h0 + h) * a.D, a.q_scale, [&](int d, float v) {
-                v *= a.scale;
-                oh[d] = __float2bfloat16_rn(v);
-                ol[d] = __float2bfloat16_rn(v - __bfloat162float(oh[d]));
-            });
-    }
-    if ((tiles - 1) % active == (int)blockIdx.x && warp == kWarps - 1) append<bf16>(a, g, pos);
-    __syncthreads();
+    if (!CL && (int)blockIdx.x >= active) return;
 
     const size_t W = (size_t)a.G * (a.D + a.E);
     const bf16* K = reinterpret_cast<const bf16*>(a.ring) + (size_t)g * a.D;
     const bf16* V = reinterpret_cast<const bf16*>(a.ring) + (size_t)a.G * a.D + (size_t)g * a.E;
-    float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f, o[EB][8][4];
-#pragma unroll
-    for (int c = 0; c < EB; ++c)
-#pragma unroll
-        for (int j = 0; j < 8; ++j) o[c][j][0] = o[c][j][1] = o[c][j][2] = o[c][j][3] = 0.f;
-    for (int tile = blockIdx.x + warp * active; tile < tiles; tile += active * kWarps) {
-        const int p0 = low + tile * kTile;
-        auto row = [&](int i) { return (size_t)(min(p0 + i, (int)pos) % a.ring_rows) * W; };      // positions beyond the current one: any row, weight zero
-        uint4 k[NB][2], v[EB][4];
+    uint4 k[NB][2], v[EB][4];
+    auto load = [&](int p0) {
+        const int base = p0 % a.ring_rows;
+        auto row = [&](int i) {               // positions beyond the current one: any row, weight zero
+            const int r = base + min(i, (int)pos - p0);
+            return (size_t)(r < a.ring_rows ? r : r - a.ring_rows) * W;
+        };
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
             const bf16* src = K + row(i * 8 + gr);
@@ -180,6 +199,63 @@ __global__ void __launch_bounds__(kThreads) grouped_step_mma_kernel(const Args a
                 v[c][i] = e < a.E ? *reinterpret_cast<const uint4*>(src + e) : make_uint4(0u, 0u, 0u, 0u);
             }
         }
+    };
+    const int first = (int)blockIdx.x + warp * active, step = active * kWarps;
+    const bool mine = (int)blockIdx.x < active && first < tiles, early = mine && low + first * kTile + kTile <= (int)pos;
+    if (early) load(low + first * kTile);     // cached rows only: they travel while the queries are prepared
+
+    // norm and rotation of a head in registers
+    auto prepare = [&](float2(&x)[KP], const float2(&scale)[KP]) {
+        float q = 0.f;
+#pragma unroll
+        for (int i = 0; i < KP; ++i) q += x[i].x * x[i].x + x[i].y * x[i].y;
+        const float rstd = 1.0f / sqrtf(warp_sum(q) / (float)a.D + a.eps);
+#pragma unroll
+        for (int i = 0; i < KP; ++i) {
+            const float u = x[i].x * rstd * scale[i].x, w = x[i].y * rstd * scale[i].y;
+            x[i] = make_float2(u * cs[i].x - w * cs[i].y, w * cs[i].x + u * cs[i].y);
+        }
+    };
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+        const int h = warp + x * kWarps;
+        if (h >= nh) break;
+        prepare(xq[x], qs);
+#pragma unroll
+        for (int i = 0; i < KP; ++i) {
+            const int d = 2 * (lane + 32 * i);
+            uint32_t hi, lo;
+            lm::split2(xq[x][i].x * a.scale, xq[x][i].y * a.scale, hi, lo);
+            if (d < a.D) {
+                *reinterpret_cast<uint32_t*>(qh + h * ldq + d) = hi;
+                *reinterpret_cast<uint32_t*>(ql + h * ldq + d) = lo;
+            }
+        }
+    }
+    if (warp == kWarps - 1 && (tiles - 1) % active == (int)blockIdx.x) {
+        bf16* dst = reinterpret_cast<bf16*>(a.ring) + (size_t)(pos % (uint32_t)a.ring_rows) * W;
+        prepare(xk, ks);
+#pragma unroll
+        for (int i = 0; i < KP; ++i) {
+            const int d = 2 * (lane + 32 * i);
+            if (d < a.D) *reinterpret_cast<__nv_bfloat162*>(dst + (size_t)g * a.D + d) = __floats2bfloat162_rn(xk[i].x, xk[i].y);
+        }
+        const float* xv = a.mix + (size_t)(a.H + a.G) * a.D + (size_t)g * a.E;
+        for (int e = 2 * lane; e < a.E; e += 64) {
+            const float2 u = *reinterpret_cast<const float2*>(xv + e);
+            *reinterpret_cast<__nv_bfloat162*>(dst + (size_t)a.G * a.D + (size_t)g * a.E + e) = __floats2bfloat162_rn(u.x, u.y);
+        }
+    }
+    __syncthreads();
+
+    float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f, o[EB][8][4];
+#pragma unroll
+    for (int c = 0; c < EB; ++c)
+#pragma unroll
+        for (int j = 0; j < 8; ++j) o[c][j][0] = o[c][j][1] = o[c][j][2] = o[c][j][3] = 0.f;
+    for (int tile = mine ? first : tiles; tile < tiles; tile += step) {
+        const int p0 = low + tile * kTile;
+        if (tile != first || !early) load(p0);
         float s0[4] = {}, s1[4] = {};
 #pragma unroll
         for (int b = 0; b < NB; ++b)
@@ -250,38 +326,89 @@ __global__ void __launch_bounds__(kThreads) grouped_step_mma_kernel(const Args a
         l_s[warp][gr] = l0; l_s[warp][gr + 8] = l1;
     }
     // column 2 t + (e & 1) of product j is value feature c * 64 + 8 (2 t + (e & 1)) + j
+    if (mine)
 #pragma unroll
-    for (int c = 0; c < EB; ++c)
+        for (int c = 0; c < EB; ++c)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            const int h = gr + (e >> 1) * 8, col = c * 64 + (2 * t + (e & 1)) * 8;
-            if (h < nh && col < a.E) {
-                float4* dst = reinterpret_cast<float4*>(acc_s + ((size_t)warp * nh + h) * a.E + col);
-                dst[0] = make_float4(o[c][0][e], o[c][1][e], o[c][2][e], o[c][3][e]);
-                dst[1] = make_float4(o[c][4][e], o[c][5][e], o[c][6][e], o[c][7][e]);
+            for (int e = 0; e < 4; ++e) {
+                const int h = gr + (e >> 1) * 8, col = c * 64 + (2 * t + (e & 1)) * 8;
+                if (h < nh && col < a.E) {
+                    float4* dst = reinterpret_cast<float4*>(acc_s + ((size_t)warp * nh + h) * a.E + col);
+                    dst[0] = make_float4(o[c][0][e], o[c][1][e], o[c][2][e], o[c][3][e]);
+                    dst[1] = make_float4(o[c][4][e], o[c][5][e], o[c][6][e], o[c][7][e]);
+                }
             }
-        }
     __syncthreads();
+    // the warps' parts of a head, four features per thread; a warp without a tile has the maximum -inf and left no sums
+    const int quads = a.E / 4;
     const int pitch = pitch_of(a.E);
-    float* part = a.partial + ((size_t)blockIdx.x * a.H + h0) * pitch;
-    for (int i = threadIdx.x; i < nh * a.E; i += kThreads) {
-        const int h = i / a.E, e = i - h * a.E;
-        float M = -INFINITY, s = 0.f, l = 0.f;
+    float* part = CL ? acc_s : a.partial + ((size_t)blockIdx.x * a.H + h0) * pitch;
+    for (int i = threadIdx.x; i < nh * quads; i += kThreads) {
+        const int h = i / quads, e = (i - h * quads) * 4;
+        float M = -INFINITY, l = 0.f;
+        float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
         for (int w = 0; w < kWarps; ++w) M = fmaxf(M, m_s[w][h]);
 #pragma unroll
         for (int w = 0; w < kWarps; ++w) {
-            const float f = expf(m_s[w][h] - M);              // 0 for warps without a tile
-            s = fmaf(f, acc_s[((size_t)w * nh + h) * a.E + e], s);
+            if (m_s[w][h] == -INFINITY) continue;
+            const float f = expf(m_s[w][h] - M);
+            const float4 x = *reinterpret_cast<const float4*>(acc_s + ((size_t)w * nh + h) * a.E + e);
+            s.x = fmaf(f, x.x, s.x);
+            s.y = fmaf(f, x.y, s.y);
+            s.z = fmaf(f, x.z, s.z);
+            s.w = fmaf(f, x.w, s.w);
             l = fmaf(f, l_s[w][h], l);
         }
-        part[(size_t)h * pitch + e] = s;
+        *reinterpret_cast<float4*>(part + (CL ? (size_t)h * a.E : (size_t)h * pitch) + e) = s;      // CL: over warp 0's part, read by this thread only
         if (e == 0) {
-            part[(size_t)h * pitch + pitch - 2] = M;
-            part[(size_t)h * pitch + pitch - 1] = l;
+            if (CL) {
+                cta_m[h] = M;
+                cta_l[h] = l;
+            } else {
+                part[(size_t)h * pitch + pitch - 2] = M;
+                part[(size_t)h * pitch + pitch - 1] = l;
+            }
         }
     }
-    merge(a, h0, nh, active, weights);
+    if (!CL) {
+        merge(a, h0, nh, active, weights);
+        return;
+    }
+    namespace cg = cooperative_groups;
+    cg::cluster_group cluster = cg::this_cluster();
+    cluster.sync();
+    // every CTA merges a share of the outputs
+    for (int i = (int)blockIdx.x * kThreads + threadIdx.x; i < nh * quads; i += (int)gridDim.x * kThreads) {
+        const int h = i / quads, e = (i - h * quads) * 4;
+        float M = -INFINITY, ms[kCluster], ls[kCluster];
+        float4 x[kCluster];
+#pragma unroll
+        for (int j = 0; j < kCluster; ++j)
+            if (j < active) {
+                ms[j] = *cluster.map_shared_rank(&cta_m[h], j);
+                ls[j] = *cluster.map_shared_rank(&cta_l[h], j);
+                x[j] = *reinterpret_cast<const float4*>(cluster.map_shared_rank(acc_s + (size_t)h * a.E + e, j));
+            }
+#pragma unroll
+        for (int j = 0; j < kCluster; ++j)
+            if (j < active) M = fmaxf(M, ms[j]);
+        float l = a.sink ? expf(a.sink[h0 + h] - M) : 0.f;
+        float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int j = 0; j < kCluster; ++j)
+            if (j < active) {
+                const float f = expf(ms[j] - M);
+                l = fmaf(f, ls[j], l);
+                s.x = fmaf(f, x[j].x, s.x);
+                s.y = fmaf(f, x[j].y, s.y);
+                s.z = fmaf(f, x[j].z, s.z);
+                s.w = fmaf(f, x[j].w, s.w);
+            }
+        const float inv = 1.0f / l;
+        *reinterpret_cast<float4*>(a.out + (size_t)(h0 + h) * a.E + e) = make_float4(s.x * inv, s.y * inv, s.z * inv, s.w * inv);
+    }
+    cluster.sync();                       // no CTA leaves while its shared memory is being read
 }
 
 // A warp per head; tiles of positions staged in shared memory and shared by the heads; a lane owns every 32nd feature.
@@ -367,31 +494,38 @@ inline bool takes_mma(int dt, int D, int E, const void* ring) {
     return dt == RCU_BF16 && D % 8 == 0 && E % 8 == 0 && D <= 256 && E <= 256 && (reinterpret_cast<uintptr_t>(ring) & 15) == 0;
 }
 
-// CTAs (grid.x) of a layer whose positions see at most `most` rows
-inline int splits(int sm_count, int rows_y, uint64_t most) {
-    const int tiles = (int)((most + kTile - 1) / kTile);
-    const int want = (tiles + kWarps - 1) / kWarps, room = sm_count / (rows_y > 0 ? rows_y : 1), spread = (tiles + 1) / 2 < room ? (tiles + 1) / 2 : room;
-    const int n = want > spread ? want : spread;
-    return n < 1 ? 1 : n > kMaxSplits ? kMaxSplits : n;
+// CTAs (grid.x) of a layer whose tokens see at most `most` rows: one tile per warp, as far as a cluster goes (`clusters`), beyond that
+// as many as the device holds
+inline int splits(int sm_count, int rows_y, uint64_t most, bool clusters) {
+    const int tiles = (int)std::min<uint64_t>((most + kTile - 1) / kTile, 1u << 26), want = (tiles + kWarps - 1) / kWarps;
+    if (clusters && want <= 4 * kCluster) return std::min(kCluster, std::max(1, (tiles + 1) / 2));
+    const int room = std::max(1, 2 * sm_count / std::max(1, rows_y));
+    return std::max(1, std::min(std::min(kMaxSplits, room), want));
 }
 
 inline rcu_status launch(rcu_device* dev, int dt, const Args& a, int n_splits) {
     const bool mma = takes_mma(dt, a.D, a.E, a.ring);
     const int heads = mma ? kMmaHeads : kFmaHeads, nh = a.H / a.G < heads ? a.H / a.G : heads;
     const dim3 grid(n_splits, a.G * head_groups(a.H, a.G, heads));
+    const bool cluster = mma && n_splits <= kCluster;
 #define RCU_GS(KERN_)                                                                                                            \
     do {                                                                                                                         \
         RCU_CUDA(dev, cudaFuncSetAttribute(KERN_, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)(smem > 48 * 1024 ? smem : 48 * 1024))); \
-        RCU_CUDA(dev, rcu_launch(dev, KERN_, grid, kThreads, smem, a));                                                          \
+        RCU_CUDA(dev, rcu_launch_cluster(dev, KERN_, grid, kThreads, smem, cluster ? n_splits : 0, a));                          \
+    } while (0)
+#define RCU_GS_C(NB_, EB_)                                              \
+    do {                                                                \
+        if (cluster) RCU_GS((grouped_step_mma_kernel<NB_, EB_, true>)); \
+        else RCU_GS((grouped_step_mma_kernel<NB_, EB_, false>));        \
     } while (0)
     if (mma) {
         const int nb = a.D <= 64 ? 2 : a.D <= 128 ? 4 : 8;
         const size_t smem = (size_t)2 * kMmaHeads * (nb * 32 + 8) * 2 + (size_t)kWarps * nh * a.E * 4;
 #define RCU_GS_E(NB_)                                                                     \
     do {                                                                                  \
-        if (a.E <= 64) RCU_GS((grouped_step_mma_kernel<NB_, 1>));                         \
-        else if (a.E <= 128) RCU_GS((grouped_step_mma_kernel<NB_, 2>));                   \
-        else RCU_GS((grouped_step_mma_kernel<NB_, 4>));                                   \
+        if (a.E <= 64) RCU_GS_C(NB_, 1);                                                  \
+        else if (a.E <= 128) RCU_GS_C(NB_, 2);                                            \
+        else RCU_GS_C(NB_, 4);                                                            \
     } while (0)
         if (nb == 2) RCU_GS_E(2);
         else if (nb == 4) RCU_GS_E(4);
@@ -411,6 +545,7 @@ inline rcu_status launch(rcu_device* dev, int dt, const Args& a, int n_splits) {
 #undef RCU_GS_T
     }
 #undef RCU_GS
+#undef RCU_GS_C
     RCU_LAUNCH_CHECK(dev);
     return RCU_OK;
 }

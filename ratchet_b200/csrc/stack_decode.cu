@@ -1000,8 +1000,9 @@ uint64_t grouped_seen(const rcu_stack_run& r) {      // rows a token can see at 
     return std::min<uint64_t>(most, r.ring_rows);
 }
 int grouped_splits(const rcu_device* dev, const rcu_stack_run& r, int dt) {
-    const int per = gstep::takes_mma(dt, (int)r.dim, (int)r.vdim, r.state) ? gstep::kMmaHeads : gstep::kFmaHeads;
-    return gstep::splits(dev->sm_count, (int)r.kv_heads * gstep::head_groups((int)r.heads, (int)r.kv_heads, per), grouped_seen(r));
+    const bool mma = gstep::takes_mma(dt, (int)r.dim, (int)r.vdim, r.state);
+    const int groups = gstep::head_groups((int)r.heads, (int)r.kv_heads, mma ? gstep::kMmaHeads : gstep::kFmaHeads);
+    return gstep::splits(dev->sm_count, (int)r.kv_heads * groups, grouped_seen(r), mma);
 }
 
 // Warps per team.  A CTA's time is bound below by the memory system (its units' items, one after the other) and by the longest
