@@ -18,27 +18,48 @@ struct KvArgs {
     uint32_t pos;              // position of the block's first token
 };
 
-// A group of lanes per (row, kv head): rows [0, L - T) come from the ring, the others from the block.
+constexpr int kKvHeads = 2;           // kv heads of a row that a group of lanes takes
+
+// A group of lanes per (row, kKvHeads kv heads), or (V == 1) a warp per (row, kv head): rows [0, L - T) come from the ring, the
+// others from the block.
 template <class T, int V>
 __global__ void __launch_bounds__(256) kv_rows_kernel(const KvArgs a, const T* __restrict__ x, T* ring, T* __restrict__ out, long long n, int lanes) {
     rcu_kernel_entry();
-    const int lane = threadIdx.x & 31, s = lane & (lanes - 1), D = a.norm.dim;
+    using Vec = lm::HeadVec<T, V>;
+    constexpr int N = V == 1 ? 1 : kKvHeads;
+    const int lane = threadIdx.x & 31, s = lane & (lanes - 1), D = a.norm.dim, per = (a.G + N - 1) / N;
     const long long item = ((long long)blockIdx.x * 8 + (threadIdx.x >> 5)) * (32 / lanes) + lane / lanes;
     const bool live = item < n;
-    const int r = live ? (int)(item / a.G) : 0, g = live ? (int)(item - (long long)r * a.G) : 0;
+    const int r = live ? (int)(item / per) : 0, g = live ? (int)(item - (long long)r * per) * N : 0, heads = live ? min(N, a.G - g) : 0;
     const int old = a.L - a.T, t = r - old;
     const long long W = (long long)a.G * (D + a.E), kc = (long long)g * D, vc = (long long)a.G * D + (long long)g * a.E;
     T* orow = out + r * W;
     const bool fresh = live && t >= 0;
     const T* src = fresh ? x + t * a.pitch : ring + (size_t)((a.pos - (uint32_t)(old - r)) % (uint32_t)a.ring_rows) * W;
     T* store = fresh && a.direct && t >= a.T - a.keep ? ring + (size_t)((a.pos + (uint32_t)t) % (uint32_t)a.ring_rows) * W : nullptr;
-    lm::head_norm_rotate<T, V>(a.norm, fresh ? src + kc : x, reinterpret_cast<const float2*>(a.norm.angles) + (long long)(fresh ? t : 0) * a.norm.pairs,
-                               orow + kc, store ? store + kc : nullptr, s, lanes, fresh);
-    if (!live) return;
-    using Vec = lm::HeadVec<T, V>;
-    if (!fresh)
-        for (int c = s * V; c < D; c += lanes * V) *reinterpret_cast<Vec*>(orow + kc + c) = *reinterpret_cast<const Vec*>(src + kc + c);
-    for (int c = s * V; c < a.E; c += lanes * V) {
+    if constexpr (V == 1) {
+        lm::head_norm_rotate<T>(a.norm, fresh ? src + kc : x, fresh ? t : 0, orow + kc, store ? store + kc : nullptr, s, fresh);
+        if (live && !fresh)
+            for (int c = s; c < D; c += 32) orow[kc + c] = src[kc + c];
+    } else {
+        lm::HeadPart<T, V> part;
+        part.load(a.norm, fresh ? t : 0, s, live);
+        Vec k[N];
+#pragma unroll
+        for (int j = 0; j < N; ++j) k[j] = part.in && j < heads ? *reinterpret_cast<const Vec*>(src + kc + j * D + part.c) : Vec{};
+#pragma unroll
+        for (int j = 0; j < N; ++j) {
+            const Vec y = part.apply(a.norm, k[j], lanes);
+            if (fresh) k[j] = y;
+            if (part.in && j < heads) {
+                *reinterpret_cast<Vec*>(orow + kc + j * D + part.c) = k[j];
+                if (store) *reinterpret_cast<Vec*>(store + kc + j * D + part.c) = k[j];
+            }
+        }
+    }
+    // the values of these heads lie side by side
+#pragma unroll 4
+    for (int c = s * V; c < heads * a.E; c += lanes * V) {
         const Vec v = *reinterpret_cast<const Vec*>(src + vc + c);
         *reinterpret_cast<Vec*>(orow + vc + c) = v;
         if (store) *reinterpret_cast<Vec*>(store + vc + c) = v;
@@ -62,12 +83,13 @@ rcu_status launch_kv_append(rcu_device* dev, KvArgs a, const void* x, void* ring
     constexpr int V = 16 / (int)sizeof(T);
     const int D = a.norm.dim, old = a.L - a.T;
     const size_t W = (size_t)a.G * (D + a.E);
-    const long long n = (long long)a.L * a.G;
     // the rows read and the rows written are different ones when together they fit the ring
     a.direct = a.keep > 0 && (old == 0 || a.L <= a.ring_rows);
-    const bool aligned = ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(ring) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+    const bool aligned = ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(ring) | reinterpret_cast<uintptr_t>(out) |
+                           reinterpret_cast<uintptr_t>(a.norm.scale) | reinterpret_cast<uintptr_t>(a.norm.angles)) & 15) == 0;
     const bool vec = D % V == 0 && a.E % V == 0 && D <= 32 * V && a.pitch % V == 0 && aligned;
     const int lanes = vec ? lm::head_lanes(D, V) : 32, per = 8 * (32 / lanes);
+    const long long n = (long long)a.L * (vec ? (a.G + kKvHeads - 1) / kKvHeads : a.G);
     const unsigned grid = (unsigned)((n + per - 1) / per);
     if (vec) rcu_launch(dev, kv_rows_kernel<T, V>, grid, 256, 0, a, (const T*)x, (T*)ring, (T*)out, n, lanes);
     else rcu_launch(dev, kv_rows_kernel<T, 1>, grid, 256, 0, a, (const T*)x, (T*)ring, (T*)out, n, lanes);

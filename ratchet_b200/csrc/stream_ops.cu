@@ -311,7 +311,9 @@ __global__ void __launch_bounds__(128) rotary_angles_kernel(const float* __restr
     if (i < n) out[i] = lm::rotary_angle(freqs, pairs, (int)(i % pairs), position + (uint32_t)(i / pairs), magnitude);
 }
 
-// dst[t, h] = rotate(rms_norm(x[t, head h])); a group of lanes per (token, head)
+constexpr int kHeadsPerGroup = 4;        // heads of a token that a group of lanes takes, their loads in flight together
+
+// dst[t, h] = rotate(rms_norm(x[t, head h])); a group of lanes per (token, kHeadsPerGroup heads), or (V == 1) a warp per head
 template <class T, int V>
 __global__ void __launch_bounds__(256) norm_rotary_kernel(const lm::HeadNorm a, const T* __restrict__ x, long long pitch, T* __restrict__ out, int H, long long n,
                                                           int lanes) {
@@ -319,17 +321,37 @@ __global__ void __launch_bounds__(256) norm_rotary_kernel(const lm::HeadNorm a, 
     const int lane = threadIdx.x & 31;
     const long long item = ((long long)blockIdx.x * 8 + (threadIdx.x >> 5)) * (32 / lanes) + lane / lanes;
     const bool live = item < n;
-    const long long t = live ? item / H : 0;
-    const int h = live ? (int)(item - t * H) : 0;
-    lm::head_norm_rotate<T, V>(a, x + t * pitch + (long long)h * a.dim, reinterpret_cast<const float2*>(a.angles) + t * a.pairs,
-                               out + (t * H + h) * a.dim, (T*)nullptr, lane & (lanes - 1), lanes, live);
+    if constexpr (V == 1) {
+        const long long t = live ? item / H : 0;
+        const int h = live ? (int)(item - t * H) : 0;
+        lm::head_norm_rotate<T>(a, x + t * pitch + (long long)h * a.dim, t, out + (t * H + h) * a.dim, (T*)nullptr, lane, live);
+    } else {
+        using Vec = lm::HeadVec<T, V>;
+        constexpr int N = kHeadsPerGroup;
+        const int per = (H + N - 1) / N;
+        const long long t = live ? item / per : 0;
+        const int h0 = live ? (int)(item - t * per) * N : 0;
+        lm::HeadPart<T, V> part;
+        part.load(a, t, lane & (lanes - 1), live);
+        const T* src = x + t * pitch + (long long)h0 * a.dim + part.c;
+        T* dst = out + (t * H + h0) * a.dim + part.c;
+        Vec v[N];
+#pragma unroll
+        for (int j = 0; j < N; ++j) v[j] = part.in && h0 + j < H ? *reinterpret_cast<const Vec*>(src + (long long)j * a.dim) : Vec{};
+#pragma unroll
+        for (int j = 0; j < N; ++j) {
+            const Vec y = part.apply(a, v[j], lanes);
+            if (part.in && h0 + j < H) *reinterpret_cast<Vec*>(dst + (long long)j * a.dim) = y;
+        }
+    }
 }
 
 template <class T>
 void launch_norm_rotary(rcu_device* dev, const lm::HeadNorm& a, const void* x, long long pitch, void* out, int H, long long T_) {
-    constexpr int V = 16 / (int)sizeof(T);
-    const long long n = T_ * H;
-    const bool vec = a.dim % V == 0 && a.dim <= 32 * V && pitch % V == 0 && ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(out)) & 15) == 0;
+    constexpr int V = 16 / (int)sizeof(T), N = kHeadsPerGroup;
+    const bool vec = a.dim % V == 0 && a.dim <= 32 * V && pitch % V == 0 &&
+                     ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(out) | reinterpret_cast<uintptr_t>(a.scale) | reinterpret_cast<uintptr_t>(a.angles)) & 15) == 0;
+    const long long n = vec ? T_ * ((H + N - 1) / N) : T_ * H;
     const int lanes = vec ? lm::head_lanes(a.dim, V) : 32, per = 8 * (32 / lanes);
     const unsigned grid = (unsigned)((n + per - 1) / per);
     if (vec) rcu_launch(dev, norm_rotary_kernel<T, V>, grid, 256, 0, a, (const T*)x, pitch, (T*)out, H, n, lanes);

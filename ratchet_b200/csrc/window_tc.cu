@@ -4,14 +4,16 @@
 // CTA = 256 queries of one head, in two tiles of 128 that take turns: while the softmax warps of one tile work, the tensor core
 // runs the other tile's products.
 //   warp 0 (one lane)   TMA producer: the queries once, then 64 keys (own and shared features) and their values per stage;
-//   warp 1 (one lane)   per key tile n and query tile w: S_w = Q_w K^T into tensor memory, then O_w += P_w V of tile n - 1 with
+//   warp 1              per key tile n and query tile w: S_w = Q_w K^T into tensor memory, then O_w += P_w V of tile n - 1 with
 //                       P_w read from tensor memory - its value and its remainder, two products, so that attention weights
-//                       keep 16 bits of mantissa;
+//                       keep 16 bits of mantissa.  S and P of consecutive key tiles have buffers of their own, so the scores of a
+//                       tile are there before the weights of the one before are;
 //   warps 2-5, 6-9      softmax of tile 0 / 1, a query per thread: scores from tensor memory, mask, running maximum, weights
-//                       back to tensor memory.  The maximum that weights are taken against only moves when a score exceeds it
+//                       back over the scores.  The maximum that weights are taken against only moves when a score exceeds it
 //                       by more than 2^8, so that O_w is rescaled rarely; all of it is f32.
-// Tensor memory per query tile: 64 columns S, 64 columns P, up to 128 columns O.  A query tile passes over key tiles none of its
-// queries sees.  Every wait is bounded; one that gives up raises RCU_DEVFLAG_TIMEOUT and ends all others of the CTA.
+// Tensor memory per query tile: two buffers of 64 columns (S, then P), up to 128 columns O.  A query tile passes over key tiles none
+// of its queries sees.  CTAs with many key tiles start first.  Every wait is bounded; one that gives up raises RCU_DEVFLAG_TIMEOUT and
+// ends all others of the CTA.
 #include <cuda.h>
 
 #include "lm_mma.cuh"
@@ -40,21 +42,33 @@ __device__ __forceinline__ float ex2(float x) {
     return y;
 }
 
+// The i-th query block to start of n: blocks late in a chunk (without chunks: late in the sequence) see the most keys and go first.
+__device__ __forceinline__ int heavy_first(int i, int n, int chunk) {
+    const int p = chunk > 0 ? min(n, max(1, (chunk + kTileQ) / (2 * kTileQ))) : n;        // blocks per chunk
+    const int full = n / p, more = n - full * p, head = (p - more) * full;               // `more` places of a chunk occur once more than the others
+    if (i < head) return i % full * p + p - 1 - i / full;
+    i -= head;
+    return i % (full + 1) * p + more - 1 - i / (full + 1);
+}
+
+// NB: 64-column blocks of a query (own features, then shared ones; columns beyond the features are zero)
+template <int NB>
 __global__ void __launch_bounds__(kThreadsW, 1)
 window_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_constant__ CUtensorMap qrmap, const __grid_constant__ CUtensorMap kmap,
                  const __grid_constant__ CUtensorMap krmap, const __grid_constant__ CUtensorMap vmap, const TcArgs a) {
     rcu_kernel_entry_wait_only();
     extern __shared__ unsigned char smem_dyn[];
-    const int nd = (a.D + 63) / 64, nb = nd + (a.R + 63) / 64, eb = (a.E + 63) / 64;      // 64-column blocks
+    constexpr int nb = NB;
+    const int nd = (a.D + 63) / 64, eb = (a.E + 63) / 64;      // 64-column blocks
     unsigned char* qs = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_dyn) + 1023) & ~(uintptr_t)1023);
     unsigned char* ks = qs + 2 * nb * kBlockQ;
     unsigned char* vs = ks + 2 * nb * kBlockK;
-    __shared__ __align__(8) uint64_t q_full, k_full[2], k_empty[2], v_full[2], v_empty[2], s_full[2], p_full[2], pv_done[2], drained;
+    __shared__ __align__(8) uint64_t q_full, k_full[2], k_empty[2], v_full[2], v_empty[2], s_full[2][2], p_full[2][2], pv_done[2], drained;
     __shared__ uint32_t tmem_slot;
     __shared__ volatile int abort_flag;
 
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int h = blockIdx.y, hk = h / (a.H / a.G), i0 = blockIdx.x * 2 * kTileQ;
+    const int h = blockIdx.x, hk = h / (a.H / a.G), i0 = heavy_first(blockIdx.y, gridDim.y, a.see.chunk) * 2 * kTileQ;
     const int base = a.L - a.T + i0, nq = min(2 * kTileQ, a.T - i0);    // key row of the CTA's first query; its queries
     const int first = a.see.first(base);
     const int tiles = (base + nq - 1 - first) / kTileK + 1;
@@ -70,8 +84,10 @@ window_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_constant
             mbar_init(&k_empty[i], 1);
             mbar_init(&v_full[i], 1);
             mbar_init(&v_empty[i], 1);
-            mbar_init(&s_full[i], 1);
-            mbar_init(&p_full[i], 4);
+            for (int b = 0; b < 2; ++b) {
+                mbar_init(&s_full[i][b], 1);
+                mbar_init(&p_full[i][b], 4);
+            }
             mbar_init(&pv_done[i], 1);
         }
         abort_flag = 0;
@@ -92,60 +108,91 @@ window_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_constant
             for (int w = 0; w < 2; ++w)
                 for (int b = 0; b < nb; ++b)
                     tma_load_3d(qs + (w * nb + b) * kBlockQ, b < nd ? &qmap : &qrmap, (b < nd ? b : b - nd) * 64, h, i0 + w * kTileQ, &q_full);
-            for (int n = 0; n < tiles; ++n) {
-                const int s = n & 1, j0 = first + n * kTileK;
-                if (n >= 2 && !mbar_wait(&k_empty[s], ((n >> 1) - 1) & 1, &abort_flag, a.status)) break;
-                mbar_expect_tx(&k_full[s], nb * kBlockK);
-                for (int b = 0; b < nd; ++b) tma_load_3d(ks + (s * nb + b) * kBlockK, &kmap, b * 64, hk, j0, &k_full[s]);
-                for (int b = nd; b < nb; ++b) tma_load_2d(ks + (s * nb + b) * kBlockK, &krmap, (b - nd) * 64, j0, &k_full[s]);
-                if (n >= 2 && !mbar_wait(&v_empty[s], ((n >> 1) - 1) & 1, &abort_flag, a.status)) break;
-                mbar_expect_tx(&v_full[s], eb * kBlockK);
-                for (int b = 0; b < eb; ++b) tma_load_3d(vs + (s * eb + b) * kBlockK, &vmap, b * 64, hk, j0, &v_full[s]);
+            // keys run one tile ahead of values
+            for (int n = 0; n <= tiles; ++n) {
+                if (n < tiles) {
+                    const int s = n & 1, j0 = first + n * kTileK;
+                    if (n >= 2 && !mbar_wait(&k_empty[s], ((n >> 1) - 1) & 1, &abort_flag, a.status)) break;
+                    mbar_expect_tx(&k_full[s], nb * kBlockK);
+                    for (int b = 0; b < nd; ++b) tma_load_3d(ks + (s * nb + b) * kBlockK, &kmap, b * 64, hk, j0, &k_full[s]);
+                    for (int b = nd; b < nb; ++b) tma_load_2d(ks + (s * nb + b) * kBlockK, &krmap, (b - nd) * 64, j0, &k_full[s]);
+                }
+                if (n > 0) {
+                    const int v = n - 1, s = v & 1, j0 = first + v * kTileK;
+                    if (v >= 2 && !mbar_wait(&v_empty[s], ((v >> 1) - 1) & 1, &abort_flag, a.status)) break;
+                    mbar_expect_tx(&v_full[s], eb * kBlockK);
+                    for (int b = 0; b < eb; ++b) tma_load_3d(vs + (s * eb + b) * kBlockK, &vmap, b * 64, hk, j0, &v_full[s]);
+                }
             }
         }
     } else if (warp == 1) {
-        if (lane == 0) {
-            const uint32_t idesc_s = umma_idesc_f16(kTileQ, kTileK, true);
-            const uint32_t idesc_o = umma_idesc_f16(kTileQ, (a.E + 15) & ~15, true) | (1u << 16);     // V is stored with its columns contiguous
-            const int lo[2] = {lo_of(0), lo_of(1)}, hi[2] = {hi_of(0), hi_of(1)};
-            bool ok = mbar_wait(&q_full, 0, &abort_flag, a.status);
-            tc_fence_after();
-            for (int n = 0; n <= tiles && ok; ++n) {
-                const int s = n & 1, p = s ^ 1;
-                if (n < tiles) ok = mbar_wait_spin(&k_full[s], (n >> 1) & 1, &abort_flag, a.status);
-                if (n > 0) ok = ok && mbar_wait_spin(&v_full[p], ((n - 1) >> 1) & 1, &abort_flag, a.status);
-                for (int w = 0; w < 2 && ok; ++w) {
-                    const bool pv = n - 1 >= lo[w] && n - 1 < hi[w], sc = n >= lo[w] && n < hi[w];
-                    const uint32_t t = tmem + (uint32_t)w * 256;
-                    if (pv) {           // the tile's weights are written, hence its scores read
-                        ok = mbar_wait_spin(&p_full[w], (n - 1 - lo[w]) & 1, &abort_flag, a.status);
-                        if (!ok) break;
-                    }
+        // the whole warp keeps step, one elected lane issues
+        const uint32_t idesc_s = umma_idesc_f16(kTileQ, kTileK, true);
+        const uint32_t idesc_o = umma_idesc_f16(kTileQ, (a.E + 15) & ~15, true) | (1u << 16);     // V is stored with its columns contiguous
+        const int lo[2] = {lo_of(0), lo_of(1)}, hi[2] = {hi_of(0), hi_of(1)};
+        const uint64_t qd = umma_desc_sw128(qs), kd = umma_desc_sw128(ks), vd = umma_desc_sw128_mn(vs, kBlockK);
+        const bool leader = elect_one();
+        auto wait = [&](uint64_t* bar, int phase) { return (bool)__all_sync(0xffffffffu, mbar_wait_spin(bar, phase & 1, &abort_flag, a.status)); };
+        bool ok = wait(&q_full, 0);
+        tc_fence_after();
+        for (int n = 0; n <= tiles && ok; ++n) {
+            const int s = n & 1, p = s ^ 1;
+            if (n < tiles) {
+                ok = wait(&k_full[s], n >> 1);
+#pragma unroll
+                for (int w = 0; w < 2; ++w) {
+                    if (!ok || n < lo[w] || n >= hi[w]) continue;
+                    // the buffer's last weights have been read
+                    if (n - 2 >= lo[w]) ok = wait(&pv_done[w], n - 2 - lo[w]);
+                    if (!ok) continue;
                     tc_fence_after();
-                    if (sc) {
-                        for (int b = 0; b < nb; ++b) {
-                            const uint64_t ad = umma_desc_sw128(qs + (w * nb + b) * kBlockQ), bd = umma_desc_sw128(ks + (s * nb + b) * kBlockK);
-                            const int cols = min(64, b < nd ? a.D - 64 * b : a.R - 64 * (b - nd));
-                            for (int k = 0; k * 16 < cols; ++k) umma_f16(t, ad + 2 * k, bd + 2 * k, idesc_s, (b > 0 || k > 0) ? 1u : 0u);
-                        }
-                        umma_commit(&s_full[w]);
+                    if (leader) {
+                        const uint32_t t = tmem + (uint32_t)w * 256 + 64 * s;
+                        const uint64_t bd = kd + (uint64_t)(s * NB * (kBlockK >> 4));
+#pragma unroll
+                        for (int b = 0; b < NB; ++b)
+#pragma unroll
+                            for (int k = 0; k < 4; ++k)
+                                umma_f16(t, qd + (w * NB + b) * (kBlockQ >> 4) + 2 * k, bd + b * (kBlockK >> 4) + 2 * k, idesc_s, (b > 0 || k > 0) ? 1u : 0u);
+                        umma_commit(&s_full[w][s]);
                     }
-                    if (pv) {
-                        const uint64_t vd = umma_desc_sw128_mn(vs + p * eb * kBlockK, kBlockK);
+                    __syncwarp();
+                }
+                if (!ok) break;
+                if (leader) umma_commit(&k_empty[s]);
+                __syncwarp();
+            }
+            if (n > 0) {
+                ok = wait(&v_full[p], (n - 1) >> 1);
+#pragma unroll
+                for (int w = 0; w < 2; ++w) {
+                    if (!ok || n - 1 < lo[w] || n - 1 >= hi[w]) continue;
+                    ok = wait(&p_full[w][p], (n - 1 - lo[w]) >> 1);
+                    if (!ok) continue;
+                    tc_fence_after();
+                    if (leader) {
+                        const uint32_t t = tmem + (uint32_t)w * 256;
+                        const uint64_t bd = vd + (uint64_t)(p * eb * (kBlockK >> 4));
+                        const uint32_t more = n - 1 > lo[w] ? 1u : 0u;
+#pragma unroll
                         for (int half = 0; half < 2; ++half)          // weights, then their remainders
+#pragma unroll
                             for (int k = 0; k < kTileK / 16; ++k)      // 16 keys are two 1024-byte groups of V, eight columns of P
-                                umma_f16_ta(t + 128, t + 64 + 32 * half + 8 * k, vd + 128 * k, idesc_o, (n - 1 > lo[w] || half > 0 || k > 0) ? 1u : 0u);
+                                umma_f16_ta(t + 128, t + 64 * p + 32 * half + 8 * k, bd + 128 * k, idesc_o, half > 0 || k > 0 ? 1u : more);
                         umma_commit(&pv_done[w]);
                     }
+                    __syncwarp();
                 }
-                if (n < tiles) umma_commit(&k_empty[s]);
-                if (n > 0) umma_commit(&v_empty[p]);
-            }
-            if (!ok) {                  // given up: let the products in flight end before tensor memory is freed
-                umma_commit(&drained);
-                for (int i = 0; i < (1 << 20) && !gemvq8::mbar_test_wait(&drained, 0); ++i) {}
+                if (!ok) break;
+                if (leader) umma_commit(&v_empty[p]);
+                __syncwarp();
             }
         }
+        if (!ok && leader) {            // given up: let the products in flight end before tensor memory is freed
+            umma_commit(&drained);
+            for (int i = 0; i < (1 << 20) && !gemvq8::mbar_test_wait(&drained, 0); ++i) {}
+        }
+        __syncwarp();
     } else {
         const int w = warp < 6 ? 0 : 1, quarter = warp & 3;
         const int r = w * kTileQ + quarter * 32 + lane, row = base + r;        // query of the CTA, its key row
@@ -158,45 +205,44 @@ window_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_constant
         float m = -INFINITY, l = 0.f;
         bool ok = true;
         for (int n = lo; n < hi; ++n) {
-            ok = __all_sync(0xffffffffu, mbar_wait_spin(&s_full[w], (n - lo) & 1, &abort_flag, a.status));
+            const int b = n & 1;
+            ok = __all_sync(0xffffffffu, mbar_wait_spin(&s_full[w][b], ((n - lo) >> 1) & 1, &abort_flag, a.status));
             if (!ok) break;
             tc_fence_after();
             float s[64];
-            tmem_ld_32x32(t, s);
-            tmem_ld_32x32(t + 32, s + 32);
+            tmem_ld_32x64(t + 64 * b, s);
             const int j0 = first + n * kTileK;
-            float top = -INFINITY;
-            if (j0 + kTileK - 1 <= row0 && j0 >= low1) {
+            if (j0 + kTileK - 1 > row0 || j0 < low1) {
 #pragma unroll
-                for (int j = 0; j < 64; ++j) {
-                    s[j] *= sc;
-                    top = fmaxf(top, s[j]);
-                }
-            } else {
-#pragma unroll
-                for (int j = 0; j < 64; ++j) {
-                    s[j] = j0 + j <= row && j0 + j >= low ? s[j] * sc : -INFINITY;
-                    top = fmaxf(top, s[j]);
-                }
+                for (int j = 0; j < 64; ++j)
+                    if (j0 + j > row || j0 + j < low) s[j] = -INFINITY;
             }
+            float top4[4] = {s[0], s[1], s[2], s[3]};
+#pragma unroll
+            for (int j = 4; j < 64; ++j) top4[j & 3] = fmaxf(top4[j & 3], s[j]);
+            const float top = fmaxf(fmaxf(top4[0], top4[1]), fmaxf(top4[2], top4[3])) * sc;      // sc > 0
             const bool move = top > m + 8.f || (m == -INFINITY && top > -INFINITY);
             const float next = move ? top : m;
             const float corr = move ? ex2(m - next) : 1.f;                    // 0 while no key has been seen
             m = next;
-            l *= corr;
-            const float z = m == -INFINITY ? 0.f : m;
-            uint32_t ph[32], pl[32];
+            const float z = m == -INFINITY ? 0.f : -m;
+            float l4[4] = {l * corr, 0.f, 0.f, 0.f};
+            uint32_t pw[64];                                                  // weights, then their remainders
 #pragma unroll
             for (int j = 0; j < 32; ++j) {
-                const float x = ex2(s[2 * j] - z), y = ex2(s[2 * j + 1] - z);
-                l += x + y;
-                lm::split2(x, y, ph[j], pl[j]);
+                const float x = ex2(fmaf(s[2 * j], sc, z)), y = ex2(fmaf(s[2 * j + 1], sc, z));
+                l4[j & 3] += x + y;
+                lm::split2(x, y, pw[j], pw[32 + j]);
             }
-            if (n > lo) {               // the product of the tile before has read P and written O
+            l = (l4[0] + l4[1]) + (l4[2] + l4[3]);
+            // O may be rescaled once the product of the tile before has been added.  The last tile always waits for that: a wait for
+            // the last product then never looks two completions back.
+            const bool any = __any_sync(0xffffffffu, move);
+            if (n > lo && (any || n == hi - 1)) {
                 ok = __all_sync(0xffffffffu, mbar_wait_spin(&pv_done[w], (n - lo - 1) & 1, &abort_flag, a.status));
                 if (!ok) break;
                 tc_fence_after();
-                if (__any_sync(0xffffffffu, move)) {
+                if (any) {
                     for (int c = 0; c < ocols; c += 32) {
                         float o[32];
                         tmem_ld_32x32(t + 128 + c, o);
@@ -206,11 +252,10 @@ window_tc_kernel(const __grid_constant__ CUtensorMap qmap, const __grid_constant
                     }
                 }
             }
-            tmem_st_32x32(t + 64, ph);
-            tmem_st_32x32(t + 96, pl);
+            tmem_st_32x64(t + 64 * b, pw);
             tc_fence_before();
             __syncwarp();
-            if (lane == 0) mbar_arrive(&p_full[w]);
+            if (lane == 0) mbar_arrive(&p_full[w][b]);
         }
         if (ok && hi > lo) {
             ok = __all_sync(0xffffffffu, mbar_wait(&pv_done[w], (hi - lo - 1) & 1, &abort_flag, a.status));
@@ -269,7 +314,7 @@ bool make_row_map(CUtensorMap* map, const void* base, uint64_t cols, uint64_t ro
 
 rcu_status rcu_window_tc(rcu_device* dev, const WindowArgs& a) {
     const int Q = a.D + a.R, nb = (a.D + 63) / 64 + (a.R + 63) / 64, eb = (a.E + 63) / 64;
-    if (a.T < 256 || a.D < 8 || a.D % 8 || a.R % 8 || a.E % 8 || a.E > 128 || nb > 4 || a.shared_pitch % 8) return RCU_ERR_UNSUPPORTED;
+    if (!(a.scale > 0.f) || a.T < 256 || a.T > 65535 * 2 * kTileQ || a.D < 8 || a.D % 8 || a.R % 8 || a.E % 8 || a.E > 128 || nb > 4 || a.shared_pitch % 8) return RCU_ERR_UNSUPPORTED;
     if ((reinterpret_cast<uintptr_t>(a.q) | reinterpret_cast<uintptr_t>(a.kv) | reinterpret_cast<uintptr_t>(a.shared) | reinterpret_cast<uintptr_t>(a.out)) & 15)
         return RCU_ERR_UNSUPPORTED;
     const size_t smem = 1024 + (size_t)2 * nb * kBlockQ + (size_t)2 * (nb + eb) * kBlockK;
@@ -285,10 +330,12 @@ rcu_status rcu_window_tc(rcu_device* dev, const WindowArgs& a) {
         kr = km;
     } else if (!make_head_map(&qr, q + a.D, a.R, a.H, a.T, Q, qp, kTileQ) || !make_row_map(&kr, a.shared, a.R, a.L, a.shared_pitch, kTileK))
         return rcu_fail(dev, RCU_ERR_CUDA, "window_attention: cuTensorMapEncodeTiled failed (T=%d L=%d H=%d)", a.T, a.L, a.H);
-    RCU_CUDA(dev, cudaFuncSetAttribute(window_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     const TcArgs t{(__nv_bfloat16*)a.out, a.T, a.L, a.H, a.G, a.D, a.R, a.E, a.see, a.scale, a.sink, dev->d_status};
-    const dim3 grid((a.T + 2 * kTileQ - 1) / (2 * kTileQ), a.H);
-    RCU_CUDA(dev, rcu_launch(dev, window_tc_kernel, grid, kThreadsW, smem, qm, qr, km, kr, vm, t));
+    const dim3 grid(a.H, (a.T + 2 * kTileQ - 1) / (2 * kTileQ));
+    void (*kern)(CUtensorMap, CUtensorMap, CUtensorMap, CUtensorMap, CUtensorMap, TcArgs) =
+        nb == 1 ? window_tc_kernel<1> : nb == 2 ? window_tc_kernel<2> : nb == 3 ? window_tc_kernel<3> : window_tc_kernel<4>;
+    RCU_CUDA(dev, cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    RCU_CUDA(dev, rcu_launch(dev, kern, grid, kThreadsW, smem, qm, qr, km, kr, vm, t));
     RCU_LAUNCH_CHECK(dev);
     return RCU_OK;
 }

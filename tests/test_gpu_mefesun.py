@@ -92,6 +92,18 @@ def test_a_loud_token_is_seen_in_its_chunk_only(dev, tmp_path, dtype, chunk, siz
         assert rel(got, want[:len(got)]) < limit, first
 
 
+@pytest.mark.parametrize("sizes", [{}, dict(dim=128, vdim=64, heads=6), dict(dim=18, vdim=10)])
+def test_caches_of_thousands_of_rows(dev, tmp_path, sizes):
+    """The decode attention of a cache that more CTAs share than a cluster holds."""
+    cfg, W = B.loud_case(6000, **sizes)
+    tokens = [1 if k in (0, 130) else 2 + k % 30 for k in range(300)]
+    want = mp.forward(cfg, W, tokens)
+    m = load(dev, B.write_model(str(tmp_path), cfg, W), "bfloat16")
+    st = m.new_state()
+    got = [m.prefill(tokens[:100], st, list(range(100)))] + [m.decode(st, t)[0].to_numpy() for t in tokens[100:]]
+    assert rel(np.concatenate(got), want) < LIMIT["bfloat16"]
+
+
 def test_without_a_mask_every_position_is_seen(dev, tmp_path):
     cfg, W = B.loud_case(7)
     del cfg["layers"][0]["mixer"]["mask"]
