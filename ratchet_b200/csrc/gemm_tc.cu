@@ -125,13 +125,15 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant__
             }
         }
     } else if (warp == 1) {
-        if (lane == 0) {
-            bool ok = true;
-            for (int it = 0; it < nk && ok; ++it) {
-                const int s = it % STAGES;
-                ok = mbar_wait(&full[s], (it / STAGES) & 1, abort_flag, status);
-                if (!ok) break;
-                tc_fence_after();
+        // the whole warp keeps step, one elected lane issues
+        const bool leader = elect_one();
+        bool ok = true;
+        for (int it = 0; it < nk && ok; ++it) {
+            const int s = it % STAGES;
+            ok = __all_sync(0xffffffffu, mbar_wait(&full[s], (it / STAGES) & 1, abort_flag, status));
+            if (!ok) break;
+            tc_fence_after();
+            if (leader) {
                 unsigned char* st = smem + s * STAGE;
                 const uint64_t adesc = umma_desc_sw128(st);
                 const uint64_t bdesc = umma_desc_sw128(st + A_BYTES);
@@ -142,8 +144,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant__
                 }
                 umma_commit(&empty[s]);      // the stage may be refilled once these MMAs have read it
             }
-            umma_commit(accum_bar);          // accumulators complete (arrives even after an abort so the epilogue ends)
+            __syncwarp();
         }
+        if (leader) umma_commit(accum_bar);          // accumulators complete (arrives even after an abort so the epilogue ends)
+        __syncwarp();
     } else if (warp < 6) {
         // epilogue warps 2..5: tensor-memory lane quarter = warp index modulo 4
         const int q = warp & 3;

@@ -135,30 +135,34 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant_
             }
         }
     } else if (warp == 1) {
-        if (lane == 0 && rank == 0) {
-            int it = 0, i = 0;
+        if (rank == 0) {               // the whole warp keeps step, one elected lane issues
+            const bool leader = elect_one();
+            const uint64_t desc0 = umma_desc_sw128(smem);
+            int s = 0, phase = 0, i = 0;
             bool ok = true;
             for (int t = pair; t < n_tiles && ok; t += n_pairs, ++i) {
                 const int b = i & 1;
                 if (i >= 2) {
-                    ok = mbar_wait(&acc_empty[b], ((i >> 1) - 1) & 1, abort_flag, status);
+                    ok = __all_sync(0xffffffffu, mbar_wait(&acc_empty[b], ((i >> 1) - 1) & 1, abort_flag, status));
                     if (!ok) break;
                     tc_fence_after();
                 }
                 const uint32_t acc = tmem_base + (uint32_t)(b * kAccCols);
-                for (int k = 0; k < nk; ++k, ++it) {
-                    const int s = it % kStages2;
-                    ok = mbar_wait(&full[s], (it / kStages2) & 1, abort_flag, status);
+                for (int k = 0; k < nk; ++k) {
+                    ok = __all_sync(0xffffffffu, mbar_wait(&full[s], phase, abort_flag, status));
                     if (!ok) break;
                     tc_fence_after();
-                    unsigned char* st = smem + s * kStageBytes2;
-                    const uint64_t adesc = umma_desc_sw128(st);
-                    const uint64_t bdesc = umma_desc_sw128(st + TM * TK * 2);
+                    if (leader) {
+                        const uint64_t adesc = desc0 + (uint64_t)(s * (kStageBytes2 >> 4)), bdesc = adesc + (TM * TK * 2 >> 4);
 #pragma unroll
-                    for (int kk = 0; kk < TK / 16; ++kk) umma2_f16(acc, adesc + 2 * kk, bdesc + 2 * kk, idesc, (k > 0 || kk > 0) ? 1u : 0u);
-                    umma2_commit_both(&empty[s]);
+                        for (int kk = 0; kk < TK / 16; ++kk) umma2_f16(acc, adesc + 2 * kk, bdesc + 2 * kk, idesc, (k > 0 || kk > 0) ? 1u : 0u);
+                        umma2_commit_both(&empty[s]);
+                    }
+                    __syncwarp();
+                    if (++s == kStages2) { s = 0; phase ^= 1; }
                 }
-                umma2_commit_both(&acc_full[b]);      // also after an abort, so that the epilogues end
+                if (leader) umma2_commit_both(&acc_full[b]);      // also after an abort, so that the epilogues end
+                __syncwarp();
             }
         }
     } else {
