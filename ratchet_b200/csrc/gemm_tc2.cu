@@ -36,6 +36,7 @@ constexpr int kStages2 = 6;
 constexpr int kTileN2 = 256;                       // weight rows per pair tile (128 per CTA)
 constexpr int kStageBytes2 = 2 * TM * TK * 2;      // 128 x 64 f16 of X + 128 x 64 f16 of W = 32 KiB
 constexpr int kAccCols = 256;                      // f32 accumulator columns per buffer
+constexpr int kTurnPitch = 9;        // float4s per row of an epilogue piece: 32 columns and a pad against bank conflicts
 
 __device__ __forceinline__ uint32_t cluster_ctarank() {
     uint32_t r;
@@ -90,6 +91,7 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant_
     uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(acc_empty + 2);
     volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
+    __shared__ float4 turn[4][32 * kTurnPitch];              // one piece of an accumulator per epilogue warp
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const uint32_t rank = cluster_ctarank();                 // 0 = leader
     const int pair = blockIdx.x >> 1, n_pairs = gridDim.x >> 1;
@@ -176,24 +178,37 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant_
             ok = mbar_wait(&acc_full[b], (i >> 1) & 1, abort_flag, status);
             if (!ok) break;
             tc_fence_after();
-            const int row = (t % tiles_m) * 2 * TM + (int)rank * TM + q * 32 + lane;
+            const int row0 = (t % tiles_m) * 2 * TM + (int)rank * TM + q * 32;
             const int n0 = (t / tiles_m) * kTileN2;
+            // 32 x 32 pieces: a thread reads a row from tensor memory; turned around in shared memory, eight lanes write (and
+            // read, for the residual) 32 consecutive columns of a row.  Rows are kilobytes apart: a lane per row wrote
+            // 128-byte lines in sixteen-byte pieces at 0.5 TB/s.
+            float4* mine = turn[q];
+            const int r = lane >> 3, quad = lane & 7;
 #pragma unroll 1
             for (int c = 0; c < kTileN2; c += 32) {
+                const int col = n0 + c + quad * 4;              // N is a multiple of 8
+                const bool in = col < N;
+                const float4 bias = in ? epi.bias4(col) : make_float4(0.f, 0.f, 0.f, 0.f);
+                float4 resid[8];
+#pragma unroll
+                for (int i = 0; i < 8; ++i) {
+                    const int row = row0 + 4 * i + r;
+                    resid[i] = sizeof(Out) == 4 && epi.resid && in && row < M ? *reinterpret_cast<const float4*>(epi.resid + (size_t)row * N + col)
+                                                                             : make_float4(0.f, 0.f, 0.f, 0.f);
+                }
                 float v[32];
                 tmem_ld_32x32(tmem_base + ((uint32_t)(q * 32) << 16) + (uint32_t)(b * kAccCols + c), v);
-                if (row < M) {
-                    const size_t base = (size_t)row * N + n0 + c;
 #pragma unroll
-                    for (int j = 0; j < 32; j += 8) {
-                        const int col = n0 + c + j;
-                        if (col + 8 <= N) {
-                            epi.store8(out, base + j, v + j, col);
-                        } else {
-                            for (int e = 0; e < 8 && col + e < N; ++e) out[base + j + e] = epi(v[j + e], col + e, base + j + e);
-                        }
-                    }
+                for (int j = 0; j < 8; ++j) mine[lane * kTurnPitch + j] = make_float4(v[4 * j], v[4 * j + 1], v[4 * j + 2], v[4 * j + 3]);
+                __syncwarp();
+#pragma unroll
+                for (int i = 0; i < 8; ++i) {
+                    const int row = row0 + 4 * i + r;
+                    const float4 x = mine[(4 * i + r) * kTurnPitch + quad];
+                    if (in && row < M) epi.store4(out, (size_t)row * N + col, x, bias, resid[i], col);
                 }
+                __syncwarp();
             }
             // this warp has read its part of the buffer: tell the leader's MMA thread
             tc_fence_before();

@@ -172,6 +172,28 @@ template <class Out> struct GemmEpilogue {
         if (sizeof(Out) == 4) v = resid ? fmaf(alpha, v, resid[idx]) : alpha * v;
         return from_f32<Out>(v);
     }
+    // four consecutive columns whose bias, and residual (f32 output), the caller has loaded; `col` a multiple of 4
+    struct alignas(4 * sizeof(Out)) Quad { Out v[4]; };
+    __device__ __forceinline__ float4 bias4(int col) const {
+        return bias ? make_float4(to_f32<Out>(bias[col]), to_f32<Out>(bias[col + 1]), to_f32<Out>(bias[col + 2]), to_f32<Out>(bias[col + 3])) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    __device__ __forceinline__ void store4(Out* out, size_t idx, const float4& acc, const float4& b, const float4& r, int col) const {
+        float v[4] = {acc.x + b.x, acc.y + b.y, acc.z + b.z, acc.w + b.w};
+        if (col < act.cols) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) v[e] = col + e < act.cols ? act(v[e]) : v[e];
+        }
+        if (sizeof(Out) == 4) {
+            v[0] = resid ? fmaf(alpha, v[0], r.x) : alpha * v[0];
+            v[1] = resid ? fmaf(alpha, v[1], r.y) : alpha * v[1];
+            v[2] = resid ? fmaf(alpha, v[2], r.z) : alpha * v[2];
+            v[3] = resid ? fmaf(alpha, v[3], r.w) : alpha * v[3];
+        }
+        Quad q;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) q.v[e] = from_f32<Out>(v[e]);
+        *reinterpret_cast<Quad*>(out + idx) = q;
+    }
     // eight consecutive columns, 16-byte aligned
     __device__ __forceinline__ void store8(Out* out, size_t idx, const float* acc, int col) const {
         __align__(16) Out h[8];
