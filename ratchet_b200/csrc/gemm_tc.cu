@@ -153,37 +153,30 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant__
         const int q = warp & 3;
         const bool ok = mbar_wait(accum_bar, 0, abort_flag, status);
         tc_fence_after();
-        const int row = m0 + q * 32 + lane;
         if (ok) {
+            // every stage has been read: their memory turns the pieces around.  N is a multiple of 4 (checked by the host)
+            float4* turn = reinterpret_cast<float4*>(smem) + q * 32 * kTurnPitch;
+            const int row0 = m0 + q * 32, r = lane >> 3;
 #pragma unroll 1
             for (int c = 0; c < BN; c += 32) {
+                const int col = n0 + c + (lane & 7) * 4;
+                const bool in = col < N, whole = splits == 1;      // not whole: a K slice leaves f32 partial sums, the summing kernel does the rest
+                const float4 bias = in && whole ? epi.bias4(col) : make_float4(0.f, 0.f, 0.f, 0.f);
+                float4 resid[8];
+#pragma unroll
+                for (int i = 0; i < 8; ++i) {
+                    const int row = row0 + 4 * i + r;
+                    resid[i] = sizeof(Out) == 4 && whole && epi.resid && in && row < M ? *reinterpret_cast<const float4*>(epi.resid + (size_t)row * N + col)
+                                                                                      : make_float4(0.f, 0.f, 0.f, 0.f);
+                }
                 float v[32];
                 tmem_ld_32x32(tmem_base + ((uint32_t)(q * 32) << 16) + (uint32_t)c, v);
-                if (row < M && splits > 1) {         // a K slice: f32 partial sums, bias and rounding in the summing kernel (N % 8 == 0)
-                    float* prow = partial + ((size_t)sp * M + row) * N + n0 + c;
-#pragma unroll
-                    for (int j = 0; j < 32; j += 4)
-                        if (n0 + c + j + 4 <= N) *reinterpret_cast<float4*>(prow + j) = make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]);
-                } else if (row < M) {
-                    const size_t base = (size_t)row * N + n0 + c;
-                    if ((N & 7) == 0) {              // rows start on 16-byte boundaries
-#pragma unroll
-                        for (int j = 0; j < 32; j += 8)
-                            if (n0 + c + j + 8 <= N) epi.store8(out, base + j, v + j, n0 + c + j);
-                    } else {                         // N a multiple of 4 (checked by the host): 4-element stores
-#pragma unroll
-                        for (int j = 0; j < 32; j += 4) {
-                            const int col = n0 + c + j;
-                            if (col + 4 <= N) {
-                                __align__(16) Out h[4];
-#pragma unroll
-                                for (int e = 0; e < 4; ++e) h[e] = epi(v[j + e], col + e, base + j + e);
-#pragma unroll
-                                for (int e = 0; e < (int)sizeof(Out) / 2; ++e) reinterpret_cast<uint2*>(out + base + j)[e] = reinterpret_cast<const uint2*>(h)[e];
-                            }
-                        }
-                    }
-                }
+                turn_piece(turn, v, [&](int i, int piece_row, const float4& x) {
+                    const int row = row0 + piece_row;
+                    if (!in || row >= M) return;
+                    if (whole) epi.store4(out, (size_t)row * N + col, x, bias, resid[i], col);
+                    else *reinterpret_cast<float4*>(partial + ((size_t)sp * M + row) * N + col) = x;
+                });
             }
         }
     } else if (WK != WK_F16) {

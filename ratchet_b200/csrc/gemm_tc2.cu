@@ -36,7 +36,6 @@ constexpr int kStages2 = 6;
 constexpr int kTileN2 = 256;                       // weight rows per pair tile (128 per CTA)
 constexpr int kStageBytes2 = 2 * TM * TK * 2;      // 128 x 64 f16 of X + 128 x 64 f16 of W = 32 KiB
 constexpr int kAccCols = 256;                      // f32 accumulator columns per buffer
-constexpr int kTurnPitch = 9;        // float4s per row of an epilogue piece: 32 columns and a pad against bank conflicts
 
 __device__ __forceinline__ uint32_t cluster_ctarank() {
     uint32_t r;
@@ -180,9 +179,6 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant_
             tc_fence_after();
             const int row0 = (t % tiles_m) * 2 * TM + (int)rank * TM + q * 32;
             const int n0 = (t / tiles_m) * kTileN2;
-            // 32 x 32 pieces: a thread reads a row from tensor memory; turned around in shared memory, eight lanes write (and
-            // read, for the residual) 32 consecutive columns of a row.  Rows are kilobytes apart: a lane per row wrote
-            // 128-byte lines in sixteen-byte pieces at 0.5 TB/s.
             float4* mine = turn[q];
             const int r = lane >> 3, quad = lane & 7;
 #pragma unroll 1
@@ -199,16 +195,10 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant_
                 }
                 float v[32];
                 tmem_ld_32x32(tmem_base + ((uint32_t)(q * 32) << 16) + (uint32_t)(b * kAccCols + c), v);
-#pragma unroll
-                for (int j = 0; j < 8; ++j) mine[lane * kTurnPitch + j] = make_float4(v[4 * j], v[4 * j + 1], v[4 * j + 2], v[4 * j + 3]);
-                __syncwarp();
-#pragma unroll
-                for (int i = 0; i < 8; ++i) {
-                    const int row = row0 + 4 * i + r;
-                    const float4 x = mine[(4 * i + r) * kTurnPitch + quad];
+                turn_piece(mine, v, [&](int i, int piece_row, const float4& x) {
+                    const int row = row0 + piece_row;
                     if (in && row < M) epi.store4(out, (size_t)row * N + col, x, bias, resid[i], col);
-                }
-                __syncwarp();
+                });
             }
             // this warp has read its part of the buffer: tell the leader's MMA thread
             tc_fence_before();

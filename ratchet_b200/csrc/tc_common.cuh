@@ -155,6 +155,20 @@ __device__ __forceinline__ uint64_t umma_desc_sw128_mn(const void* smem_ptr, uin
     return (uint64_t)((addr & 0x3FFFF) >> 4) | (uint64_t)(block_bytes >> 4) << 16 | (uint64_t)(1024 >> 4) << 32 | (uint64_t)1 << 46 | (uint64_t)2 << 61;
 }
 
+// One 32 x 32 piece of an accumulator on its way to memory: a lane holds a row; turned around in shared memory, eight lanes handle 32
+// consecutive columns of a row (four rows per pass), because rows are kilobytes apart and a lane per row writes 128-byte lines in
+// sixteen-byte pieces (0.5 TB/s measured).  put(i, row of the piece, four values of this lane's columns 4 (lane % 8)..).
+constexpr int kTurnPitch = 9;        // float4s per row: 32 columns and a pad against bank conflicts
+template <class Put> __device__ __forceinline__ void turn_piece(float4* turn, const float* v, Put put) {
+    const int lane = threadIdx.x & 31, r = lane >> 3, quad = lane & 7;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) turn[lane * kTurnPitch + j] = make_float4(v[4 * j], v[4 * j + 1], v[4 * j + 2], v[4 * j + 3]);
+    __syncwarp();
+#pragma unroll
+    for (int i = 0; i < 8; ++i) put(i, 4 * i + r, turn[(4 * i + r) * kTurnPitch + quad]);
+    __syncwarp();
+}
+
 // What the epilogue of a tensor-core GEMM does with an accumulator: Out = f16 / bf16: round(acc + bias);
 // Out = f32: residual + alpha * (acc + bias), the residual stream of a model that keeps it in 32 bits
 // (`resid` may be the output itself: every element is read by the thread that writes it).
