@@ -155,7 +155,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant__
         tc_fence_after();
         if (ok) {
             // every stage has been read: their memory turns the pieces around.  N is a multiple of 4 (checked by the host)
-            float4* turn = reinterpret_cast<float4*>(smem) + q * 32 * kTurnPitch;
+            float4* turn = reinterpret_cast<float4*>(smem) + q * kTurnQuads;
             const int row0 = m0 + q * 32, r = lane >> 3;
 #pragma unroll 1
             for (int c = 0; c < BN; c += 32) {

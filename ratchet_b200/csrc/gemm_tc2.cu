@@ -35,6 +35,8 @@ using namespace tc;
 constexpr int kStages2 = 6;
 constexpr int kTileN2 = 256;                       // weight rows per pair tile (128 per CTA)
 constexpr int kStageBytes2 = 2 * TM * TK * 2;      // 128 x 64 f16 of X + 128 x 64 f16 of W = 32 KiB
+constexpr int kEpilogueWarps = 8;                  // two per tensor-memory lane quarter, half of the columns each
+constexpr int kThreads2 = 64 + kEpilogueWarps * 32;
 constexpr int kAccCols = 256;                      // f32 accumulator columns per buffer
 
 __device__ __forceinline__ uint32_t cluster_ctarank() {
@@ -78,7 +80,7 @@ __device__ __forceinline__ void umma2_commit_both(uint64_t* bar) {
 }
 
 template <class Out>
-__global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(kThreadsTc, 1)
+__global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(kThreads2, 1)
 gemm_tc2_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant__ CUtensorMap wmap, const GemmEpilogue<Out> epi,
                 Out* out, int M, int N, int K, int tiles_m, int n_tiles, int* status, uint32_t idesc) {
     extern __shared__ unsigned char smem_dyn[];
@@ -90,7 +92,7 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant_
     uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(acc_empty + 2);
     volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
-    __shared__ float4 turn[4][32 * kTurnPitch];              // one piece of an accumulator per epilogue warp
+    __shared__ float4 turn[kEpilogueWarps][kTurnQuads];      // one piece of an accumulator per epilogue warp
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const uint32_t rank = cluster_ctarank();                 // 0 = leader
     const int pair = blockIdx.x >> 1, n_pairs = gridDim.x >> 1;
@@ -103,7 +105,7 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant_
         }
         for (int b = 0; b < 2; ++b) {
             mbar_init(&acc_full[b], 1);
-            mbar_init(&acc_empty[b], 8);           // four epilogue warps in each CTA
+            mbar_init(&acc_empty[b], 2 * kEpilogueWarps);           // both CTAs'
         }
         *abort_flag = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
@@ -167,8 +169,8 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant_
             }
         }
     } else {
-        // epilogue warps 2..5: tensor-memory lane quarter = warp index modulo 4
-        const int q = warp & 3;
+        // epilogue warps 2..9: tensor-memory lane quarter = warp index modulo 4
+        const int q = warp & 3, c0 = (warp - 2) / 4 * (kTileN2 / 2);
         const uint32_t acc_empty_leader0 = map_to_cta(smem_u32(&acc_empty[0]), 0);
         int i = 0;
         bool ok = true;
@@ -179,10 +181,10 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant_
             tc_fence_after();
             const int row0 = (t % tiles_m) * 2 * TM + (int)rank * TM + q * 32;
             const int n0 = (t / tiles_m) * kTileN2;
-            float4* mine = turn[q];
+            float4* mine = turn[warp - 2];
             const int r = lane >> 3, quad = lane & 7;
 #pragma unroll 1
-            for (int c = 0; c < kTileN2; c += 32) {
+            for (int c = c0; c < c0 + kTileN2 / 2; c += 32) {
                 const int col = n0 + c + quad * 4;              // N is a multiple of 8
                 const bool in = col < N;
                 const float4 bias = in ? epi.bias4(col) : make_float4(0.f, 0.f, 0.f, 0.f);
@@ -245,7 +247,7 @@ rcu_status launch_pair(rcu_device* dev, const CUtensorMap& xmap, const CUtensorM
     const int n_pairs = std::min(n_tiles, dev->sm_count / 2);
     const size_t smem = (size_t)kStages2 * kStageBytes2 + 1024 + 256;
     RCU_CUDA(dev, cudaFuncSetAttribute(gemm_tc2_kernel<Out>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    gemm_tc2_kernel<Out><<<2 * n_pairs, kThreadsTc, smem, dev->stream>>>(xmap, wmap, epi, (Out*)y, (int)M, (int)N, (int)K, tiles_m, n_tiles,
+    gemm_tc2_kernel<Out><<<2 * n_pairs, kThreads2, smem, dev->stream>>>(xmap, wmap, epi, (Out*)y, (int)M, (int)N, (int)K, tiles_m, n_tiles,
                                                                        dev->d_status, umma_idesc_f16(2 * TM, kTileN2, bf16));
     RCU_LAUNCH_CHECK(dev);
     return RCU_OK;

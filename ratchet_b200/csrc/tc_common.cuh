@@ -158,14 +158,15 @@ __device__ __forceinline__ uint64_t umma_desc_sw128_mn(const void* smem_ptr, uin
 // One 32 x 32 piece of an accumulator on its way to memory: a lane holds a row; turned around in shared memory, eight lanes handle 32
 // consecutive columns of a row (four rows per pass), because rows are kilobytes apart and a lane per row writes 128-byte lines in
 // sixteen-byte pieces (0.5 TB/s measured).  put(i, row of the piece, four values of this lane's columns 4 (lane % 8)..).
-constexpr int kTurnPitch = 9;        // float4s per row: 32 columns and a pad against bank conflicts
+// `turn`: 256 float4s of the warp's own, places swizzled against bank conflicts.
+constexpr int kTurnQuads = 32 * 8;
 template <class Put> __device__ __forceinline__ void turn_piece(float4* turn, const float* v, Put put) {
     const int lane = threadIdx.x & 31, r = lane >> 3, quad = lane & 7;
 #pragma unroll
-    for (int j = 0; j < 8; ++j) turn[lane * kTurnPitch + j] = make_float4(v[4 * j], v[4 * j + 1], v[4 * j + 2], v[4 * j + 3]);
+    for (int j = 0; j < 8; ++j) turn[lane * 8 + (j ^ (lane & 7))] = make_float4(v[4 * j], v[4 * j + 1], v[4 * j + 2], v[4 * j + 3]);
     __syncwarp();
 #pragma unroll
-    for (int i = 0; i < 8; ++i) put(i, 4 * i + r, turn[(4 * i + r) * kTurnPitch + quad]);
+    for (int i = 0; i < 8; ++i) put(i, 4 * i + r, turn[(4 * i + r) * 8 + (quad ^ ((4 * i + r) & 7))]);
     __syncwarp();
 }
 
@@ -194,8 +195,16 @@ template <class Out> struct GemmEpilogue {
     __device__ __forceinline__ void store4(Out* out, size_t idx, const float4& acc, const float4& b, const float4& r, int col) const {
         float v[4] = {acc.x + b.x, acc.y + b.y, acc.z + b.z, acc.w + b.w};
         if (col < act.cols) {
+            if (act.kind == RCU_ACT_RELU_SQUARED) {      // without branches: the others are dear enough to hide them
 #pragma unroll
-            for (int e = 0; e < 4; ++e) v[e] = col + e < act.cols ? act(v[e]) : v[e];
+                for (int e = 0; e < 4; ++e) {
+                    const float p = fmaxf(v[e], 0.f);
+                    v[e] = col + e < act.cols ? p * p : v[e];
+                }
+            } else {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) v[e] = col + e < act.cols ? act(v[e]) : v[e];
+            }
         }
         if (sizeof(Out) == 4) {
             v[0] = resid ? fmaf(alpha, v[0], r.x) : alpha * v[0];
