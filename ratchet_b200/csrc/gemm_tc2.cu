@@ -11,11 +11,12 @@
 //
 //   warp 0 (one lane)  TMA producer: its CTA's 128 x 64 X tile and 128 x 64 W tile per stage, completion
 //                      counted on the LEADER CTA's `full` barrier (the leader expects both CTAs' bytes);
-//   warp 1 (one lane, leader CTA only)  issues four tcgen05.mma.cta_group::2 per stage and commits them
+//   warp 1 (leader CTA only; one elected lane)  issues four tcgen05.mma.cta_group::2 per stage and commits them
 //                      to the stage's `empty` barrier of both CTAs, and at the end of a tile to both CTAs'
 //                      `acc_full` barrier;
-//   warps 2-5          epilogue of the CTA's own 128 rows: tcgen05.ld, bias, f16, 16-byte stores; then
-//                      one arrival per warp on the leader's `acc_empty` barrier.
+//   warps 2-9          epilogue of the CTA's own 128 rows, two warps per tensor-memory lane quarter: tcgen05.ld, 32 x 32
+//                      pieces turned around in shared memory, bias, activation, residual, whole lines to memory; then one
+//                      arrival per warp on the leader's `acc_empty` barrier.
 // The kernel is persistent: a pair walks over tiles pair, pair + n_pairs, ...; the accumulator is
 // double-buffered (2 x 256 of the 512 tensor-memory columns), so the epilogue of tile i overlaps the
 // MMAs of tile i + 1.  Tiles that share a weight tile run on neighbouring pairs at the same time (the
@@ -105,7 +106,7 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap xmap, const __grid_constant_
         }
         for (int b = 0; b < 2; ++b) {
             mbar_init(&acc_full[b], 1);
-            mbar_init(&acc_empty[b], 2 * kEpilogueWarps);           // both CTAs'
+            mbar_init(&acc_empty[b], 2 * kEpilogueWarps);       // both CTAs'
         }
         *abort_flag = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");

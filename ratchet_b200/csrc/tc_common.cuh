@@ -140,8 +140,8 @@ __device__ __forceinline__ void umma_f16_ta(uint32_t tmem_d, uint32_t tmem_a, ui
         : "memory");
 }
 // One lane of a converged warp.  A branch on it keeps the warp uniform for the compiler: the operands of the tensor-core instructions
-// behind it go straight into uniform registers (behind `lane == 0` every instruction pays for moving them there: 140 cycles per
-// tcgen05.mma were measured, against about 30).
+// behind it go straight into uniform registers (behind `lane == 0` every instruction pays for moving them there: 140 to 190 cycles
+// per tcgen05.mma were measured).
 __device__ __forceinline__ bool elect_one() {
     uint32_t pred;
     asm volatile("{\n\t.reg .pred p;\n\telect.sync _|p, 0xffffffff;\n\tselp.u32 %0, 1, 0, p;\n\t}" : "=r"(pred));
