@@ -40,7 +40,7 @@ def mefesun_config(c):
                                             "rot": {"base": 10000.0, "dims": 128,
                                                     "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}},
              "mlp": {"kind": "dense", "ff": c["ff"]}}
-    return {"architecture": "Mefesun", "width": d, "vocab": c["vocab"], "norm": {"eps": 1e-5}, "logit_softcap": 30.0, "layers": [layer] * c["layers"]}
+    return {"architecture": "Mefesun", "width": d, "vocab": c["vocab"], "norm": {"eps": 1e-5}, "logit_softcap": 50.0, "layers": [layer] * c["layers"]}
 
 
 def mefesun_shapes(config):

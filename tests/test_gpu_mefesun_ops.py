@@ -101,7 +101,7 @@ def test_rotary_angles_near_and_far(dev):
 
 
 @pytest.mark.parametrize("dt", [F32, BF16])
-@pytest.mark.parametrize("T,H,D,dims", [(1, 1, 2, 2), (5, 3, 9, 4), (6, 2, 24, 8), (33, 4, 64, 64), (7, 5, 128, 96), (3, 2, 256, 64), (4, 1, 300, 128)])
+@pytest.mark.parametrize("T,H,D,dims", [(1, 1, 2, 2), (5, 3, 9, 4), (6, 2, 24, 8), (6, 7, 24, 6), (9, 5, 64, 14), (33, 4, 64, 64), (7, 5, 128, 96), (3, 2, 256, 64), (4, 1, 300, 128)])
 def test_head_norm_and_rotation(dev, dt, T, H, D, dims):
     g = rng(D)
     rot = {"dims": dims, "base": 1000.0, "scaling": YARN}
